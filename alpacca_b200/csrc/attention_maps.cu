@@ -14,6 +14,9 @@
 //             out_scale.  The softmax is the running form, in key order; nothing is shared between warps, so
 //             a token's result does not depend on the rest of the batch.
 //
+//             `dist`: a penalty on distance, r1_h ln(1 + r2_h (p - s)), is taken off each scaled score (Chi et al.,
+//             "KERPLE: Kernelized Relative Positional Embedding for Length Extrapolation", the logarithmic form).
+//
 //   combine   the last step of `attend` alone, for maps that another kernel has attended (float [T, H*M, Dv]).
 //
 // Mixing of the softmax weights across heads (Shazeer et al., "Talking-Heads Attention", mix the weights of all heads
@@ -282,6 +285,151 @@ attention_prepare_vec_kernel(PrepareArgs a, int P, int vec_per_warp, long long q
   *reinterpret_cast<uint4*>(dst) = out;
 }
 
+// The query and key norm over the whole projection: all n_q query vectors of a token are divided by ONE root mean square
+// (over n_q * Dk numbers) and multiplied by a weight of that size, likewise its n_k key vectors.  A block per token.
+// The rest is as in the kernels above.  This form serves every size, dtype and rotation: the token's query and key rows
+// wait in shared memory as float32 between norm and rotation.
+template <typename T>
+__global__ void __launch_bounds__(256)
+attention_prepare_rows_kernel(PrepareArgs a) {
+  extern __shared__ float pr_rows[];                  // [(n_q + n_k) * Dk]
+  __shared__ float scratch[64];
+  pdl_wait();
+  pdl_trigger();
+  const int t = blockIdx.x;
+  const int b = a.tok_seq[t];
+  if (b < 0) return;
+  const int pos = a.tok_pos[t];
+  const int D = a.Dk, NQ = a.n_q * D, NK = a.write_cache ? a.n_k * D : 0;
+  T* row = reinterpret_cast<T*>(a.buf) + (size_t)t * a.stride;
+  const int page = a.write_cache ? a.block_table[(size_t)b * a.table_width + pos / a.page_size] : 0;
+  const int in_page = pos % a.page_size;
+  float sq = 0.f, sk = 0.f;
+  for (int i = threadIdx.x; i < NQ + NK; i += blockDim.x) {
+    const int col = i < NQ ? a.off_q + i : a.off_k + i - NQ;
+    const float v = to_f32(row[col]) + (a.bias != nullptr ? a.bias[col] : 0.f);
+    pr_rows[i] = v;
+    if (i < NQ) sq += v * v; else sk += v * v;
+  }
+  sq = block_sum(sq, scratch);
+  sk = block_sum(sk, scratch + 32);
+  const float iq = 1.0f / sqrtf(sq / (float)NQ + a.eps), ik = NK > 0 ? 1.0f / sqrtf(sk / (float)NK + a.eps) : 0.f;
+  for (int i = threadIdx.x; i < NQ + NK; i += blockDim.x)      // a thread's own elements
+    pr_rows[i] = i < NQ ? pr_rows[i] * iq * a.q_weight[i] : pr_rows[i] * ik * a.k_weight[i - NQ];
+  __syncthreads();
+  const int half = a.n_rot >> 1;
+  const float* cr = a.cos_t ? a.cos_t + (size_t)pos * half : nullptr;
+  const float* sr = a.cos_t ? a.sin_t + (size_t)pos * half : nullptr;
+  for (int i = threadIdx.x; i < NQ + NK; i += blockDim.x) {
+    const int vec = i / D, d = i - vec * D;
+    float v = pr_rows[i];
+    if (cr != nullptr && d < a.n_rot) {
+      int f, partner;
+      bool first;
+      if (a.pairing == 0) { f = d >> 1; first = (d & 1) == 0; partner = d ^ 1; }
+      else { first = d < half; f = first ? d : d - half; partner = first ? d + half : d - half; }
+      const float p = pr_rows[vec * D + partner], c = cr[f], s = sr[f];
+      v = first ? v * c - p * s : v * c + p * s;
+    }
+    if (i < NQ) row[a.off_q + i] = from_f32<T>(v);
+    else
+      reinterpret_cast<T*>(a.k_pages)[(((size_t)page * a.n_k + (vec - a.n_q)) * a.page_size + in_page) * D + d] = from_f32<T>(v);
+  }
+  if (!a.write_cache) return;
+  for (int i = threadIdx.x; i < a.n_v * a.Dv; i += blockDim.x) {
+    const int g = i / a.Dv, d = i - g * a.Dv;
+    const int col = a.off_v + i;
+    const float v = to_f32(row[col]) + (a.bias != nullptr ? a.bias[col] : 0.f);
+    reinterpret_cast<T*>(a.v_pages)[(((size_t)page * a.n_v + g) * a.page_size + in_page) * a.Dv + d] = from_f32<T>(v);
+  }
+}
+
+// The same for bfloat16 rows in 16-byte pieces held in registers (no rotation, no bias): NP pieces of 8 numbers per
+// thread over the token's query, key and value pieces one after another.
+template <int NP>
+__global__ void __launch_bounds__(256)
+attention_prepare_rows_vec_kernel(PrepareArgs a) {
+  __shared__ float scratch[64];
+  const int t = blockIdx.x;
+  const int b = a.tok_seq[t];
+  const int pq = a.n_q * a.Dk / 8, pk = a.write_cache ? a.n_k * a.Dk / 8 : 0, pv = a.write_cache ? a.n_v * a.Dv / 8 : 0;
+  float4 w0[NP], w1[NP];
+#pragma unroll
+  for (int j = 0; j < NP; ++j) {                      // constants: before the wait
+    const int i = threadIdx.x + j * blockDim.x;
+    if (i < pq + pk) {
+      const float4* w = reinterpret_cast<const float4*>(i < pq ? a.q_weight + i * 8 : a.k_weight + (i - pq) * 8);
+      w0[j] = w[0];
+      w1[j] = w[1];
+    }
+  }
+  pdl_wait();
+  pdl_trigger();
+  if (b < 0) return;
+  const int pos = a.tok_pos[t];
+  bf16* row = reinterpret_cast<bf16*>(a.buf) + (size_t)t * a.stride;
+  const int page = a.write_cache ? a.block_table[(size_t)b * a.table_width + pos / a.page_size] : 0;
+  const int in_page = pos % a.page_size;
+  uint4 raw[NP];
+  float sq = 0.f, sk = 0.f;
+#pragma unroll
+  for (int j = 0; j < NP; ++j) {
+    const int i = threadIdx.x + j * blockDim.x;
+    if (i < pq + pk + pv) {
+      const int col = i < pq ? a.off_q + i * 8 : i < pq + pk ? a.off_k + (i - pq) * 8 : a.off_v + (i - pq - pk) * 8;
+      raw[j] = *reinterpret_cast<const uint4*>(row + col);
+    }
+  }
+#pragma unroll
+  for (int j = 0; j < NP; ++j) {
+    const int i = threadIdx.x + j * blockDim.x;
+    if (i < pq + pk) {
+      const uint32_t wd[4] = {raw[j].x, raw[j].y, raw[j].z, raw[j].w};
+      float s = 0.f;
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const float lo = __uint_as_float(wd[e] << 16), hi = __uint_as_float(wd[e] & 0xffff0000u);
+        s += lo * lo + hi * hi;
+      }
+      if (i < pq) sq += s; else sk += s;
+    }
+  }
+  sq = block_sum(sq, scratch);
+  if (pk > 0) sk = block_sum(sk, scratch + 32);
+  const float iq = 1.0f / sqrtf(sq / (float)(pq * 8) + a.eps), ik = pk > 0 ? 1.0f / sqrtf(sk / (float)(pk * 8) + a.eps) : 0.f;
+#pragma unroll
+  for (int j = 0; j < NP; ++j) {
+    const int i = threadIdx.x + j * blockDim.x;
+    if (i >= pq + pk + pv) continue;
+    if (i >= pq + pk) {                               // a value piece: as projected
+      const int at = (i - pq - pk) * 8, g = at / a.Dv, d = at - g * a.Dv;
+      *reinterpret_cast<uint4*>(reinterpret_cast<bf16*>(a.v_pages) +
+                                (((size_t)page * a.n_v + g) * a.page_size + in_page) * a.Dv + d) = raw[j];
+      continue;
+    }
+    const float inv = i < pq ? iq : ik;
+    const uint32_t wd[4] = {raw[j].x, raw[j].y, raw[j].z, raw[j].w};
+    float x[8];
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      x[2 * e] = __uint_as_float(wd[e] << 16) * inv;
+      x[2 * e + 1] = __uint_as_float(wd[e] & 0xffff0000u) * inv;
+    }
+    uint4 o;
+    o.x = pack2(x[0] * w0[j].x, x[1] * w0[j].y);
+    o.y = pack2(x[2] * w0[j].z, x[3] * w0[j].w);
+    o.z = pack2(x[4] * w1[j].x, x[5] * w1[j].y);
+    o.w = pack2(x[6] * w1[j].z, x[7] * w1[j].w);
+    if (i < pq) {
+      *reinterpret_cast<uint4*>(row + a.off_q + i * 8) = o;
+    } else {
+      const int at = (i - pq) * 8, g = at / a.Dk, d = at - g * a.Dk;
+      *reinterpret_cast<uint4*>(reinterpret_cast<bf16*>(a.k_pages) +
+                                (((size_t)page * a.n_k + g) * a.page_size + in_page) * a.Dk + d) = o;
+    }
+  }
+}
+
 struct AttendArgs {
   const void* q; int q_stride;      // query vectors of token t at q + t*q_stride + (h*M + m)*Dk
   void* out;                        // [T, H*Dv]
@@ -293,6 +441,7 @@ struct AttendArgs {
   const float* sink;                // [H] or null
   float coef;                       // weight of every map after the first
   int unit_norm; float eps, out_scale;
+  const float* dist;                // [2, H] or null: r1, r2 of a penalty r1 ln(1 + r2 (p - s)) taken off each score
 };
 
 template <typename T, int KPL, int VPL>
@@ -317,6 +466,7 @@ attention_maps_kernel(AttendArgs a) {
   const int* bt = a.block_table + (size_t)b * a.table_width;
   const T* kp = reinterpret_cast<const T*>(a.k_pages);
   const T* vp = reinterpret_cast<const T*>(a.v_pages);
+  const float r1 = a.dist != nullptr ? a.dist[h] : 0.f, r2 = a.dist != nullptr ? a.dist[a.H + h] : 0.f;
   float total[VPL];
 #pragma unroll
   for (int j = 0; j < VPL; ++j) total[j] = 0.f;
@@ -342,7 +492,8 @@ attention_maps_kernel(AttendArgs a) {
         const int d = lane + 32 * j;
         if (d < Dk) part += qr[j] * to_f32(kv[d]);
       }
-      const float score = warp_sum(part) * a.scale;
+      float score = warp_sum(part) * a.scale;
+      if (a.dist != nullptr) score -= r1 * log1pf(r2 * (float)(pos - s));
       const float m_new = fmaxf(mx, score);
       const float corr = expf(mx - m_new);   // exp(-inf) = 0 on the first key
       const float p = expf(score - m_new);
@@ -490,6 +641,52 @@ AB_API int ab_attention_prepare_opts(void* buf, int dtype, int stride, int off_q
   return ab_launch_status();
 }
 
+// The query and key norm over the whole projection (see attention_prepare_rows_kernel): q_weight [n_q * Dk], k_weight
+// [n_k * Dk].  With write_cache 0 the key and value vectors are not touched.
+AB_API int ab_attention_prepare_rows(void* buf, int dtype, int stride, int off_q, int off_k, int off_v, int n_q, int n_k,
+                                     int n_v, int Dk, int Dv, const float* q_weight, const float* k_weight, float eps,
+                                     const float* cos_t, const float* sin_t, int n_rot, int pairing, const int* tok_pos,
+                                     const int* tok_seq, const int* block_table, int table_width, void* k_pages,
+                                     void* v_pages, int page_size, int n_tokens, int write_cache, const float* bias,
+                                     cudaStream_t stream) {
+  if (n_tokens <= 0) return AB_OK;
+  if (Dk <= 0 || Dv <= 0 || n_q <= 0 || n_k < 0 || n_v < 0 || page_size <= 0) return AB_BAD_ARG;
+  if (n_rot < 0 || n_rot > Dk || (n_rot & 1) || pairing < 0 || pairing > 1) return AB_BAD_ARG;
+  if (!q_weight || (write_cache && (!k_weight || !k_pages || !v_pages))) return AB_BAD_ARG;
+  if (!cos_t || !sin_t || n_rot == 0) { cos_t = sin_t = nullptr; n_rot = 0; }
+  PrepareArgs a{buf, stride, off_q, off_k, off_v, n_q, n_k, n_v, Dk, Dv, q_weight, k_weight, eps, cos_t, sin_t, n_rot,
+                pairing, tok_pos, tok_seq, block_table, table_width, k_pages, v_pages, page_size, n_tokens, write_cache,
+                bias, 0, 0};
+  const int pieces = write_cache ? (n_q * Dk + n_k * Dk + n_v * Dv) / 8 : n_q * Dk / 8;
+  if (dtype == AB_BF16 && bias == nullptr && n_rot == 0 && Dk % 8 == 0 && Dv % 8 == 0 && stride % 8 == 0 && off_q % 8 == 0 &&
+      off_k % 8 == 0 && off_v % 8 == 0 && pieces <= 1024) {
+    const int threads = pieces <= 128 ? 128 : 256;
+    if (pieces <= threads)
+      ab_launch(attention_prepare_rows_vec_kernel<1>, dim3((unsigned)n_tokens), dim3(threads), 0, stream, a);
+    else if (pieces <= 2 * threads)
+      ab_launch(attention_prepare_rows_vec_kernel<2>, dim3((unsigned)n_tokens), dim3(threads), 0, stream, a);
+    else
+      ab_launch(attention_prepare_rows_vec_kernel<4>, dim3((unsigned)n_tokens), dim3(threads), 0, stream, a);
+    return ab_launch_status();
+  }
+  const size_t smem = (size_t)(n_q + (write_cache ? n_k : 0)) * Dk * sizeof(float);
+  if (smem > 200 * 1024) return AB_BAD_ARG;
+#define AB_GO(T)                                                                                                        \
+  {                                                                                                                     \
+    if (smem > 40 * 1024) {                                                                                             \
+      cudaError_t e = cudaFuncSetAttribute(attention_prepare_rows_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, \
+                                           (int)smem);                                                                  \
+      if (e != cudaSuccess) return AB_CUDA_ERR + (int)e;                                                                \
+    }                                                                                                                   \
+    ab_launch(attention_prepare_rows_kernel<T>, dim3((unsigned)n_tokens), dim3(256), smem, stream, a);                  \
+  }
+  if (dtype == AB_F32) AB_GO(float)
+  else if (dtype == AB_BF16) AB_GO(bf16)
+  else return AB_BAD_ARG;
+#undef AB_GO
+  return ab_launch_status();
+}
+
 template <typename T>
 static int launch_attend(const AttendArgs& a, cudaStream_t stream) {
   const long long warps = (long long)a.n_tokens * a.H;
@@ -509,19 +706,30 @@ static int launch_attend(const AttendArgs& a, cudaStream_t stream) {
   return ab_launch_status();
 }
 
+// `dist`: float [2, H] or null (see AttendArgs).
+AB_API int ab_attention_maps_dist(const void* q, int q_stride, void* out, int dtype, const void* k_pages,
+                                  const void* v_pages, const int* block_table, int table_width, const int* tok_pos,
+                                  const int* tok_seq, int n_tokens, int H, int G, int M, int Dk, int Dv, int page_size,
+                                  float scale, int window, const float* sink, float coef, int unit_norm, float eps,
+                                  float out_scale, const float* dist, cudaStream_t stream) {
+  if (n_tokens <= 0) return AB_OK;
+  if (Dk <= 0 || Dk > AM_MAX_DIM || Dv <= 0 || Dv > AM_MAX_DIM || H <= 0 || G <= 0 || H % G || M <= 0 || page_size <= 0)
+    return AB_BAD_ARG;
+  AttendArgs a{q, q_stride, out, k_pages, v_pages, block_table, table_width, tok_pos, tok_seq, n_tokens, H, G, M, Dk,
+               Dv, page_size, scale, window, sink, coef, unit_norm, eps, out_scale, dist};
+  if (dtype == AB_F32) return launch_attend<float>(a, stream);
+  if (dtype == AB_BF16) return launch_attend<bf16>(a, stream);
+  return AB_BAD_ARG;
+}
+
 AB_API int ab_attention_maps(const void* q, int q_stride, void* out, int dtype, const void* k_pages,
                              const void* v_pages, const int* block_table, int table_width, const int* tok_pos,
                              const int* tok_seq, int n_tokens, int H, int G, int M, int Dk, int Dv, int page_size,
                              float scale, int window, const float* sink, float coef, int unit_norm, float eps,
                              float out_scale, cudaStream_t stream) {
-  if (n_tokens <= 0) return AB_OK;
-  if (Dk <= 0 || Dk > AM_MAX_DIM || Dv <= 0 || Dv > AM_MAX_DIM || H <= 0 || G <= 0 || H % G || M <= 0 || page_size <= 0)
-    return AB_BAD_ARG;
-  AttendArgs a{q, q_stride, out, k_pages, v_pages, block_table, table_width, tok_pos, tok_seq, n_tokens, H, G, M, Dk,
-               Dv, page_size, scale, window, sink, coef, unit_norm, eps, out_scale};
-  if (dtype == AB_F32) return launch_attend<float>(a, stream);
-  if (dtype == AB_BF16) return launch_attend<bf16>(a, stream);
-  return AB_BAD_ARG;
+  return ab_attention_maps_dist(q, q_stride, out, dtype, k_pages, v_pages, block_table, table_width, tok_pos, tok_seq,
+                                n_tokens, H, G, M, Dk, Dv, page_size, scale, window, sink, coef, unit_norm, eps, out_scale,
+                                nullptr, stream);
 }
 
 

@@ -21,6 +21,9 @@
 // Scores: (q.k) * scale; key s is seen by a token at position p iff
 // lo <= s <= p, lo = max(0, p - window + 1) (window 0: all)
 // (alpacca/model.py:447-467).  Head sizes: multiples of 16 up to 256.
+// A penalty on distance may be taken off each scaled score (template parameter DIST): r1_h ln(1 + r2_h (p - s)), a head's
+// numbers from `dist` [2, heads] (r1 of all heads, then r2).  In the kernels' units (scores times log2 e) it is
+// r1 log2(1 + r2 (p - s)), one logarithm of the hardware's approximation (relative error 2^-22) per score.
 #include "attention_common.cuh"
 #include "launch.cuh"
 #include <cooperative_groups.h>
@@ -42,14 +45,30 @@ struct RowState {
   float l[2];   // running sum of 2^(score' - m)
 };
 
+// What the penalty on distance needs of one row or column: r1, r2 of its head and 1 + r2 * (its position - the tile's
+// first key), so that key number c of the tile costs one fused multiply-add and one logarithm.
+struct DistRow {
+  float r1, r2, base;
+};
+__device__ __forceinline__ float fast_log2(float x) {
+  float y;
+  asm("lg2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+// score - r1 log2(1 + r2 (distance - c)); negative distances (keys that are masked afterwards) may give NaN
+__device__ __forceinline__ float less_distance(float score, const DistRow& d, float c) {
+  return fmaf(-d.r1, fast_log2(fmaf(-d.r2, c, d.base)), score);
+}
+
 // One key tile (64 keys) for one warp.
 //   qs: this warp's 16 query rows in shared memory, pitch `pitch` elements
 //   ks, vs: the key tile [64][pitch] of D dims and the value tile [64][pitch_v] of Dv dims
 //   pos0/pos1, lo0/lo1: last and first visible key of rows g and g+8; key0: position of the tile's first key
-template <int DMAX>
+template <int DMAX, bool DIST>
 __device__ __forceinline__ void attend_tile(RowState<DMAX>& st, const bf16* qs, const bf16* ks, const bf16* vs,
                                             int pitch, int pitch_v, int D, int Dv, float scale_log2, int key0,
-                                            int pos0, int pos1, int lo0, int lo1, bool need_mask) {
+                                            int pos0, int pos1, int lo0, int lo1, bool need_mask, const DistRow& d0,
+                                            const DistRow& d1) {
   const int lane = threadIdx.x & 31;
   const int t = lane & 3;
   float s[8][4];
@@ -81,6 +100,7 @@ __device__ __forceinline__ void attend_tile(RowState<DMAX>& st, const bf16* qs, 
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
       float v = s[nt][j] * scale_log2;
+      if (DIST) v = less_distance(v, j < 2 ? d0 : d1, (float)(nt * 8 + (j & 1)));     // the lane's 2t is in `base`
       if (need_mask) {
         const int key = key0 + nt * 8 + 2 * t + (j & 1);
         const bool ok = (j < 2) ? (key <= pos0 && key >= lo0) : (key <= pos1 && key >= lo1);
@@ -189,7 +209,7 @@ __device__ __forceinline__ float sum_with_sink(float l, float m, const float* __
 // for itself) and group c the columns c*group_cols .. (c+1)*group_cols of the launch's Dv: one copy of the key tile
 // and of a value tile of all Dv columns serves NG times the warps, where a value row is too wide for one warp's
 // registers.  DMAX then covers D and group_cols.
-template <int DMAX, int NG>
+template <int DMAX, int NG, bool DIST>
 __global__ void __launch_bounds__(128 * NG)
 attention_prefill_kernel(const bf16* __restrict__ qkv, int q_stride, void* __restrict__ out_any, int out_f32,
                          const bf16* __restrict__ k_pages, const bf16* __restrict__ v_pages,
@@ -197,7 +217,7 @@ attention_prefill_kernel(const bf16* __restrict__ qkv, int q_stride, void* __res
                          const int* __restrict__ cu_q, const int* __restrict__ tok_seq,
                          const int* __restrict__ tile_seq, const int* __restrict__ tile_q0, int H, int K, int M, int D,
                          int Dv, float scale_log2, int window, int tokens_per_tile, const float* __restrict__ sink,
-                         int v_row, int v_col0, int group_cols) {
+                         int v_row, int v_col0, int group_cols, const float* __restrict__ dist) {
   extern __shared__ __align__(16) unsigned char smem_raw[];
   constexpr int NT = 128 * NG;
   const int pitch = D + 8, pitch_v = Dv + 8;
@@ -246,6 +266,12 @@ attention_prefill_kernel(const bf16* __restrict__ qkv, int q_stride, void* __res
   const int kb_begin = (window > 0 && pos_first - window + 1 > 0) ? (pos_first - window + 1) / PAGE : 0;
   const int kb_end = pos_last / PAGE + 1;
   const int* bt = block_table + (size_t)b * table_width;
+  float ra0 = 0.f, rb0 = 0.f, ra1 = 0.f, rb1 = 0.f;      // r1, r2 of the heads of this thread's two rows
+  if (DIST) {
+    const int n_heads = H / M;
+    if (r0 < n_rows) { ra0 = dist[grp * G + r0 % G]; rb0 = dist[n_heads + grp * G + r0 % G]; }
+    if (r1 < n_rows) { ra1 = dist[grp * G + r1 % G]; rb1 = dist[n_heads + grp * G + r1 % G]; }
+  }
 
   RowState<DMAX> st;
   init_state(st);
@@ -266,8 +292,14 @@ attention_prefill_kernel(const bf16* __restrict__ qkv, int q_stride, void* __res
     // rows of this warp that exist at all; a warp without rows still joins the barriers
     if (warp * 16 < n_rows && n_cols > 0) {
       const bool need_mask = (key0 + PAGE - 1 > pos_first) || (window > 0);
-      attend_tile<DMAX>(st, qs + warp * 16 * pitch, kbuf + stage * 64 * pitch, vbuf + stage * 64 * pitch_v + col_first,
-                        pitch, pitch_v, D, n_cols, scale_log2, key0, pos0, pos1, lo0, lo1, need_mask);
+      DistRow d0{0.f, 0.f, 1.f}, d1{0.f, 0.f, 1.f};
+      if (DIST) {
+        d0 = DistRow{ra0, rb0, fmaf(rb0, (float)(pos0 - key0 - 2 * t4), 1.f)};
+        d1 = DistRow{ra1, rb1, fmaf(rb1, (float)(pos1 - key0 - 2 * t4), 1.f)};
+      }
+      attend_tile<DMAX, DIST>(st, qs + warp * 16 * pitch, kbuf + stage * 64 * pitch,
+                              vbuf + stage * 64 * pitch_v + col_first, pitch, pitch_v, D, n_cols, scale_log2, key0, pos0,
+                              pos1, lo0, lo1, need_mask, d0, d1);
     }
     __syncthreads();
   }
@@ -325,10 +357,10 @@ struct DecodeState {
 
 // One run of `nt` (1..DECODE_RUN) 16-key tiles; ks, vs: the run's keys and values [nt*16][pitch];
 // qb: Q^T as the second operand, per 16 columns of the head; key0: position of the run's first key.
-template <int DMAX>
+template <int DMAX, bool DIST>
 __device__ __forceinline__ void attend_run(DecodeState<DMAX>& st, const uint32_t (&qb)[DMAX / 16][2], const bf16* ks,
                                            const bf16* vs, int pitch, int D, float scale_log2, int nt, int key0,
-                                           int pos, int lo) {
+                                           int pos, int lo, const DistRow& h0, const DistRow& h1) {
   const int lane = threadIdx.x & 31;
   const int g = lane >> 2;
   const int a_row = (lane & 7) + ((lane >> 3) & 1) * 8, a_col = (lane >> 4) * 8;
@@ -348,10 +380,15 @@ __device__ __forceinline__ void attend_run(DecodeState<DMAX>& st, const uint32_t
       }
       const int ka = key0 + i * 16 + g, kb = ka + 8;
       const bool oka = ka <= pos && ka >= lo, okb = kb <= pos && kb >= lo;
-      s[i][0] = oka ? s[i][0] * scale_log2 : -INFINITY;
-      s[i][1] = oka ? s[i][1] * scale_log2 : -INFINITY;
-      s[i][2] = okb ? s[i][2] * scale_log2 : -INFINITY;
-      s[i][3] = okb ? s[i][3] * scale_log2 : -INFINITY;
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        float v = s[i][j] * scale_log2;
+        if (DIST) {
+          const DistRow& hd = (j & 1) ? h1 : h0;
+          v = fmaf(-hd.r1, fast_log2(fmaf(hd.r2, (float)(pos - (j < 2 ? ka : kb)), 1.f)), v);
+        }
+        s[i][j] = (j < 2 ? oka : okb) ? v : -INFINITY;
+      }
     } else {
       s[i][0] = s[i][1] = s[i][2] = s[i][3] = -INFINITY;
     }
@@ -429,7 +466,7 @@ __device__ __forceinline__ void load_run_async(bf16* ks, bf16* vs, const bf16* _
 // rotation kernel ran); 1 = this kernel rotates q; the step's key and value are in the cache (a layer
 // that reads the cache of another); 2 = this kernel rotates q and k, takes this step's key and value
 // from qkv and writes them to their place in the cache.
-template <int DMAX, int NWARPS>
+template <int DMAX, int NWARPS, bool DIST>
 __global__ void __launch_bounds__(NWARPS * 32)
 attention_decode_kernel(const bf16* __restrict__ qkv, int q_stride, bf16* __restrict__ out,
                         float* __restrict__ part_o, float* __restrict__ part_ml, int* __restrict__ arrivals,
@@ -437,7 +474,8 @@ attention_decode_kernel(const bf16* __restrict__ qkv, int q_stride, bf16* __rest
                         const int* __restrict__ block_table, int table_width, const int* __restrict__ tok_seq,
                         const int* __restrict__ kv_len, int H, int K, int D, float scale_log2, int window,
                         int pages_per_cta, int n_chunks, int cluster_merge, bf16* k_out, bf16* v_out, const float* __restrict__ cos_t, const float* __restrict__ sin_t,
-                        int n_rot, int pairing, int fuse, const float* __restrict__ sink) {
+                        int n_rot, int pairing, int fuse, const float* __restrict__ sink,
+                        const float* __restrict__ dist) {
   extern __shared__ __align__(16) unsigned char smem_raw[];
   const int pitch = D + 8;
   bf16* qs = reinterpret_cast<bf16*>(smem_raw);                 // [8][pitch] q, [2][pitch] this step's k, v
@@ -467,6 +505,12 @@ attention_decode_kernel(const bf16* __restrict__ qkv, int q_stride, bf16* __rest
   const bool active = chunk >= first_chunk && chunk <= last_chunk;
   if (!active && !cluster_merge) { pdl_wait(); pdl_trigger(); return; }
   const int n_heads = min(8, G - rt * 8);
+  DistRow hd0{0.f, 0.f, 1.f}, hd1{0.f, 0.f, 1.f};      // of this thread's two heads (columns 2t, 2t + 1 of the tiles)
+  if (DIST) {
+    const int h = kh * G + rt * 8 + 2 * t4;
+    if (2 * t4 < n_heads) { hd0.r1 = dist[h]; hd0.r2 = dist[H + h]; }
+    if (2 * t4 + 1 < n_heads) { hd1.r1 = dist[h + 1]; hd1.r2 = dist[H + h + 1]; }
+  }
 
   // this chunk's 16-key tiles, dealt to the warps in equal runs of at most DECODE_RUN, round after round
   const int tile_begin = max(chunk * pages_per_cta * (PAGE / 16), lo / 16);
@@ -568,7 +612,7 @@ attention_decode_kernel(const bf16* __restrict__ qkv, int q_stride, bf16* __rest
       }
     }
     __syncwarp();
-    if (t0 < t1) attend_run<DMAX>(st, qb, ks, vs, pitch, D, scale_log2, t1 - t0, t0 * 16, pos, lo);
+    if (t0 < t1) attend_run<DMAX, DIST>(st, qb, ks, vs, pitch, D, scale_log2, t1 - t0, t0 * 16, pos, lo, hd0, hd1);
     __syncwarp();      // every lane is done reading the run before the next one overwrites it
   }
   float l0 = st.l[0], l1 = st.l[1];
@@ -717,13 +761,14 @@ AB_API int ab_attention_decode_round_pages(int D) { return ab_attention_decode_r
 // `v_row`, `v_col0`: columns v_col0 .. v_col0 + Dv of value rows and output vectors of v_row numbers (both multiples
 // of 8: 16-byte pieces).  `group_cols`: the columns of Dv that one group of four warps takes (a multiple of 16, up to
 // 256); ceil(Dv / group_cols) must be 1, 2 or 4 (four groups: D and group_cols up to 128).
-AB_API int ab_attention_prefill_maps_groups_bf16(const void* qkv, int q_stride, void* out, int out_f32,
-                                                 const void* k_pages, const void* v_pages, const int* block_table,
-                                                 int table_width, const int* tok_pos, const int* cu_q,
-                                                 const int* tok_seq, const int* tile_seq, const int* tile_q0, int n_tiles,
-                                                 int tokens_per_tile, int H, int K, int M, int D, int Dv, float scale,
-                                                 int window, const float* sink, int v_row, int v_col0, int group_cols,
-                                                 cudaStream_t stream) {
+// `dist`: float [2, H / M] or null, the penalty on distance (one group of columns then).
+AB_API int ab_attention_prefill_maps_dist_bf16(const void* qkv, int q_stride, void* out, int out_f32,
+                                               const void* k_pages, const void* v_pages, const int* block_table,
+                                               int table_width, const int* tok_pos, const int* cu_q,
+                                               const int* tok_seq, const int* tile_seq, const int* tile_q0, int n_tiles,
+                                               int tokens_per_tile, int H, int K, int M, int D, int Dv, float scale,
+                                               int window, const float* sink, int v_row, int v_col0, int group_cols,
+                                               const float* dist, cudaStream_t stream) {
   if (n_tiles <= 0) return AB_OK;
   if (D <= 0 || D > 256 || (D % 16) || Dv <= 0 || (Dv % 16) || K <= 0 || H % K || K > 65535 || M <= 0 || K % M)
     return AB_BAD_ARG;
@@ -739,19 +784,27 @@ AB_API int ab_attention_prefill_maps_groups_bf16(const void* qkv, int q_stride, 
   if ((long long)n_tiles * K > 0x7fffffffLL) return AB_BAD_ARG;
   dim3 grid((unsigned)n_tiles * K);
   const float sl = scale * LOG2E;
-#define AB_GO(DM, NG)                                                                                               \
+#define AB_GO_D(DM, NG, DS)                                                                                         \
   {                                                                                                                 \
-    cudaError_t e = cudaFuncSetAttribute(attention_prefill_kernel<DM, NG>,                                          \
+    cudaError_t e = cudaFuncSetAttribute(attention_prefill_kernel<DM, NG, DS>,                                      \
                                          cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);                   \
     if (e != cudaSuccess) return AB_CUDA_ERR + (int)e;                                                              \
-    ab_launch(attention_prefill_kernel<DM, NG>, grid, dim3(128 * NG), smem, stream,                                 \
+    ab_launch(attention_prefill_kernel<DM, NG, DS>, grid, dim3(128 * NG), smem, stream,                             \
         (const bf16*)qkv, q_stride, out, out_f32, (const bf16*)k_pages, (const bf16*)v_pages, block_table,          \
         table_width, tok_pos, cu_q, tok_seq, tile_seq, tile_q0, H, K, M, D, Dv, sl, window, tokens_per_tile, sink,  \
-        v_row, v_col0, group_cols);                                                                                 \
+        v_row, v_col0, group_cols, dist);                                                                           \
   }
+#define AB_GO(DM, NG) AB_GO_D(DM, NG, false)
   const int widest = groups == 1 ? Dv : group_cols;
   const int dm = dmax_of(D > widest ? D : widest);
-  if (groups == 1) {
+  if (dist != nullptr) {
+    if (groups != 1) return AB_BAD_ARG;
+    switch (dm) {
+      case 64: AB_GO_D(64, 1, true); break;
+      case 128: AB_GO_D(128, 1, true); break;
+      default: AB_GO_D(256, 1, true); break;
+    }
+  } else if (groups == 1) {
     switch (dm) {
       case 64: AB_GO(64, 1); break;
       case 128: AB_GO(128, 1); break;
@@ -764,7 +817,20 @@ AB_API int ab_attention_prefill_maps_groups_bf16(const void* qkv, int q_stride, 
     AB_GO(128, 4)
   }
 #undef AB_GO
+#undef AB_GO_D
   return ab_launch_status();
+}
+
+AB_API int ab_attention_prefill_maps_groups_bf16(const void* qkv, int q_stride, void* out, int out_f32,
+                                                 const void* k_pages, const void* v_pages, const int* block_table,
+                                                 int table_width, const int* tok_pos, const int* cu_q,
+                                                 const int* tok_seq, const int* tile_seq, const int* tile_q0, int n_tiles,
+                                                 int tokens_per_tile, int H, int K, int M, int D, int Dv, float scale,
+                                                 int window, const float* sink, int v_row, int v_col0, int group_cols,
+                                                 cudaStream_t stream) {
+  return ab_attention_prefill_maps_dist_bf16(qkv, q_stride, out, out_f32, k_pages, v_pages, block_table, table_width,
+                                             tok_pos, cu_q, tok_seq, tile_seq, tile_q0, n_tiles, tokens_per_tile, H, K, M,
+                                             D, Dv, scale, window, sink, v_row, v_col0, group_cols, nullptr, stream);
 }
 
 // One group of warps: up to 256 columns per launch.
@@ -885,13 +951,14 @@ AB_API int ab_attention_decode_rope_bf16(const void* qkv, int q_stride, void* ou
                                        n_chunks, small, cos_t, sin_t, n_rot, pairing, fuse, nullptr, stream);
 }
 
-// The same with a sink per head in the softmax's denominator (`sink`: float [H] or null).
-AB_API int ab_attention_decode_sink_bf16(const void* qkv, int q_stride, void* out, float* part_o, float* part_ml,
+// The same with a sink per head in the softmax's denominator (`sink`: float [H] or null) and a penalty on distance
+// (`dist`: float [2, H] or null).
+AB_API int ab_attention_decode_dist_bf16(const void* qkv, int q_stride, void* out, float* part_o, float* part_ml,
                                          int* arrivals, void* k_pages, void* v_pages, const int* block_table,
                                          int table_width, const int* tok_seq, const int* kv_len, int n_tokens, int H,
                                          int K, int D, float scale, int window, int pages_per_cta, int n_chunks,
                                          int small, const float* cos_t, const float* sin_t, int n_rot, int pairing,
-                                         int fuse, const float* sink, cudaStream_t stream) {
+                                         int fuse, const float* sink, const float* dist, cudaStream_t stream) {
   if (n_tokens <= 0) return AB_OK;
   if (D <= 0 || D > 256 || (D % 16) || H % K || n_chunks < 1 || n_chunks > 65535 || pages_per_cta < 1)
     return AB_BAD_ARG;
@@ -906,19 +973,20 @@ AB_API int ab_attention_decode_sink_bf16(const void* qkv, int q_stride, void* ou
   const float sl = scale * LOG2E;
   const int cluster_merge = (n_chunks > 1 && n_chunks <= AB_DECODE_MAX_CLUSTER) ? 1 : 0;
   dim3 grid(n_tokens, K * row_tiles, n_chunks);
-#define AB_GO(DM, NW)                                                                                               \
+#define AB_GO(DM, NW) { if (dist != nullptr) AB_GO_D(DM, NW, true) else AB_GO_D(DM, NW, false) }
+#define AB_GO_D(DM, NW, DS)                                                                                         \
   {                                                                                                                 \
     size_t tiles = (size_t)(10 + NW * 2 * 16 * DECODE_RUN) * pitch * sizeof(bf16);                                  \
     size_t merge = (size_t)10 * pitch * sizeof(bf16) + (size_t)(NW * 8 * (D + 6) + 8 * (D + 2)) * sizeof(float);    \
     size_t smem = tiles > merge ? tiles : merge;                                                                    \
-    cudaError_t e = cudaFuncSetAttribute(attention_decode_kernel<DM, NW>,                                           \
+    cudaError_t e = cudaFuncSetAttribute(attention_decode_kernel<DM, NW, DS>,                                       \
                                          cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);                   \
     if (e != cudaSuccess) return AB_CUDA_ERR + (int)e;                                                              \
-    launch_clustered(attention_decode_kernel<DM, NW>, grid, dim3(NW * 32), smem, stream,                            \
+    launch_clustered(attention_decode_kernel<DM, NW, DS>, grid, dim3(NW * 32), smem, stream,                            \
         cluster_merge ? (unsigned)n_chunks : 1u,                                                                    \
         (const bf16*)qkv, q_stride, (bf16*)out, part_o, part_ml, arrivals, (const bf16*)k_pages,                    \
         (const bf16*)v_pages, block_table, table_width, tok_seq, kv_len, H, K, D, sl, window, pages_per_cta,        \
-        n_chunks, cluster_merge, (bf16*)k_pages, (bf16*)v_pages, cos_t, sin_t, n_rot, pairing, fuse, sink);         \
+        n_chunks, cluster_merge, (bf16*)k_pages, (bf16*)v_pages, cos_t, sin_t, n_rot, pairing, fuse, sink, dist);   \
   }
   if (n_chunks > AB_DECODE_MAX_CLUSTER && (!part_o || !part_ml || !arrivals)) return AB_BAD_ARG;
   switch (dmax_of(D)) {
@@ -934,7 +1002,19 @@ AB_API int ab_attention_decode_sink_bf16(const void* qkv, int q_stride, void* ou
       break;
   }
 #undef AB_GO
+#undef AB_GO_D
   return ab_launch_status();
+}
+
+AB_API int ab_attention_decode_sink_bf16(const void* qkv, int q_stride, void* out, float* part_o, float* part_ml,
+                                         int* arrivals, void* k_pages, void* v_pages, const int* block_table,
+                                         int table_width, const int* tok_seq, const int* kv_len, int n_tokens, int H,
+                                         int K, int D, float scale, int window, int pages_per_cta, int n_chunks,
+                                         int small, const float* cos_t, const float* sin_t, int n_rot, int pairing,
+                                         int fuse, const float* sink, cudaStream_t stream) {
+  return ab_attention_decode_dist_bf16(qkv, q_stride, out, part_o, part_ml, arrivals, k_pages, v_pages, block_table,
+                                       table_width, tok_seq, kv_len, n_tokens, H, K, D, scale, window, pages_per_cta,
+                                       n_chunks, small, cos_t, sin_t, n_rot, pairing, fuse, sink, nullptr, stream);
 }
 
 // ---------------------------------------------------------------------------

@@ -26,6 +26,12 @@
 // (q.k) * scale, key s visible to position p iff lo <= s <= p
 // (alpacca/model.py:457-467).
 //
+// A penalty on distance (template parameter DIST) is taken off each scaled score: r1_h ln(1 + r2_h (p - s)) with a head's
+// numbers from `dist` [2, H].  The exponentials already fill the unit that forms logarithms, so a tile's penalties are
+// not formed per score: along a tile they depend on the head and on p - s alone, G x (tokens + 63) numbers instead of
+// 128 x 64.  The softmax threads form them for the next tile into one of two tables in shared memory, one named barrier
+// of their 128 threads per tile, and read one number per score (neighbouring rows meet different banks).
+//
 // Every mbarrier wait is bounded (see gemm_tc.cu): on a timeout the thread records a
 // code in `status` and all roles fall through to the end, where TMEM is given back.
 #include "common.cuh"
@@ -158,14 +164,27 @@ template <int HD> struct AtSmem {
   static constexpr int TOTAL = BAR_OFF + 256 + 1024;
 };
 
-template <int HD>
+// what a head's table of penalties takes, in numbers: a tile's tokens + 63 of them, rounded up so that the rows of a
+// warp (32 / G tokens of G heads) read different banks
+__host__ __device__ __forceinline__ int at_dist_stride(int tokens_per_tile, int G) {
+  const int n = (tokens_per_tile + AT_KEYS - 1 + 31) / 32 * 32;
+  return n + (G >= 32 ? 1 : 32 / G);
+}
+__device__ __forceinline__ float at_log2(float x) {
+  float y;
+  asm("lg2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+
+template <int HD, bool DIST>
 __global__ void __launch_bounds__(AT_THREADS, 2)
 attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                             const __grid_constant__ CUtensorMap map_v, bf16* __restrict__ out,
                             const int* __restrict__ block_table, int table_width, const int* __restrict__ tok_pos,
                             const int* __restrict__ cu_q, const int* __restrict__ tile_seq,
                             const int* __restrict__ tile_q0, int H, int K, float scale_log2, int window,
-                            int tokens_per_tile, int* __restrict__ status, const float* __restrict__ sink) {
+                            int tokens_per_tile, int* __restrict__ status, const float* __restrict__ sink,
+                            const float* __restrict__ dist) {
   extern __shared__ unsigned char smem_raw[];
   unsigned char* base = reinterpret_cast<unsigned char*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~(uintptr_t)1023);
   using Sm = AtSmem<HD>;
@@ -290,11 +309,34 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
     }
     float m_ref = -INFINITY, l_run = 0.f;       // the row's reference and its sum of 2^(s - m_ref)
     bool ok = true;
+    // the tables of penalties: entry e of head g in the table of tile j is for the distance
+    // (pos_first - first key) - 63 + e: token i of the tile and key c read e = i + 63 - c
+    const int d_stride = DIST ? at_dist_stride(tokens_per_tile, G) : 0;
+    float* d_tab = reinterpret_cast<float*>(base + Sm::BAR_OFF + 256);
+    const float* d_row = d_tab + (DIST && row_ok ? (r % G) * d_stride + r / G + AT_KEYS - 1 : AT_KEYS - 1);
+    auto form_penalties = [&](int j) {
+      const int n = tokens_per_tile + AT_KEYS - 1;
+      const int d0 = pos_first - (kb_begin + j) * AT_KEYS - (AT_KEYS - 1);
+      float* tab = d_tab + (j & 1) * G * d_stride;
+      for (int i = threadIdx.x - 64; i < G * n; i += 128) {
+        const int hg = i / n, e = i - hg * n;
+        const float d = (float)max(d0 + e, 0);
+        tab[hg * d_stride + e] = -dist[kh * G + hg] * at_log2(fmaf(dist[H + kh * G + hg], d, 1.f));
+      }
+    };
+    if (DIST && n_tiles > 0) form_penalties(0);
 
-    for (int j = 0; j < n_tiles && ok; ++j) {
+    for (int j = 0; j < n_tiles && (ok || DIST); ++j) {
+      if (DIST) {
+        // the table of tile j is complete, and nobody reads the other one any more; a warp that gave up on a barrier
+        // still meets the others here until the last tile
+        asm volatile("bar.sync 1, 128;" ::: "memory");
+        if (!ok) continue;
+        if (j + 1 < n_tiles) form_penalties(j + 1);
+      }
       if (!at_wait(s_full + (j & 1), (j >> 1) & 1)) { atomicExch(status, 16); ok = false; }
       ok = __all_sync(0xffffffffu, ok);
-      if (!ok) break;
+      if (!ok) { if (DIST) continue; else break; }
       asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
       float sc[AT_KEYS];
 #pragma unroll
@@ -305,6 +347,11 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
       // the maximum is taken on the raw scores (the scale is positive), and scale and shift ride in
       // the exponent's fused multiply-add: p = 2^(s * scale - m)
       // four running maxima (and below four running sums) keep the dependent chains short
+      if (DIST) {
+        const float* pen = d_row + (j & 1) * G * d_stride;
+#pragma unroll
+        for (int c = 0; c < AT_KEYS; ++c) sc[c] = fmaf(sc[c], scale_log2, pen[-c]);
+      }
       if (need_mask) {
 #pragma unroll
         for (int c = 0; c < AT_KEYS; ++c)
@@ -318,7 +365,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
         mx4[2] = fmaxf(mx4[2], sc[c + 2]);
         mx4[3] = fmaxf(mx4[3], sc[c + 3]);
       }
-      const float mx = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3])) * scale_log2;
+      const float mx = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3])) * (DIST ? 1.f : scale_log2);
       // move the reference only when the maximum has outgrown it by a lot (or there was none yet)
       const bool move = (mx > m_ref + AT_LAZY) || (m_ref == -INFINITY && mx > -INFINITY);
       float corr = 1.f;
@@ -331,7 +378,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
         // rescale this warp's rows of O in TMEM, after the product before this tile has landed there
         if (!at_wait(o_done, (j - 1) & 1)) { atomicExch(status, 15); ok = false; }
         ok = __all_sync(0xffffffffu, ok);
-        if (!ok) break;
+        if (!ok) { if (DIST) continue; else break; }
         asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
 #pragma unroll
         for (int c0 = 0; c0 < HD; c0 += 32) {
@@ -351,8 +398,9 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
       uint32_t packed[AT_KEYS / 2];
 #pragma unroll
       for (int c = 0; c < AT_KEYS; c += 4) {
-        const float p0 = at_exp2(fmaf(sc[c], scale_log2, -sub)), p1 = at_exp2(fmaf(sc[c + 1], scale_log2, -sub));
-        const float p2 = at_exp2(fmaf(sc[c + 2], scale_log2, -sub)), p3 = at_exp2(fmaf(sc[c + 3], scale_log2, -sub));
+        const float sl = DIST ? 1.f : scale_log2;
+        const float p0 = at_exp2(fmaf(sc[c], sl, -sub)), p1 = at_exp2(fmaf(sc[c + 1], sl, -sub));
+        const float p2 = at_exp2(fmaf(sc[c + 2], sl, -sub)), p3 = at_exp2(fmaf(sc[c + 3], sl, -sub));
         sum4[0] += p0; sum4[1] += p1; sum4[2] += p2; sum4[3] += p3;
         __nv_bfloat162 pa = __floats2bfloat162_rn(p0, p1), pb = __floats2bfloat162_rn(p2, p3);
         packed[c >> 1] = *reinterpret_cast<uint32_t*>(&pa);
@@ -453,11 +501,14 @@ AB_API int ab_attention_prefill_tc_supports(int H, int K, int D) {
 // (q part read); out [n_tokens, H*D], cache pages [n_pages, K, 64, D].  `sink`: float [H] or null, one more term
 // exp(sink_h) in every softmax's denominator.
 // tile_seq / tile_q0: the tiles of floor(128 / G) tokens (sequence, first packed token), as for the mma kernel.
-AB_API int ab_attention_prefill_tc_sink(const void* qkv, int row_heads, int n_tokens, void* out, const void* k_pages,
+// `dist`: float [2, H] or null, the penalty on distance (G up to AT_DIST_MAX_GROUP: the tables' shared memory).
+#define AT_DIST_MAX_GROUP 16
+AB_API int ab_attention_prefill_tc_dist_max_group() { return AT_DIST_MAX_GROUP; }
+AB_API int ab_attention_prefill_tc_dist(const void* qkv, int row_heads, int n_tokens, void* out, const void* k_pages,
                                         const void* v_pages, int n_pages, const int* block_table, int table_width,
                                         const int* tok_pos, const int* cu_q, const int* tile_seq, const int* tile_q0,
                                         int n_tiles, int H, int K, int D, float scale, int window, const float* sink,
-                                        cudaStream_t stream) {
+                                        const float* dist, cudaStream_t stream) {
   if (n_tiles <= 0) return AB_OK;
   if (!ab_attention_prefill_tc_supports(H, K, D) || (long long)n_tiles * K > 0x7fffffffLL || row_heads < H)
     return AB_BAD_ARG;
@@ -465,6 +516,8 @@ AB_API int ab_attention_prefill_tc_sink(const void* qkv, int row_heads, int n_to
   int* status = at_status_word();
   if (!enc || !status) return AB_BAD_ARG;
   const int G = H / K, tpt = AT_ROWS / G;
+  if (dist != nullptr && G > AT_DIST_MAX_GROUP) return AB_BAD_ARG;
+  const size_t d_bytes = dist != nullptr ? (size_t)2 * G * at_dist_stride(tpt, G) * sizeof(float) : 0;
   CUtensorMap mq, mk, mv;
   {
     cuuint64_t dims[3] = {(cuuint64_t)D, (cuuint64_t)row_heads, (cuuint64_t)n_tokens};
@@ -487,19 +540,31 @@ AB_API int ab_attention_prefill_tc_sink(const void* qkv, int row_heads, int n_to
       return AB_BAD_ARG;
   }
   cudaError_t e;
-#define AT_GO(HDV)                                                                                                   \
+#define AT_GO(HDV, DS)                                                                                               \
   {                                                                                                                 \
-    e = cudaFuncSetAttribute(attention_prefill_tc_kernel<HDV>, cudaFuncAttributeMaxDynamicSharedMemorySize,         \
-                             AtSmem<HDV>::TOTAL);                                                                   \
+    const size_t smem = (size_t)AtSmem<HDV>::TOTAL + d_bytes;                                                       \
+    e = cudaFuncSetAttribute(attention_prefill_tc_kernel<HDV, DS>, cudaFuncAttributeMaxDynamicSharedMemorySize,     \
+                             (int)smem);                                                                            \
     if (e != cudaSuccess) return AB_CUDA_ERR + (int)e;                                                              \
-    e = ab_launch(attention_prefill_tc_kernel<HDV>, dim3((unsigned)n_tiles * K), dim3(AT_THREADS), (size_t)AtSmem<HDV>::TOTAL, \
+    e = ab_launch(attention_prefill_tc_kernel<HDV, DS>, dim3((unsigned)n_tiles * K), dim3(AT_THREADS), smem,        \
                   stream, mq, mk, mv, (bf16*)out, block_table, table_width, tok_pos, cu_q, tile_seq, tile_q0, H, K, \
-                  scale * AT_LOG2E, window, tpt, status, sink);                                                     \
+                  scale * AT_LOG2E, window, tpt, status, sink, dist);                                               \
   }
-  if (D == 64) AT_GO(64) else AT_GO(128)
+  if (dist != nullptr) { if (D == 64) AT_GO(64, true) else AT_GO(128, true) }
+  else { if (D == 64) AT_GO(64, false) else AT_GO(128, false) }
 #undef AT_GO
   if (e != cudaSuccess) return AB_CUDA_ERR + (int)e;
   return ab_launch_status();
+}
+
+AB_API int ab_attention_prefill_tc_sink(const void* qkv, int row_heads, int n_tokens, void* out, const void* k_pages,
+                                        const void* v_pages, int n_pages, const int* block_table, int table_width,
+                                        const int* tok_pos, const int* cu_q, const int* tile_seq, const int* tile_q0,
+                                        int n_tiles, int H, int K, int D, float scale, int window, const float* sink,
+                                        cudaStream_t stream) {
+  return ab_attention_prefill_tc_dist(qkv, row_heads, n_tokens, out, k_pages, v_pages, n_pages, block_table, table_width,
+                                      tok_pos, cu_q, tile_seq, tile_q0, n_tiles, H, K, D, scale, window, sink, nullptr,
+                                      stream);
 }
 
 // qkv [n_tokens, (H+2K)*D]: q | k | v of a token side by side; no sink.

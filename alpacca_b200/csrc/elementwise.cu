@@ -589,6 +589,62 @@ AB_API int ab_gated_act(const void* gu, void* act, int dtype, int n_rows, int F,
 }
 
 // ---------------------------------------------------------------------------
+// y[i] = act(y[i]) in place (kind 0: GELU in its erf form), and for logits
+// y[i] = cap * tanh(y[i] / cap).
+// ---------------------------------------------------------------------------
+__device__ __forceinline__ float gelu_exact(float z) { return 0.5f * z * (1.0f + erff(z * 0.70710678118654752440f)); }
+
+template <typename T>
+__global__ void act_kernel(T* __restrict__ y, size_t total) {
+  pdl_wait();
+  pdl_trigger();
+  const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
+  if (i < total) y[i] = from_f32<T>(gelu_exact(to_f32(y[i])));
+}
+__global__ void act_bf16x8_kernel(uint4* __restrict__ y, size_t n8) {
+  pdl_wait();
+  pdl_trigger();
+  const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
+  if (i >= n8) return;
+  uint4 v = y[i];
+  uint32_t* w = reinterpret_cast<uint32_t*>(&v);
+#pragma unroll
+  for (int j = 0; j < 4; ++j) {
+    __nv_bfloat162 r = __floats2bfloat162_rn(gelu_exact(__uint_as_float(w[j] << 16)), gelu_exact(__uint_as_float(w[j] & 0xffff0000u)));
+    w[j] = *reinterpret_cast<uint32_t*>(&r);
+  }
+  y[i] = v;
+}
+
+AB_API int ab_act(void* y, int dtype, long long total, int kind, cudaStream_t stream) {
+  if (total <= 0) return AB_OK;
+  if (kind != 0) return AB_BAD_ARG;
+  if (dtype == AB_BF16 && total % 8 == 0 && (((uintptr_t)y) & 15) == 0)
+    ab_launch(act_bf16x8_kernel, (unsigned)((total / 8 + 255) / 256), 256, 0, stream, (uint4*)y, (size_t)(total / 8));
+  else if (dtype == AB_BF16)
+    ab_launch(act_kernel<bf16>, (unsigned)((total + 255) / 256), 256, 0, stream, (bf16*)y, (size_t)total);
+  else if (dtype == AB_F32)
+    ab_launch(act_kernel<float>, (unsigned)((total + 255) / 256), 256, 0, stream, (float*)y, (size_t)total);
+  else
+    return AB_BAD_ARG;
+  return ab_launch_status();
+}
+
+__global__ void softcap_kernel(float* __restrict__ y, float cap, size_t total) {
+  pdl_wait();
+  pdl_trigger();
+  const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
+  if (i < total) y[i] = cap * tanhf(y[i] / cap);
+}
+
+AB_API int ab_softcap(float* y, float cap, long long total, cudaStream_t stream) {
+  if (total <= 0) return AB_OK;
+  if (!(cap > 0.f)) return AB_BAD_ARG;
+  ab_launch(softcap_kernel, (unsigned)((total + 255) / 256), 256, 0, stream, y, cap, (size_t)total);
+  return ab_launch_status();
+}
+
+// ---------------------------------------------------------------------------
 // After a decode step whose tokens were sampled on the device: feed them back.
 // For every live row b (tok_seq[b] >= 0): tokens[b] = sampled[b]; position,
 // length and the sampler's step counter go up by one; the token enters the

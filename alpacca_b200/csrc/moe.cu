@@ -71,6 +71,21 @@ __global__ void moe_logits_kernel(const T* __restrict__ h, int ld, const float* 
   if (lane == 0) z[id] = part + (bias != nullptr ? bias[e] : 0.f);
 }
 
+// z[t, e] alone (float32), without a choice: gate logits of a part that reads the stream
+AB_API int ab_moe_logits(const void* h, int dtype, int ld, const float* wr, int n_tokens, int width, int E, float* z,
+                         cudaStream_t stream) {
+  if (n_tokens <= 0) return AB_OK;
+  if (E <= 0 || width <= 0) return AB_BAD_ARG;
+  const unsigned blocks = (unsigned)(((long long)n_tokens * E + 7) / 8);
+  if (dtype == AB_F32)
+    ab_launch(moe_logits_kernel<float>, dim3(blocks), dim3(256), 0, stream, (const float*)h, ld, wr, n_tokens, width, E, z, nullptr);
+  else if (dtype == AB_BF16)
+    ab_launch(moe_logits_kernel<bf16>, dim3(blocks), dim3(256), 0, stream, (const bf16*)h, ld, wr, n_tokens, width, E, z, nullptr);
+  else
+    return AB_BAD_ARG;
+  return ab_launch_status();
+}
+
 // the choice, one warp per token, from the logits z [T, E]
 __global__ void moe_route_kernel(const float* __restrict__ z, int n_tokens, int E, int groups, int keep, int top,
                                  float scale, int* __restrict__ idx, float* __restrict__ wts) {
@@ -469,4 +484,235 @@ AB_API int ab_moe_weigh_all_gated(void* up, int dtype, const int* idx, const flo
 AB_API int ab_moe_weigh_all(void* up, int dtype, const int* idx, const float* wts, int n_tokens, int top, int ff, int E,
                             int activation, cudaStream_t stream) {
   return ab_moe_weigh_all_gated(up, dtype, idx, wts, n_tokens, top, ff, E, activation, 0, stream);
+}
+
+// ---------------------------------------------------------------------------
+// Gated experts behind any choice, with a shared expert.
+//
+//   y_t = sum_k weight_k W_down[e_k] (silu(W_gate[e_k] h_t) * (W_up[e_k] h_t))
+//         + sigmoid(z_t) W_down_s (silu(W_gate_s h_t) * (W_up_s h_t))               (if there is a shared expert)
+//
+// The choice comes from a router (`idx`, `wts`) or from the token's id: row token_t of a table [vocab, top] names its
+// experts, each with the same constant weight.  The matrices lie together: gate_up [2, C, width] with C = E * ff + fs
+// (the gates of all experts, then the shared expert's; then the up-projections likewise), down [width, C].
+// z [T] are the shared expert's gate logits (float32, formed elsewhere).
+// ---------------------------------------------------------------------------
+struct Choice {
+  const int* idx; const float* wts;       // [T, top], from a router
+  const int* table; const int* tokens;    // [vocab, top], [T]: by token id (idx null)
+  float weight;                           // of every expert chosen by table
+};
+__device__ __forceinline__ int chosen_expert(const Choice& c, int t, int k, int top) {
+  return c.idx != nullptr ? c.idx[(size_t)t * top + k] : c.table[(size_t)c.tokens[t] * top + k];
+}
+__device__ __forceinline__ float chosen_weight(const Choice& c, int t, int k, int top) {
+  return c.idx != nullptr ? c.wts[(size_t)t * top + k] : c.weight;
+}
+__device__ __forceinline__ float activate(float z, int kind) { return kind == 0 ? gelu_erf(z) : silu(z); }
+
+__device__ __forceinline__ void fma8(float& part, uint4 x, uint4 y) {
+  const uint32_t a[4] = {x.x, x.y, x.z, x.w}, b[4] = {y.x, y.y, y.z, y.w};
+#pragma unroll
+  for (int j = 0; j < 4; ++j) {
+    part = fmaf(__uint_as_float(a[j] << 16), __uint_as_float(b[j] << 16), part);
+    part = fmaf(__uint_as_float(a[j] & 0xffff0000u), __uint_as_float(b[j] & 0xffff0000u), part);
+  }
+}
+// A warp's shares of x . g and x . u (rows of n numbers): the rows' 16-byte pieces are asked for four at a time each.
+__device__ __forceinline__ void lane_dot2(const bf16* __restrict__ x, const bf16* __restrict__ g, const bf16* __restrict__ u,
+                                          int n, int lane, float& pg, float& pu) {
+  pg = pu = 0.f;
+  if ((n & 7) == 0 && ((((uintptr_t)x) | ((uintptr_t)g) | ((uintptr_t)u)) & 15) == 0) {
+    for (int k0 = lane * 8; k0 < n; k0 += 1024) {
+      uint4 gv[4], uv[4];
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        const int k = k0 + j * 256;
+        gv[j] = uv[j] = make_uint4(0, 0, 0, 0);
+        if (k < n) {
+          gv[j] = __ldg(reinterpret_cast<const uint4*>(g + k));
+          uv[j] = __ldg(reinterpret_cast<const uint4*>(u + k));
+        }
+      }
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        const int k = k0 + j * 256;
+        if (k < n) {
+          const uint4 xv = *reinterpret_cast<const uint4*>(x + k);
+          fma8(pg, xv, gv[j]);
+          fma8(pu, xv, uv[j]);
+        }
+      }
+    }
+    return;
+  }
+  for (int k = lane; k < n; k += 32) {
+    const float v = __bfloat162float(x[k]);
+    pg = fmaf(v, __bfloat162float(g[k]), pg);
+    pu = fmaf(v, __bfloat162float(u[k]), pu);
+  }
+}
+__device__ __forceinline__ void lane_dot2(const float* __restrict__ x, const float* __restrict__ g, const float* __restrict__ u,
+                                          int n, int lane, float& pg, float& pu) {
+  pg = pu = 0.f;
+  for (int k = lane; k < n; k += 32) {
+    pg = fmaf(x[k], g[k], pg);
+    pu = fmaf(x[k], u[k], pu);
+  }
+}
+
+// act: [T, top * ff + fs].  A block of eight warps takes one unit of an expert for eight (token, choice) pairs, or one
+// unit of the shared expert for eight tokens, whose warps then read the same two rows at the same time.
+template <typename T>
+__global__ void __launch_bounds__(256)
+moe_shared_up_kernel(const T* __restrict__ h, int ld, const T* __restrict__ gate_up, Choice c, T* __restrict__ act,
+                     int n_tokens, int top, int width, int ff, int fs, int E, int activation, long long pair_blocks) {
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  pdl_wait();
+  pdl_trigger();
+  const size_t C = (size_t)E * ff + fs;
+  const int row_len = top * ff + fs;
+  int t;
+  size_t row, dst;
+  long long blk = blockIdx.x;
+  if (blk < pair_blocks) {
+    const long long group = blk / ff;
+    const int j = (int)(blk - group * ff);
+    const long long p = group * 8 + warp;
+    if (p >= (long long)n_tokens * top) return;
+    t = (int)(p / top);
+    const int k = (int)(p - (long long)t * top);
+    row = (size_t)chosen_expert(c, t, k, top) * ff + j;
+    dst = (size_t)t * row_len + (size_t)k * ff + j;
+  } else {
+    blk -= pair_blocks;
+    const int chunk = (int)(blk / fs), j = (int)(blk - (long long)chunk * fs);
+    t = chunk * 8 + warp;
+    if (t >= n_tokens) return;
+    row = (size_t)E * ff + j;
+    dst = (size_t)t * row_len + (size_t)top * ff + j;
+  }
+  float pg, pu;
+  lane_dot2(h + (size_t)t * ld, gate_up + row * width, gate_up + (C + row) * width, width, lane, pg, pu);
+  pg = warp_sum(pg);
+  pu = warp_sum(pu);
+  if (lane == 0) act[dst] = from_f32<T>(activate(pg, activation) * pu);
+}
+
+// out[t, i], float32 or T.  A block of eight warps takes one column i for eight tokens (the shared expert's row is then
+// read by all of them together).
+template <typename T, typename TO>
+__global__ void __launch_bounds__(256)
+moe_shared_down_kernel(const T* __restrict__ act, const T* __restrict__ down, Choice c, const float* __restrict__ z,
+                       TO* __restrict__ out, int n_tokens, int top, int width, int ff, int fs, int E) {
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  pdl_wait();
+  pdl_trigger();
+  const int i = blockIdx.x, t = blockIdx.y * 8 + warp;
+  if (t >= n_tokens) return;
+  const size_t C = (size_t)E * ff + fs;
+  const T* a = act + (size_t)t * (top * ff + fs);
+  const T* w = down + (size_t)i * C;
+  float total = 0.f;
+#pragma unroll 4
+  for (int k = 0; k < top; ++k) {
+    const int e = chosen_expert(c, t, k, top);
+    const float part = lane_dot(a + (size_t)k * ff, w + (size_t)e * ff, ff, lane);
+    total = fmaf(chosen_weight(c, t, k, top), part, total);
+  }
+  if (fs > 0) {
+    const float part = lane_dot(a + (size_t)top * ff, w + (size_t)E * ff, fs, lane);
+    total = fmaf(1.0f / (1.0f + expf(-z[t])), part, total);
+  }
+  total = warp_sum(total);
+  if (lane == 0) out[(size_t)t * width + i] = from_f32<TO>(total);
+}
+
+static bool choice_ok(const Choice& c) { return c.idx ? c.wts != nullptr : (c.table != nullptr && c.tokens != nullptr); }
+
+// act: scratch [n_tokens, top * ff + fs] of `dtype`; out of `out_dtype`.
+AB_API int ab_moe_shared_pairs(const void* h, int dtype, int ld, const void* gate_up, const void* down, const int* idx,
+                               const float* wts, const int* table, const int* tokens, float weight, const float* z, void* act,
+                               void* out, int out_dtype, int n_tokens, int top, int width, int ff, int fs, int E,
+                               int activation, cudaStream_t stream) {
+  if (n_tokens <= 0) return AB_OK;
+  const Choice c{idx, wts, table, tokens, weight};
+  if (top <= 0 || width <= 0 || ff <= 0 || fs < 0 || E <= 0 || (activation != 0 && activation != 1) || !choice_ok(c) ||
+      (fs > 0 && !z))
+    return AB_BAD_ARG;
+  const long long pair_blocks = ((long long)n_tokens * top + 7) / 8 * ff;
+  const long long blocks = pair_blocks + ((long long)n_tokens + 7) / 8 * fs;
+  if (blocks > 0x7fffffffLL || width > 0x7fffffff || (n_tokens + 7) / 8 > 65535) return AB_BAD_ARG;
+  const dim3 dgrid((unsigned)width, (unsigned)((n_tokens + 7) / 8));
+#define AB_GO(T, TO)                                                                                                   \
+  {                                                                                                                    \
+    ab_launch(moe_shared_up_kernel<T>, dim3((unsigned)blocks), dim3(256), 0, stream, (const T*)h, ld, (const T*)gate_up, c, \
+              (T*)act, n_tokens, top, width, ff, fs, E, activation, pair_blocks);                                      \
+    ab_launch(moe_shared_down_kernel<T, TO>, dgrid, dim3(256), 0, stream, (const T*)act, (const T*)down, c, z, (TO*)out, \
+              n_tokens, top, width, ff, fs, E);                                                                        \
+  }
+  if (dtype == AB_F32 && out_dtype == AB_F32) AB_GO(float, float)
+  else if (dtype == AB_BF16 && out_dtype == AB_F32) AB_GO(bf16, float)
+  else if (dtype == AB_BF16 && out_dtype == AB_BF16) AB_GO(bf16, bf16)
+  else return AB_BAD_ARG;
+#undef AB_GO
+  return ab_launch_status();
+}
+
+// All experts at once, for steps of many tokens: a row of `up` holds the gates of all C units and then their
+// up-projections (2 C numbers); the gates' place becomes act(gate) * up * weight, weight 0 for experts that were not
+// chosen and sigmoid(z_t) for the shared expert.
+template <int NC>
+__global__ void __launch_bounds__(256)
+moe_shared_weigh_kernel(bf16* __restrict__ up, Choice c, const float* __restrict__ z, int top, int ff, int fs, int E,
+                        int activation) {
+  const int t = blockIdx.y;
+  const int C = E * ff + fs;
+  const int col = (blockIdx.x * blockDim.x + threadIdx.x) * NC;
+  if (col >= C) return;
+  float g = 0.f;
+  if (col >= E * ff) {
+    g = 1.0f / (1.0f + expf(-z[t]));
+  } else {
+    const int e = col / ff;
+    for (int k = 0; k < top; ++k)
+      if (chosen_expert(c, t, k, top) == e) g = chosen_weight(c, t, k, top);
+  }
+  bf16* x = up + (size_t)t * 2 * C + col;
+  if (NC == 8) {
+    uint4 v = make_uint4(0, 0, 0, 0);
+    if (g != 0.f) {
+      const uint4 gv = *reinterpret_cast<const uint4*>(x), uv = *reinterpret_cast<const uint4*>(x + C);
+      const uint32_t a[4] = {gv.x, gv.y, gv.z, gv.w}, b[4] = {uv.x, uv.y, uv.z, uv.w};
+      uint32_t* o = reinterpret_cast<uint32_t*>(&v);
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        const float lo = g * activate(__uint_as_float(a[j] << 16), activation) * __uint_as_float(b[j] << 16);
+        const float hi = g * activate(__uint_as_float(a[j] & 0xffff0000u), activation) * __uint_as_float(b[j] & 0xffff0000u);
+        __nv_bfloat162 r = __floats2bfloat162_rn(lo, hi);
+        o[j] = *reinterpret_cast<uint32_t*>(&r);
+      }
+    }
+    *reinterpret_cast<uint4*>(x) = v;
+  } else {
+    x[0] = __float2bfloat16_rn(g != 0.f ? g * activate(__bfloat162float(x[0]), activation) * __bfloat162float(x[C]) : 0.f);
+  }
+}
+
+AB_API int ab_moe_shared_weigh(void* up, const int* idx, const float* wts, const int* table, const int* tokens, float weight,
+                               const float* z, int n_tokens, int top, int ff, int fs, int E, int activation,
+                               cudaStream_t stream) {
+  if (n_tokens <= 0) return AB_OK;
+  const Choice c{idx, wts, table, tokens, weight};
+  if (top <= 0 || ff <= 0 || fs < 0 || E <= 0 || n_tokens > 65535 || (activation != 0 && activation != 1) || !choice_ok(c) ||
+      (fs > 0 && !z))
+    return AB_BAD_ARG;
+  const long long C = (long long)E * ff + fs;
+  if (ff % 8 == 0 && fs % 8 == 0 && (((uintptr_t)up) & 15) == 0)
+    moe_shared_weigh_kernel<8><<<dim3((unsigned)((C / 8 + 255) / 256), (unsigned)n_tokens), 256, 0, stream>>>(
+        (bf16*)up, c, z, top, ff, fs, E, activation);
+  else
+    moe_shared_weigh_kernel<1><<<dim3((unsigned)((C + 255) / 256), (unsigned)n_tokens), 256, 0, stream>>>(
+        (bf16*)up, c, z, top, ff, fs, E, activation);
+  return ab_launch_status();
 }

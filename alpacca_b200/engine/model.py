@@ -21,7 +21,7 @@ from dataclasses import dataclass, field
 
 import torch
 
-from ..parts.base import BuildOptions, Norm, Part, PositionEncoding, block_cache_specs
+from ..parts.base import BuildOptions, Norm, Part, PositionEncoding, block_cache_specs, readable_entries
 from ..parts.block import HiddenStream
 from ..parts.embedding import TokenEmbedding, VocabHead
 from ..weights.loader import Fetcher, check_names
@@ -73,12 +73,21 @@ class DecoderModel(Part):
         self.entries_of_run: list[list[int]] = []
         for i, r in enumerate(spec.schedule):
             if r.reads_entry_of is not None:
-                theirs = self.entries_of_run[r.reads_entry_of]
-                mine = block_cache_specs(spec.layers[r.layer])
-                if [self._entry_specs[e] for e in theirs] != mine:
+                # the readable entries are the other run's, what else the block keeps is this run's own
+                other, block = spec.layers[spec.schedule[r.reads_entry_of].layer], spec.layers[r.layer]
+                theirs = [self.entries_of_run[r.reads_entry_of][k] for k in readable_entries(other)]
+                mine, shared = block_cache_specs(block), readable_entries(block)
+                if [self._entry_specs[e] for e in theirs] != [mine[k] for k in shared]:
                     raise ValueError(f"run {i} reads the cache of run {r.reads_entry_of}, which keeps "
                                      "something else than this run's layer would")
-                self.entries_of_run.append(theirs)
+                entries = []
+                for k, s in enumerate(mine):
+                    if k in shared:
+                        entries.append(theirs[shared.index(k)])
+                    else:
+                        entries.append(len(self._entry_specs))
+                        self._entry_specs.append(s)
+                self.entries_of_run.append(entries)
                 continue
             specs = block_cache_specs(spec.layers[r.layer])
             self.entries_of_run.append(list(range(len(self._entry_specs), len(self._entry_specs) + len(specs))))
@@ -86,6 +95,7 @@ class DecoderModel(Part):
         # an embedding that keeps something per sequence (its last token, say) has an entry after the runs'
         own = getattr(spec.embedding, "cache_spec", None)
         own = own() if own is not None else None
+        self.averages_depth = any(getattr(b, "average", None) is not None for b in spec.layers)
         self.embedding_entry = None
         if own is not None:
             self.embedding_entry = len(self._entry_specs)
@@ -150,26 +160,42 @@ class DecoderModel(Part):
         first = getattr(s.layers[s.schedule[i + 1].layer], "first_plain_norm", None)
         return first() if first is not None else None
 
+    def _front_after(self, i: int, views, ctx):
+        """(part, cache view) that opens the next block, if that block lets the block before it run the part and the step
+        brings one token per sequence."""
+        s = self.spec
+        if not ctx.is_decode or i + 1 >= len(s.schedule) or s.schedule[i + 1].enter is not None:
+            return None
+        front = getattr(s.layers[s.schedule[i + 1].layer], "front_part", None)
+        return front(views[i + 1]) if front is not None else None
+
     def forward(self, ctx, cache) -> torch.Tensor:
         """Runs the step described by `ctx`; returns float32 logits [n_want, vocab]."""
         s = self.spec
+        more: dict = {}
+        history = None
+        if self.averages_depth:       # what the embedding and every run leave, for blocks that average over depth
+            history = torch.empty((len(s.schedule) + 1, ctx.n_tokens, s.embedding.width), dtype=torch.float32,
+                                  device=ctx.tokens.device)
+            more["out"] = history[0]
         if self.embedding_entry is not None:
-            kept = cache.entry_view(self.embedding_entry, ctx.block_tables)
-            stream = HiddenStream(s.embedding.forward(ctx.tokens, ctx.n_tokens, ctx=ctx, cache=kept))
-        elif getattr(s.embedding, "scale", 1.0) != 1.0:
-            stream = HiddenStream(s.embedding.forward(ctx.tokens, ctx.n_tokens, ctx=ctx))
-        else:
-            stream = HiddenStream(s.embedding.forward(ctx.tokens, ctx.n_tokens))
+            more.update(ctx=ctx, cache=cache.entry_view(self.embedding_entry, ctx.block_tables))
+        elif getattr(s.embedding, "needs_context", False):
+            more["ctx"] = ctx
+        stream = HiddenStream(s.embedding.forward(ctx.tokens, ctx.n_tokens, **more), history=history,
+                              depth=0 if history is None else 1)
         if s.position is not None:
             s.position.add_to_embeddings(stream.residual, ctx)
+        views = [self._views(i, cache, ctx.block_tables) for i in range(len(s.schedule))]
         for i, run in enumerate(s.schedule):
-            view = self._views(i, cache, ctx.block_tables)
+            view = views[i]
             if run.enter is not None:
                 s.stream_parts[run.enter[0]].forward(stream, ctx, run.enter[1])
             stream.next_norm = self._reader_after(i, ctx)
             stream.next_plain = self._plain_reader_after(i)
+            stream.next_front = self._front_after(i, views, ctx)
             s.layers[run.layer].forward(stream, ctx, view, write_cache=run.reads_entry_of is None)
-        stream.next_norm = stream.next_plain = None
+        stream.next_norm = stream.next_plain = stream.next_front = None
         if ctx.n_want == 0:
             return torch.empty((0, s.vocab_size), dtype=torch.float32, device=stream.residual.device)
         if stream.owed is not None:

@@ -338,13 +338,17 @@ def _sm_count(device) -> int:
     return n
 
 
+PLAIN_ACTIVATIONS = {None: 0, "gelu": 1}      # on a product without a gate ("gelu": the erf form)
+
+
 def gemv_bf16(x, w, out, bias=None, n_rows=None, swiglu=False, slices=None, start_early=True, owed=None,
-              residual=None, norm_weight=None, activation="silu"):
+              residual=None, norm_weight=None, activation="silu", act=None, cap=0.0):
     """out[:n] = x[:n] @ w^T (+ bias) for n <= 32 rows, bfloat16 x [M,K], w [N,K].
 
     out bfloat16 or float32 [M,N]; with `swiglu`, w is the 8-row interleaved gate|up
     matrix [2F,K] and out is bfloat16 [M,F] = act(gate) * up (`activation`: "silu", "relu",
-    "gelu_tanh").  `start_early` off: the kernel is
+    "gelu_tanh").  Without it `act` ("gelu") is applied to the stored result, and `cap` > 0 bounds float32 results:
+    cap * tanh(y / cap).  `start_early` off: the kernel is
     launched without programmatic dependent launch, i.e. after the kernel before it has ended (for
     the product that follows the decode attention, see csrc/launch.cuh).
 
@@ -382,6 +386,9 @@ def gemv_bf16(x, w, out, bias=None, n_rows=None, swiglu=False, slices=None, star
     else:
         _need(out.shape[-1] == N and out.dtype in (torch.bfloat16, torch.float32), "gemv_bf16: out [M,N]")
         epi = 1 if out.dtype == torch.float32 else 0
+    _need(act in PLAIN_ACTIVATIONS, f"gemv_bf16: activation {act!r} is not one of {tuple(PLAIN_ACTIVATIONS)}")
+    _need(act is None or epi <= 1, "gemv_bf16: an activation without a gate belongs to a plain store")
+    _need(not cap or epi == 1, "gemv_bf16: a bound on the result belongs to a float32 store")
     if bias is not None:
         _need(bias.dtype == torch.float32 and bias.numel() == N and bias.is_contiguous(), "gemv_bf16: bias f32 [N]")
     ss_in, n_part, inv_width, eps = None, 0, 0.0, 0.0
@@ -403,10 +410,11 @@ def gemv_bf16(x, w, out, bias=None, n_rows=None, swiglu=False, slices=None, star
     if not start_early:
         lib.ab_pdl_hold(1)
     try:
-        _check(lib.ab_gemv_bf16_gated(_p(x), _p(w), _p(bias), _p(out), _p(partials), _p(arrivals), n, N, K,
-                                      out.shape[-1], epi, slices, _p(ss_in), n_part, ctypes.c_float(inv_width),
-                                      ctypes.c_float(eps), _p(residual), _p(norm_weight), _p(ss_out),
-                                      GATE_ACTIVATIONS[activation], _stream()), "gemv_bf16")
+        _check(lib.ab_gemv_bf16_act(_p(x), _p(w), _p(bias), _p(out), _p(partials), _p(arrivals), n, N, K,
+                                    out.shape[-1], epi, slices, _p(ss_in), n_part, ctypes.c_float(inv_width),
+                                    ctypes.c_float(eps), _p(residual), _p(norm_weight), _p(ss_out),
+                                    GATE_ACTIVATIONS[activation], PLAIN_ACTIVATIONS[act], ctypes.c_float(cap), _stream()),
+               "gemv_bf16")
     finally:
         if not start_early:
             lib.ab_pdl_hold(0)
@@ -509,15 +517,24 @@ def _stream_scratch(device, n_partial: int, n_counters: int):
     return have
 
 
+def _check_dist(dist, H):
+    """The penalty on distance of H heads: float32 [2, H], r1 of all heads and then r2."""
+    if dist is not None:
+        _cuda(dist)
+        _need(dist.dtype == torch.float32 and dist.is_contiguous() and tuple(dist.shape) == (2, H),
+              f"the penalty on distance must be float32 [2, {H}]")
+
+
 def attention_stream(qkv, out, cache, ctx, H, K, D, scale, window=0, rot=None, fuse=0, pages_per_cta=8,
-                     merge="memory", ring=1):
+                     merge="memory", ring=1, dist=None):
     """Decode attention that streams the cache through a ring of pages filled by TMA
     (csrc/attention_stream.cu): head sizes 64 and 128, bfloat16.  A CTA takes `pages_per_cta` pages of
     one (sequence, KV head); the chunks of a sequence are merged in chunk order, through scratch memory
     (`merge` "memory") or inside a cluster of up to 8 ("cluster").  `ring`: 0 a short ring (four CTAs per
     processor), 1 the usual one (two), 2 a deep one (one).  `fuse` as for the other decode kernel: 1 rotates q, 2 also rotates k
-    and appends k, v to the cache."""
+    and appends k, v to the cache.  `dist` (float32 [2, H]): a penalty on distance, see `attention_maps`."""
     lib = _lib("attention_stream")
+    _check_dist(dist, H)
     k_pages, v_pages, table = cache.k, cache.v, cache.block_table
     _cuda(qkv, out, k_pages, v_pages, table)
     T = ctx.n_tokens
@@ -554,11 +571,11 @@ def attention_stream(qkv, out, cache, ctx, H, K, D, scale, window=0, rot=None, f
             kind = 2
             part_o, part_ml, arrivals = _stream_scratch(qkv.device, T * H * n_chunks * D, T * K * -(-(H // K) // 8))
     _tc_unchecked["attention_stream"] = True
-    _check(lib.ab_attention_stream_bf16(
+    _check(lib.ab_attention_stream_dist_bf16(
         _p(qkv), qkv.shape[-1], _p(out), _p(part_o), _p(part_ml), _p(arrivals), _p(k_pages), _p(v_pages),
         k_pages.shape[0], _p(table), table.shape[1], _p(ctx.tok_seq), _p(ctx.kv_len), _p(order), T, H, K, D,
         ctypes.c_float(scale), int(window or 0), ppc, n_chunks, kind, int(ring), _p(cos), _p(sin), n_rot,
-        pairing, fuse, _stream()), "attention_stream")
+        pairing, fuse, _p(dist), _stream()), "attention_stream")
     return out
 
 
@@ -734,8 +751,31 @@ def owed_norm_pays(n_rows: int, out_features: int, in_features: int, device) -> 
     return (defers_norm(n_rows, in_features) and -(-out_features // 16) <= 2 * _sm_count(device))
 
 
-def linear_bf16(x, w, out, n_rows=None, bias=None, start_early=True, owed=None):
+def softcap(y, cap, n_rows=None):
+    """y[:n] = cap * tanh(y[:n] / cap) in place; y float32 [M, N]."""
+    _cuda(y)
+    n = y.shape[0] if n_rows is None else n_rows
+    _need(y.dtype == torch.float32 and y.is_contiguous() and y.dim() == 2 and n <= y.shape[0] and cap > 0,
+          "softcap: y float32 [M, N], cap > 0")
+    _check(_lib("elementwise").ab_softcap(_p(y), ctypes.c_float(cap), ctypes.c_longlong(n * y.shape[1]), _stream()), "softcap")
+    return y
+
+
+def plain_act(y, activation, n_rows=None):
+    """y[:n] = act(y[:n]) in place ("gelu": the erf form); y [M, N]."""
+    _cuda(y)
+    n = y.shape[0] if n_rows is None else n_rows
+    _need(activation in PLAIN_ACTIVATIONS and activation is not None,
+          f"plain_act: activation {activation!r} is not one of {tuple(PLAIN_ACTIVATIONS)}")
+    _need(y.is_contiguous() and y.dim() == 2 and n <= y.shape[0], "plain_act: y [M, N]")
+    _check(_lib("elementwise").ab_act(_p(y), _dt(y), ctypes.c_longlong(n * y.shape[1]), PLAIN_ACTIVATIONS[activation] - 1,
+                                      _stream()), "plain_act")
+    return y
+
+
+def linear_bf16(x, w, out, n_rows=None, bias=None, start_early=True, owed=None, act=None, cap=0.0):
     """out[:n] = x[:n] @ w^T (+ bias) for bfloat16 x [M,K], w [N,K]; out bfloat16 or float32 [M,N].
+    `act` ("gelu"): applied to the result; `cap` > 0 (float32 results): cap * tanh(result / cap).
 
     Up to GEMV_MAX_ROWS rows (decode steps; GEMV_NARROW_MAX_ROWS for narrow matrices): the
     skinny-matrix kernel, which reads the weights once.  More rows: the library matrix product (as
@@ -747,7 +787,9 @@ def linear_bf16(x, w, out, n_rows=None, bias=None, start_early=True, owed=None):
           "linear_bf16: x [M,K], w [N,K], out [M,N]")
     if x.shape[1] % 8 == 0 and (n <= GEMV_MAX_ROWS or (n <= GEMV_NARROW_MAX_ROWS
                                                        and -(-w.shape[0] // 16) <= _sm_count(x.device))):
-        return gemv_bf16(x, w, out, bias=bias, n_rows=n, start_early=start_early, owed=owed)
+        return gemv_bf16(x, w, out, bias=bias, n_rows=n, start_early=start_early, owed=owed, act=act, cap=cap)
+    if act is not None and out.dtype == torch.bfloat16 and x.shape[1] % 8 == 0 and n >= TC_PERSISTENT_MIN_ROWS:
+        return gemm_tc(x, w, out, bias=bias, n_rows=n, swap=False, act=act)     # the activation in the product's tail
     _need(owed is None, "linear_bf16: only the skinny product finishes a norm that its input owes")
     xs, ys = (x, out) if n == x.shape[0] == out.shape[0] else (x[:n], out[:n])
     if out.dtype == torch.float32:
@@ -757,6 +799,10 @@ def linear_bf16(x, w, out, n_rows=None, bias=None, start_early=True, owed=None):
     _mark("library product")
     if bias is not None:
         add_bias(ys, bias)
+    if act is not None:
+        plain_act(out, act, n_rows=n)
+    if cap:
+        softcap(out, cap, n_rows=n)
     return out
 
 
@@ -828,12 +874,13 @@ def decode_advance(tokens, tok_pos, kv_len, rng_step, tok_seq, sampled, recent, 
 
 
 def gemm_tc(x, w, out, bias=None, n_rows=None, swiglu=False, swap=None, bn=None, slices=None, persistent=True,
-            pair=None, activation="silu"):
+            pair=None, activation="silu", act=None):
     """out[:n] = x[:n] @ w^T (+ bias) on the tcgen05 tensor cores (TMA-fed, TMEM accumulators).
 
     x [M,K], w [N,K] bfloat16; out bfloat16 or float32 [M,N]; with `swiglu`, w is the 8-row
     interleaved gate|up matrix and out is bfloat16 [M, N/2] (`activation` on the gate: "silu"; "relu" and
-    "gelu_tanh" in the persistent forms only).  `swap` puts the weights on the
+    "gelu_tanh" in the persistent forms only).  `act` ("gelu", bfloat16, persistent forms only): an activation
+    on a product without a gate.  `swap` puts the weights on the
     128-row side of the MMA (the batch, up to 256 rows, becomes the columns): the shape for decode
     steps.  `bn` is the MMA's column count per tile, `slices` the number of K slices.  Without `swap`,
     256-wide tiles and one slice run as the persistent kernel (one CTA per SM walks the tiles) unless
@@ -862,6 +909,10 @@ def gemm_tc(x, w, out, bias=None, n_rows=None, swiglu=False, swap=None, bn=None,
     else:
         _need(out.shape[-1] == N and out.dtype in (torch.bfloat16, torch.float32), "gemm_tc: out [M,N]")
         epi = 1 if out.dtype == torch.float32 else 0
+        if act is not None:
+            _need(act == "gelu" and epi == 0 and not swap and bn == 256 and slices in (None, 1) and persistent,
+                  "gemm_tc: an activation without a gate is GELU on a bfloat16 store of the persistent forms")
+            epi = 5
     if bias is not None:
         _need(bias.dtype == torch.float32 and bias.numel() == N and bias.is_contiguous(), "gemm_tc: bias f32 [N]")
     _tc_unchecked["gemm_tc"] = True
@@ -1342,7 +1393,7 @@ ATTENTION_MAPS_MAX_DIM = 256
 
 
 def attention_prepare(buf, offsets, H, G, M, Dk, Dv, cache, ctx, q_weight=None, k_weight=None, eps=0.0, rot=None,
-                      write_cache=True, bias=None, v_norm=False, v_side_by_side=False):
+                      write_cache=True, bias=None, v_norm=False, v_side_by_side=False, norm_rows=False):
     """Query and key norm, position rotation and the append of keys and values to the cache, for an attention
     whose heads have M score maps (csrc/attention_maps.cu).
 
@@ -1352,7 +1403,9 @@ def attention_prepare(buf, offsets, H, G, M, Dk, Dv, cache, ctx, q_weight=None, 
     [n_pages, G*M, page, Dk] and value pages [n_pages, G, page, Dv]).  `bias` float32 [N]: the projection's
     bias where the product left it out; it is added first.  `v_norm`: every value vector is divided by its root mean
     square (eps inside the root) before it is stored.  `v_side_by_side`: the value pages are [n_pages, 1, page,
-    G*Dv], a token's value heads in one row."""
+    G*Dv], a token's value heads in one row.  `norm_rows`: the norm runs over ALL query vectors of a token at once
+    (q_weight [H*M*Dk]), and over all its key vectors (k_weight [G*M*Dk]), instead of vector by vector.  With
+    `write_cache` off the rows need not hold key and value vectors."""
     k_pages, v_pages, table = cache.k, cache.v, cache.block_table
     cos, sin, n_rot, pairing = rot if rot is not None else (None, None, 0, 0)
     _cuda(buf, k_pages, v_pages, table, q_weight, k_weight, cos, sin)
@@ -1360,7 +1413,7 @@ def attention_prepare(buf, offsets, H, G, M, Dk, Dv, cache, ctx, q_weight=None, 
     off_q, off_k, off_v = (int(o) for o in offsets)
     N = buf.shape[-1]
     _need(buf.is_contiguous() and buf.numel() >= T * N and min(off_q, off_k, off_v) >= 0
-          and max(off_q + H * M * Dk, off_k + G * M * Dk, off_v + G * Dv) <= N,
+          and max([off_q + H * M * Dk] + ([off_k + G * M * Dk, off_v + G * Dv] if write_cache or not norm_rows else [])) <= N,
           "attention_prepare: buf [T, N] must hold the query, key and value vectors at their offsets")
     _need(0 < Dk <= ATTENTION_MAPS_MAX_DIM and 0 < Dv <= ATTENTION_MAPS_MAX_DIM,
           f"attention_prepare: head sizes {Dk}, {Dv} are outside 1..{ATTENTION_MAPS_MAX_DIM}")
@@ -1372,10 +1425,10 @@ def attention_prepare(buf, offsets, H, G, M, Dk, Dv, cache, ctx, q_weight=None, 
           f"attention_prepare: cache pages [n, {G * M}, page, {Dk}] and [n, {G}, page, {Dv}] of buf's dtype")
     _need(table.dtype == torch.int32 and table.dim() == 2 and table.is_contiguous()
           and ctx.max_kv_len <= table.shape[1] * page, "attention_prepare: the block table does not cover the step")
-    for wgt in (q_weight, k_weight):
+    for wgt, vectors in ((q_weight, H * M), (k_weight, G * M)):
         if wgt is not None:
-            _need(wgt.dtype == torch.float32 and wgt.numel() == Dk and wgt.is_contiguous(),
-                  "attention_prepare: norm weights float32 [Dk]")
+            _need(wgt.dtype == torch.float32 and wgt.numel() == (vectors * Dk if norm_rows else Dk) and wgt.is_contiguous(),
+                  "attention_prepare: norm weights float32 [Dk], or one number per column of the rows with norm_rows")
     if cos is not None:
         _need(sin is not None and cos.dtype == torch.float32 and sin.dtype == torch.float32 and cos.is_contiguous()
               and sin.is_contiguous() and cos.shape == sin.shape and cos.shape[-1] == n_rot // 2 and n_rot % 2 == 0
@@ -1388,6 +1441,16 @@ def attention_prepare(buf, offsets, H, G, M, Dk, Dv, cache, ctx, q_weight=None, 
               "attention_prepare: bias float32 [N]")
     _i32(ctx.tok_pos, T, "tok_pos")
     _i32(ctx.tok_seq, T, "tok_seq")
+    if norm_rows:
+        _need(q_weight is not None and (k_weight is not None or not write_cache) and not v_norm and not v_side_by_side,
+              "attention_prepare: a norm over whole rows has weights, and stands alone")
+        _need((H + G) * M * Dk * 4 <= 200 * 1024, "attention_prepare: the rows to be normed do not fit shared memory")
+        _check(_lib("attention_maps").ab_attention_prepare_rows(
+            _p(buf), _dt(buf), N, off_q, off_k, off_v, H * M, G * M, G, Dk, Dv, _p(q_weight), _p(k_weight),
+            ctypes.c_float(eps), _p(cos), _p(sin), n_rot, pairing, _p(ctx.tok_pos), _p(ctx.tok_seq), _p(table),
+            table.shape[1], _p(k_pages), _p(v_pages), page, T, 1 if write_cache else 0, _p(bias), _stream()),
+            "attention_prepare")
+        return
     _check(_lib("attention_maps").ab_attention_prepare_opts(
         _p(buf), _dt(buf), N, off_q, off_k, off_v, H * M, G * M, G, Dk, Dv, _p(q_weight), _p(k_weight),
         ctypes.c_float(eps), _p(cos), _p(sin), n_rot, pairing, _p(ctx.tok_pos), _p(ctx.tok_seq), _p(table),
@@ -1396,11 +1459,13 @@ def attention_prepare(buf, offsets, H, G, M, Dk, Dv, cache, ctx, q_weight=None, 
 
 
 def attention_maps(q, q_stride, out, cache, ctx, H, G, M, Dk, Dv, scale, window=0, sink=None, coef=0.0,
-                   unit_norm=False, eps=0.0, out_scale=1.0):
+                   unit_norm=False, eps=0.0, out_scale=1.0, dist=None):
     """Attention of every token over its sequence's cached keys and values, one warp per (token, head), 32-bit
     arithmetic (csrc/attention_maps.cu): M score maps per head, combined as a_0 + coef * (a_1 + ..), optionally
     divided by the head's root mean square, times `out_scale`.  q: the prepared rows (query vectors at the
-    start of each row of `q_stride` elements); out [T, H*Dv] of q's dtype."""
+    start of each row of `q_stride` elements); out [T, H*Dv] of q's dtype.  `dist` (float32 [2, H], r1 and r2): a
+    penalty r1_h ln(1 + r2_h (p - s)) is taken off the scaled score of a key at s for a token at p."""
+    _check_dist(dist, H)
     k_pages, v_pages, table = cache.k, cache.v, cache.block_table
     _cuda(q, out, k_pages, v_pages, table, sink)
     T = ctx.n_tokens
@@ -1419,10 +1484,10 @@ def attention_maps(q, q_stride, out, cache, ctx, H, G, M, Dk, Dv, scale, window=
         _need(sink.dtype == torch.float32 and sink.numel() == H and sink.is_contiguous(), "sink must be float32 [H]")
     _i32(ctx.tok_pos, T, "tok_pos")
     _i32(ctx.tok_seq, T, "tok_seq")
-    _check(_lib("attention_maps").ab_attention_maps(
+    _check(_lib("attention_maps").ab_attention_maps_dist(
         _p(q), q_stride, _p(out), _dt(q), _p(k_pages), _p(v_pages), _p(table), table.shape[1], _p(ctx.tok_pos),
         _p(ctx.tok_seq), T, H, G, M, Dk, Dv, page, ctypes.c_float(scale), int(window or 0), _p(sink),
-        ctypes.c_float(coef), 1 if unit_norm else 0, ctypes.c_float(eps), ctypes.c_float(out_scale), _stream()),
+        ctypes.c_float(coef), 1 if unit_norm else 0, ctypes.c_float(eps), ctypes.c_float(out_scale), _p(dist), _stream()),
         "attention_maps")
     return out
 
@@ -1451,12 +1516,13 @@ def _row_index(device, n: int):
 
 
 def attention_maps_mma(q, q_stride, out, cache, ctx, H, G, M, Dk, Dv, scale, window=0, sink=None, coef=0.0,
-                       unit_norm=False, eps=0.0, out_scale=1.0):
+                       unit_norm=False, eps=0.0, out_scale=1.0, dist=None):
     """`attention_maps` on the tensor-core kernels (bfloat16 operands, float32 scores, softmax and sums): q holds
     the prepared query vectors at the start of each row, keys and values are in the cache already.  One map with
     equal key and value sizes in a step of one token each takes the decode kernel; everything else the kernel that
     tiles query rows (a step of one token each then has one token per tile).  Several maps leave their outputs
-    in float32 and are combined by `ab_maps_combine`."""
+    in float32 and are combined by `ab_maps_combine`.  `dist`: see `attention_maps`."""
+    _check_dist(dist, H)
     k_pages, v_pages, table = cache.k, cache.v, cache.block_table
     _cuda(q, out, k_pages, v_pages, table, sink)
     T = ctx.n_tokens
@@ -1477,26 +1543,31 @@ def attention_maps_mma(q, q_stride, out, cache, ctx, H, G, M, Dk, Dv, scale, win
     _i32(ctx.tok_seq, T, "tok_seq")
     if ctx.is_decode and M == 1 and Dk == Dv:
         width = max(int(table.shape[1]), 1)
+        plan = _stream_plan(T, H, G, Dk, width, _sm_count(q.device)) if dist is not None and sink is None else None
+        if plan is not None:
+            return attention_stream(q, out, cache, ctx, H, G, Dk, scale, window, pages_per_cta=plan[0], merge=plan[1],
+                                    ring=plan[2], dist=dist)
         small, n_chunks = _decode_attention_plan(T * G * -(-(H // G) // 8), width, Dk, _sm_count(q.device))
         _i32(ctx.kv_len, ctx.n_seqs, "kv_len")
-        _check(lib.ab_attention_decode_sink_bf16(
+        _check(lib.ab_attention_decode_dist_bf16(
             _p(q), q_stride, _p(out), None, None, None, _p(k_pages), _p(v_pages), _p(table), table.shape[1],
             _p(ctx.tok_seq), _p(ctx.kv_len), T, H, G, Dk, ctypes.c_float(scale), int(window or 0),
-            -(-width // n_chunks), n_chunks, small, None, None, 0, 0, 0, _p(sink), _stream()), "attention_decode")
+            -(-width // n_chunks), n_chunks, small, None, None, 0, 0, 0, _p(sink), _p(dist), _stream()), "attention_decode")
         return out
     _i32(ctx.tok_pos, T, "tok_pos")
     _i32(ctx.cu_q, ctx.n_seqs + 1, "cu_q")
     if (USE_TCGEN05_ATTENTION and not ctx.is_decode and M == 1 and Dk == Dv and Dk in (64, 128) and T >= 128
             and q.shape[0] >= T and q_stride % Dk == 0):
         tc = _lib("attention_tc")
-        if tc.ab_attention_prefill_tc_supports(H, G, Dk):
+        if (tc.ab_attention_prefill_tc_supports(H, G, Dk)
+                and (dist is None or H // G <= tc.ab_attention_prefill_tc_dist_max_group())):
             # long prompts, one map, head size 64 or 128: the tcgen05 kernel (a sink in its last step)
             _tc_unchecked["attention_tc"] = True
             tile_seq, tile_q0, n_tiles, _ = _prefill_tiles(ctx, H // G, q.device, rows=128)
-            _check(tc.ab_attention_prefill_tc_sink(
+            _check(tc.ab_attention_prefill_tc_dist(
                 _p(q), q_stride // Dk, T, _p(out), _p(k_pages), _p(v_pages), k_pages.shape[0], _p(table), table.shape[1],
                 _p(ctx.tok_pos), _p(ctx.cu_q), _p(tile_seq), _p(tile_q0), n_tiles, H, G, Dk, ctypes.c_float(scale),
-                int(window or 0), _p(sink), _stream()), "attention_prefill_tc")
+                int(window or 0), _p(sink), _p(dist), _stream()), "attention_prefill_tc")
             return out
     if ctx.is_decode:
         # one token per sequence: a tile per token; the rows are the batch rows themselves
@@ -1505,10 +1576,10 @@ def attention_maps_mma(q, q_stride, out, cache, ctx, H, G, M, Dk, Dv, scale, win
     else:
         tile_seq, tile_q0, n_tiles, tpt = _prefill_tiles(ctx, H // G, q.device)
     maps = out if M == 1 else torch.empty((q.shape[0], H * M * Dv), dtype=torch.float32, device=q.device)
-    _check(lib.ab_attention_prefill_maps_bf16(
+    _check(lib.ab_attention_prefill_maps_dist_bf16(
         _p(q), q_stride, _p(maps), 0 if M == 1 else 1, _p(k_pages), _p(v_pages), _p(table), table.shape[1],
         _p(ctx.tok_pos), _p(ctx.cu_q), _p(ctx.tok_seq), _p(tile_seq), _p(tile_q0), n_tiles, tpt, H * M, G * M, M, Dk, Dv,
-        ctypes.c_float(scale), int(window or 0), _p(sink), _stream()), "attention_prefill")
+        ctypes.c_float(scale), int(window or 0), _p(sink), Dv, 0, Dv, _p(dist), _stream()), "attention_prefill")
     if M > 1:
         _check(_lib("attention_maps").ab_maps_combine(
             _p(maps), _p(out), _dt(out), _p(ctx.tok_seq), T, H, M, Dv, ctypes.c_float(coef),
@@ -1945,4 +2016,155 @@ def head_norm_gate(o, weight, gate, gate_act, eps, out, ctx, H, V):
     _check(_lib("gated_recurrence").ab_head_norm_gate(
         _p(o), _p(weight), _p(gate), ldg, HEAD_GATES[gate_act if gate is not None else None], _p(out), _dt(out),
         _p(ctx.tok_seq), T, H, V, ctypes.c_float(eps), _stream()), "head_norm_gate")
+    return out
+
+
+# ---------------------------------------------------------------------------
+# blocks whose norms act on the sub-layers' outputs, whose mixers see the stream through a short convolution and whose
+# results are averaged over depth (csrc/depth_stream.cu); experts chosen by token id and a shared expert (csrc/moe.cu)
+
+def embed_positions(table, pos, out, ctx):
+    """out[t] = table[token of t] + pos[place of t in its sequence] as float32; table [V, E], pos [P, E] of one dtype."""
+    _cuda(table, pos, out)
+    T, E = ctx.n_tokens, table.shape[1]
+    _need(table.dim() == 2 and pos.dim() == 2 and table.is_contiguous() and pos.is_contiguous() and pos.shape[1] == E
+          and pos.dtype == table.dtype, "embed_positions: table [V, E], pos [P, E] of one dtype")
+    _need(ctx.max_kv_len <= pos.shape[0], f"embed_positions: {pos.shape[0]} positions, the step reaches {ctx.max_kv_len}")
+    _need(out.dtype == torch.float32 and out.is_contiguous() and out.shape[-1] == E and out.numel() >= T * E,
+          "embed_positions: out float32 [T, E]")
+    for t, name in ((ctx.tokens, "tokens"), (ctx.tok_seq, "tok_seq"), (ctx.tok_pos, "tok_pos")):
+        _i32(t, T, name)
+    _check(_lib("depth_stream").ab_embed_positions(_p(table), _p(pos), _dt(table), _p(ctx.tokens), _p(ctx.tok_seq),
+                                                   _p(ctx.tok_pos), _p(out), T, E, _stream()), "embed_positions")
+    return out
+
+
+def _check_conv(w, state, E):
+    _need(w.dtype == torch.float32 and w.dim() == 2 and w.shape[1] == E and w.is_contiguous(),
+          "the convolution's weights must be float32 [taps, E]")
+    taps = w.shape[0]
+    if taps > 1:
+        _need(state is not None and state.dtype == torch.float32 and state.is_contiguous()
+              and tuple(state.shape[1:]) == (taps - 1, E), f"the convolution's state must be float32 [slots, {taps - 1}, {E}]")
+    return taps
+
+
+def input_conv(x, w, state, out, ctx, write_state=True):
+    """out[t] = x[t] + sum_j w[j] * x[t - taps + 1 + j] per channel, over each sequence's tokens; x float32 [T, E], w
+    float32 [taps, E] (the last tap meets the token itself), out [T, E].  state float32 [slots, taps - 1, E] (None for
+    one tap): the sequence's last rows of x before the step, and after it (`write_state`)."""
+    _cuda(x, w, state, out)
+    T, E = ctx.n_tokens, x.shape[-1]
+    taps = _check_conv(w, state, E)
+    _need(x.dtype == torch.float32 and x.is_contiguous() and x.numel() >= T * E and out.is_contiguous()
+          and out.shape[-1] == E and out.numel() >= T * E, "input_conv: x float32 [T, E], out [T, E]")
+    _i32(ctx.tok_seq, T, "tok_seq")
+    _i32(ctx.cu_q, ctx.n_seqs + 1, "cu_q")
+    _i32(ctx.slots, ctx.n_seqs, "slots")
+    _check(_lib("depth_stream").ab_input_conv(_p(x), _p(w), _p(state), _p(out), _dt(out), _p(ctx.tok_seq), _p(ctx.cu_q),
+                                              _p(ctx.slots), T, E, taps, 1 if write_state else 0, _stream()), "input_conv")
+    return out
+
+
+def post_norm_stream(x, y, weight, eps, ctx, v_out=None, dot_weight=None, dots=None, history=None, n_history=0, coef=None,
+                     avg_out=None, out=None, conv=None):
+    """v = x + y / sqrt(mean(y^2) + eps) * weight for every token of the step (a sub-layer's output joins the stream).
+    Then, each if it is given: `v_out` = v; `dots` [T] = v . dot_weight; `avg_out` = coef[n] v + sum_(j < n) coef[j]
+    history[j] with n = `n_history` and history float32 [.., T, E] (m = v without it); `out` = m in out's dtype, or, with
+    `conv` = (w [taps, E], state) and one token per sequence, `input_conv` of m with the state moved on."""
+    w_conv, state = conv if conv is not None else (None, None)
+    _cuda(x, y, weight, v_out, dot_weight, dots, history, coef, avg_out, out, w_conv, state)
+    T, E = ctx.n_tokens, x.shape[-1]
+    for t, name in ((x, "x"), (v_out, "v_out"), (avg_out, "avg_out")):
+        if t is not None:
+            _need(t.dtype == torch.float32 and t.is_contiguous() and t.shape[-1] == E and t.numel() >= T * E,
+                  f"post_norm_stream: {name} float32 [T, E]")
+    _need(y.is_contiguous() and y.shape[-1] == E and y.numel() >= T * E, "post_norm_stream: y [T, E]")
+    for t, name in ((weight, "weight"), (dot_weight, "dot_weight")):
+        if t is not None:
+            _need(t.dtype == torch.float32 and t.is_contiguous() and t.numel() == E, f"post_norm_stream: {name} float32 [E]")
+    if dots is not None:
+        _need(dot_weight is not None and dots.dtype == torch.float32 and dots.is_contiguous() and dots.numel() >= T,
+              "post_norm_stream: dots float32 [T] with dot_weight")
+    stride = 0
+    if coef is not None:
+        _need(coef.dtype == torch.float32 and coef.is_contiguous() and coef.numel() == n_history + 1 and avg_out is not None,
+              "post_norm_stream: coef float32 [n_history + 1] with avg_out")
+        if n_history:
+            _need(history is not None and history.dtype == torch.float32 and history.is_contiguous() and history.dim() == 3
+                  and history.shape[0] >= n_history and history.shape[1] >= T and history.shape[2] == E,
+                  "post_norm_stream: history float32 [>= n_history, >= T, E]")
+            stride = history.stride(0)
+    if out is not None:
+        _need(out.is_contiguous() and out.shape[-1] == E and out.numel() >= T * E, "post_norm_stream: out [T, E]")
+    taps = 1
+    if conv is not None:
+        _need(out is not None and ctx.is_decode, "post_norm_stream: the convolution belongs to steps of one token per sequence")
+        taps = _check_conv(w_conv, state, E)
+        _i32(ctx.slots, ctx.n_seqs, "slots")
+    _i32(ctx.tok_seq, T, "tok_seq")
+    _check(_lib("depth_stream").ab_post_norm_stream(
+        _p(x), _p(y), _dt(y), _p(weight), ctypes.c_float(eps), _p(v_out), _p(dot_weight), _p(dots), _p(history),
+        ctypes.c_longlong(stride), int(n_history), _p(coef), _p(avg_out), _p(out), _dt(out) if out is not None else 0,
+        _p(w_conv), _p(state), _p(ctx.slots), taps, _p(ctx.tok_seq), T, E, _stream()), "post_norm_stream")
+    return out
+
+
+def row_dots(h, w, n_tokens):
+    """float32 [T]: h[t] . w for h [T, E] and w float32 [E]."""
+    _cuda(h, w)
+    E = h.shape[-1]
+    _need(h.is_contiguous() and h.numel() >= n_tokens * E and w.dtype == torch.float32 and w.is_contiguous() and w.numel() == E,
+          "row_dots: h [T, E], w float32 [E]")
+    z = torch.empty((max(n_tokens, 1),), dtype=torch.float32, device=h.device)
+    _check(_lib("moe").ab_moe_logits(_p(h), _dt(h), E, _p(w), n_tokens, E, 1, _p(z), _stream()), "row_dots")
+    return z
+
+
+def moe_shared_experts(h, gate_up, down, n_experts, ff, shared_ff, top, out, ctx, activation="silu", choice=None, table=None,
+                       gate_logits=None):
+    """Gated experts and a shared expert: out[t] = sum_k weight_k E_(e_k)(h[t]) + sigmoid(gate_logits[t]) S(h[t]), an expert
+    W_down (act(W_gate h) * (W_up h)).  gate_up [2, C, width], down [width, C] with C = n_experts * ff + shared_ff: the
+    experts' units side by side, then the shared expert's (`shared_ff` 0: none).  The choice is `choice` = (experts int32
+    [T, top], weights float32 [T, top]), or row token_t of `table` int32 [vocab, top] with weight 1 / top each.
+    out [T, width] float32, or of h's dtype."""
+    idx, wts = choice if choice is not None else (None, None)
+    _cuda(h, gate_up, down, out, idx, wts, table, gate_logits)
+    T, width = ctx.n_tokens, h.shape[-1]
+    C = n_experts * ff + shared_ff
+    _need(tuple(gate_up.shape) == (2, C, width) and tuple(down.shape) == (width, C) and gate_up.is_contiguous()
+          and down.is_contiguous() and gate_up.dtype == h.dtype and down.dtype == h.dtype,
+          f"moe_shared_experts: gate_up [2, {C}, {width}], down [{width}, {C}] of h's dtype")
+    _need(h.is_contiguous() and h.numel() >= T * width and out.is_contiguous() and out.shape[-1] == width
+          and out.numel() >= T * width and out.dtype in (torch.float32, h.dtype),
+          "moe_shared_experts: h [T, width], out [T, width] float32 or of h's dtype")
+    _need((choice is None) != (table is None), "moe_shared_experts: the choice is a router's or a table's")
+    if choice is not None:
+        _i32(idx, T * top, "experts")
+        _need(wts.dtype == torch.float32 and wts.is_contiguous() and wts.numel() >= T * top, "weights float32 [T, top]")
+    else:
+        _i32(ctx.tokens, T, "tokens")
+        _need(table.dtype == torch.int32 and table.is_contiguous() and table.dim() == 2 and table.shape[1] == top,
+              "the experts' table must be contiguous int32 [vocab, top]")
+    if shared_ff:
+        _need(gate_logits is not None and gate_logits.dtype == torch.float32 and gate_logits.is_contiguous()
+              and gate_logits.numel() >= T, "moe_shared_experts: the shared expert's gate logits float32 [T]")
+    by = (_p(idx), _p(wts), _p(table), _p(ctx.tokens) if table is not None else None, ctypes.c_float(1.0 / top),
+          _p(gate_logits))
+    if h.dtype == torch.bfloat16 and MOE_ALL_EXPERTS_MIN_ROWS <= T <= 65535:
+        up = torch.empty((T, 2 * C), dtype=h.dtype, device=h.device)
+        torch.mm(h[:T], gate_up.view(2 * C, width).t(), out=up)
+        _mark("library product")
+        _check(_lib("moe").ab_moe_shared_weigh(_p(up), *by, T, top, ff, shared_ff, n_experts, MOE_ACTIVATIONS[activation],
+                                               _stream()), "moe_weigh_all")
+        if out.dtype == torch.float32:
+            torch.mm(up[:, :C], down.t(), out_dtype=torch.float32, out=out[:T])
+        else:
+            torch.mm(up[:, :C], down.t(), out=out[:T])
+        _mark("library product")
+        return out
+    act = torch.empty((max(T, 1), top * ff + shared_ff), dtype=h.dtype, device=h.device)
+    _check(_lib("moe").ab_moe_shared_pairs(_p(h), _dt(h), width, _p(gate_up), _p(down), *by, _p(act), _p(out), _dt(out), T, top,
+                                           width, ff, shared_ff, n_experts, MOE_ACTIVATIONS[activation], _stream()),
+           "moe_experts", kernels=2)
     return out

@@ -215,6 +215,13 @@ class Block(Part):
         raise NotImplementedError
 
 
+def readable_entries(block) -> list[int]:
+    """Which of a block's cache entries (places in `block_cache_specs`) a run that reads another run's cache shares with
+    it: the block's `readable_entries()`, by default all.  The others are always a run's own."""
+    own = getattr(block, "readable_entries", None)
+    return list(own()) if own is not None else list(range(len(block_cache_specs(block))))
+
+
 def block_cache_specs(block) -> list:
     """`block.cache_specs()`, or for a block that does not define it, its `.mixer`'s spec."""
     own = getattr(block, "cache_specs", None)

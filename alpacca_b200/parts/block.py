@@ -15,8 +15,9 @@ from dataclasses import dataclass
 import torch
 
 from .. import ops
-from .base import Block, FeedForward, HalfSum, Mixer, Norm, OwedNorm, WeightedSum
+from .base import Block, FeedForward, HalfSum, Mixer, Norm, OwedNorm, WeightedSum, mixer_cache_specs
 from .layer_norm import LayerNorm
+from .stream import StreamCast
 
 
 @dataclass
@@ -28,6 +29,11 @@ class HiddenStream:
                                        # if its reader accepts an OwedNorm in this step
     next_plain: Norm | None = None     # set by the model: the next block's first norm, if that block takes the
                                        # norm's finished output from the block before it (`ready`)
+    history: torch.Tensor | None = None  # float32 [runs + 1, T, E]: what every run has left so far, for blocks that
+                                       # average over depth (row 0: the embedded tokens)
+    depth: int = 0                     # how many rows of `history` are filled
+    next_front: tuple | None = None    # set by the model: (part, cache view) of the next block's `front_part`, if
+                                       # this block may run it (a step of one token per sequence)
     ready: tuple | None = None         # (norm, rows): the residual is up to date and `rows` are norm(residual)
 
 
@@ -137,6 +143,91 @@ class SandwichBlock(Block):
         rows = _post_add(last, stream.residual, y, ctx, then=after, mult=self.residual_mult)
         if after is not None:
             stream.ready = (after, rows)
+
+
+class PostNormBlock(Block):
+    """A norm on each sub-layer's output and none before it: the sub-layers read the stream itself.
+
+        h = x + conv(x) (`conv`, an `InputConv`; without one h = x);   y = x + Norm1(Mixer(h));   X = y + Norm2(FF(y))
+        x <- X, or with `average` (a `DepthAverage`) the average of X and what all runs before left
+
+    One kernel after each sub-layer (`ops.post_norm_stream`) norms its output, adds it to the float32 stream and leaves
+    the next reader's input: the feed-forward's, and after the last sub-layer the average; in steps of one token per
+    sequence it runs the NEXT block's convolution as well (`front_part`, `HiddenStream.next_front`).  A feed-forward
+    with a gate that is one product per row (`row_gate`) gets the products from that kernel too.
+
+    The convolution's kept rows and what the mixer keeps are entries of their own; another run may read the mixer's
+    entries (`readable_entries`) while the convolution's stay this run's."""
+
+    def __init__(self, mixer: Mixer, norm1: Norm, ffn: FeedForward | None = None, norm2: Norm | None = None, conv=None,
+                 average=None):
+        if (ffn is None) != (norm2 is None):
+            raise ValueError("a feed-forward comes with a norm after it")
+        self.conv, self.mixer, self.norm1, self.ffn, self.norm2, self.average = conv, mixer, norm1, ffn, norm2, average
+        self.cast = StreamCast(norm1.opts, norm1.width) if conv is None else None
+
+    def _conv_spec(self):
+        return self.conv.cache_spec() if self.conv is not None else None
+
+    def cache_specs(self) -> list:
+        own = self._conv_spec()
+        return ([own] if own is not None else []) + mixer_cache_specs(self.mixer)
+
+    def readable_entries(self) -> list[int]:
+        first = 1 if self._conv_spec() is not None else 0
+        return list(range(first, first + len(mixer_cache_specs(self.mixer))))
+
+    def _split(self, cache):
+        """(the convolution's view, the mixer's view or views) of what the model hands over."""
+        views = list(cache) if isinstance(cache, (list, tuple)) else ([] if cache is None else [cache])
+        own = views.pop(0) if self._conv_spec() is not None else None
+        return own, (views[0] if len(views) == 1 else (views or None))
+
+    def front_part(self, cache):
+        """(part, its cache view) that the kernel ending the block before may run in a step of one token per sequence."""
+        return (self.conv, self._split(cache)[0]) if self.conv is not None else None
+
+    def forward(self, stream: HiddenStream, ctx, cache, write_cache: bool = True) -> None:
+        stream.next_norm = stream.next_plain = None
+        front, stream.next_front = stream.next_front, None
+        ready, stream.ready = stream.ready, None
+        if stream.delta is not None or stream.owed is not None:
+            raise RuntimeError("a block whose sub-layers read the stream itself follows blocks that leave it complete")
+        kept, view = self._split(cache)
+        x = stream.residual
+        if ready is not None and ready[0] is self.conv:
+            h = ready[1]
+        elif self.conv is not None:
+            h = self.conv.forward(x, ctx, kept)
+        else:
+            h = self.cast.forward(x, None, n_rows=ctx.n_tokens)
+        y = self.mixer.forward(h, ctx, view, write_cache)
+        more: dict = {}              # what the kernel after the LAST sub-layer does besides
+        v = x
+        if self.average is not None:
+            if stream.history is None or stream.depth != self.average.earlier:
+                raise RuntimeError(f"an average over {self.average.earlier} earlier results, {stream.depth} are kept")
+            v = stream.history[stream.depth]
+            # the stream's own memory is free once the mixer's output has been added, unless it is the history's row 0
+            stream.residual = torch.empty_like(x) if stream.depth == 1 else x
+            more = {"history": stream.history, "n_history": stream.depth, "coef": self.average.coef,
+                    "avg_out": stream.residual}
+            stream.depth += 1
+        if front is not None and ctx.is_decode:
+            part, its_view = front
+            rows = torch.empty(x.shape, dtype=part.opts.dtype, device=x.device)
+            more.update(out=rows, conv=(part.weight, its_view.state if its_view is not None else None))
+            stream.ready = (part, rows)
+        if self.ffn is None:
+            ops.post_norm_stream(x, y, self.norm1.weight, self.norm1.eps, ctx, v_out=v, **more)
+            return
+        h = torch.empty(x.shape, dtype=self.norm1.opts.dtype, device=x.device)
+        gate = getattr(self.ffn, "row_gate", None)
+        gate = gate() if gate is not None else None
+        dots = torch.empty(x.shape[0], dtype=torch.float32, device=x.device) if gate is not None else None
+        ops.post_norm_stream(x, y, self.norm1.weight, self.norm1.eps, ctx, v_out=v, out=h, dot_weight=gate, dots=dots)
+        y = self.ffn.forward(h, ctx, gate_logits=dots) if gate is not None else self.ffn.forward(h, ctx)
+        ops.post_norm_stream(v, y, self.norm2.weight, self.norm2.eps, ctx, v_out=v, **more)
 
 
 def _post_add(post: Norm, residual, y, ctx, then: Norm | None = None, mult: float = 1.0):

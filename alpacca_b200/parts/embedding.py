@@ -1,7 +1,7 @@
-"""Token embedding (row gather, no scaling: alpacca/model.py:482; options: a constant factor, and a hashed table
-of (previous token, token) pairs whose row is added) and the
+"""Token embedding (row gather, no scaling: alpacca/model.py:482; options: a constant factor, a hashed table
+of (previous token, token) pairs whose row is added, and a table of learned positions) and the
 vocabulary head (logits = W . norm(x), alpacca/model.py:518; tied: the head is
-the embedding table itself, :320-322).  Logits are float32 in both precisions.
+the embedding table itself, :320-322; option: a bound on the logits).  Logits are float32 in both precisions.
 """
 from __future__ import annotations
 
@@ -31,12 +31,31 @@ class PairTable(Part):
         self.weight = fetch(self.own_param_specs()[0])
 
 
+class PositionTable(Part):
+    """A learned row per place in a sequence, added to the embedded token (not scaled with it)."""
+
+    def __init__(self, opts: BuildOptions, positions: int, width: int, name: str):
+        self.opts, self.positions, self.width, self.name = opts, int(positions), int(width), name
+        if opts.max_positions > self.positions:
+            raise ValueError(f"{name}: sequences of {opts.max_positions} tokens were asked for, the table has "
+                             f"{self.positions} rows")
+        self.weight = None
+
+    def own_param_specs(self):
+        return [ParamSpec(self.name, (self.positions, self.width), "matrix", "normal")]
+
+    def load_own(self, fetch):
+        self.weight = fetch(self.own_param_specs()[0])
+
+
 class TokenEmbedding(Part):
     def __init__(self, opts: BuildOptions, vocab: int, width: int, name: str, weight_suffix: str = ".weight",
-                 norm=None, scale: float = 1.0, pairs: "PairTable | None" = None):
+                 norm=None, scale: float = 1.0, pairs: "PairTable | None" = None,
+                 positions: "PositionTable | None" = None):
         """`norm`: a norm that the embedded rows pass before they become the stream (32-bit).  `scale`: a factor on
         the embedded row.  `pairs`: a `PairTable` whose row for (previous token, token) is added (not scaled); the
-        sequence's last token is then part of what it keeps from step to step (`cache_spec`)."""
+        sequence's last token is then part of what it keeps from step to step (`cache_spec`).  `positions`: a
+        `PositionTable` whose row for the token's place is added."""
         self.opts, self.vocab, self.width, self.name = opts, int(vocab), int(width), name
         self.weight_suffix = weight_suffix
         self.weight = None
@@ -44,6 +63,14 @@ class TokenEmbedding(Part):
         self.scale, self.pairs = float(scale), pairs
         if norm is not None and (pairs is not None or self.scale != 1.0):
             raise ValueError(f"{name}: a normed embedding has no factor and no pair table")
+        self.positions = positions
+        if positions is not None and (norm is not None or pairs is not None or self.scale != 1.0):
+            raise ValueError(f"{name}: an embedding with learned positions has no norm, factor or pair table")
+
+    @property
+    def needs_context(self) -> bool:
+        """Whether `forward` wants the step's context (places, sequences), not the token ids alone."""
+        return self.pairs is not None or self.scale != 1.0 or self.positions is not None
 
     def cache_spec(self):
         """What the embedding keeps per sequence: its last token, for the pair of the next step's first token."""
@@ -55,8 +82,14 @@ class TokenEmbedding(Part):
     def load_own(self, fetch):
         self.weight = fetch(self.own_param_specs()[0])
 
-    def forward(self, tokens: torch.Tensor, n_rows: int, ctx=None, cache=None) -> torch.Tensor:
-        out = torch.empty((n_rows, self.width), dtype=torch.float32, device=tokens.device)
+    def forward(self, tokens: torch.Tensor, n_rows: int, ctx=None, cache=None, out=None) -> torch.Tensor:
+        """float32 [n_rows, width]; `out`: where to put it."""
+        if out is None:
+            out = torch.empty((n_rows, self.width), dtype=torch.float32, device=tokens.device)
+        if self.positions is not None:
+            if ctx is None:
+                raise ValueError(f"{self.name}: the embedding needs the step's context")
+            return ops.embed_positions(self.weight, self.positions.weight, out, ctx)
         if self.pairs is not None or self.scale != 1.0:
             if ctx is None or (self.pairs is not None and cache is None):
                 raise ValueError(f"{self.name}: the embedding needs the step's context (and the sequences' last tokens)")
@@ -73,7 +106,11 @@ class TokenEmbedding(Part):
 
 class VocabHead(Part):
     def __init__(self, opts: BuildOptions, vocab: int, width: int, name: str,
-                 tied_to: TokenEmbedding | None = None, weight_suffix: str = ".weight"):
+                 tied_to: TokenEmbedding | None = None, weight_suffix: str = ".weight", softcap: float | None = None):
+        """`softcap` c: logits -> c * tanh(logits / c)."""
+        self.softcap = float(softcap) if softcap else 0.0
+        if self.softcap < 0:
+            raise ValueError(f"{name}: a bound on the logits must be positive, got {softcap}")
         self.opts, self.vocab, self.width, self.name = opts, int(vocab), int(width), name
         self.tied_to, self.weight_suffix = tied_to, weight_suffix
         self.proj = Linear(opts, width, [(name, vocab)], out_dtype=torch.float32, weight_suffix=weight_suffix)
@@ -92,4 +129,4 @@ class VocabHead(Part):
     def forward(self, h: torch.Tensor, n_rows: int | None = None) -> torch.Tensor:
         if self.tied_to is not None and self.proj.weight is not self.tied_to.weight:
             self.proj.share_weight(self.tied_to.weight)
-        return self.proj.forward(h, n_rows=n_rows)
+        return self.proj.forward(h, n_rows=n_rows, cap=self.softcap)

@@ -27,7 +27,7 @@ from __future__ import annotations
 import torch
 
 from .. import ops
-from ..weights.loader import ParamSpec
+from ..weights.loader import ParamSpec, WeightError
 from .base import BuildOptions, FeedForward
 
 
@@ -89,3 +89,77 @@ class RoutedExperts(FeedForward):
                                  renorm=self.renorm)
         out = torch.empty((h.shape[0], self.width), dtype=h.dtype, device=h.device)
         return ops.moe_experts(h, self.w_up, self.w_down, idx, wts, out, T, self.activation, gate_up=self.w_gate_up)
+
+
+class TableExperts(FeedForward):
+    """Gated experts that the token's id chooses: row token of a table [vocab, top] names a token's experts (all different),
+    each with weight 1 / top; there is no router.
+
+        out = sum_k E_(e_k)(h) / top + sigmoid(w_s . h) S(h),       E(h) = W_down (act(W_gate h) * (W_up h))
+
+    `shared_inner` > 0: the shared expert S, of that inner size, runs for every token; its gate is one number per token,
+    formed in 32-bit.  A block whose kernel has the stream's row in registers may form it there: `row_gate()` is the
+    vector w_s, and `forward` takes the products as `gate_logits`.
+
+    The matrices lie side by side (the experts' units, then the shared expert's), the inner sizes padded with zero units to
+    multiples of 8, so that few tokens read their experts' rows per (token, expert) pair together with the shared expert's
+    and many tokens run everything in two library products with the units of experts that were not chosen set to zero
+    (csrc/moe.cu).  The table is read by the kernels: routing never reaches the host."""
+
+    def __init__(self, opts: BuildOptions, width: int, inner: int, n_experts: int, top: int, vocab: int, prefix: str,
+                 activation: str = "silu", shared_inner: int = 0, table_name: str = "table",
+                 expert_names=("e{}.gate", "e{}.up", "e{}.down"), shared_names=("shared.gate", "shared.up", "shared.down"),
+                 shared_gate: str = "shared.sg", out_dtype=None):
+        if activation not in ops.MOE_ACTIVATIONS:
+            raise ValueError(f"activation must be one of {tuple(ops.MOE_ACTIVATIONS)}, got {activation!r}")
+        if not 0 < top <= n_experts:
+            raise ValueError(f"{prefix}: {top} of {n_experts} experts cannot be chosen")
+        self.opts, self.width, self.inner, self.E, self.top = opts, int(width), int(inner), int(n_experts), int(top)
+        self.vocab, self.prefix, self.activation, self.shared_inner = int(vocab), prefix, activation, int(shared_inner)
+        self.table_name, self.expert_names, self.shared_names, self.shared_gate = table_name, expert_names, shared_names, shared_gate
+        self.out_dtype = out_dtype or opts.dtype
+        self.ff, self.fs = -(-self.inner // 8) * 8, -(-self.shared_inner // 8) * 8
+        self.table = self.gate_up = self.down = self.w_sg = None
+
+    def own_param_specs(self):
+        p = self.prefix
+        specs = [ParamSpec(f"{p}.{self.table_name}", (self.vocab, self.top), "int", f"choice:{self.E}")]
+        gate, up, down = self.expert_names
+        for e in range(self.E):
+            specs += [ParamSpec(f"{p}.{gate.format(e)}", (self.inner, self.width)),
+                      ParamSpec(f"{p}.{up.format(e)}", (self.inner, self.width)),
+                      ParamSpec(f"{p}.{down.format(e)}", (self.width, self.inner))]
+        if self.shared_inner:
+            gate, up, down = self.shared_names
+            specs += [ParamSpec(f"{p}.{gate}", (self.shared_inner, self.width)),
+                      ParamSpec(f"{p}.{up}", (self.shared_inner, self.width)),
+                      ParamSpec(f"{p}.{down}", (self.width, self.shared_inner)),
+                      ParamSpec(f"{p}.{self.shared_gate}", (1, self.width), "vector")]
+        return specs
+
+    def load_own(self, fetch):
+        specs = self.own_param_specs()
+        self.table = fetch(specs[0])
+        if int(self.table.min()) < 0 or int(self.table.max()) >= self.E:
+            raise WeightError(f"{specs[0].name} names experts outside 0..{self.E - 1}")
+        C = self.E * self.ff + self.fs
+        for i in range(self.E + (1 if self.shared_inner else 0)):
+            g, u, d = (fetch(s) for s in specs[1 + 3 * i:4 + 3 * i])
+            if self.gate_up is None:
+                self.gate_up = torch.zeros((2, C, self.width), dtype=g.dtype, device=g.device)
+                self.down = torch.zeros((self.width, C), dtype=g.dtype, device=g.device)
+            at, n = i * self.ff, g.shape[0]
+            self.gate_up[0, at:at + n], self.gate_up[1, at:at + n], self.down[:, at:at + n] = g, u, d
+        if self.shared_inner:
+            self.w_sg = fetch(specs[-1]).reshape(-1).contiguous()
+
+    def row_gate(self):
+        """The vector (float32 [width]) whose product with this part's input is the shared expert's gate logit."""
+        return self.w_sg
+
+    def forward(self, h, ctx, gate_logits=None):
+        if self.shared_inner and gate_logits is None:
+            gate_logits = ops.row_dots(h, self.w_sg, ctx.n_tokens)
+        out = torch.empty((h.shape[0], self.width), dtype=self.out_dtype, device=h.device)
+        return ops.moe_shared_experts(h, self.gate_up, self.down, self.E, self.ff, self.fs, self.top, out, ctx,
+                                      activation=self.activation, table=self.table, gate_logits=gate_logits)

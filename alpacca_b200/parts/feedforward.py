@@ -38,3 +38,22 @@ class SwiGLU(FeedForward):
         T = ctx.n_tokens
         act = self.gate_up.forward_swiglu(h, n_rows=T, activation=self.activation)
         return self.down.forward(act, n_rows=T, then=then)
+
+
+class PlainFeedForward(FeedForward):
+    """Two matrices and no gate: out = W_down act(W_up h); `activation` "gelu" is the erf form.  An inner width that is no
+    multiple of 8 is padded with zero rows when the weights are loaded (act(0) = 0)."""
+
+    def __init__(self, opts: BuildOptions, width: int, inner: int, prefix: str, names=("up", "down"),
+                 weight_suffix: str = "", out_dtype=None, activation: str = "gelu"):
+        if activation is None or activation not in ops.PLAIN_ACTIVATIONS:
+            raise ValueError(f"activation {activation!r} is not one of {[a for a in ops.PLAIN_ACTIVATIONS if a]}")
+        self.opts, self.width, self.inner, self.activation = opts, int(width), int(inner), activation
+        up, down = names
+        self.up = Linear(opts, width, [(f"{prefix}.{up}", inner)], weight_suffix=weight_suffix, pad_rows_to=8)
+        self.down = Linear(opts, inner, [(f"{prefix}.{down}", width)], weight_suffix=weight_suffix, out_dtype=out_dtype,
+                           pad_in_to=8)
+
+    def forward(self, h, ctx):
+        T = ctx.n_tokens
+        return self.down.forward(self.up.forward(h, n_rows=T, act=self.activation), n_rows=T)

@@ -89,12 +89,14 @@ class Linear(Part):
         return (self.opts.dtype == torch.bfloat16 and self.weight is not None
                 and ops.owed_norm_pays(n_rows, self.out_features, self.in_features, self.weight.device))
 
-    def forward(self, x, n_rows: int | None = None, start_early: bool = True, then=None, with_bias: bool = True):
+    def forward(self, x, n_rows: int | None = None, start_early: bool = True, then=None, with_bias: bool = True,
+                act: str | None = None, cap: float = 0.0):
         """`start_early` off: the product's kernel may not start before the kernel before it has ended
         (see `ops.gemv_bf16`).  `x` may be an `OwedNorm` (the division by the rms is applied to the
         sums).  `then` = (residual, norm): where the step has few enough rows, the result is added to
         the residual here and an `OwedNorm` for `norm` is returned instead of the result.  `with_bias` off: the
-        caller adds `self.bias` itself (in a kernel that touches the result anyway)."""
+        caller adds `self.bias` itself (in a kernel that touches the result anyway).  `act` ("gelu"): an activation
+        on the result; `cap` > 0: float32 results are bounded, cap * tanh(y / cap)."""
         n = x.shape[0] if n_rows is None else n_rows
         owed = None
         if isinstance(x, OwedNorm):
@@ -112,8 +114,10 @@ class Linear(Part):
         bias = self.bias if with_bias else None
         if x.dtype == torch.float32:
             ops.gemm_f32(x, self.weight, out, bias=bias, n_rows=n)
-            return out
-        return ops.linear_bf16(x, self.weight, out, n_rows=n, bias=bias, start_early=start_early, owed=owed)
+            if act is not None:
+                ops.plain_act(out, act, n_rows=n)
+            return ops.softcap(out, cap, n_rows=n) if cap else out
+        return ops.linear_bf16(x, self.weight, out, n_rows=n, bias=bias, start_early=start_early, owed=owed, act=act, cap=cap)
 
     def forward_swiglu(self, x, n_rows: int | None = None, activation: str = "silu") -> torch.Tensor:
         """act(gate) * up of the interleaved gate|up product, [M, out_features / 2] (`activation`: "silu",

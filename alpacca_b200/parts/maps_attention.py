@@ -29,6 +29,16 @@ Options, each a constructor argument:
     head_gate        every head's output is multiplied by sigmoid(W_g h)_h, ONE number per head and token (tensor
                      `<prefix>.<head_gate>` [H, width]), before W_o; its rows ride in the projections' product
 
+    qk_norm_rows     with qk_norm: ONE root mean square over all query vectors of a token together and one over all its key
+                     vectors, with weights of those sizes (tensors `<prefix>.<q>.norm` [H*M*dim], `<prefix>.<k>.norm`)
+    distance         names of two tensors [H], r1 and r2: r1_h ln(1 + r2_h (p - s)) is taken off each scaled score (Chi et
+                     al., "KERPLE: Kernelized Relative Positional Embedding for Length Extrapolation")
+    own_kv           off: the layer has no W_k and W_v (nor a key norm); it reads the keys, as cached, and values of another
+                     layer with the same key/value heads and sizes (the schedule's run names that layer's run), with its
+                     own queries, window and penalty
+    keep_window      what the cache keeps, where it must be more than this layer reads because another layer reads it with
+                     a window of its own ("all": everything); None: the window
+
 The rotation turns the first n_rot dims of every query and key vector (each map by itself).  In bfloat16 with key
 and value sizes in steps of 16, prompts and decode steps run on the tensor-core kernels of csrc/attention_mma.cu
 (several maps leave their outputs in float32, which one more kernel combines); everything else runs
@@ -53,7 +63,8 @@ class MapsAttention(Mixer):
                  sink: bool = False, difference: float | None = None, names=("q", "k", "v", "o"),
                  weight_suffix: str = "", bias_suffix: str = ".b", out_dtype=None, qk_norm_weight: bool = True,
                  value_norm: bool = False, head_mix: str | None = None, gate: str | None = None,
-                 head_gate: str | None = None):
+                 head_gate: str | None = None, qk_norm_rows: bool = False, distance: tuple | None = None,
+                 own_kv: bool = True, keep_window: int | str | None = None):
         if n_heads % n_kv_heads:
             raise ValueError(f"{prefix}: {n_heads} heads cannot share {n_kv_heads} key/value heads")
         self.opts, self.prefix = opts, prefix
@@ -81,16 +92,31 @@ class MapsAttention(Mixer):
             if self.G * self.Dv > ops.talk_max_row():
                 raise ValueError(f"{prefix}: {self.G} value heads of {self.Dv} are more than {ops.talk_max_row()} numbers per token")
         self.window = int(window) if window else None
+        self.own_kv, self.qk_norm_rows, self.distance = bool(own_kv), bool(qk_norm_rows), distance
+        if self.window is None or keep_window == "all":
+            self.keep_window = None            # a layer that reads everything keeps everything
+        else:
+            self.keep_window = int(keep_window) if keep_window else self.window
+            if self.keep_window < self.window:
+                raise ValueError(f"{prefix}: the cache keeps {self.keep_window} tokens, the window reads {self.window}")
+        if self.qk_norm_rows and not (qk_norm and qk_norm_weight and head_mix is None and not value_norm):
+            raise ValueError(f"{prefix}: a norm over whole rows is a query/key norm with weights, without mixed heads")
+        if not self.own_kv and not (self.qk_norm_rows and head_mix is None and not self.values_are_keys and not bias):
+            raise ValueError(f"{prefix}: a layer that reads another layer's keys has a query norm over whole rows")
+        if distance is not None and head_mix is not None:
+            raise ValueError(f"{prefix}: a penalty on distance does not go with mixed heads")
         self.scale, self.eps = float(scale), float(eps)
         self.position, self.qk_norm, self.has_sink = position, bool(qk_norm), bool(sink)
         self.difference = None if difference is None else float(difference)
         q, k, v, o = names
         self.names = names
         n_q, n_k = self.H * self.M * self.Dk, self.G * self.M * self.Dk
-        sources = [(f"{prefix}.{q}", n_q), (f"{prefix}.{k}", n_k)]
-        if not self.values_are_keys:
-            sources.append((f"{prefix}.{v}", self.G * self.Dv))
-        self.offsets = (0, n_q, n_q if self.values_are_keys else n_q + n_k)
+        sources = [(f"{prefix}.{q}", n_q)]
+        if self.own_kv:
+            sources.append((f"{prefix}.{k}", n_k))
+            if not self.values_are_keys:
+                sources.append((f"{prefix}.{v}", self.G * self.Dv))
+        self.offsets = (0, n_q, n_q if self.values_are_keys else n_q + n_k) if self.own_kv else (0, 0, 0)
         self.gate_offset = None
         if gate is not None:
             self.gate_offset = sum(r for _, r in sources)
@@ -108,7 +134,7 @@ class MapsAttention(Mixer):
             self.gate_offset = sum(r for _, r in self.qkv.sources[:-1])
         self.out = Linear(opts, self.H * self.Dv, [(f"{prefix}.{o}", width)], weight_suffix=weight_suffix,
                           out_dtype=out_dtype)
-        self.q_weight = self.k_weight = self.sink = self.talk = None
+        self.q_weight = self.k_weight = self.sink = self.talk = self.penalty = None
         self.coef = 0.0
 
     def own_param_specs(self):
@@ -117,12 +143,18 @@ class MapsAttention(Mixer):
         if self.difference is not None:
             specs += [ParamSpec(f"{p}.{n}", (self.Dk,), "vector", "normal") for n in ("lq1", "lk1", "lq2", "lk2")]
         if self.qk_norm and self.qk_norm_weight:
-            specs += [ParamSpec(f"{p}.{q}.norm", (self.Dk,), "vector", "one_plus_normal"),
-                      ParamSpec(f"{p}.{k}.norm", (self.Dk,), "vector", "one_plus_normal")]
+            whole = self.qk_norm_rows
+            specs.append(ParamSpec(f"{p}.{q}.norm", (self.H * self.M * self.Dk if whole else self.Dk,), "vector",
+                                   "one_plus_normal"))
+            if self.own_kv:
+                specs.append(ParamSpec(f"{p}.{k}.norm", (self.G * self.M * self.Dk if whole else self.Dk,), "vector",
+                                       "one_plus_normal"))
         if self.head_mix is not None:
             specs.append(ParamSpec(f"{p}.{self.head_mix}", (self.H, self.H), "vector", "normal"))
         if self.has_sink:
             specs.append(ParamSpec(f"{p}.sink", (self.H,), "vector", "normal"))
+        if self.distance is not None:
+            specs += [ParamSpec(f"{p}.{n}", (self.H,), "vector", "positive") for n in self.distance]
         return specs
 
     def load_own(self, fetch):
@@ -133,13 +165,15 @@ class MapsAttention(Mixer):
                    + self.difference)
             self.coef = -lam
         if self.qk_norm and self.qk_norm_weight:
-            self.q_weight, self.k_weight = got[f"{self.names[0]}.norm"], got[f"{self.names[1]}.norm"]
+            self.q_weight, self.k_weight = got[f"{self.names[0]}.norm"], got.get(f"{self.names[1]}.norm")
         elif self.qk_norm:
             self.q_weight = self.k_weight = torch.ones(self.Dk, dtype=torch.float32, device=self.opts.device)
         if self.head_mix is not None:
             self.talk = got[self.head_mix].contiguous()
         if self.has_sink:
             self.sink = got["sink"]
+        if self.distance is not None:
+            self.penalty = torch.stack([got[n] for n in self.distance]).contiguous()
 
     def load(self, fetch):
         super().load(fetch)
@@ -154,8 +188,8 @@ class MapsAttention(Mixer):
 
     def cache_spec(self):
         if self.head_mix is not None:       # a token's value heads side by side in one row
-            return KVSpec(self.G, self.Dk, self.window, value_heads=1, value_dim=self.G * self.Dv)
-        return KVSpec(self.G * self.M, self.Dk, self.window, value_heads=self.G, value_dim=self.Dv)
+            return KVSpec(self.G, self.Dk, self.keep_window, value_heads=1, value_dim=self.G * self.Dv)
+        return KVSpec(self.G * self.M, self.Dk, self.keep_window, value_heads=self.G, value_dim=self.Dv)
 
     def _on_tensor_cores(self, buf) -> bool:
         return ops.attention_maps_mma_supports(self.H, self.G, self.M, self.Dk, self.Dv, buf.shape[-1], buf.dtype)
@@ -168,11 +202,14 @@ class MapsAttention(Mixer):
         # touches every projected value anyway; few rows and the 32-bit path add it in the product
         later = self.qkv.bias is not None and h.dtype == torch.bfloat16 and T > ops.GEMV_NARROW_MAX_ROWS
         buf = self.qkv.forward(h, n_rows=T, with_bias=not later)
+        if write_cache and not self.own_kv:
+            raise ValueError(f"{self.prefix}: a layer without W_k and W_v writes no cache; its run reads another run's")
         rot = self.position.rotation() if self.position is not None else None
         ops.attention_prepare(buf, self.offsets, self.H, self.G, self.M, self.Dk, self.Dv, cache, ctx,
                               q_weight=self.q_weight, k_weight=self.k_weight, eps=self.eps, rot=rot,
                               write_cache=write_cache, bias=self.qkv.bias if later else None,
-                              v_norm=self.value_norm, v_side_by_side=self.head_mix is not None)
+                              v_norm=self.value_norm, v_side_by_side=self.head_mix is not None,
+                              norm_rows=self.qk_norm_rows)
         att = torch.empty((buf.shape[0], self.H * self.Dv), dtype=buf.dtype, device=buf.device)
         if self.head_mix is not None:
             gate_rows = buf.reshape(-1)[self.gate_offset:] if self.gate_offset is not None else None
@@ -184,7 +221,7 @@ class MapsAttention(Mixer):
         attend = ops.attention_maps_mma if self._on_tensor_cores(buf) else ops.attention_maps
         attend(buf, buf.shape[-1], att, cache, ctx, self.H, self.G, self.M, self.Dk, self.Dv, self.scale,
                self.window or 0, self.sink, coef=self.coef, unit_norm=unit, eps=self.eps,
-               out_scale=(1.0 - self.difference) if unit else 1.0)
+               out_scale=(1.0 - self.difference) if unit else 1.0, dist=self.penalty)
         if self.head_gate is not None:
             ops.head_gate(att, buf.reshape(-1)[self.gate_offset:], buf.shape[-1], T, self.H, self.Dv)
         # after a kernel that fills the processors' shared memory the product starts when that kernel has ended

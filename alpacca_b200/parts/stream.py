@@ -11,6 +11,12 @@
                weight is 1 and whose division nobody owes: in a step of a few rows the product before it adds its
                result to the stream and leaves bf16(stream) behind (the skinny product's residual tail), and the
                kernel that casts the stream is not launched.
+`InputConv`    what a mixer reads is the stream plus a causal convolution of it over time, channel by channel:
+               h_t = x_t + sum_j w[:, j] x_(t - taps + 1 + j), zeros before the sequence's start.  The last taps - 1 rows
+               of x (float32) are part of a sequence's state.
+`DepthAverage` what a layer hands on: x = sum_(j <= n) c_j X_j with X_0 the embedded tokens, X_j the result of run j
+               before this average, and one learned coefficient per j (Pagliardini et al., "DenseFormer: Enhancing
+               Information Flow in Transformers via Depth Weighted Averaging").
 """
 from __future__ import annotations
 
@@ -18,7 +24,7 @@ import torch
 
 from .. import ops
 from ..weights.loader import ParamSpec
-from .base import BuildOptions, Norm, Part
+from .base import BuildOptions, Norm, Part, StateSpec
 from .linear import Linear
 
 
@@ -39,6 +45,42 @@ class StreamCast(Norm):
         if out is None:
             out = torch.empty(residual.shape, dtype=self.opts.dtype, device=residual.device)
         return ops.stream_cast(residual, delta, out, n_rows=n_rows)
+
+
+class InputConv(Part):
+    def __init__(self, opts: BuildOptions, width: int, taps: int, name: str):
+        self.opts, self.width, self.taps, self.name = opts, int(width), int(taps), name
+        if self.taps < 1:
+            raise ValueError(f"{name}: a convolution over {taps} tokens")
+        self.weight = None
+
+    def own_param_specs(self):
+        return [ParamSpec(self.name, (self.width, self.taps), "vector", "normal")]
+
+    def load_own(self, fetch):
+        self.weight = fetch(self.own_param_specs()[0]).t().contiguous()      # [taps, width]: what the kernels read
+
+    def cache_spec(self):
+        return StateSpec((self.taps - 1, self.width), torch.float32) if self.taps > 1 else None
+
+    def forward(self, residual, ctx, cache, write_state: bool = True):
+        out = torch.empty(residual.shape, dtype=self.opts.dtype, device=residual.device)
+        return ops.input_conv(residual, self.weight, cache.state if cache is not None else None, out, ctx,
+                              write_state=write_state)
+
+
+class DepthAverage(Part):
+    """`earlier`: how many results come before the layer's own (the embedding output and the earlier layers')."""
+
+    def __init__(self, opts: BuildOptions, earlier: int, name: str):
+        self.opts, self.earlier, self.name = opts, int(earlier), name
+        self.coef = None
+
+    def own_param_specs(self):
+        return [ParamSpec(self.name, (self.earlier + 1,), "vector", "last_one")]
+
+    def load_own(self, fetch):
+        self.coef = fetch(self.own_param_specs()[0])
 
 
 class PassOffset(Part):

@@ -28,7 +28,9 @@ class ParamSpec:
     name: str                 # full tensor name in the checkpoint
     shape: tuple
     role: str = "matrix"      # "matrix" | "vector" | "int" | "keep32"
-    init: str = "normal"      # random-weights mode: "normal" | "one_plus_normal" | "zeros"
+    init: str = "normal"      # random-weights mode: "normal" | "one_plus_normal" | "zeros" | "positive" (|normal|) |
+                              # "last_one" (normal, the last number near 1) | "choice:<n>" (integers: every row holds
+                              # different numbers below n)
     absent: bool = False      # declared but not stored (a tied head): must NOT be in the source
 
 

@@ -88,6 +88,9 @@ class RandomSource:
         g = torch.Generator(device=self.device)
         g.manual_seed(_name_seed(self.seed, name))
         if spec.role == "int":
+            if spec.init.startswith("choice:"):
+                order = torch.rand((spec.shape[0], int(spec.init.split(":")[1])), generator=g, device=self.device)
+                return order.argsort(dim=1)[:, :spec.shape[1]].to(torch.int32).contiguous()
             return torch.zeros(spec.shape, dtype=torch.int32, device=self.device)
         if spec.init == "zeros":
             t = torch.zeros(spec.shape, dtype=torch.float32, device=self.device)
@@ -95,6 +98,10 @@ class RandomSource:
             t = torch.randn(spec.shape, generator=g, dtype=torch.float32, device=self.device) * self.std
             if spec.init == "one_plus_normal":
                 t += 1.0
+            elif spec.init == "positive":
+                t = t.abs()
+            elif spec.init == "last_one":
+                t[-1] += 1.0
         return t.to(self._stored_dtype(spec))
 
     def close(self):
