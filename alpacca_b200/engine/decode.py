@@ -339,6 +339,20 @@ class GraphDecoder:
         done.record()
         return {"live": list(live), "rows": rows, "done": done, "host": host}
 
+    def _adopt(self, live) -> bool:
+        """Whether the next step in flight is the one the caller asks for, apart from sequences that it has ended since
+        (a stop token): their rows are then simply not read.  Nothing is taken back, so this serves models that keep a
+        state, which has no earlier value, as well."""
+        flight = self._flights[0]
+        have = {(slot, tok): (i, st) for i, (slot, tok, st) in enumerate(flight["live"])}
+        found = [have.get((slot, tok)) for slot, tok, _ in live]
+        if len(self._flights) != 1 or any(f is None or f[1] is not st for f, (_, _, st) in zip(found, live)):
+            return False
+        flight["live"] = list(live)
+        flight["rows"] = [flight["rows"][i] for i, _ in found]
+        self._last_slots = None          # the next launch masks the ended sequences' rows
+        return True
+
     def _drop_flights(self, live):
         """Gives up the steps that ran ahead for sequences the caller did not bring back: their tokens
         are dropped, the lengths they were counted with are taken back, the device state is uploaded
@@ -348,6 +362,9 @@ class GraphDecoder:
         # a sequence is known by its sampler state: one that the caller still brings has the steps
         # that ran ahead in its length; one that is gone has given its slot back
         here = {id(st) for _, _, st in live}
+        if self.engine.cache.state_groups and any(id(st) in here for f in flights for _, _, st in f["live"]):
+            raise RuntimeError("a step that ran ahead cannot be taken back for a model that keeps a state of fixed size: the "
+                               "caller comes back with the forecast sequences and tokens, less those that have ended")
         for f in flights:
             self.engine.cache.commit([(slot, -1) for slot, _, st in f["live"] if id(st) in here])
         sampler = self.sampler
@@ -368,10 +385,11 @@ class GraphDecoder:
         that the device never waits for the host: the next step of all sequences that have room for
         one is enqueued before this step's tokens are even known (it feeds on the tokens on the
         device), provided that needs nothing from the host but the replay.  If one of them then
-        samples a stop token, the caller comes back without it, and the step that ran ahead is given
-        up: one step's worth of device time for each sequence end by a stop token."""
+        samples a stop token, the caller comes back without it, and the step that ran ahead serves the
+        others (`_adopt`).  A caller that comes back with anything else makes the decoder give the step up."""
         q = self._flights
-        if q and [(slot, tok) for slot, tok, _ in q[0]["live"]] != [(slot, tok) for slot, tok, _ in live]:
+        if (q and [(slot, tok) for slot, tok, _ in q[0]["live"]] != [(slot, tok) for slot, tok, _ in live]
+                and not self._adopt(live)):
             self._drop_flights(live)
             q = self._flights
         if not q:
