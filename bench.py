@@ -41,6 +41,10 @@ layer reading another's cache; attention with a sink beside the gated delta rule
 scores in every layer; layer norms around every sub-layer), beside the Sazepel decoder (the closest: recurrent mixers,
 two mixers side by side, routed gated experts of the same sizes, norms around every sub-layer), the Lefatar decoder
 (the same latent-attention kernels) and the Llama decoder.
+`--design ponusun` does the same for the Ponusun decoder (attention with a window and a penalty on distance, every second
+layer reading the keys of the layer before; experts chosen by token id beside a shared one; norms on the sub-layers'
+outputs, an input convolution and an average over depth in every layer), beside the Sazepel decoder (routed gated
+experts of the same sizes), the Buguzen decoder (attention with a window and a query/key norm) and the Llama decoder.
 
 One JSON line goes to standard output.  With --gpus N > 1 it prints a line that says so and exits
 with 2: this library runs on one GPU.
@@ -547,7 +551,7 @@ def run_reference(args):
 
 
 # ---------------------------------------------------------------------------------------------------------
-# --design lefatar | buguzen | sazepel | mavidra: that decoder beside the Llama decoder of the same width, depth and dense
+# --design lefatar | buguzen | sazepel | mavidra | ponusun: that decoder beside the Llama decoder of the same width, depth and dense
 # feed-forward, at sizes that resemble a real model's layers (random weights).
 
 def _lefatar_layers(E, mlstm, latent, dense_ff, moe, n_layers):
@@ -649,6 +653,25 @@ def _mavidra_config(z):
             "layers": layers[:z["layers"]]}
 
 
+def _ponusun_config(z):
+    """Eight layers of attention with a window, every second one reading the keys of the layer before with half the window;
+    a dense feed-forward in the first layer, then experts of the size of the other decoders' beside a shared one of twice
+    that size."""
+    rt = z["moe"]["router"]
+    ff = z["moe"]["expert"]["ff"]
+    moe = {"kind": "moe", "expert": {"ff": ff}, "router": {"experts": rt["experts"], "top": rt["top"]}, "shared": {"ff": 2 * ff}}
+    window = z["buguzen"]["window"]
+    layers = []
+    for i in range(z["layers"]):
+        mx = {"heads": z["heads"], "kv_heads": z["kv_heads"], "dim": z["head_dim"], "vdim": z["head_dim"],
+              "scale": z["head_dim"] ** -0.5, "mask": {"size": window if i % 2 == 0 else window // 2}}
+        if i % 2:
+            mx["kv_from"] = i - 1
+        layers.append({"type": "attention", "mixer": mx, "mlp": moe if i else {"kind": "dense", "ff": z["dense_ff"]}})
+    return {"architecture": "Ponusun", "vocab": z["vocab"], "width": z["width"], "max_positions": 8192, "norm": {"eps": 1e-6},
+            "canon": {"taps": 4}, "logit_softcap": 30.0, "layers": layers}
+
+
 def design_configs(size, design="lefatar"):
     z = DESIGN_SIZES[size]
     llama = {"architectures": ["LlamaForCausalLM"], "num_hidden_layers": z["layers"], "hidden_size": z["width"],
@@ -664,6 +687,8 @@ def design_configs(size, design="lefatar"):
         return {"sazepel": _sazepel_config(z), "lefatar": lefatar, "llama": llama}
     if design == "mavidra":
         return {"mavidra": _mavidra_config(z), "sazepel": _sazepel_config(z), "lefatar": lefatar, "llama": llama}
+    if design == "ponusun":
+        return {"ponusun": _ponusun_config(z), "sazepel": _sazepel_config(z), "buguzen": _buguzen_config(z), "llama": llama}
     return {"lefatar": lefatar, "llama": llama}
 
 
@@ -744,7 +769,7 @@ def main():
                     help="with --only decode: equal prompts of this many tokens instead of the workload's")
     ap.add_argument("--prefill-tokens", type=int, default=0,
                     help="with --only prefill: one prompt of this many tokens instead of the workload's")
-    ap.add_argument("--design", default="", choices=["", "lefatar", "buguzen", "sazepel", "mavidra"],
+    ap.add_argument("--design", default="", choices=["", "lefatar", "buguzen", "sazepel", "mavidra", "ponusun"],
                     help="instead of the benchmark workload: prefill and decode throughput of this design beside the "
                          "Llama decoder of the same width and depth (random weights), one JSON line")
     ap.add_argument("--size", default="", choices=[""] + sorted(DESIGN_SIZES), help="with --design: one size only")
