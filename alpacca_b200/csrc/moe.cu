@@ -12,6 +12,7 @@
 // weights stream from memory once and every token adds its experts in the order of its choices.
 #include "common.cuh"
 #include "launch.cuh"
+#include "moe_choice.cuh"
 
 #define MOE_MAX_EXPERTS 1024
 
@@ -317,8 +318,6 @@ AB_API int ab_moe_route_scores(const void* h, int dtype, int ld, const float* wr
   return ab_launch_status();
 }
 
-__device__ __forceinline__ float gelu_erf(float z) { return 0.5f * z * (1.0f + erff(z * 0.70710678118654752440f)); }
-__device__ __forceinline__ float silu(float z) { return z / (1.0f + expf(-z)); }
 
 // act[p, j] = f(W_up[e_p][j] . h[t_p]) for pair p = t * top + k, or, gated (w_gate given),
 // f(W_gate[e_p][j] . h[t_p]) * (W_up[e_p][j] . h[t_p]).  One warp per (pair, j).
@@ -492,24 +491,13 @@ AB_API int ab_moe_weigh_all(void* up, int dtype, const int* idx, const float* wt
 //   y_t = sum_k weight_k W_down[e_k] (silu(W_gate[e_k] h_t) * (W_up[e_k] h_t))
 //         + sigmoid(z_t) W_down_s (silu(W_gate_s h_t) * (W_up_s h_t))               (if there is a shared expert)
 //
-// The choice comes from a router (`idx`, `wts`) or from the token's id: row token_t of a table [vocab, top] names its
-// experts, each with the same constant weight.  The matrices lie together: gate_up [2, C, width] with C = E * ff + fs
-// (the gates of all experts, then the shared expert's; then the up-projections likewise), down [width, C].
+// The choice comes from a router (`idx`, `wts`) or from the token's id: a row of a table names its experts, each with the
+// same constant weight (moe_choice.cuh).  The matrices lie together, C = E * ff + fs units (the experts' one after another,
+// then the shared expert's; ff and fs multiples of 8): gate_up [2 C, width] in groups of 16 rows, the gates of 8 units and
+// then their up-projections, and down [width, C].
 // z [T] are the shared expert's gate logits (float32, formed elsewhere).
+// The kernels here take any width and the 32-bit path; bfloat16 steps of a few tokens run csrc/moe_gemv.cu.
 // ---------------------------------------------------------------------------
-struct Choice {
-  const int* idx; const float* wts;       // [T, top], from a router
-  const int* table; const int* tokens;    // [vocab, top], [T]: by token id (idx null)
-  float weight;                           // of every expert chosen by table
-};
-__device__ __forceinline__ int chosen_expert(const Choice& c, int t, int k, int top) {
-  return c.idx != nullptr ? c.idx[(size_t)t * top + k] : c.table[(size_t)c.tokens[t] * top + k];
-}
-__device__ __forceinline__ float chosen_weight(const Choice& c, int t, int k, int top) {
-  return c.idx != nullptr ? c.wts[(size_t)t * top + k] : c.weight;
-}
-__device__ __forceinline__ float activate(float z, int kind) { return kind == 0 ? gelu_erf(z) : silu(z); }
-
 __device__ __forceinline__ void fma8(float& part, uint4 x, uint4 y) {
   const uint32_t a[4] = {x.x, x.y, x.z, x.w}, b[4] = {y.x, y.y, y.z, y.w};
 #pragma unroll
@@ -570,10 +558,9 @@ moe_shared_up_kernel(const T* __restrict__ h, int ld, const T* __restrict__ gate
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   pdl_wait();
   pdl_trigger();
-  const size_t C = (size_t)E * ff + fs;
   const int row_len = top * ff + fs;
   int t;
-  size_t row, dst;
+  size_t unit, dst;
   long long blk = blockIdx.x;
   if (blk < pair_blocks) {
     const long long group = blk / ff;
@@ -582,18 +569,19 @@ moe_shared_up_kernel(const T* __restrict__ h, int ld, const T* __restrict__ gate
     if (p >= (long long)n_tokens * top) return;
     t = (int)(p / top);
     const int k = (int)(p - (long long)t * top);
-    row = (size_t)chosen_expert(c, t, k, top) * ff + j;
+    unit = (size_t)chosen_expert(c, t, k, top) * ff + j;
     dst = (size_t)t * row_len + (size_t)k * ff + j;
   } else {
     blk -= pair_blocks;
     const int chunk = (int)(blk / fs), j = (int)(blk - (long long)chunk * fs);
     t = chunk * 8 + warp;
     if (t >= n_tokens) return;
-    row = (size_t)E * ff + j;
+    unit = (size_t)E * ff + j;
     dst = (size_t)t * row_len + (size_t)top * ff + j;
   }
+  const T* gate = gate_up + ((unit >> 3) * 16 + (unit & 7)) * width;
   float pg, pu;
-  lane_dot2(h + (size_t)t * ld, gate_up + row * width, gate_up + (C + row) * width, width, lane, pg, pu);
+  lane_dot2(h + (size_t)t * ld, gate, gate + (size_t)8 * width, width, lane, pg, pu);
   pg = warp_sum(pg);
   pu = warp_sum(pu);
   if (lane == 0) act[dst] = from_f32<T>(activate(pg, activation) * pu);
@@ -628,8 +616,6 @@ moe_shared_down_kernel(const T* __restrict__ act, const T* __restrict__ down, Ch
   if (lane == 0) out[(size_t)t * width + i] = from_f32<TO>(total);
 }
 
-static bool choice_ok(const Choice& c) { return c.idx ? c.wts != nullptr : (c.table != nullptr && c.tokens != nullptr); }
-
 // act: scratch [n_tokens, top * ff + fs] of `dtype`; out of `out_dtype`.
 AB_API int ab_moe_shared_pairs(const void* h, int dtype, int ld, const void* gate_up, const void* down, const int* idx,
                                const float* wts, const int* table, const int* tokens, float weight, const float* z, void* act,
@@ -637,7 +623,7 @@ AB_API int ab_moe_shared_pairs(const void* h, int dtype, int ld, const void* gat
                                int activation, cudaStream_t stream) {
   if (n_tokens <= 0) return AB_OK;
   const Choice c{idx, wts, table, tokens, weight};
-  if (top <= 0 || width <= 0 || ff <= 0 || fs < 0 || E <= 0 || (activation != 0 && activation != 1) || !choice_ok(c) ||
+  if (top <= 0 || width <= 0 || ff <= 0 || ff % 8 || fs < 0 || fs % 8 || E <= 0 || (activation != 0 && activation != 1) || !choice_ok(c) ||
       (fs > 0 && !z))
     return AB_BAD_ARG;
   const long long pair_blocks = ((long long)n_tokens * top + 7) / 8 * ff;
@@ -659,16 +645,15 @@ AB_API int ab_moe_shared_pairs(const void* h, int dtype, int ld, const void* gat
   return ab_launch_status();
 }
 
-// All experts at once, for steps of many tokens: a row of `up` holds the gates of all C units and then their
-// up-projections (2 C numbers); the gates' place becomes act(gate) * up * weight, weight 0 for experts that were not
-// chosen and sigmoid(z_t) for the shared expert.
-template <int NC>
+// All experts at once, for steps of many tokens: a row of `up` holds all 2 C columns of the first product (8 gates, 8
+// up-projections, ..); act [T, C] becomes act(gate) * up * weight, weight 0 for experts that were not chosen and
+// sigmoid(z_t) for the shared expert.  Eight units per thread.
 __global__ void __launch_bounds__(256)
-moe_shared_weigh_kernel(bf16* __restrict__ up, Choice c, const float* __restrict__ z, int top, int ff, int fs, int E,
-                        int activation) {
+moe_shared_weigh_kernel(const bf16* __restrict__ up, bf16* __restrict__ act, Choice c, const float* __restrict__ z, int top,
+                        int ff, int fs, int E, int activation) {
   const int t = blockIdx.y;
   const int C = E * ff + fs;
-  const int col = (blockIdx.x * blockDim.x + threadIdx.x) * NC;
+  const int col = (blockIdx.x * blockDim.x + threadIdx.x) * 8;
   if (col >= C) return;
   float g = 0.f;
   if (col >= E * ff) {
@@ -678,41 +663,33 @@ moe_shared_weigh_kernel(bf16* __restrict__ up, Choice c, const float* __restrict
     for (int k = 0; k < top; ++k)
       if (chosen_expert(c, t, k, top) == e) g = chosen_weight(c, t, k, top);
   }
-  bf16* x = up + (size_t)t * 2 * C + col;
-  if (NC == 8) {
-    uint4 v = make_uint4(0, 0, 0, 0);
-    if (g != 0.f) {
-      const uint4 gv = *reinterpret_cast<const uint4*>(x), uv = *reinterpret_cast<const uint4*>(x + C);
-      const uint32_t a[4] = {gv.x, gv.y, gv.z, gv.w}, b[4] = {uv.x, uv.y, uv.z, uv.w};
-      uint32_t* o = reinterpret_cast<uint32_t*>(&v);
+  uint4 v = make_uint4(0, 0, 0, 0);
+  if (g != 0.f) {
+    const uint4* x = reinterpret_cast<const uint4*>(up + (size_t)t * 2 * C + (size_t)col * 2);
+    const uint4 gv = x[0], uv = x[1];
+    const uint32_t a[4] = {gv.x, gv.y, gv.z, gv.w}, b[4] = {uv.x, uv.y, uv.z, uv.w};
+    uint32_t* o = reinterpret_cast<uint32_t*>(&v);
 #pragma unroll
-      for (int j = 0; j < 4; ++j) {
-        const float lo = g * activate(__uint_as_float(a[j] << 16), activation) * __uint_as_float(b[j] << 16);
-        const float hi = g * activate(__uint_as_float(a[j] & 0xffff0000u), activation) * __uint_as_float(b[j] & 0xffff0000u);
-        __nv_bfloat162 r = __floats2bfloat162_rn(lo, hi);
-        o[j] = *reinterpret_cast<uint32_t*>(&r);
-      }
+    for (int j = 0; j < 4; ++j) {
+      const float lo = g * activate(__uint_as_float(a[j] << 16), activation) * __uint_as_float(b[j] << 16);
+      const float hi = g * activate(__uint_as_float(a[j] & 0xffff0000u), activation) * __uint_as_float(b[j] & 0xffff0000u);
+      __nv_bfloat162 r = __floats2bfloat162_rn(lo, hi);
+      o[j] = *reinterpret_cast<uint32_t*>(&r);
     }
-    *reinterpret_cast<uint4*>(x) = v;
-  } else {
-    x[0] = __float2bfloat16_rn(g != 0.f ? g * activate(__bfloat162float(x[0]), activation) * __bfloat162float(x[C]) : 0.f);
   }
+  *reinterpret_cast<uint4*>(act + (size_t)t * C + col) = v;
 }
 
-AB_API int ab_moe_shared_weigh(void* up, const int* idx, const float* wts, const int* table, const int* tokens, float weight,
-                               const float* z, int n_tokens, int top, int ff, int fs, int E, int activation,
-                               cudaStream_t stream) {
+AB_API int ab_moe_shared_weigh(const void* up, void* act, const int* idx, const float* wts, const int* table,
+                               const int* tokens, float weight, const float* z, int n_tokens, int top, int ff, int fs, int E,
+                               int activation, cudaStream_t stream) {
   if (n_tokens <= 0) return AB_OK;
   const Choice c{idx, wts, table, tokens, weight};
-  if (top <= 0 || ff <= 0 || fs < 0 || E <= 0 || n_tokens > 65535 || (activation != 0 && activation != 1) || !choice_ok(c) ||
-      (fs > 0 && !z))
+  if (top <= 0 || ff <= 0 || ff % 8 || fs < 0 || fs % 8 || E <= 0 || n_tokens > 65535 || (activation != 0 && activation != 1) ||
+      !choice_ok(c) || (fs > 0 && !z) || ((((uintptr_t)up) | ((uintptr_t)act)) & 15))
     return AB_BAD_ARG;
   const long long C = (long long)E * ff + fs;
-  if (ff % 8 == 0 && fs % 8 == 0 && (((uintptr_t)up) & 15) == 0)
-    moe_shared_weigh_kernel<8><<<dim3((unsigned)((C / 8 + 255) / 256), (unsigned)n_tokens), 256, 0, stream>>>(
-        (bf16*)up, c, z, top, ff, fs, E, activation);
-  else
-    moe_shared_weigh_kernel<1><<<dim3((unsigned)((C + 255) / 256), (unsigned)n_tokens), 256, 0, stream>>>(
-        (bf16*)up, c, z, top, ff, fs, E, activation);
+  moe_shared_weigh_kernel<<<dim3((unsigned)((C / 8 + 255) / 256), (unsigned)n_tokens), 256, 0, stream>>>(
+      (const bf16*)up, (bf16*)act, c, z, top, ff, fs, E, activation);
   return ab_launch_status();
 }

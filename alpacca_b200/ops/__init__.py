@@ -2124,17 +2124,19 @@ def row_dots(h, w, n_tokens):
 def moe_shared_experts(h, gate_up, down, n_experts, ff, shared_ff, top, out, ctx, activation="silu", choice=None, table=None,
                        gate_logits=None):
     """Gated experts and a shared expert: out[t] = sum_k weight_k E_(e_k)(h[t]) + sigmoid(gate_logits[t]) S(h[t]), an expert
-    W_down (act(W_gate h) * (W_up h)).  gate_up [2, C, width], down [width, C] with C = n_experts * ff + shared_ff: the
-    experts' units side by side, then the shared expert's (`shared_ff` 0: none).  The choice is `choice` = (experts int32
+    W_down (act(W_gate h) * (W_up h)).  gate_up [2 C, width] and down [width, C] with C = n_experts * ff + shared_ff units,
+    the experts' one after another, then the shared expert's (`shared_ff` 0: none); gate_up in groups of 16 rows, the
+    gates of 8 units and then their up-projections.  The choice is `choice` = (experts int32
     [T, top], weights float32 [T, top]), or row token_t of `table` int32 [vocab, top] with weight 1 / top each.
     out [T, width] float32, or of h's dtype."""
     idx, wts = choice if choice is not None else (None, None)
     _cuda(h, gate_up, down, out, idx, wts, table, gate_logits)
     T, width = ctx.n_tokens, h.shape[-1]
     C = n_experts * ff + shared_ff
-    _need(tuple(gate_up.shape) == (2, C, width) and tuple(down.shape) == (width, C) and gate_up.is_contiguous()
-          and down.is_contiguous() and gate_up.dtype == h.dtype and down.dtype == h.dtype,
-          f"moe_shared_experts: gate_up [2, {C}, {width}], down [{width}, {C}] of h's dtype")
+    _need(tuple(gate_up.shape) == (2 * C, width) and tuple(down.shape) == (width, C) and gate_up.is_contiguous()
+          and down.is_contiguous() and gate_up.dtype == h.dtype and down.dtype == h.dtype and ff % 8 == 0
+          and shared_ff % 8 == 0,
+          f"moe_shared_experts: gate_up [{2 * C}, {width}], down [{width}, {C}] of h's dtype, inner sizes multiples of 8")
     _need(h.is_contiguous() and h.numel() >= T * width and out.is_contiguous() and out.shape[-1] == width
           and out.numel() >= T * width and out.dtype in (torch.float32, h.dtype),
           "moe_shared_experts: h [T, width], out [T, width] float32 or of h's dtype")
@@ -2153,17 +2155,26 @@ def moe_shared_experts(h, gate_up, down, n_experts, ff, shared_ff, top, out, ctx
           _p(gate_logits))
     if h.dtype == torch.bfloat16 and MOE_ALL_EXPERTS_MIN_ROWS <= T <= 65535:
         up = torch.empty((T, 2 * C), dtype=h.dtype, device=h.device)
-        torch.mm(h[:T], gate_up.view(2 * C, width).t(), out=up)
+        torch.mm(h[:T], gate_up.t(), out=up)
         _mark("library product")
-        _check(_lib("moe").ab_moe_shared_weigh(_p(up), *by, T, top, ff, shared_ff, n_experts, MOE_ACTIVATIONS[activation],
+        act = torch.empty((T, C), dtype=h.dtype, device=h.device)
+        _check(_lib("moe").ab_moe_shared_weigh(_p(up), _p(act), *by, T, top, ff, shared_ff, n_experts, MOE_ACTIVATIONS[activation],
                                                _stream()), "moe_weigh_all")
         if out.dtype == torch.float32:
-            torch.mm(up[:, :C], down.t(), out_dtype=torch.float32, out=out[:T])
+            torch.mm(act, down.t(), out_dtype=torch.float32, out=out[:T])
         else:
-            torch.mm(up[:, :C], down.t(), out=out[:T])
+            torch.mm(act, down.t(), out=out[:T])
         _mark("library product")
         return out
     act = torch.empty((max(T, 1), top * ff + shared_ff), dtype=h.dtype, device=h.device)
+    if h.dtype == torch.bfloat16 and out.dtype == torch.float32 and width % 8 == 0 and T <= 32 and n_experts <= 512:
+        # few tokens: weights read once for all tokens that chose an expert
+        slabs, slices = -(-width // 16), 1
+        while slices < 8 and slabs * slices * 4 < 3 * _sm_count(h.device):
+            slices *= 2
+        _check(_lib("moe_gemv").ab_moe_gemv(_p(h), _p(gate_up), _p(down), *by, _p(act), _p(out), T, top, width, ff, shared_ff,
+                                            n_experts, MOE_ACTIVATIONS[activation], slices, _stream()), "moe_experts", kernels=2)
+        return out
     _check(_lib("moe").ab_moe_shared_pairs(_p(h), _dt(h), width, _p(gate_up), _p(down), *by, _p(act), _p(out), _dt(out), T, top,
                                            width, ff, shared_ff, n_experts, MOE_ACTIVATIONS[activation], _stream()),
            "moe_experts", kernels=2)

@@ -101,10 +101,10 @@ class TableExperts(FeedForward):
     formed in 32-bit.  A block whose kernel has the stream's row in registers may form it there: `row_gate()` is the
     vector w_s, and `forward` takes the products as `gate_logits`.
 
-    The matrices lie side by side (the experts' units, then the shared expert's), the inner sizes padded with zero units to
-    multiples of 8, so that few tokens read their experts' rows per (token, expert) pair together with the shared expert's
-    and many tokens run everything in two library products with the units of experts that were not chosen set to zero
-    (csrc/moe.cu).  The table is read by the kernels: routing never reaches the host."""
+    The matrices lie together (the experts' units one after another, then the shared expert's; gates and up-projections
+    interleaved in groups of 8 rows), the inner sizes padded with zero units to multiples of 8, so that few tokens run two
+    skinny products that read the chosen experts' weights once (csrc/moe_gemv.cu) and many tokens two library products
+    with the units of experts that were not chosen set to zero (csrc/moe.cu).  The table is read by the kernels: routing never reaches the host."""
 
     def __init__(self, opts: BuildOptions, width: int, inner: int, n_experts: int, top: int, vocab: int, prefix: str,
                  activation: str = "silu", shared_inner: int = 0, table_name: str = "table",
@@ -145,11 +145,13 @@ class TableExperts(FeedForward):
         C = self.E * self.ff + self.fs
         for i in range(self.E + (1 if self.shared_inner else 0)):
             g, u, d = (fetch(s) for s in specs[1 + 3 * i:4 + 3 * i])
-            if self.gate_up is None:
-                self.gate_up = torch.zeros((2, C, self.width), dtype=g.dtype, device=g.device)
+            if i == 0:
+                gate_up = torch.zeros((2, C, self.width), dtype=g.dtype, device=g.device)
                 self.down = torch.zeros((self.width, C), dtype=g.dtype, device=g.device)
             at, n = i * self.ff, g.shape[0]
-            self.gate_up[0, at:at + n], self.gate_up[1, at:at + n], self.down[:, at:at + n] = g, u, d
+            gate_up[0, at:at + n], gate_up[1, at:at + n], self.down[:, at:at + n] = g, u, d
+        # groups of 16 rows: the gates of 8 units, then their up-projections
+        self.gate_up = gate_up.view(2, C // 8, 8, self.width).transpose(0, 1).reshape(2 * C, self.width).contiguous()
         if self.shared_inner:
             self.w_sg = fetch(specs[-1]).reshape(-1).contiguous()
 
