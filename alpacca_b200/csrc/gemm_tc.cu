@@ -404,11 +404,15 @@ __device__ __forceinline__ void tp_tile_origin(int tile, int tiles_m, int tiles_
   n0 = col * TP_BN;
 }
 
-template <int EPI>
+// GROUPED: the rows come in groups that start on tiles, each with a matrix of its own (routed experts): row tile i belongs
+// to group tile_group[i] and meets the rows group * N .. of W.  How many row tiles there are (*row_tiles, at most
+// tiles_m) is known on the device only, from kernels before this one; so everything waits for those.
+template <int EPI, bool GROUPED>
 __global__ void __launch_bounds__(TC_THREADS)
 gemm_tc_persistent_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant__ CUtensorMap map_w,
                           void* __restrict__ Y, const float* __restrict__ bias, int* __restrict__ status, int M, int N,
-                          int K, int ldy, int tiles_m, int n_tiles) {
+                          int K, int ldy, int tiles_m, int n_tiles, const int* __restrict__ tile_group,
+                          const int* __restrict__ row_tiles) {
   extern __shared__ unsigned char smem_raw[];
   unsigned char* base = reinterpret_cast<unsigned char*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~(uintptr_t)1023);
   uint64_t* full = reinterpret_cast<uint64_t*>(base + TP_STAGES * TP_STAGE_BYTES);
@@ -419,6 +423,13 @@ gemm_tc_persistent_kernel(const __grid_constant__ CUtensorMap map_x, const __gri
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int nkb = (K + TC_BK - 1) / TC_BK;
   const int tiles_n = n_tiles / tiles_m;
+  if (GROUPED) {
+    pdl_wait();
+    tiles_m = min(*row_tiles, tiles_m);
+    n_tiles = tiles_m * tiles_n;
+    M = min(M, tiles_m * TC_BM);
+  }
+  auto w_row = [&](int m0, int n0) { return GROUPED ? tile_group[m0 / TC_BM] * N + n0 : n0; };
 
   if (threadIdx.x == 0) {
     for (int s = 0; s < TP_STAGES; ++s) { mbar_init(full + s, 1); mbar_init(empty + s, 1); }
@@ -445,7 +456,7 @@ gemm_tc_persistent_kernel(const __grid_constant__ CUtensorMap map_x, const __gri
       if (first < n_tiles) tp_tile_origin(first, tiles_m, tiles_n, m0_first, n0_first);
       for (int i = 0; i < early; ++i) {
         mbar_expect_tx(full + i, TP_STAGE_BYTES);
-        tma_load_2d(base + i * TP_STAGE_BYTES + TP_A_BYTES, &map_w, i * TC_BK, n0_first, full + i);
+        tma_load_2d(base + i * TP_STAGE_BYTES + TP_A_BYTES, &map_w, i * TC_BK, w_row(m0_first, n0_first), full + i);
       }
       pdl_wait();
       pdl_trigger();
@@ -453,12 +464,13 @@ gemm_tc_persistent_kernel(const __grid_constant__ CUtensorMap map_x, const __gri
       for (int tile = first; tile < n_tiles && ok; tile += gridDim.x) {
         int m0, n0;
         tp_tile_origin(tile, tiles_m, tiles_n, m0, n0);
+        const int wy = w_row(m0, n0);
         for (int kb = (tile == first ? early : 0); kb < nkb; ++kb) {
           const int i = it + kb;
           const int s = i % TP_STAGES;
           if (i >= TP_STAGES && !mbar_wait(empty + s, ((i / TP_STAGES) - 1) & 1)) { atomicExch(status, 11); ok = false; break; }
           mbar_expect_tx(full + s, TP_STAGE_BYTES);
-          tma_load_2d(base + s * TP_STAGE_BYTES + TP_A_BYTES, &map_w, kb * TC_BK, n0, full + s);
+          tma_load_2d(base + s * TP_STAGE_BYTES + TP_A_BYTES, &map_w, kb * TC_BK, wy, full + s);
           tma_load_2d(base + s * TP_STAGE_BYTES, &map_x, kb * TC_BK, m0, full + s);
         }
         it += nkb;
@@ -852,10 +864,10 @@ AB_API int ab_gemm_tc_persistent(const void* X, const void* W, const float* bias
   const int grid = n_tiles < sms ? n_tiles : sms;
 #define AB_GO(E)                                                                                                   \
   {                                                                                                                \
-    cudaError_t e = cudaFuncSetAttribute(gemm_tc_persistent_kernel<E>, cudaFuncAttributeMaxDynamicSharedMemorySize, TP_SMEM); \
+    cudaError_t e = cudaFuncSetAttribute(gemm_tc_persistent_kernel<E, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, TP_SMEM); \
     if (e != cudaSuccess) return AB_CUDA_ERR + (int)e;                                                             \
-    e = ab_launch(gemm_tc_persistent_kernel<E>, dim3(grid), dim3(TC_THREADS), (size_t)TP_SMEM, stream, mx, mw, Y,  \
-                  bias, status, M, N, K, ldy, tiles_m, n_tiles);                                                   \
+    e = ab_launch(gemm_tc_persistent_kernel<E, false>, dim3(grid), dim3(TC_THREADS), (size_t)TP_SMEM, stream, mx, mw, Y, \
+                  bias, status, M, N, K, ldy, tiles_m, n_tiles, (const int*)nullptr, (const int*)nullptr);         \
     if (e != cudaSuccess) return AB_CUDA_ERR + (int)e;                                                             \
     return ab_launch_status();                                                                                     \
   }
@@ -866,6 +878,47 @@ AB_API int ab_gemm_tc_persistent(const void* X, const void* W, const float* bias
     case EPI_RELUGLU_BF16: AB_GO(EPI_RELUGLU_BF16)
     case EPI_GELUGLU_BF16: AB_GO(EPI_GELUGLU_BF16)
     case EPI_GELU_BF16: AB_GO(EPI_GELU_BF16)
+  }
+#undef AB_GO
+  return AB_BAD_ARG;
+}
+
+// Rows in groups with a matrix each (see the kernel): X [max_rows, K] in row tiles of 128 (max_rows a multiple of 128), W
+// [groups * N, K], Y [max_rows, ..]; tile_group int [max_rows / 128], row_tiles int [1] on the device.  Epilogue kinds 0
+// (bfloat16) and 2 (SwiGLU).
+AB_API int ab_gemm_tc_grouped(const void* X, const void* W, void* Y, int max_rows, int N, int K, int groups, int ldy,
+                              int epilogue_kind, const int* tile_group, const int* row_tiles, cudaStream_t stream) {
+  if (max_rows <= 0 || N <= 0) return AB_OK;
+  if (K <= 0 || (K % 8) || groups <= 0 || (max_rows % TC_BM) || (long long)groups * N > 0x7fffffffLL || !tile_group || !row_tiles)
+    return AB_BAD_ARG;
+  if (epilogue_kind == EPI_SWIGLU_BF16 && (N % 16)) return AB_BAD_ARG;
+  int* status = status_word();
+  if (!status) return AB_BAD_ARG;
+  CUtensorMap mx, mw;
+  if (!make_map(&mx, X, max_rows, K, TC_BM)) return AB_BAD_ARG;
+  if (!make_map(&mw, W, groups * N, K, TP_BN)) return AB_BAD_ARG;
+  static int sms = 0;
+  if (!sms) {
+    int dev = 0;
+    cudaGetDevice(&dev);
+    cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, dev);
+  }
+  const int tiles_m = max_rows / TC_BM, tiles_n = (N + TP_BN - 1) / TP_BN;
+  if ((long long)tiles_m * tiles_n > 0x7fffffffLL) return AB_BAD_ARG;
+  const int n_tiles = tiles_m * tiles_n;
+  const int grid = n_tiles < sms ? n_tiles : sms;
+#define AB_GO(E)                                                                                                   \
+  {                                                                                                                \
+    cudaError_t e = cudaFuncSetAttribute(gemm_tc_persistent_kernel<E, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, TP_SMEM); \
+    if (e != cudaSuccess) return AB_CUDA_ERR + (int)e;                                                             \
+    e = ab_launch(gemm_tc_persistent_kernel<E, true>, dim3(grid), dim3(TC_THREADS), (size_t)TP_SMEM, stream, mx, mw, Y, \
+                  (const float*)nullptr, status, max_rows, N, K, ldy, tiles_m, n_tiles, tile_group, row_tiles);    \
+    if (e != cudaSuccess) return AB_CUDA_ERR + (int)e;                                                             \
+    return ab_launch_status();                                                                                     \
+  }
+  switch (epilogue_kind) {
+    case EPI_STORE_BF16: AB_GO(EPI_STORE_BF16)
+    case EPI_SWIGLU_BF16: AB_GO(EPI_SWIGLU_BF16)
   }
 #undef AB_GO
   return AB_BAD_ARG;

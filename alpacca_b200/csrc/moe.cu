@@ -492,11 +492,12 @@ AB_API int ab_moe_weigh_all(void* up, int dtype, const int* idx, const float* wt
 //         + sigmoid(z_t) W_down_s (silu(W_gate_s h_t) * (W_up_s h_t))               (if there is a shared expert)
 //
 // The choice comes from a router (`idx`, `wts`) or from the token's id: a row of a table names its experts, each with the
-// same constant weight (moe_choice.cuh).  The matrices lie together, C = E * ff + fs units (the experts' one after another,
-// then the shared expert's; ff and fs multiples of 8): gate_up [2 C, width] in groups of 16 rows, the gates of 8 units and
-// then their up-projections, and down [width, C].
-// z [T] are the shared expert's gate logits (float32, formed elsewhere).
-// The kernels here take any width and the 32-bit path; bfloat16 steps of a few tokens run csrc/moe_gemv.cu.
+// same constant weight (moe_choice.cuh).  Layouts (ff and fs multiples of 8): gate_up [E, 2 ff, width], an expert's rows in
+// groups of 16, the gates of 8 units and then their up-projections; down [E, width, ff]; the shared expert's likewise,
+// [2 fs, width] and [width, fs].  z [T] are the shared expert's gate logits (float32, formed elsewhere).
+// The pair kernels here take any width and the 32-bit path.  bfloat16 steps of a few tokens run csrc/moe_gemv.cu; steps of
+// many tokens sort their (token, expert) pairs by expert (moe_plan), copy the tokens' rows into that order (moe_gather),
+// run two grouped products (csrc/gemm_tc.cu) and add up each token's outputs (moe_combine).
 // ---------------------------------------------------------------------------
 __device__ __forceinline__ void fma8(float& part, uint4 x, uint4 y) {
   const uint32_t a[4] = {x.x, x.y, x.z, x.w}, b[4] = {y.x, y.y, y.z, y.w};
@@ -553,14 +554,15 @@ __device__ __forceinline__ void lane_dot2(const float* __restrict__ x, const flo
 // unit of the shared expert for eight tokens, whose warps then read the same two rows at the same time.
 template <typename T>
 __global__ void __launch_bounds__(256)
-moe_shared_up_kernel(const T* __restrict__ h, int ld, const T* __restrict__ gate_up, Choice c, T* __restrict__ act,
-                     int n_tokens, int top, int width, int ff, int fs, int E, int activation, long long pair_blocks) {
+moe_shared_up_kernel(const T* __restrict__ h, int ld, const T* __restrict__ gate_up, const T* __restrict__ gate_up_s, Choice c,
+                     T* __restrict__ act, int n_tokens, int top, int width, int ff, int fs, int E, int activation, long long pair_blocks) {
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   pdl_wait();
   pdl_trigger();
   const int row_len = top * ff + fs;
   int t;
   size_t unit, dst;
+  const T* w = gate_up;
   long long blk = blockIdx.x;
   if (blk < pair_blocks) {
     const long long group = blk / ff;
@@ -576,10 +578,11 @@ moe_shared_up_kernel(const T* __restrict__ h, int ld, const T* __restrict__ gate
     const int chunk = (int)(blk / fs), j = (int)(blk - (long long)chunk * fs);
     t = chunk * 8 + warp;
     if (t >= n_tokens) return;
-    unit = (size_t)E * ff + j;
+    unit = j;
+    w = gate_up_s;
     dst = (size_t)t * row_len + (size_t)top * ff + j;
   }
-  const T* gate = gate_up + ((unit >> 3) * 16 + (unit & 7)) * width;
+  const T* gate = w + ((unit >> 3) * 16 + (unit & 7)) * width;
   float pg, pu;
   lane_dot2(h + (size_t)t * ld, gate, gate + (size_t)8 * width, width, lane, pg, pu);
   pg = warp_sum(pg);
@@ -591,25 +594,23 @@ moe_shared_up_kernel(const T* __restrict__ h, int ld, const T* __restrict__ gate
 // read by all of them together).
 template <typename T, typename TO>
 __global__ void __launch_bounds__(256)
-moe_shared_down_kernel(const T* __restrict__ act, const T* __restrict__ down, Choice c, const float* __restrict__ z,
-                       TO* __restrict__ out, int n_tokens, int top, int width, int ff, int fs, int E) {
+moe_shared_down_kernel(const T* __restrict__ act, const T* __restrict__ down, const T* __restrict__ down_s, Choice c,
+                       const float* __restrict__ z, TO* __restrict__ out, int n_tokens, int top, int width, int ff, int fs, int E) {
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   pdl_wait();
   pdl_trigger();
   const int i = blockIdx.x, t = blockIdx.y * 8 + warp;
   if (t >= n_tokens) return;
-  const size_t C = (size_t)E * ff + fs;
   const T* a = act + (size_t)t * (top * ff + fs);
-  const T* w = down + (size_t)i * C;
   float total = 0.f;
 #pragma unroll 4
   for (int k = 0; k < top; ++k) {
     const int e = chosen_expert(c, t, k, top);
-    const float part = lane_dot(a + (size_t)k * ff, w + (size_t)e * ff, ff, lane);
+    const float part = lane_dot(a + (size_t)k * ff, down + ((size_t)e * width + i) * ff, ff, lane);
     total = fmaf(chosen_weight(c, t, k, top), part, total);
   }
   if (fs > 0) {
-    const float part = lane_dot(a + (size_t)top * ff, w + (size_t)E * ff, fs, lane);
+    const float part = lane_dot(a + (size_t)top * ff, down_s + (size_t)i * fs, fs, lane);
     total = fmaf(1.0f / (1.0f + expf(-z[t])), part, total);
   }
   total = warp_sum(total);
@@ -617,14 +618,14 @@ moe_shared_down_kernel(const T* __restrict__ act, const T* __restrict__ down, Ch
 }
 
 // act: scratch [n_tokens, top * ff + fs] of `dtype`; out of `out_dtype`.
-AB_API int ab_moe_shared_pairs(const void* h, int dtype, int ld, const void* gate_up, const void* down, const int* idx,
-                               const float* wts, const int* table, const int* tokens, float weight, const float* z, void* act,
+AB_API int ab_moe_shared_pairs(const void* h, int dtype, int ld, const void* gate_up, const void* down, const void* gate_up_s,
+                               const void* down_s, const int* idx, const float* wts, const int* table, const int* tokens, float weight, const float* z, void* act,
                                void* out, int out_dtype, int n_tokens, int top, int width, int ff, int fs, int E,
                                int activation, cudaStream_t stream) {
   if (n_tokens <= 0) return AB_OK;
   const Choice c{idx, wts, table, tokens, weight};
   if (top <= 0 || width <= 0 || ff <= 0 || ff % 8 || fs < 0 || fs % 8 || E <= 0 || (activation != 0 && activation != 1) || !choice_ok(c) ||
-      (fs > 0 && !z))
+      (fs > 0 && (!z || !gate_up_s || !down_s)))
     return AB_BAD_ARG;
   const long long pair_blocks = ((long long)n_tokens * top + 7) / 8 * ff;
   const long long blocks = pair_blocks + ((long long)n_tokens + 7) / 8 * fs;
@@ -632,9 +633,9 @@ AB_API int ab_moe_shared_pairs(const void* h, int dtype, int ld, const void* gat
   const dim3 dgrid((unsigned)width, (unsigned)((n_tokens + 7) / 8));
 #define AB_GO(T, TO)                                                                                                   \
   {                                                                                                                    \
-    ab_launch(moe_shared_up_kernel<T>, dim3((unsigned)blocks), dim3(256), 0, stream, (const T*)h, ld, (const T*)gate_up, c, \
-              (T*)act, n_tokens, top, width, ff, fs, E, activation, pair_blocks);                                      \
-    ab_launch(moe_shared_down_kernel<T, TO>, dgrid, dim3(256), 0, stream, (const T*)act, (const T*)down, c, z, (TO*)out, \
+    ab_launch(moe_shared_up_kernel<T>, dim3((unsigned)blocks), dim3(256), 0, stream, (const T*)h, ld, (const T*)gate_up, \
+              (const T*)gate_up_s, c, (T*)act, n_tokens, top, width, ff, fs, E, activation, pair_blocks);                                      \
+    ab_launch(moe_shared_down_kernel<T, TO>, dgrid, dim3(256), 0, stream, (const T*)act, (const T*)down, (const T*)down_s, c, z, (TO*)out, \
               n_tokens, top, width, ff, fs, E);                                                                        \
   }
   if (dtype == AB_F32 && out_dtype == AB_F32) AB_GO(float, float)
@@ -645,51 +646,117 @@ AB_API int ab_moe_shared_pairs(const void* h, int dtype, int ld, const void* gat
   return ab_launch_status();
 }
 
-// All experts at once, for steps of many tokens: a row of `up` holds all 2 C columns of the first product (8 gates, 8
-// up-projections, ..); act [T, C] becomes act(gate) * up * weight, weight 0 for experts that were not chosen and
-// sigmoid(z_t) for the shared expert.  Eight units per thread.
-__global__ void __launch_bounds__(256)
-moe_shared_weigh_kernel(const bf16* __restrict__ up, bf16* __restrict__ act, Choice c, const float* __restrict__ z, int top,
-                        int ff, int fs, int E, int activation) {
-  const int t = blockIdx.y;
-  const int C = E * ff + fs;
-  const int col = (blockIdx.x * blockDim.x + threadIdx.x) * 8;
-  if (col >= C) return;
-  float g = 0.f;
-  if (col >= E * ff) {
-    g = 1.0f / (1.0f + expf(-z[t]));
-  } else {
-    const int e = col / ff;
-    for (int k = 0; k < top; ++k)
-      if (chosen_expert(c, t, k, top) == e) g = chosen_weight(c, t, k, top);
-  }
-  uint4 v = make_uint4(0, 0, 0, 0);
-  if (g != 0.f) {
-    const uint4* x = reinterpret_cast<const uint4*>(up + (size_t)t * 2 * C + (size_t)col * 2);
-    const uint4 gv = x[0], uv = x[1];
-    const uint32_t a[4] = {gv.x, gv.y, gv.z, gv.w}, b[4] = {uv.x, uv.y, uv.z, uv.w};
-    uint32_t* o = reinterpret_cast<uint32_t*>(&v);
+// ---------------------------------------------------------------------------
+// many tokens: the pairs in order of their experts
+// ---------------------------------------------------------------------------
+#define MOE_TILE 128           // rows of a row tile of the grouped product
+
+// pos[t * top + k]: the row of a pair; an expert's rows start on a row tile.  tile_group[i]: the expert of row tile i,
+// row_tiles[0]: how many row tiles there are.  One block; the order of an expert's rows among themselves is whatever the
+// counters give (a row's result does not depend on its place).
+__global__ void __launch_bounds__(1024)
+moe_plan_kernel(Choice c, int n_tokens, int top, int E, int* __restrict__ pos, int* __restrict__ tile_group,
+                int* __restrict__ row_tiles) {
+  __shared__ int count[MOE_MAX_EXPERTS], first[MOE_MAX_EXPERTS];
+  pdl_wait();
+  pdl_trigger();
+  for (int e = threadIdx.x; e < E; e += blockDim.x) count[e] = 0;
+  __syncthreads();
+  const int n_pairs = n_tokens * top;
+  for (int p = threadIdx.x; p < n_pairs; p += blockDim.x) atomicAdd(&count[chosen_expert(c, p / top, p % top, top)], 1);
+  __syncthreads();
+  if (threadIdx.x < 32) {                      // the experts' first row tiles: a running sum over lanes
+    int before = 0;
+    for (int e0 = 0; e0 < E; e0 += 32) {
+      const int e = e0 + threadIdx.x;
+      const int tiles = e < E ? (count[e] + MOE_TILE - 1) / MOE_TILE : 0;
+      int incl = tiles;
 #pragma unroll
-    for (int j = 0; j < 4; ++j) {
-      const float lo = g * activate(__uint_as_float(a[j] << 16), activation) * __uint_as_float(b[j] << 16);
-      const float hi = g * activate(__uint_as_float(a[j] & 0xffff0000u), activation) * __uint_as_float(b[j] & 0xffff0000u);
-      __nv_bfloat162 r = __floats2bfloat162_rn(lo, hi);
-      o[j] = *reinterpret_cast<uint32_t*>(&r);
+      for (int o = 1; o < 32; o <<= 1) {
+        const int up = __shfl_up_sync(0xffffffffu, incl, o);
+        if ((int)threadIdx.x >= o) incl += up;
+      }
+      if (e < E) {
+        first[e] = (before + incl - tiles) * MOE_TILE;
+        for (int i = 0; i < tiles; ++i) tile_group[before + incl - tiles + i] = e;
+      }
+      before += __shfl_sync(0xffffffffu, incl, 31);
     }
+    if (threadIdx.x == 0) *row_tiles = before;
   }
-  *reinterpret_cast<uint4*>(act + (size_t)t * C + col) = v;
+  __syncthreads();
+  for (int p = threadIdx.x; p < n_pairs; p += blockDim.x)
+    pos[p] = atomicAdd(&first[chosen_expert(c, p / top, p % top, top)], 1);
 }
 
-AB_API int ab_moe_shared_weigh(const void* up, void* act, const int* idx, const float* wts, const int* table,
-                               const int* tokens, float weight, const float* z, int n_tokens, int top, int ff, int fs, int E,
-                               int activation, cudaStream_t stream) {
+// rows[pos[t, k]] = h[t] for every choice k; 16-byte pieces (width a multiple of 8)
+__global__ void __launch_bounds__(256)
+moe_gather_kernel(const bf16* __restrict__ h, const int* __restrict__ pos, bf16* __restrict__ rows, int top, int width) {
+  pdl_wait();
+  pdl_trigger();
+  const int t = blockIdx.x;
+  for (int i = threadIdx.x * 8; i < width; i += blockDim.x * 8) {
+    const uint4 v = *reinterpret_cast<const uint4*>(h + (size_t)t * width + i);
+    for (int k = 0; k < top; ++k)
+      *reinterpret_cast<uint4*>(rows + (size_t)pos[(size_t)t * top + k] * width + i) = v;
+  }
+}
+
+// out[t] = sum_k weight_k y[pos[t, k]] + sigmoid(z_t) ys[t]   (ys null: no shared expert)
+__global__ void __launch_bounds__(256)
+moe_combine_kernel(const bf16* __restrict__ y, const int* __restrict__ pos, Choice c, const bf16* __restrict__ ys,
+                   const float* __restrict__ z, float* __restrict__ out, int top, int width) {
+  pdl_wait();
+  pdl_trigger();
+  const int t = blockIdx.x;
+  const float g = ys != nullptr ? 1.0f / (1.0f + expf(-z[t])) : 0.f;
+  for (int i = threadIdx.x * 8; i < width; i += blockDim.x * 8) {
+    float s[8];
+#pragma unroll
+    for (int j = 0; j < 8; ++j) s[j] = 0.f;
+    auto add = [&](const bf16* p, float w) {
+      const uint4 v = *reinterpret_cast<const uint4*>(p);
+      const uint32_t a[4] = {v.x, v.y, v.z, v.w};
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        s[2 * j] = fmaf(w, __uint_as_float(a[j] << 16), s[2 * j]);
+        s[2 * j + 1] = fmaf(w, __uint_as_float(a[j] & 0xffff0000u), s[2 * j + 1]);
+      }
+    };
+#pragma unroll 4
+    for (int k = 0; k < top; ++k) add(y + (size_t)pos[(size_t)t * top + k] * width + i, chosen_weight(c, t, k, top));
+    if (ys != nullptr) add(ys + (size_t)t * width + i, g);
+    float4* o = reinterpret_cast<float4*>(out + (size_t)t * width + i);
+    o[0] = make_float4(s[0], s[1], s[2], s[3]);
+    o[1] = make_float4(s[4], s[5], s[6], s[7]);
+  }
+}
+
+// pos int [n_tokens * top], tile_group int [n_tokens * top / 128 + E], row_tiles int [1]; rows bfloat16
+// [(n_tokens * top / 128 + E) * 128, width].
+AB_API int ab_moe_gather(const void* h, const int* idx, const float* wts, const int* table, const int* tokens, float weight,
+                         int* pos, int* tile_group, int* row_tiles, void* rows, int n_tokens, int top, int width, int E,
+                         cudaStream_t stream) {
   if (n_tokens <= 0) return AB_OK;
   const Choice c{idx, wts, table, tokens, weight};
-  if (top <= 0 || ff <= 0 || ff % 8 || fs < 0 || fs % 8 || E <= 0 || n_tokens > 65535 || (activation != 0 && activation != 1) ||
-      !choice_ok(c) || (fs > 0 && !z) || ((((uintptr_t)up) | ((uintptr_t)act)) & 15))
+  if (top <= 0 || E <= 0 || E > MOE_MAX_EXPERTS || width <= 0 || width % 8 || !choice_ok(c) ||
+      (long long)n_tokens * top > 0x3fffffffLL || ((((uintptr_t)h) | ((uintptr_t)rows)) & 15))
     return AB_BAD_ARG;
-  const long long C = (long long)E * ff + fs;
-  moe_shared_weigh_kernel<<<dim3((unsigned)((C / 8 + 255) / 256), (unsigned)n_tokens), 256, 0, stream>>>(
-      (const bf16*)up, (bf16*)act, c, z, top, ff, fs, E, activation);
+  ab_launch(moe_plan_kernel, dim3(1), dim3(1024), 0, stream, c, n_tokens, top, E, pos, tile_group, row_tiles);
+  ab_launch(moe_gather_kernel, dim3((unsigned)n_tokens), dim3(width >= 2048 ? 256 : 128), 0, stream, (const bf16*)h,
+            (const int*)pos, (bf16*)rows, top, width);
+  return ab_launch_status();
+}
+
+AB_API int ab_moe_combine(const void* y, const int* pos, const int* idx, const float* wts, const int* table, const int* tokens,
+                          float weight, const void* ys, const float* z, float* out, int n_tokens, int top, int width,
+                          cudaStream_t stream) {
+  if (n_tokens <= 0) return AB_OK;
+  const Choice c{idx, wts, table, tokens, weight};
+  if (top <= 0 || width <= 0 || width % 8 || !choice_ok(c) || (ys && !z) ||
+      ((((uintptr_t)y) | ((uintptr_t)ys) | ((uintptr_t)out)) & 15))
+    return AB_BAD_ARG;
+  ab_launch(moe_combine_kernel, dim3((unsigned)n_tokens), dim3(width >= 2048 ? 256 : 128), 0, stream, (const bf16*)y, pos, c,
+            (const bf16*)ys, z, out, top, width);
   return ab_launch_status();
 }

@@ -21,6 +21,7 @@
 #define MG_U 8                 // k-groups (32 numbers) a thread asks for before it uses any
 #define MG_MAX_TOKENS 32
 #define MG_MAX_EXPERTS 512
+#define MG_MAX_TOP 32
 
 __device__ __forceinline__ void mg_mma(float* c, uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3, uint32_t b0, uint32_t b1) {
   asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, "
@@ -44,7 +45,7 @@ __device__ __forceinline__ uint4 mg_act(const bf16* p) {
 
 template <int NT>
 __global__ void __launch_bounds__(256)
-moe_gemv_up_kernel(const bf16* __restrict__ X, const bf16* __restrict__ W, Choice c, const float* __restrict__ z,
+moe_gemv_up_kernel(const bf16* __restrict__ X, const bf16* __restrict__ W, const bf16* __restrict__ Ws, Choice c, const float* __restrict__ z,
                    bf16* __restrict__ act, int M, int K, int top, int ff, int fs, int E, int activation) {
   constexpr int WARPS = 8;
   __shared__ float red[WARPS][NT][32][4];
@@ -76,7 +77,7 @@ moe_gemv_up_kernel(const bf16* __restrict__ X, const bf16* __restrict__ W, Choic
     if (!waited) { pdl_wait(); pdl_trigger(); }
     return;
   }
-  const bf16* w_lo = W + ((size_t)slab * 16 + g) * K;
+  const bf16* w_lo = (shared ? Ws + (size_t)(slab - E * per_expert) * 16 * K : W + (size_t)slab * 16 * K) + (size_t)g * K;
   const bf16* w_hi = w_lo + (size_t)8 * K;
   const bf16* x_row[NT];
   bool x_ok[NT];
@@ -148,30 +149,36 @@ moe_gemv_up_kernel(const bf16* __restrict__ X, const bf16* __restrict__ W, Choic
 
 template <int NT, int WARPS>
 __global__ void __launch_bounds__(WARPS * 32)
-moe_gemv_down_kernel(const bf16* __restrict__ act, const bf16* __restrict__ W, Choice c, float* __restrict__ out, int M, int N,
+moe_gemv_down_kernel(const bf16* __restrict__ act, const bf16* __restrict__ W, const bf16* __restrict__ Ws, Choice c, float* __restrict__ out, int M, int N,
                      int top, int ff, int fs, int E, int slices) {
   namespace cg = cooperative_groups;
   __shared__ float red[WARPS][NT][32][4];
   __shared__ float tile[NT][32][4];                          // this slice's sums, read by the cluster's first CTA
   __shared__ signed char slot_of[MG_MAX_EXPERTS][NT * 8];    // a token's slot of an expert, -1: not chosen
   __shared__ short active[MG_MAX_EXPERTS];
+  __shared__ bool picked[MG_MAX_EXPERTS];
   __shared__ int n_active;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int g = lane >> 2, t = lane & 3;
   const int n0 = blockIdx.x * 16, slice = blockIdx.y;
-  for (int i = tid; i < E * NT * 8; i += WARPS * 32) (&slot_of[0][0])[i] = -1;
+  __shared__ short chosen[MG_MAX_TOKENS * MG_MAX_TOP];
+  for (int i = tid; i < M * top; i += WARPS * 32) chosen[i] = (short)chosen_expert(c, i / top, i % top, top);
   __syncthreads();
-  for (int i = tid; i < M * top; i += WARPS * 32) {
-    const int tok = i / top, k = i - tok * top;
-    slot_of[chosen_expert(c, tok, k, top)][tok] = (signed char)k;
+  for (int e0 = 0; e0 < E; e0 += WARPS * 32) {               // a thread looks for its expert among the choices
+    const int e = e0 + tid;
+    if (e >= E) continue;
+    bool any = false;
+#pragma unroll
+    for (int i = 0; i < NT * 8; ++i) slot_of[e][i] = -1;
+    for (int i = 0; i < M * top; ++i)
+      if (chosen[i] == e) { slot_of[e][i / top] = (signed char)(i % top); any = true; }
+    picked[e] = any;
   }
   __syncthreads();
   if (warp == 0) {                                           // the experts that some token chose, in order
     int have = 0;
     for (int e0 = 0; e0 < E; e0 += 32) {
-      bool any = false;
-      if (e0 + lane < E)
-        for (int i = 0; i < M; ++i) any |= slot_of[e0 + lane][i] >= 0;
+      const bool any = e0 + lane < E && picked[e0 + lane];
       const unsigned who = __ballot_sync(0xffffffffu, any);
       if (any) active[have + __popc(who & ((1u << lane) - 1u))] = (short)(e0 + lane);
       have += __popc(who);
@@ -180,13 +187,11 @@ moe_gemv_down_kernel(const bf16* __restrict__ act, const bf16* __restrict__ W, C
   }
   __syncthreads();
   // the walk: groups of 32 units (an expert's last one may be short), active experts one after another, then the shared one
-  const size_t C = (size_t)E * ff + fs;
   const int ge = (ff + 31) / 32, gs = (fs + 31) / 32;
   const int total = n_active * ge + gs;
   const int runs = slices * WARPS, run = slice * WARPS + warp;
   const int begin = (int)((long long)total * run / runs), end = (int)((long long)total * (run + 1) / runs);
-  const bf16* w_lo = W + (size_t)min(n0 + g, N - 1) * C;     // rows past N read row N - 1 again; their sums are not stored
-  const bf16* w_hi = W + (size_t)min(n0 + g + 8, N - 1) * C;
+  const size_t lo = min(n0 + g, N - 1), hi = min(n0 + g + 8, N - 1);      // rows past N read row N - 1 again, unstored
   const int row_len = top * ff + fs;
   float acc[NT][4];
 #pragma unroll
@@ -203,9 +208,9 @@ moe_gemv_down_kernel(const bf16* __restrict__ act, const bf16* __restrict__ W, C
         const bool sh = ai >= n_active;
         const int k = (sh ? at - n_active * ge : at - ai * ge) * 32 + t * 8;
         if (k < (sh ? fs : ff)) {
-          const size_t col = (sh ? (size_t)E * ff : (size_t)active[ai] * ff) + k;
-          wl[u] = mg_stream(w_lo + col);
-          wh[u] = mg_stream(w_hi + col);
+          const bf16* w = sh ? Ws + k : W + (size_t)active[ai] * N * ff + k;
+          wl[u] = mg_stream(w + lo * (sh ? fs : ff));
+          wh[u] = mg_stream(w + hi * (sh ? fs : ff));
         }
       }
     }
@@ -283,16 +288,18 @@ AB_API int ab_moe_gemv_max_tokens() { return MG_MAX_TOKENS; }
 AB_API int ab_moe_gemv_max_experts() { return MG_MAX_EXPERTS; }
 
 // act: scratch bfloat16 [M, top * ff + fs]; out: float32 [M, width].  `slices` (1, 2, 4 or 8): CTAs per 16 output columns.
-AB_API int ab_moe_gemv(const void* h, const void* gate_up, const void* down, const int* idx, const float* wts, const int* table,
+AB_API int ab_moe_gemv_max_top() { return MG_MAX_TOP; }
+AB_API int ab_moe_gemv(const void* h, const void* gate_up, const void* down, const void* gate_up_s, const void* down_s, const int* idx, const float* wts, const int* table,
                        const int* tokens, float weight, const float* z, void* act, float* out, int M, int top, int width, int ff,
                        int fs, int E, int activation, int slices, cudaStream_t stream) {
   if (M <= 0) return AB_OK;
   const Choice c{idx, wts, table, tokens, weight};
-  if (M > MG_MAX_TOKENS || E <= 0 || E > MG_MAX_EXPERTS || top <= 0 || top > 126 || top > E || width <= 0 || width % 8 || ff <= 0 ||
-      ff % 8 || fs < 0 || fs % 8 || (activation != 0 && activation != 1) || !choice_ok(c) || (fs > 0 && !z))
+  if (M > MG_MAX_TOKENS || E <= 0 || E > MG_MAX_EXPERTS || top <= 0 || top > MG_MAX_TOP || top > E || width <= 0 || width % 8 || ff <= 0 ||
+      ff % 8 || fs < 0 || fs % 8 || (activation != 0 && activation != 1) || !choice_ok(c) || (fs > 0 && (!z || !gate_up_s || !down_s)))
     return AB_BAD_ARG;
   if (slices != 1 && slices != 2 && slices != 4 && slices != 8) return AB_BAD_ARG;
-  if ((((uintptr_t)h) | ((uintptr_t)gate_up) | ((uintptr_t)down) | ((uintptr_t)act)) & 15) return AB_BAD_ARG;
+  if ((((uintptr_t)h) | ((uintptr_t)gate_up) | ((uintptr_t)down) | ((uintptr_t)gate_up_s) | ((uintptr_t)down_s) |
+       ((uintptr_t)act)) & 15) return AB_BAD_ARG;
   const unsigned up_blocks = (unsigned)(E * (ff / 8) + fs / 8);
   cudaLaunchConfig_t cfg = {};
   cfg.gridDim = dim3((unsigned)((width + 15) / 16), (unsigned)slices);
@@ -316,11 +323,11 @@ AB_API int ab_moe_gemv(const void* h, const void* gate_up, const void* down, con
   cudaError_t e = cudaSuccess;
 #define AB_GO(NT, WARPS)                                                                                               \
   {                                                                                                                    \
-    ab_launch(moe_gemv_up_kernel<NT>, dim3(up_blocks), dim3(256), 0, stream, (const bf16*)h, (const bf16*)gate_up, c, z, \
-              (bf16*)act, M, width, top, ff, fs, E, activation);                                                       \
+    ab_launch(moe_gemv_up_kernel<NT>, dim3(up_blocks), dim3(256), 0, stream, (const bf16*)h, (const bf16*)gate_up, \
+              (const bf16*)gate_up_s, c, z, (bf16*)act, M, width, top, ff, fs, E, activation);                                                       \
     cfg.blockDim = dim3(WARPS * 32);                                                                                   \
-    e = cudaLaunchKernelEx(&cfg, moe_gemv_down_kernel<NT, WARPS>, (const bf16*)act, (const bf16*)down, c, out, M, width, top, \
-                           ff, fs, E, slices);                                                                         \
+    e = cudaLaunchKernelEx(&cfg, moe_gemv_down_kernel<NT, WARPS>, (const bf16*)act, (const bf16*)down, (const bf16*)down_s, c, out, \
+                           M, width, top, ff, fs, E, slices);                                                                         \
   }
   if (M <= 8) AB_GO(1, 16)
   else if (M <= 16) AB_GO(2, 16)

@@ -60,7 +60,7 @@ def build_ponusun(cfg: PonusunConfig, opts: BuildOptions) -> DecoderSpec:
         elif mlp is not None:
             shared = mlp.get("shared")
             ffn = TableExperts(opts, E, mlp["expert"]["ff"], mlp["router"]["experts"], mlp["router"]["top"], cfg.vocab,
-                               f"{p}.mlp", shared_inner=shared["ff"] if shared else 0, out_dtype=torch.float32)
+                               f"{p}.mlp", shared_inner=shared["ff"] if shared else 0)
         layers.append(PostNormBlock(mixer, norm(f"{p}.norm1"), ffn, norm(f"{p}.norm2") if ffn is not None else None,
                                     conv=InputConv(opts, E, cfg.canon["taps"], f"{p}.canon1"),
                                     average=DepthAverage(opts, i + 1, f"{p}.dwa")))

@@ -2121,26 +2121,59 @@ def row_dots(h, w, n_tokens):
     return z
 
 
-def moe_shared_experts(h, gate_up, down, n_experts, ff, shared_ff, top, out, ctx, activation="silu", choice=None, table=None,
+MOE_GEMV_MAX_ROWS = 32             # up to here the skinny products of csrc/moe_gemv.cu
+
+
+def gemm_tc_grouped(x, w, out, n_groups, tile_group, row_tiles, swiglu=False):
+    """Rows in groups with a matrix each, on the tcgen05 tensor cores: row tile i (128 rows) of x [R, K] belongs to group
+    tile_group[i] and is multiplied with w [n_groups * N, K]'s rows of that group; out [R, N], or [R, N / 2] with `swiglu`
+    (an 8-row interleaved gate|up matrix per group).  row_tiles int32 [1]: how many row tiles there are, on the device;
+    rows past them are left alone.  All bfloat16."""
+    _cuda(x, w, out, tile_group, row_tiles)
+    R, K = x.shape
+    N = w.shape[0] // n_groups
+    _need(x.dtype == w.dtype == out.dtype == torch.bfloat16 and x.is_contiguous() and w.is_contiguous() and out.is_contiguous()
+          and w.dim() == 2 and w.shape[1] == K and w.shape[0] == n_groups * N and R % 128 == 0 and K % 8 == 0
+          and out.shape[0] == R and out.shape[1] == (N // 2 if swiglu else N) and (not swiglu or N % 16 == 0),
+          "gemm_tc_grouped: x [R, K] with R a multiple of 128, w [groups * N, K], out [R, N] (or N / 2), bfloat16")
+    _need(x.data_ptr() % 16 == 0 and w.data_ptr() % 16 == 0, "gemm_tc_grouped: operands must be 16-byte aligned")
+    _i32(tile_group, R // 128, "tile_group")
+    _i32(row_tiles, 1, "row_tiles")
+    _tc_unchecked["gemm_tc"] = True
+    _check(_lib("gemm_tc").ab_gemm_tc_grouped(_p(x), _p(w), _p(out), R, N, K, n_groups, out.shape[1], 2 if swiglu else 0,
+                                              _p(tile_group), _p(row_tiles), _stream()), "gemm_tc_grouped")
+    return out
+
+
+def moe_shared_experts(h, gate_up, down, n_experts, top, out, ctx, activation="silu", choice=None, table=None, shared=None,
                        gate_logits=None):
     """Gated experts and a shared expert: out[t] = sum_k weight_k E_(e_k)(h[t]) + sigmoid(gate_logits[t]) S(h[t]), an expert
-    W_down (act(W_gate h) * (W_up h)).  gate_up [2 C, width] and down [width, C] with C = n_experts * ff + shared_ff units,
-    the experts' one after another, then the shared expert's (`shared_ff` 0: none); gate_up in groups of 16 rows, the
-    gates of 8 units and then their up-projections.  The choice is `choice` = (experts int32
-    [T, top], weights float32 [T, top]), or row token_t of `table` int32 [vocab, top] with weight 1 / top each.
-    out [T, width] float32, or of h's dtype."""
+    W_down (act(W_gate h) * (W_up h)).  gate_up [n_experts * 2 ff, width]: an expert's rows in groups of 16, the gates of 8
+    units and then their up-projections; down [n_experts * width, ff].  `shared` = (gate_up [2 fs, width], down [width, fs])
+    likewise, or None.  The choice is `choice` = (experts int32 [T, top], weights float32 [T, top]), or row token_t of
+    `table` int32 [vocab, top] with weight 1 / top each.  out [T, width] float32.
+
+    bfloat16: up to MOE_GEMV_MAX_ROWS tokens two skinny products that read the chosen experts' weights once; more tokens
+    grouped products over the (token, expert) pairs in order of their experts, the shared expert beside them as a dense
+    feed-forward.  Everything else (32-bit, widths that are no multiples of 8): a warp per (pair, unit)."""
     idx, wts = choice if choice is not None else (None, None)
-    _cuda(h, gate_up, down, out, idx, wts, table, gate_logits)
+    gate_up_s, down_s = shared if shared is not None else (None, None)
+    _cuda(h, gate_up, down, out, idx, wts, table, gate_logits, gate_up_s, down_s)
     T, width = ctx.n_tokens, h.shape[-1]
-    C = n_experts * ff + shared_ff
-    _need(tuple(gate_up.shape) == (2 * C, width) and tuple(down.shape) == (width, C) and gate_up.is_contiguous()
-          and down.is_contiguous() and gate_up.dtype == h.dtype and down.dtype == h.dtype and ff % 8 == 0
-          and shared_ff % 8 == 0,
-          f"moe_shared_experts: gate_up [{2 * C}, {width}], down [{width}, {C}] of h's dtype, inner sizes multiples of 8")
+    ff, fs = down.shape[1], 0 if shared is None else down_s.shape[1]
+    _need(tuple(gate_up.shape) == (n_experts * 2 * ff, width) and tuple(down.shape) == (n_experts * width, ff) and ff % 8 == 0
+          and gate_up.is_contiguous() and down.is_contiguous() and gate_up.dtype == h.dtype and down.dtype == h.dtype,
+          "moe_shared_experts: gate_up [experts * 2 ff, width], down [experts * width, ff] of h's dtype, ff a multiple of 8")
+    if shared is not None:
+        _need(tuple(gate_up_s.shape) == (2 * fs, width) and tuple(down_s.shape) == (width, fs) and fs % 8 == 0
+              and gate_up_s.is_contiguous() and down_s.is_contiguous() and gate_up_s.dtype == h.dtype and down_s.dtype == h.dtype,
+              "moe_shared_experts: the shared expert's gate_up [2 fs, width], down [width, fs] of h's dtype, fs a multiple of 8")
+        _need(gate_logits is not None and gate_logits.dtype == torch.float32 and gate_logits.is_contiguous()
+              and gate_logits.numel() >= T, "moe_shared_experts: the shared expert's gate logits float32 [T]")
     _need(h.is_contiguous() and h.numel() >= T * width and out.is_contiguous() and out.shape[-1] == width
-          and out.numel() >= T * width and out.dtype in (torch.float32, h.dtype),
-          "moe_shared_experts: h [T, width], out [T, width] float32 or of h's dtype")
+          and out.numel() >= T * width and out.dtype == torch.float32, "moe_shared_experts: h [T, width], out float32 [T, width]")
     _need((choice is None) != (table is None), "moe_shared_experts: the choice is a router's or a table's")
+    _need(0 < top <= n_experts <= 1024, f"moe_shared_experts: {top} of {n_experts} experts (up to 1024)")
     if choice is not None:
         _i32(idx, T * top, "experts")
         _need(wts.dtype == torch.float32 and wts.is_contiguous() and wts.numel() >= T * top, "weights float32 [T, top]")
@@ -2148,34 +2181,39 @@ def moe_shared_experts(h, gate_up, down, n_experts, ff, shared_ff, top, out, ctx
         _i32(ctx.tokens, T, "tokens")
         _need(table.dtype == torch.int32 and table.is_contiguous() and table.dim() == 2 and table.shape[1] == top,
               "the experts' table must be contiguous int32 [vocab, top]")
-    if shared_ff:
-        _need(gate_logits is not None and gate_logits.dtype == torch.float32 and gate_logits.is_contiguous()
-              and gate_logits.numel() >= T, "moe_shared_experts: the shared expert's gate logits float32 [T]")
-    by = (_p(idx), _p(wts), _p(table), _p(ctx.tokens) if table is not None else None, ctypes.c_float(1.0 / top),
-          _p(gate_logits))
-    if h.dtype == torch.bfloat16 and MOE_ALL_EXPERTS_MIN_ROWS <= T <= 65535:
-        up = torch.empty((T, 2 * C), dtype=h.dtype, device=h.device)
-        torch.mm(h[:T], gate_up.t(), out=up)
-        _mark("library product")
-        act = torch.empty((T, C), dtype=h.dtype, device=h.device)
-        _check(_lib("moe").ab_moe_shared_weigh(_p(up), _p(act), *by, T, top, ff, shared_ff, n_experts, MOE_ACTIVATIONS[activation],
-                                               _stream()), "moe_weigh_all")
-        if out.dtype == torch.float32:
-            torch.mm(act, down.t(), out_dtype=torch.float32, out=out[:T])
-        else:
-            torch.mm(act, down.t(), out=out[:T])
-        _mark("library product")
+    by = (_p(idx), _p(wts), _p(table), _p(ctx.tokens) if table is not None else None, ctypes.c_float(1.0 / top))
+    z = _p(gate_logits) if shared is not None else None
+    dev, code = h.device, MOE_ACTIVATIONS[activation]
+    fast = h.dtype == torch.bfloat16 and width % 8 == 0
+    if fast and T > MOE_GEMV_MAX_ROWS and activation == "silu":
+        n_tiles = T * top // 128 + n_experts
+        pos = torch.empty(T * top, dtype=torch.int32, device=dev)
+        plan = torch.empty(n_tiles + 1, dtype=torch.int32, device=dev)
+        rows = torch.empty((n_tiles * 128, width), dtype=h.dtype, device=dev)
+        _check(_lib("moe").ab_moe_gather(_p(h), *by, _p(pos), _p(plan), _p(plan[n_tiles:]), _p(rows), T, top, width, n_experts,
+                                         _stream()), "moe_gather", kernels=2)
+        act = torch.empty((n_tiles * 128, ff), dtype=h.dtype, device=dev)
+        gemm_tc_grouped(rows, gate_up, act, n_experts, plan[:n_tiles], plan[n_tiles:], swiglu=True)
+        gemm_tc_grouped(act, down, rows, n_experts, plan[:n_tiles], plan[n_tiles:])
+        ys = None
+        if shared is not None:
+            act_s = torch.empty((T, fs), dtype=h.dtype, device=dev)
+            if T >= TC_PERSISTENT_MIN_ROWS:
+                gemm_tc(h, gate_up_s, act_s, n_rows=T, swiglu=True, swap=False)
+            else:
+                gated_act(linear_bf16(h, gate_up_s, torch.empty((T, 2 * fs), dtype=h.dtype, device=dev), n_rows=T), act_s, n_rows=T)
+            ys = linear_bf16(act_s, down_s, torch.empty((T, width), dtype=h.dtype, device=dev), n_rows=T)
+        _check(_lib("moe").ab_moe_combine(_p(rows), _p(pos), *by, _p(ys), z, _p(out), T, top, width, _stream()), "moe_combine")
         return out
-    act = torch.empty((max(T, 1), top * ff + shared_ff), dtype=h.dtype, device=h.device)
-    if h.dtype == torch.bfloat16 and out.dtype == torch.float32 and width % 8 == 0 and T <= 32 and n_experts <= 512:
-        # few tokens: weights read once for all tokens that chose an expert
+    act = torch.empty((max(T, 1), top * ff + fs), dtype=h.dtype, device=dev)
+    if fast and T <= MOE_GEMV_MAX_ROWS and n_experts <= 512 and top <= 32:
         slabs, slices = -(-width // 16), 1
-        while slices < 8 and slabs * slices * 4 < 3 * _sm_count(h.device):
+        while slices < 8 and slabs * slices * 4 < 3 * _sm_count(dev):
             slices *= 2
-        _check(_lib("moe_gemv").ab_moe_gemv(_p(h), _p(gate_up), _p(down), *by, _p(act), _p(out), T, top, width, ff, shared_ff,
-                                            n_experts, MOE_ACTIVATIONS[activation], slices, _stream()), "moe_experts", kernels=2)
+        _check(_lib("moe_gemv").ab_moe_gemv(_p(h), _p(gate_up), _p(down), _p(gate_up_s), _p(down_s), *by, z, _p(act), _p(out), T,
+                                            top, width, ff, fs, n_experts, code, slices, _stream()), "moe_experts", kernels=2)
         return out
-    _check(_lib("moe").ab_moe_shared_pairs(_p(h), _dt(h), width, _p(gate_up), _p(down), *by, _p(act), _p(out), _dt(out), T, top,
-                                           width, ff, shared_ff, n_experts, MOE_ACTIVATIONS[activation], _stream()),
+    _check(_lib("moe").ab_moe_shared_pairs(_p(h), _dt(h), width, _p(gate_up), _p(down), _p(gate_up_s), _p(down_s), *by, z, _p(act),
+                                           _p(out), _dt(out), T, top, width, ff, fs, n_experts, code, _stream()),
            "moe_experts", kernels=2)
     return out

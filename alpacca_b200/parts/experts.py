@@ -93,7 +93,7 @@ class RoutedExperts(FeedForward):
 
 class TableExperts(FeedForward):
     """Gated experts that the token's id chooses: row token of a table [vocab, top] names a token's experts (all different),
-    each with weight 1 / top; there is no router.
+    each with weight 1 / top; there is no router.  The output is float32.
 
         out = sum_k E_(e_k)(h) / top + sigmoid(w_s . h) S(h),       E(h) = W_down (act(W_gate h) * (W_up h))
 
@@ -101,15 +101,15 @@ class TableExperts(FeedForward):
     formed in 32-bit.  A block whose kernel has the stream's row in registers may form it there: `row_gate()` is the
     vector w_s, and `forward` takes the products as `gate_logits`.
 
-    The matrices lie together (the experts' units one after another, then the shared expert's; gates and up-projections
-    interleaved in groups of 8 rows), the inner sizes padded with zero units to multiples of 8, so that few tokens run two
-    skinny products that read the chosen experts' weights once (csrc/moe_gemv.cu) and many tokens two library products
-    with the units of experts that were not chosen set to zero (csrc/moe.cu).  The table is read by the kernels: routing never reaches the host."""
+    The experts' matrices are stacked, gates and up-projections interleaved in groups of 8 rows, the inner sizes padded with
+    zero units to multiples of 8.  Few tokens run two skinny products that read the chosen experts' weights once
+    (csrc/moe_gemv.cu); many tokens grouped products over the (token, expert) pairs in order of their experts (csrc/moe.cu,
+    csrc/gemm_tc.cu).  The table is read by the kernels: routing never reaches the host."""
 
     def __init__(self, opts: BuildOptions, width: int, inner: int, n_experts: int, top: int, vocab: int, prefix: str,
                  activation: str = "silu", shared_inner: int = 0, table_name: str = "table",
                  expert_names=("e{}.gate", "e{}.up", "e{}.down"), shared_names=("shared.gate", "shared.up", "shared.down"),
-                 shared_gate: str = "shared.sg", out_dtype=None):
+                 shared_gate: str = "shared.sg"):
         if activation not in ops.MOE_ACTIVATIONS:
             raise ValueError(f"activation must be one of {tuple(ops.MOE_ACTIVATIONS)}, got {activation!r}")
         if not 0 < top <= n_experts:
@@ -117,9 +117,7 @@ class TableExperts(FeedForward):
         self.opts, self.width, self.inner, self.E, self.top = opts, int(width), int(inner), int(n_experts), int(top)
         self.vocab, self.prefix, self.activation, self.shared_inner = int(vocab), prefix, activation, int(shared_inner)
         self.table_name, self.expert_names, self.shared_names, self.shared_gate = table_name, expert_names, shared_names, shared_gate
-        self.out_dtype = out_dtype or opts.dtype
-        self.ff, self.fs = -(-self.inner // 8) * 8, -(-self.shared_inner // 8) * 8
-        self.table = self.gate_up = self.down = self.w_sg = None
+        self.table = self.gate_up = self.down = self.shared = self.w_sg = None
 
     def own_param_specs(self):
         p = self.prefix
@@ -142,18 +140,25 @@ class TableExperts(FeedForward):
         self.table = fetch(specs[0])
         if int(self.table.min()) < 0 or int(self.table.max()) >= self.E:
             raise WeightError(f"{specs[0].name} names experts outside 0..{self.E - 1}")
-        C = self.E * self.ff + self.fs
-        for i in range(self.E + (1 if self.shared_inner else 0)):
-            g, u, d = (fetch(s) for s in specs[1 + 3 * i:4 + 3 * i])
-            if i == 0:
-                gate_up = torch.zeros((2, C, self.width), dtype=g.dtype, device=g.device)
-                self.down = torch.zeros((self.width, C), dtype=g.dtype, device=g.device)
-            at, n = i * self.ff, g.shape[0]
-            gate_up[0, at:at + n], gate_up[1, at:at + n], self.down[:, at:at + n] = g, u, d
-        # groups of 16 rows: the gates of 8 units, then their up-projections
-        self.gate_up = gate_up.view(2, C // 8, 8, self.width).transpose(0, 1).reshape(2 * C, self.width).contiguous()
+        ff = -(-self.inner // 8) * 8
+        for e in range(self.E):
+            gate_up, down = self._laid_out(*(fetch(s) for s in specs[1 + 3 * e:4 + 3 * e]))
+            if e == 0:
+                self.gate_up = torch.empty((self.E, 2 * ff, self.width), dtype=down.dtype, device=down.device)
+                self.down = torch.empty((self.E, self.width, ff), dtype=down.dtype, device=down.device)
+            self.gate_up[e], self.down[e] = gate_up, down
+        self.gate_up, self.down = self.gate_up.view(-1, self.width), self.down.view(-1, ff)
+        if self.shared_inner:
+            self.shared = self._laid_out(*(fetch(s) for s in specs[1 + 3 * self.E:4 + 3 * self.E]))
         if self.shared_inner:
             self.w_sg = fetch(specs[-1]).reshape(-1).contiguous()
+
+    def _laid_out(self, gate, up, down):
+        """(gate|up in groups of 16 rows: the gates of 8 units, then their up-projections; down), padded to whole groups."""
+        more = -gate.shape[0] % 8
+        gate, up = (torch.nn.functional.pad(w, (0, 0, 0, more)).view(-1, 8, self.width) for w in (gate, up))
+        return (torch.cat([gate, up], dim=1).reshape(-1, self.width).contiguous(),
+                torch.nn.functional.pad(down, (0, more)).contiguous())
 
     def row_gate(self):
         """The vector (float32 [width]) whose product with this part's input is the shared expert's gate logit."""
@@ -162,6 +167,6 @@ class TableExperts(FeedForward):
     def forward(self, h, ctx, gate_logits=None):
         if self.shared_inner and gate_logits is None:
             gate_logits = ops.row_dots(h, self.w_sg, ctx.n_tokens)
-        out = torch.empty((h.shape[0], self.width), dtype=self.out_dtype, device=h.device)
-        return ops.moe_shared_experts(h, self.gate_up, self.down, self.E, self.ff, self.fs, self.top, out, ctx,
-                                      activation=self.activation, table=self.table, gate_logits=gate_logits)
+        out = torch.empty((h.shape[0], self.width), dtype=torch.float32, device=h.device)
+        return ops.moe_shared_experts(h, self.gate_up, self.down, self.E, self.top, out, ctx, activation=self.activation,
+                                      table=self.table, shared=self.shared, gate_logits=gate_logits)

@@ -422,24 +422,25 @@ def test_plain_feed_forward(dtype, rows, width, ff):
 
 MOES = [  # width, experts, ff, top, shared
     (40, 6, 20, 3, 28), (64, 5, 24, 5, None), (48, 3, 9, 2, 17), (128, 16, 64, 4, 96), (37, 1, 8, 1, 8), (256, 8, 40, 1, 200),
+    (136, 70, 24, 6, 72),
 ]
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
-@pytest.mark.parametrize("rows", [1, 7, 9, 32, 33, 260])
+@pytest.mark.parametrize("rows", [1, 7, 9, 32, 33, 260, 1100])
 @pytest.mark.parametrize("width,E,ff,top,shared", MOES)
 def test_experts_by_token(dtype, rows, width, E, ff, top, shared):
-    """Few rows (per pair of token and expert) and many (all experts in two products), with the gate's logit formed by
-    the part itself and handed over."""
+    """Few rows (skinny products), many (grouped products, experts that nobody chose among them) and sizes that take the
+    kernels per pair, with the gate's logit formed by the part itself and handed over."""
     from alpacca_b200 import ops
     from alpacca_b200.engine.step import StepEntry
     from alpacca_b200.parts import TableExperts
     vocab = 30
-    part = TableExperts(opts_of(dtype), width, ff, E, top, vocab, "m", shared_inner=shared or 0, out_dtype=torch.float32)
+    part = TableExperts(opts_of(dtype, 2048), width, ff, E, top, vocab, "m", shared_inner=shared or 0)
     w = short(load_part(part, seed=E, dtype=dtype, std=0.3), "m")
     rng = np.random.default_rng(rows)
-    hs = PartHarness([], dtype)
-    toks = rng.integers(0, vocab, rows).tolist()
+    hs = PartHarness([], dtype, max_positions=2048)
+    toks = rng.integers(0, vocab if rows > 40 else 4, rows).tolist()
     ctx = hs.builder.build([StepEntry(hs.cache.alloc_slot(), toks, [])], [0], hs.cache)
     x, x64 = hidden(rng, rows, width, dtype)
     mlp = {"router": {"experts": E, "top": top}, "shared": {"ff": shared} if shared else None}
@@ -453,9 +454,13 @@ def test_experts_by_token(dtype, rows, width, E, ff, top, shared):
     # the same experts behind a choice that a router would hand over
     idx = part.table[torch.tensor(toks, device="cuda").long()].contiguous()
     out = torch.empty((rows, width), dtype=torch.float32, device="cuda")
-    ops.moe_shared_experts(x, part.gate_up, part.down, E, part.ff, part.fs, top, out, ctx,
-                           choice=(idx, torch.full((rows, top), 1.0 / top, device="cuda")),
+    share = rng.uniform(0.2, 1.5, (rows, top))
+    ops.moe_shared_experts(x, part.gate_up, part.down, E, top, out, ctx, choice=(idx, dev(share)), shared=part.shared,
                            gate_logits=dev(x64 @ w["shared.sg"][0]) if shared else None)
+    want = plain.shared_expert(x64, w) if shared else np.zeros((rows, width))
+    for t in range(rows):
+        for k, e in enumerate(idx[t].tolist()):
+            want[t] += f64(share)[t, k] * plain.gated(x64[t], w[f"e{e}.gate"], w[f"e{e}.up"], w[f"e{e}.down"])
     close(out.cpu().numpy(), want, dtype, "experts behind a router's choice", tol=tol)
 
 
