@@ -394,8 +394,15 @@ attention_prepare_rows_vec_kernel(PrepareArgs a) {
       if (i < pq) sq += s; else sk += s;
     }
   }
-  sq = block_sum(sq, scratch);
-  if (pk > 0) sk = block_sum(sk, scratch + 32);
+  {                                                   // both sums over the block at once
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = blockDim.x >> 5;
+    sq = warp_sum(sq);
+    sk = warp_sum(sk);
+    if (lane == 0) { scratch[warp] = sq; scratch[32 + warp] = sk; }
+    __syncthreads();
+    sq = warp_sum(lane < nw ? scratch[lane] : 0.f);
+    sk = warp_sum(lane < nw ? scratch[32 + lane] : 0.f);
+  }
   const float iq = 1.0f / sqrtf(sq / (float)(pq * 8) + a.eps), ik = pk > 0 ? 1.0f / sqrtf(sk / (float)(pk * 8) + a.eps) : 0.f;
 #pragma unroll
   for (int j = 0; j < NP; ++j) {

@@ -170,6 +170,95 @@ input_conv_kernel(const float* __restrict__ x, const float* __restrict__ w, floa
   }
 }
 
+// The same for steps of many tokens, TAPS of 2 to 4 and widths that are multiples of 4: a thread keeps its channels' taps and the last rows in
+// registers and walks CONV_RUN packed tokens, so that a row is read once.  The tokens whose taps reach before the step
+// are left to the block whose run holds the sequence's first token, which does them as the kernel above does.
+#define CONV_RUN 8
+template <typename T, int TAPS>
+__global__ void __launch_bounds__(256)
+input_conv_run_kernel(const float* __restrict__ x, const float* __restrict__ w, float* __restrict__ state, T* __restrict__ out,
+                      const int* __restrict__ tok_seq, const int* __restrict__ cu_q, const int* __restrict__ slots,
+                      int n_tokens, int width, int write_state) {
+  constexpr int KEEP = TAPS - 1;
+  const int c = (blockIdx.y * blockDim.x + threadIdx.x) * 4;
+  float4 wv[TAPS];
+  if (c < width)
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j) wv[j] = *reinterpret_cast<const float4*>(w + (size_t)j * width + c);
+  pdl_wait();
+  pdl_trigger();
+  if (c >= width) return;
+  const int t0 = blockIdx.x * CONV_RUN, t1 = min(t0 + CONV_RUN, n_tokens);
+  auto row = [&](int t) { return *reinterpret_cast<const float4*>(x + (size_t)t * width + c); };
+  auto emit = [&](int t, const float4 (&prev)[KEEP], float4 cur) {
+    float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+    for (int j = 0; j < KEEP; ++j) acc = fma4(wv[j], prev[j], acc);
+    acc = fma4(wv[KEEP], cur, acc);
+    Quad<T>::store(out + (size_t)t * width + c, make_float4(cur.x + acc.x, cur.y + acc.y, cur.z + acc.z, cur.w + acc.w));
+  };
+  float4 prev[KEEP];
+  {
+    // the usual case: a whole run inside one sequence, past its first KEEP tokens: every row is asked for at once
+    const int b = tok_seq[t0];
+    if (b >= 0 && t1 - t0 == CONV_RUN && tok_seq[t1 - 1] == b && t0 - cu_q[b] >= KEEP) {
+      float4 r[CONV_RUN + KEEP];
+#pragma unroll
+      for (int j = 0; j < CONV_RUN + KEEP; ++j) r[j] = row(t0 - KEEP + j);
+#pragma unroll
+      for (int q = 0; q < CONV_RUN; ++q) {
+#pragma unroll
+        for (int j = 0; j < KEEP; ++j) prev[j] = r[q + j];
+        emit(t0 + q, prev, r[q + KEEP]);
+      }
+      return;
+    }
+  }
+  bool have = false;                       // prev holds the rows before token t
+  for (int t = t0; t < t1; ++t) {
+    const int b = tok_seq[t];
+    if (b < 0) {
+      Quad<T>::store(out + (size_t)t * width + c, make_float4(0.f, 0.f, 0.f, 0.f));
+      have = false;
+      continue;
+    }
+    const int first = cu_q[b];
+    const int i = t - first;
+    if (i >= KEEP) {
+      if (!have)
+#pragma unroll
+        for (int j = 0; j < KEEP; ++j) prev[j] = row(t - KEEP + j);
+      const float4 cur = row(t);
+      emit(t, prev, cur);
+#pragma unroll
+      for (int j = 0; j + 1 < KEEP; ++j) prev[j] = prev[j + 1];
+      prev[KEEP - 1] = cur;
+      have = true;
+      continue;
+    }
+    have = false;
+    if (i > 0) continue;
+    // a sequence's first token: its first KEEP tokens from the kept rows on, then the new kept rows
+    const int n = cu_q[b + 1] - first;
+    float* st = state + (size_t)slots[b] * KEEP * width + c;
+#pragma unroll
+    for (int j = 0; j < KEEP; ++j) prev[j] = *reinterpret_cast<const float4*>(st + (size_t)j * width);
+    for (int q = 0; q < KEEP && q < n; ++q) {
+      const float4 cur = row(first + q);
+      emit(first + q, prev, cur);
+#pragma unroll
+      for (int j = 0; j + 1 < KEEP; ++j) prev[j] = prev[j + 1];
+      prev[KEEP - 1] = cur;
+    }
+    if (write_state)
+#pragma unroll
+      for (int j = 0; j < KEEP; ++j) {      // after fewer than KEEP tokens `prev` holds old and new rows, in order
+        const float4 v = n < KEEP ? prev[j] : row(first + n - KEEP + j);
+        *reinterpret_cast<float4*>(st + (size_t)j * width) = v;
+      }
+  }
+}
+
 AB_API int ab_input_conv(const float* x, const float* w, float* state, void* out, int dtype, const int* tok_seq,
                          const int* cu_q, const int* slots, int n_tokens, int width, int taps, int write_state,
                          cudaStream_t stream) {
@@ -179,6 +268,16 @@ AB_API int ab_input_conv(const float* x, const float* w, float* state, void* out
   const int units = vec ? width / 4 : width;
   const int threads = units >= 256 ? 256 : (units + 31) / 32 * 32;
   const dim3 grid((unsigned)n_tokens, (unsigned)((units + threads - 1) / threads));
+  if (n_tokens >= 256 && vec && taps >= 2 && taps <= 4 && (dtype == AB_F32 || dtype == AB_BF16)) {
+    const dim3 runs((unsigned)((n_tokens + CONV_RUN - 1) / CONV_RUN), grid.y);
+#define AB_RUN(T, TAPS)                                                                                               \
+  ab_launch(input_conv_run_kernel<T, TAPS>, runs, dim3(threads), 0, stream, x, w, state, (T*)out, tok_seq, cu_q, slots, \
+            n_tokens, width, write_state)
+    if (dtype == AB_F32) { if (taps == 2) AB_RUN(float, 2); else if (taps == 3) AB_RUN(float, 3); else AB_RUN(float, 4); }
+    else { if (taps == 2) AB_RUN(bf16, 2); else if (taps == 3) AB_RUN(bf16, 3); else AB_RUN(bf16, 4); }
+#undef AB_RUN
+    return ab_launch_status();
+  }
 #define AB_GO(T, NC)                                                                                                 \
   ab_launch(input_conv_kernel<T, NC>, grid, dim3(threads), 0, stream, x, w, state, (T*)out, tok_seq, cu_q, slots, width, taps, \
             write_state)
@@ -222,7 +321,7 @@ __device__ __forceinline__ void block_sum3(float& a, float& b, float& c, float* 
 // A block per row, the row in registers: RV x 4 numbers per thread (widths that are multiples of 4).  What earlier
 // layers left (the history, the convolution's kept rows) was written at least two kernels ago: it is asked for before
 // the wait for the kernel before this one.
-template <typename TY, typename TO, int RV>
+template <typename TY, typename TO, int RV, bool CONV>
 __global__ void __launch_bounds__(512)
 post_norm_stream_reg_kernel(const PostArgs a) {
   __shared__ float scratch[96];
@@ -260,6 +359,21 @@ post_norm_stream_reg_kernel(const PostArgs a) {
     }
     c_last = a.coef[a.n_hist];
   }
+  // the next convolution's kept rows (up to three of them; a longer convolution fetches its rows one after another below)
+  const int keep = a.taps - 1;
+  float* st = CONV && keep > 0 ? a.conv_state + (size_t)a.slots[b] * keep * width : nullptr;
+  constexpr int EARLY = CONV && RV <= 2 ? 3 : 0;
+  const bool early = CONV && keep <= EARLY;
+  float4 kept[EARLY > 0 ? EARLY : 1][RV];
+  if (early) {
+#pragma unroll
+    for (int k = 0; k < EARLY; ++k)
+#pragma unroll
+      for (int j = 0; j < RV; ++j) {
+        const int i = (threadIdx.x + j * blockDim.x) * 4;
+        if (k < keep && i < width) kept[k][j] = *reinterpret_cast<const float4*>(st + (size_t)k * width + i);
+      }
+  }
   pdl_wait();
   pdl_trigger();
   float4 yv[RV], xv[RV];
@@ -285,8 +399,6 @@ post_norm_stream_reg_kernel(const PostArgs a) {
   block_sum3(ss, xg, yg, scratch);
   const float inv = 1.0f / sqrtf(ss / (float)width + a.eps);
   if (a.dots != nullptr && threadIdx.x == 0) a.dots[t] = fmaf(inv, yg, xg);
-  const int keep = a.taps - 1;
-  float* st = a.conv_w != nullptr && keep > 0 ? a.conv_state + (size_t)a.slots[b] * keep * width : nullptr;
 #pragma unroll
   for (int j = 0; j < RV; ++j) {
     const int i = (threadIdx.x + j * blockDim.x) * 4;
@@ -298,10 +410,18 @@ post_norm_stream_reg_kernel(const PostArgs a) {
       *reinterpret_cast<float4*>(a.avg_out + row + i) = v;
     }
     if (a.out == nullptr) continue;
-    if (a.conv_w != nullptr) {
+    if (CONV) {
       // the next layer's convolution: the kept rows, then this one; the kept rows move up by one
       float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
-      for (int k = 0; k < keep; ++k) {
+      if (early) {
+#pragma unroll
+        for (int k = 0; k < EARLY; ++k)
+          if (k < keep) {
+            acc = fma4(*reinterpret_cast<const float4*>(a.conv_w + (size_t)k * width + i), kept[k][j], acc);
+            if (k > 0) *reinterpret_cast<float4*>(st + (size_t)(k - 1) * width + i) = kept[k][j];
+          }
+      }
+      for (int k = early ? keep : 0; k < keep; ++k) {
         const float4 s = *reinterpret_cast<const float4*>(st + (size_t)k * width + i);
         acc = fma4(*reinterpret_cast<const float4*>(a.conv_w + (size_t)k * width + i), s, acc);
         if (k > 0) *reinterpret_cast<float4*>(st + (size_t)(k - 1) * width + i) = s;
@@ -383,12 +503,18 @@ AB_API int ab_post_norm_stream(const float* x, const void* y, int y_dtype, const
   const bool of = !out || out_dtype == AB_F32;
   const int threads = width >= 4096 ? 512 : (width >= 1024 ? 256 : 128);
   const int rv = width % 4 == 0 ? (width / 4 + threads - 1) / threads : 99;
-#define AB_REG(TY, TO, RV) ab_launch(post_norm_stream_reg_kernel<TY, TO, RV>, dim3((unsigned)n_rows), dim3(threads), 0, stream, a)
+#define AB_REG(TY, TO, RV)                                                                                              \
+  {                                                                                                                     \
+    if (conv_w != nullptr)                                                                                              \
+      ab_launch(post_norm_stream_reg_kernel<TY, TO, RV, true>, dim3((unsigned)n_rows), dim3(threads), 0, stream, a);    \
+    else                                                                                                                \
+      ab_launch(post_norm_stream_reg_kernel<TY, TO, RV, false>, dim3((unsigned)n_rows), dim3(threads), 0, stream, a);   \
+  }
 #define AB_GO(TY, TO)                                                                                            \
   {                                                                                                              \
-    if (rv <= 1) AB_REG(TY, TO, 1);                                                                              \
-    else if (rv <= 2) AB_REG(TY, TO, 2);                                                                         \
-    else if (rv <= 4) AB_REG(TY, TO, 4);                                                                         \
+    if (rv <= 1) AB_REG(TY, TO, 1)                                                                               \
+    else if (rv <= 2) AB_REG(TY, TO, 2)                                                                          \
+    else if (rv <= 4) AB_REG(TY, TO, 4)                                                                          \
     else ab_launch(post_norm_stream_kernel<TY, TO>, dim3((unsigned)n_rows), dim3(256), 0, stream, a);            \
   }
   if (y_dtype == AB_F32) { if (of) AB_GO(float, float) else AB_GO(float, bf16) }

@@ -662,8 +662,22 @@ moe_plan_kernel(Choice c, int n_tokens, int top, int E, int* __restrict__ pos, i
   pdl_trigger();
   for (int e = threadIdx.x; e < E; e += blockDim.x) count[e] = 0;
   __syncthreads();
+  // eight pairs per thread at a time, their loads together; the first eight stay in registers for the second pass
   const int n_pairs = n_tokens * top;
-  for (int p = threadIdx.x; p < n_pairs; p += blockDim.x) atomicAdd(&count[chosen_expert(c, p / top, p % top, top)], 1);
+  int mine[8];
+  for (int p0 = threadIdx.x; p0 < n_pairs; p0 += 8 * blockDim.x) {
+    int e[8];
+#pragma unroll
+    for (int j = 0; j < 8; ++j) {
+      const int p = p0 + j * blockDim.x;
+      e[j] = p < n_pairs ? chosen_expert(c, p / top, p % top, top) : -1;
+    }
+#pragma unroll
+    for (int j = 0; j < 8; ++j) {
+      if (e[j] >= 0) atomicAdd(&count[e[j]], 1);
+      if (p0 == (int)threadIdx.x) mine[j] = e[j];
+    }
+  }
   __syncthreads();
   if (threadIdx.x < 32) {                      // the experts' first row tiles: a running sum over lanes
     int before = 0;
@@ -685,8 +699,17 @@ moe_plan_kernel(Choice c, int n_tokens, int top, int E, int* __restrict__ pos, i
     if (threadIdx.x == 0) *row_tiles = before;
   }
   __syncthreads();
-  for (int p = threadIdx.x; p < n_pairs; p += blockDim.x)
-    pos[p] = atomicAdd(&first[chosen_expert(c, p / top, p % top, top)], 1);
+  for (int p0 = threadIdx.x; p0 < n_pairs; p0 += 8 * blockDim.x) {
+    int e[8];
+#pragma unroll
+    for (int j = 0; j < 8; ++j) {
+      const int p = p0 + j * blockDim.x;
+      e[j] = p0 == (int)threadIdx.x ? mine[j] : p < n_pairs ? chosen_expert(c, p / top, p % top, top) : -1;
+    }
+#pragma unroll
+    for (int j = 0; j < 8; ++j)
+      if (e[j] >= 0) pos[p0 + j * blockDim.x] = atomicAdd(&first[e[j]], 1);
+  }
 }
 
 // rows[pos[t, k]] = h[t] for every choice k; 16-byte pieces (width a multiple of 8)

@@ -197,54 +197,55 @@ moe_gemv_down_kernel(const bf16* __restrict__ act, const bf16* __restrict__ W, c
 #pragma unroll
   for (int i = 0; i < NT; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
   bool waited = false;
-  for (int grp = begin; grp < end; grp += MG_U) {
-    uint4 wl[MG_U], wh[MG_U];
+  for (int at = begin; at < end;) {
+    // the part of this run that lies in one expert: groups g0 .. g1 of its `len` units
+    const int ai = min(at / ge, n_active);
+    const bool sh = ai == n_active;
+    const int len = sh ? fs : ff;
+    const int g0 = at - ai * ge, g1 = min(end - ai * ge, sh ? gs : ge);
+    const bf16* w = sh ? Ws : W + (size_t)active[ai] * N * ff;
+    const bf16 *w_lo = w + lo * len, *w_hi = w + hi * len;
+    const bf16* x_row[NT];
+    bool x_ok[NT];
 #pragma unroll
-    for (int u = 0; u < MG_U; ++u) {
-      wl[u] = wh[u] = make_uint4(0, 0, 0, 0);
-      const int at = grp + u;
-      if (at < end) {
-        const int ai = at / ge;
-        const bool sh = ai >= n_active;
-        const int k = (sh ? at - n_active * ge : at - ai * ge) * 32 + t * 8;
-        if (k < (sh ? fs : ff)) {
-          const bf16* w = sh ? Ws + k : W + (size_t)active[ai] * N * ff + k;
-          wl[u] = mg_stream(w + lo * (sh ? fs : ff));
-          wh[u] = mg_stream(w + hi * (sh ? fs : ff));
+    for (int i = 0; i < NT; ++i) {
+      const int tok = i * 8 + g;
+      const int slot = sh ? (tok < M ? top : -1) : slot_of[active[ai]][tok];
+      x_ok[i] = slot >= 0;
+      x_row[i] = act + (x_ok[i] ? (size_t)tok * row_len + (size_t)slot * ff : 0);
+    }
+    for (int grp = g0; grp < g1; grp += MG_U) {
+      uint4 wl[MG_U], wh[MG_U];
+#pragma unroll
+      for (int u = 0; u < MG_U; ++u) {
+        const int k = (grp + u) * 32 + t * 8;
+        wl[u] = wh[u] = make_uint4(0, 0, 0, 0);
+        if (grp + u < g1 && k < len) {
+          wl[u] = mg_stream(w_lo + k);
+          wh[u] = mg_stream(w_hi + k);
         }
       }
-    }
-    if (!waited) { pdl_wait(); pdl_trigger(); waited = true; }
+      if (!waited) { pdl_wait(); pdl_trigger(); waited = true; }
 #pragma unroll
-    for (int u0 = 0; u0 < MG_U; u0 += 4) {
-      uint4 xv[4][NT];
+      for (int u0 = 0; u0 < MG_U; u0 += 4) {
+        uint4 xv[4][NT];
 #pragma unroll
-      for (int u = 0; u < 4; ++u) {
-        const int at = grp + u0 + u;
+        for (int u = 0; u < 4; ++u) {
+          const int k = (grp + u0 + u) * 32 + t * 8;
+          const bool in = grp + u0 + u < g1 && k < len;
 #pragma unroll
-        for (int i = 0; i < NT; ++i) xv[u][i] = make_uint4(0, 0, 0, 0);
-        if (at < end) {
-          const int ai = at / ge;
-          const bool sh = ai >= n_active;
-          const int k = (sh ? at - n_active * ge : at - ai * ge) * 32 + t * 8;
-          if (k < (sh ? fs : ff)) {
+          for (int i = 0; i < NT; ++i) xv[u][i] = (in && x_ok[i]) ? mg_act(x_row[i] + k) : make_uint4(0, 0, 0, 0);
+        }
 #pragma unroll
-            for (int i = 0; i < NT; ++i) {
-              const int tok = i * 8 + g;
-              const int slot = sh ? (tok < M ? top : -1) : slot_of[active[ai]][tok];
-              if (slot >= 0) xv[u][i] = mg_act(act + (size_t)tok * row_len + (size_t)slot * ff + k);
-            }
+        for (int u = 0; u < 4; ++u)
+#pragma unroll
+          for (int i = 0; i < NT; ++i) {
+            mg_mma(acc[i], wl[u0 + u].x, wh[u0 + u].x, wl[u0 + u].y, wh[u0 + u].y, xv[u][i].x, xv[u][i].y);
+            mg_mma(acc[i], wl[u0 + u].z, wh[u0 + u].z, wl[u0 + u].w, wh[u0 + u].w, xv[u][i].z, xv[u][i].w);
           }
-        }
       }
-#pragma unroll
-      for (int u = 0; u < 4; ++u)
-#pragma unroll
-        for (int i = 0; i < NT; ++i) {
-          mg_mma(acc[i], wl[u0 + u].x, wh[u0 + u].x, wl[u0 + u].y, wh[u0 + u].y, xv[u][i].x, xv[u][i].y);
-          mg_mma(acc[i], wl[u0 + u].z, wh[u0 + u].z, wl[u0 + u].w, wh[u0 + u].w, xv[u][i].z, xv[u][i].w);
-        }
     }
+    at = ai * ge + g1;
   }
   if (!waited) { pdl_wait(); pdl_trigger(); }
 #pragma unroll

@@ -120,6 +120,35 @@ def test_input_convolution_in_portions(dtype, width, taps):
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("width,taps", [(40, 2), (64, 3), (1032, 4), (37, 3), (24, 6)])
+def test_input_convolution_of_many_tokens(dtype, width, taps):
+    """Steps of hundreds of tokens, whose rows are walked in runs: sequences that start and end inside a run, some of one
+    or two tokens, continued by a second such step."""
+    from alpacca_b200.parts import InputConv
+    part = InputConv(opts_of(dtype), width, taps, "c")
+    w = load_part(part, seed=taps, dtype=dtype, std=0.5)["c"]
+    hs = PartHarness([part.cache_spec()], dtype, max_slots=8)
+    rng = np.random.default_rng(width)
+    lens = [(131, 1), (1, 200), (2, 1), (1, 2), (90, 3), (3, 77), (40, 8), (8, 64)]
+    x = [rng.normal(0, 1, (sum(n), width)).astype(np.float32) for n in lens]
+    slots = [hs.cache.alloc_slot() for _ in x]
+    got, at = [[] for _ in x], [0] * len(x)
+    for step in range(2):
+        ctx = hs.step([(s, n[step]) for s, n in zip(slots, lens)])
+        out = part.forward(dev(np.concatenate([x[i][at[i]:at[i] + lens[i][step]] for i in range(len(x))])), ctx,
+                           hs.cache.entry_view(0, ctx.block_tables)).float().cpu().numpy()
+        hs.done()
+        r = 0
+        for i, n in enumerate(lens):
+            got[i].append(out[r:r + n[step]])
+            r += n[step]
+            at[i] += n[step]
+    for i in range(len(x)):
+        close(np.concatenate(got[i]), plain.input_conv(x[i].astype(np.float64), w), dtype, f"convolution {i}",
+              tol=(5e-6, 5e-7) if dtype == "float32" else (0.03, 0.003))
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("width", [37, 256, 1000, 2048, 4100, 9000])
 def test_the_kernel_after_a_sublayer(dtype, width):
     """Every use of the kernel: the plain addition with the product per row and the cast; the average over 0 to 7 earlier
