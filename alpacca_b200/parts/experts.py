@@ -117,7 +117,7 @@ class TableExperts(FeedForward):
         self.opts, self.width, self.inner, self.E, self.top = opts, int(width), int(inner), int(n_experts), int(top)
         self.vocab, self.prefix, self.activation, self.shared_inner = int(vocab), prefix, activation, int(shared_inner)
         self.table_name, self.expert_names, self.shared_names, self.shared_gate = table_name, expert_names, shared_names, shared_gate
-        self.table = self.gate_up = self.down = self.shared = self.w_sg = None
+        self.table = self.gate_up = self.down = self.shared_gate_up = self.shared_down = self.w_sg = None
 
     def own_param_specs(self):
         p = self.prefix
@@ -149,7 +149,7 @@ class TableExperts(FeedForward):
             self.gate_up[e], self.down[e] = gate_up, down
         self.gate_up, self.down = self.gate_up.view(-1, self.width), self.down.view(-1, ff)
         if self.shared_inner:
-            self.shared = self._laid_out(*(fetch(s) for s in specs[1 + 3 * self.E:4 + 3 * self.E]))
+            self.shared_gate_up, self.shared_down = self._laid_out(*(fetch(s) for s in specs[1 + 3 * self.E:4 + 3 * self.E]))
         if self.shared_inner:
             self.w_sg = fetch(specs[-1]).reshape(-1).contiguous()
 
@@ -160,6 +160,10 @@ class TableExperts(FeedForward):
         return (torch.cat([gate, up], dim=1).reshape(-1, self.width).contiguous(),
                 torch.nn.functional.pad(down, (0, more)).contiguous())
 
+    def shared_weights(self):
+        """(gate|up, down) of the shared expert as the kernels read them, or None."""
+        return (self.shared_gate_up, self.shared_down) if self.shared_inner else None
+
     def row_gate(self):
         """The vector (float32 [width]) whose product with this part's input is the shared expert's gate logit."""
         return self.w_sg
@@ -169,4 +173,4 @@ class TableExperts(FeedForward):
             gate_logits = ops.row_dots(h, self.w_sg, ctx.n_tokens)
         out = torch.empty((h.shape[0], self.width), dtype=torch.float32, device=h.device)
         return ops.moe_shared_experts(h, self.gate_up, self.down, self.E, self.top, out, ctx, activation=self.activation,
-                                      table=self.table, shared=self.shared, gate_logits=gate_logits)
+                                      table=self.table, shared=self.shared_weights(), gate_logits=gate_logits)

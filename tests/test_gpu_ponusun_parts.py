@@ -484,7 +484,7 @@ def test_experts_by_token(dtype, rows, width, E, ff, top, shared):
     idx = part.table[torch.tensor(toks, device="cuda").long()].contiguous()
     out = torch.empty((rows, width), dtype=torch.float32, device="cuda")
     share = rng.uniform(0.2, 1.5, (rows, top))
-    ops.moe_shared_experts(x, part.gate_up, part.down, E, top, out, ctx, choice=(idx, dev(share)), shared=part.shared,
+    ops.moe_shared_experts(x, part.gate_up, part.down, E, top, out, ctx, choice=(idx, dev(share)), shared=part.shared_weights(),
                            gate_logits=dev(x64 @ w["shared.sg"][0]) if shared else None)
     want = plain.shared_expert(x64, w) if shared else np.zeros((rows, width))
     for t in range(rows):
