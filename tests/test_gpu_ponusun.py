@@ -168,6 +168,35 @@ def test_unequal_batch_against_each_alone(dirs, name, dtype):
 
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("name", ["a", "c"])
+def test_many_sequences_decoded_together(dirs, name, dtype):
+    """Forty prompts of one to five tokens in one step, then six steps of all forty (the experts' grouped products in a step
+    of one token each, from the third step on a graph replay with other tokens)."""
+    from alpacca_b200.engine.step import StepEntry
+    eng = engine_of(dirs, name, dtype, max_tokens=64 * 40, max_slots=40)
+    full = [some_tokens(name, 7 + i % 5, 500 + i) for i in range(40)]
+    slots = [eng.alloc_slot() for _ in full]
+    try:
+        got = [[] for _ in full]
+        out = eng.step([StepEntry(s, t[:-6], list(range(len(t) - 6))) for s, t in zip(slots, full)]).cpu().numpy()
+        at = 0
+        for i, t in enumerate(full):
+            got[i].append(out[at:at + len(t) - 6])
+            at += len(t) - 6
+        for k in range(6, 0, -1):
+            out = eng.step([StepEntry(s, [t[-k]], [0]) for s, t in zip(slots, full)]).cpu().numpy()
+            for i in range(40):
+                got[i].append(out[i:i + 1])
+        eng.wait()
+        want = np.concatenate([plain_logits(name, t) for t in full])
+        check(np.concatenate([np.concatenate(g) for g in got]), want, dtype, f"{name} forty together")
+    finally:
+        for s in slots:
+            eng.free_slot(s)
+    eng.cache.check()
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("name", ["a", "c"])
 def test_slots_and_pages_used_again(dirs, name, dtype):
     """A cache of five pages and two slots: every new sequence gets a slot and pages that another one has just given back,
     with its keys still in the pages and its last rows still among the convolutions' states."""
