@@ -47,7 +47,6 @@
 #define EPI_SWIGLU_BF16 2
 #define EPI_RELUGLU_BF16 3      // the same tail with max(g, 0) on the gate
 #define EPI_GELUGLU_BF16 4      // ... with the tanh form of GELU on the gate
-#define EPI_GELU_BF16 5         // no gate: GELU in its erf form on every column (bfloat16 store)
 
 __device__ __forceinline__ uint32_t smem_addr(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
 
@@ -117,11 +116,6 @@ __device__ __forceinline__ float gate_fast(float g) {
   return silu_fast(g);
 }
 
-template <int EPI>
-__device__ __forceinline__ float plain_tail(float y) {
-  return EPI == EPI_GELU_BF16 ? 0.5f * y * (1.0f + erff(y * 0.70710678118654752440f)) : y;
-}
-
 template <int BN> struct TcShape {
   // few columns: the kernel streams weights and is bound by bytes in flight, so a deep ring;
   // many columns: bound by the tensor cores, and two CTAs per SM overlap tails with main loops
@@ -142,7 +136,7 @@ __device__ __forceinline__ void tail16(const float* v, int row_g, int col0_g, in
   if (!SWAP) {
     const int m = row_g;
     if (m >= rows_total) return;
-    if (EPI >= EPI_SWIGLU_BF16 && EPI <= EPI_GELUGLU_BF16) {
+    if (EPI >= EPI_SWIGLU_BF16) {
       // columns col0..col0+7 gate, +8..+15 up of units (col0/16)*8 + 0..7
       if (col0_g + 16 > cols_total) return;
       bf16* y = reinterpret_cast<bf16*>(Y) + (size_t)m * ldy + (col0_g >> 1);
@@ -171,8 +165,8 @@ __device__ __forceinline__ void tail16(const float* v, int row_g, int col0_g, in
         uint32_t w[8];
 #pragma unroll
         for (int j = 0; j < 8; ++j) {
-          __nv_bfloat162 r = __floats2bfloat162_rn(plain_tail<EPI>(v[2 * j] + (bias ? bias[col0_g + 2 * j] : 0.f)),
-                                                   plain_tail<EPI>(v[2 * j + 1] + (bias ? bias[col0_g + 2 * j + 1] : 0.f)));
+          __nv_bfloat162 r = __floats2bfloat162_rn(v[2 * j] + (bias ? bias[col0_g + 2 * j] : 0.f),
+                                                   v[2 * j + 1] + (bias ? bias[col0_g + 2 * j + 1] : 0.f));
           w[j] = *reinterpret_cast<uint32_t*>(&r);
         }
         *reinterpret_cast<uint4*>(y) = make_uint4(w[0], w[1], w[2], w[3]);
@@ -180,7 +174,7 @@ __device__ __forceinline__ void tail16(const float* v, int row_g, int col0_g, in
       } else {
 #pragma unroll
         for (int c = 0; c < 16; ++c)
-          if (col0_g + c < cols_total) y[c] = __float2bfloat16_rn(plain_tail<EPI>(v[c] + (bias ? bias[col0_g + c] : 0.f)));
+          if (col0_g + c < cols_total) y[c] = __float2bfloat16_rn(v[c] + (bias ? bias[col0_g + c] : 0.f));
       }
     }
   } else {
@@ -821,7 +815,7 @@ AB_API int ab_gemm_tc(const void* X, const void* W, const float* bias, void* Y, 
                       cudaStream_t stream) {
   if (M <= 0 || N <= 0) return AB_OK;
   if (K <= 0 || (K % 8) || slices < 1) return AB_BAD_ARG;
-  if (epilogue_kind >= EPI_SWIGLU_BF16 && epilogue_kind <= EPI_GELUGLU_BF16 && (N % 16)) return AB_BAD_ARG;
+  if (epilogue_kind >= EPI_SWIGLU_BF16 && (N % 16)) return AB_BAD_ARG;
   if (slices > 1 && (!partials || !arrivals)) return AB_BAD_ARG;
   int* status = status_word();
   if (!status) return AB_BAD_ARG;
@@ -847,7 +841,7 @@ AB_API int ab_gemm_tc_persistent(const void* X, const void* W, const float* bias
                                  int ldy, int epilogue_kind, cudaStream_t stream) {
   if (M <= 0 || N <= 0) return AB_OK;
   if (K <= 0 || (K % 8)) return AB_BAD_ARG;
-  if (epilogue_kind >= EPI_SWIGLU_BF16 && epilogue_kind <= EPI_GELUGLU_BF16 && (N % 16)) return AB_BAD_ARG;
+  if (epilogue_kind >= EPI_SWIGLU_BF16 && (N % 16)) return AB_BAD_ARG;
   int* status = status_word();
   if (!status) return AB_BAD_ARG;
   CUtensorMap mx, mw;
@@ -877,7 +871,6 @@ AB_API int ab_gemm_tc_persistent(const void* X, const void* W, const float* bias
     case EPI_SWIGLU_BF16: AB_GO(EPI_SWIGLU_BF16)
     case EPI_RELUGLU_BF16: AB_GO(EPI_RELUGLU_BF16)
     case EPI_GELUGLU_BF16: AB_GO(EPI_GELUGLU_BF16)
-    case EPI_GELU_BF16: AB_GO(EPI_GELU_BF16)
   }
 #undef AB_GO
   return AB_BAD_ARG;
@@ -929,7 +922,7 @@ AB_API int ab_gemm_tc_pair(const void* X, const void* W, const float* bias, void
                            int ldy, int epilogue_kind, cudaStream_t stream) {
   if (M <= 0 || N <= 0) return AB_OK;
   if (K <= 0 || (K % 8)) return AB_BAD_ARG;
-  if (epilogue_kind >= EPI_SWIGLU_BF16 && epilogue_kind <= EPI_GELUGLU_BF16 && (N % 16)) return AB_BAD_ARG;
+  if (epilogue_kind >= EPI_SWIGLU_BF16 && (N % 16)) return AB_BAD_ARG;
   int* status = status_word();
   if (!status) return AB_BAD_ARG;
   CUtensorMap mx, mw;
@@ -972,7 +965,6 @@ AB_API int ab_gemm_tc_pair(const void* X, const void* W, const float* bias, void
     case EPI_SWIGLU_BF16: AB_GO(EPI_SWIGLU_BF16)
     case EPI_RELUGLU_BF16: AB_GO(EPI_RELUGLU_BF16)
     case EPI_GELUGLU_BF16: AB_GO(EPI_GELUGLU_BF16)
-    case EPI_GELU_BF16: AB_GO(EPI_GELU_BF16)
   }
 #undef AB_GO
   return AB_BAD_ARG;

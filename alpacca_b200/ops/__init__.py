@@ -788,8 +788,6 @@ def linear_bf16(x, w, out, n_rows=None, bias=None, start_early=True, owed=None, 
     if x.shape[1] % 8 == 0 and (n <= GEMV_MAX_ROWS or (n <= GEMV_NARROW_MAX_ROWS
                                                        and -(-w.shape[0] // 16) <= _sm_count(x.device))):
         return gemv_bf16(x, w, out, bias=bias, n_rows=n, start_early=start_early, owed=owed, act=act, cap=cap)
-    if act is not None and out.dtype == torch.bfloat16 and x.shape[1] % 8 == 0 and n >= TC_PERSISTENT_MIN_ROWS:
-        return gemm_tc(x, w, out, bias=bias, n_rows=n, swap=False, act=act)     # the activation in the product's tail
     _need(owed is None, "linear_bf16: only the skinny product finishes a norm that its input owes")
     xs, ys = (x, out) if n == x.shape[0] == out.shape[0] else (x[:n], out[:n])
     if out.dtype == torch.float32:
@@ -874,13 +872,12 @@ def decode_advance(tokens, tok_pos, kv_len, rng_step, tok_seq, sampled, recent, 
 
 
 def gemm_tc(x, w, out, bias=None, n_rows=None, swiglu=False, swap=None, bn=None, slices=None, persistent=True,
-            pair=None, activation="silu", act=None):
+            pair=None, activation="silu"):
     """out[:n] = x[:n] @ w^T (+ bias) on the tcgen05 tensor cores (TMA-fed, TMEM accumulators).
 
     x [M,K], w [N,K] bfloat16; out bfloat16 or float32 [M,N]; with `swiglu`, w is the 8-row
     interleaved gate|up matrix and out is bfloat16 [M, N/2] (`activation` on the gate: "silu"; "relu" and
-    "gelu_tanh" in the persistent forms only).  `act` ("gelu", bfloat16, persistent forms only): an activation
-    on a product without a gate.  `swap` puts the weights on the
+    "gelu_tanh" in the persistent forms only).  `swap` puts the weights on the
     128-row side of the MMA (the batch, up to 256 rows, becomes the columns): the shape for decode
     steps.  `bn` is the MMA's column count per tile, `slices` the number of K slices.  Without `swap`,
     256-wide tiles and one slice run as the persistent kernel (one CTA per SM walks the tiles) unless
@@ -909,10 +906,6 @@ def gemm_tc(x, w, out, bias=None, n_rows=None, swiglu=False, swap=None, bn=None,
     else:
         _need(out.shape[-1] == N and out.dtype in (torch.bfloat16, torch.float32), "gemm_tc: out [M,N]")
         epi = 1 if out.dtype == torch.float32 else 0
-        if act is not None:
-            _need(act == "gelu" and epi == 0 and not swap and bn == 256 and slices in (None, 1) and persistent,
-                  "gemm_tc: an activation without a gate is GELU on a bfloat16 store of the persistent forms")
-            epi = 5
     if bias is not None:
         _need(bias.dtype == torch.float32 and bias.numel() == N and bias.is_contiguous(), "gemm_tc: bias f32 [N]")
     _tc_unchecked["gemm_tc"] = True
