@@ -31,8 +31,8 @@
 // Epilogues: plain store (bfloat16 or float32, + bias), or SwiGLU on the fused
 // gate|up matrix whose rows are interleaved in groups of 8 (rows 16q..16q+7
 // gate, 16q+8..16q+15 up): act[m, 8q+g] = silu(gate) * up
-// (alpacca/model.py:513), so the activation costs no pass of its own.  A plain store may apply an activation
-// (`act` 1: GELU in its erf form) or, float32, bound the result: cap * tanh(y / cap) (`cap` > 0).
+// (alpacca/model.py:513), so the activation costs no pass of its own.  A store may apply GELU or, float32,
+// bound the result: cap * tanh(y / cap).
 //
 // The norm between two products, without a kernel of its own.  An RMS norm is
 // x = r * w / rms(r) with r the residual row (alpacca/tensor.py:163-173); the division
@@ -61,6 +61,8 @@
 #define EPI_STORE_F32 1
 #define EPI_SWIGLU_BF16 2
 #define EPI_RESIDUAL_BF16 3
+#define EPI_GELU_BF16 4      // a bfloat16 store behind GELU in its erf form
+#define EPI_CAP_F32 5        // a float32 store of cap * tanh(y / cap)
 
 // What the norm fusion adds to a launch; all null / 0 without it.
 struct GemvNorm {
@@ -71,8 +73,7 @@ struct GemvNorm {
   const float* norm_w;    // EPI_RESIDUAL: float32 [N], the weight of the norm that follows
   float* ss_out;          // EPI_RESIDUAL: float32 [M, ceil(N / 16)]
   int gate_act;           // EPI_SWIGLU: the activation on the gate, 0 SiLU, 1 ReLU, 2 GELU in its tanh form
-  int act;                // EPI_STORE_*: 0 none, 1 GELU (erf)
-  float cap;              // EPI_STORE_F32: > 0: y -> cap * tanh(y / cap)
+  float cap;              // EPI_CAP_F32
 };
 
 __device__ __forceinline__ float gate_activation(float g, int kind) {
@@ -169,8 +170,9 @@ __device__ __forceinline__ void epilogue(const float acc[4], int i, int ln, int 
       const int n = (j < 2) ? na : nb, m = m0 + (j & 1);
       if (n < N && m < M) {
         float v = c[j] + (bias ? bias[n] : 0.f);
-        if (nf.act == 1) v = 0.5f * v * (1.0f + erff(v * 0.70710678118654752440f));
-        if (EPI == EPI_STORE_F32) reinterpret_cast<float*>(Y)[(size_t)m * ldy + n] = nf.cap > 0.f ? nf.cap * tanhf(v / nf.cap) : v;
+        if (EPI == EPI_GELU_BF16) v = 0.5f * v * (1.0f + erff(v * 0.70710678118654752440f));
+        if (EPI == EPI_CAP_F32) v = nf.cap * tanhf(v / nf.cap);
+        if (EPI == EPI_STORE_F32 || EPI == EPI_CAP_F32) reinterpret_cast<float*>(Y)[(size_t)m * ldy + n] = v;
         else reinterpret_cast<bf16*>(Y)[(size_t)m * ldy + n] = __float2bfloat16_rn(v);
       }
     }
@@ -388,11 +390,11 @@ AB_API int ab_gemv_bf16_slices(int N, int K, int n_sms) {
 // slices > 1 needs scratch: partials float [ceil(N/16) * slices * 128 * (1, 2 or 4 for M <= 8, 16, 32)],
 // arrivals int [ceil(N/16)], zero before the first launch and left zero by every launch.
 // gate_act (epilogue 2): the activation on the gate, 0 SiLU, 1 ReLU, 2 GELU in its tanh form.
-// act, cap (epilogues 0 and 1): see GemvNorm.
+// Epilogue 4: a bfloat16 store of GELU (erf) of the result; 5: a float32 store of cap * tanh(result / cap).
 AB_API int ab_gemv_bf16_act(const void* X, const void* W, const float* bias, void* Y, float* partials,
                             int* arrivals, int M, int N, int K, int ldy, int epilogue_kind, int slices,
                             const float* ss_in, int n_part_in, float inv_width, float eps, float* residual,
-                            const float* norm_w, float* ss_out, int gate_act, int act, float cap, cudaStream_t stream) {
+                            const float* norm_w, float* ss_out, int gate_act, float cap, cudaStream_t stream) {
   if (M <= 0 || N <= 0) return AB_OK;
   if (M > 32 || K <= 0 || (K % 8) || slices < 1 || slices > 65535) return AB_BAD_ARG;
   if (slices > 1 && (!partials || !arrivals)) return AB_BAD_ARG;
@@ -404,8 +406,7 @@ AB_API int ab_gemv_bf16_act(const void* X, const void* W, const float* bias, voi
   nf.residual = residual; nf.norm_w = norm_w; nf.ss_out = ss_out;
   if (gate_act < 0 || gate_act > 2) return AB_BAD_ARG;
   nf.gate_act = gate_act;
-  if (act < 0 || act > 1) return AB_BAD_ARG;
-  nf.act = act;
+  if (epilogue_kind == EPI_CAP_F32 && !(cap > 0.f)) return AB_BAD_ARG;
   nf.cap = cap;
   // few slabs and more than one round of loads per warp: 16 warps per CTA
   const int wide = (M <= 16 && slices == 1 && (N + 15) / 16 <= gemv_sm_count() && K > 8 * GEMV_U * 32) ? 1 : 0;
@@ -413,6 +414,8 @@ AB_API int ab_gemv_bf16_act(const void* X, const void* W, const float* bias, voi
     case EPI_STORE_BF16: return launch<EPI_STORE_BF16>(X, W, bias, Y, partials, arrivals, M, N, K, ldy, slices, wide, nf, stream);
     case EPI_STORE_F32: return launch<EPI_STORE_F32>(X, W, bias, Y, partials, arrivals, M, N, K, ldy, slices, wide, nf, stream);
     case EPI_SWIGLU_BF16: return launch<EPI_SWIGLU_BF16>(X, W, bias, Y, partials, arrivals, M, N, K, ldy, slices, wide, nf, stream);
+    case EPI_GELU_BF16: return launch<EPI_GELU_BF16>(X, W, bias, Y, partials, arrivals, M, N, K, ldy, slices, wide, nf, stream);
+    case EPI_CAP_F32: return launch<EPI_CAP_F32>(X, W, bias, Y, partials, arrivals, M, N, K, ldy, slices, wide, nf, stream);
     case EPI_RESIDUAL_BF16: return launch<EPI_RESIDUAL_BF16>(X, W, bias, Y, partials, arrivals, M, N, K, ldy, slices, wide, nf, stream);
   }
   return AB_BAD_ARG;
@@ -423,7 +426,7 @@ AB_API int ab_gemv_bf16_gated(const void* X, const void* W, const float* bias, v
                               const float* ss_in, int n_part_in, float inv_width, float eps, float* residual,
                               const float* norm_w, float* ss_out, int gate_act, cudaStream_t stream) {
   return ab_gemv_bf16_act(X, W, bias, Y, partials, arrivals, M, N, K, ldy, epilogue_kind, slices, ss_in, n_part_in,
-                          inv_width, eps, residual, norm_w, ss_out, gate_act, 0, 0.f, stream);
+                          inv_width, eps, residual, norm_w, ss_out, gate_act, 0.f, stream);
 }
 
 AB_API int ab_gemv_bf16_norm(const void* X, const void* W, const float* bias, void* Y, float* partials,

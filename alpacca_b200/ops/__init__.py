@@ -387,8 +387,9 @@ def gemv_bf16(x, w, out, bias=None, n_rows=None, swiglu=False, slices=None, star
         _need(out.shape[-1] == N and out.dtype in (torch.bfloat16, torch.float32), "gemv_bf16: out [M,N]")
         epi = 1 if out.dtype == torch.float32 else 0
     _need(act in PLAIN_ACTIVATIONS, f"gemv_bf16: activation {act!r} is not one of {tuple(PLAIN_ACTIVATIONS)}")
-    _need(act is None or epi <= 1, "gemv_bf16: an activation without a gate belongs to a plain store")
+    _need(act is None or epi == 0, "gemv_bf16: an activation without a gate belongs to a plain bfloat16 store")
     _need(not cap or epi == 1, "gemv_bf16: a bound on the result belongs to a float32 store")
+    epi = 4 if act is not None else 5 if cap else epi
     if bias is not None:
         _need(bias.dtype == torch.float32 and bias.numel() == N and bias.is_contiguous(), "gemv_bf16: bias f32 [N]")
     ss_in, n_part, inv_width, eps = None, 0, 0.0, 0.0
@@ -413,7 +414,7 @@ def gemv_bf16(x, w, out, bias=None, n_rows=None, swiglu=False, slices=None, star
         _check(lib.ab_gemv_bf16_act(_p(x), _p(w), _p(bias), _p(out), _p(partials), _p(arrivals), n, N, K,
                                     out.shape[-1], epi, slices, _p(ss_in), n_part, ctypes.c_float(inv_width),
                                     ctypes.c_float(eps), _p(residual), _p(norm_weight), _p(ss_out),
-                                    GATE_ACTIVATIONS[activation], PLAIN_ACTIVATIONS[act], ctypes.c_float(cap), _stream()),
+                                    GATE_ACTIVATIONS[activation], ctypes.c_float(cap), _stream()),
                "gemv_bf16")
     finally:
         if not start_early:
