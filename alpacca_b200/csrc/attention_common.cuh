@@ -43,6 +43,12 @@ __device__ __forceinline__ uint32_t movmatrix_trans(uint32_t x) {
 }
 
 
+// A sink: a learned logit per head whose exp joins the softmax's denominator and which has no value.  `m` is
+// the row's running maximum in the kernels' units (scaled scores times log2 e), `l` its sum of exp2(score - m).
+__device__ __forceinline__ float sum_with_sink(float l, float m, const float* __restrict__ sink, int h) {
+  return sink == nullptr ? l : l + exp2f(sink[h] * LOG2E - m);
+}
+
 // Position rotation of one unit of 16 elements of a head (the same arithmetic, in the same order, as
 // the separate rotation kernel): unit u of a rotated head covers the pairs 8u .. 8u+7, i.e. with
 // pairing 0 (neighbours) the 16 consecutive elements from 16u, with pairing 1 (halves) the pieces at 8u

@@ -14,7 +14,8 @@
 //             out_scale.  The softmax is the running form, in key order; nothing is shared between warps, so
 //             a token's result does not depend on the rest of the batch.
 //
-//             `dist`: a penalty on distance, r1_h ln(1 + r2_h (p - s)), is taken off each scaled score (Chi et al.,
+//             `kind`, `dist`, `cap` (attention_scores.cuh): each scaled score may be bounded by a tanh and have a penalty
+//             on distance taken off, r1_h ln(1 + r2_h (p - s)) or slope_h (p - s) (Chi et al.,
 //             "KERPLE: Kernelized Relative Positional Embedding for Length Extrapolation", the logarithmic form).
 //
 //   combine   the last step of `attend` alone, for maps that another kernel has attended (float [T, H*M, Dv]).
@@ -36,6 +37,7 @@
 // Key pages [n_pages, G*M, page, Dk], value pages [n_pages, G, page, Dv]; one block table for both.
 // Rotation: the first n_rot dims of a vector, pairing 0 = (2i, 2i+1), 1 = (i, i + n_rot/2); tables
 // float32 [positions, n_rot/2].  (u, v) -> (u cos - v sin, v cos + u sin).
+#include "attention_scores.cuh"
 #include "common.cuh"
 #include "launch.cuh"
 
@@ -448,7 +450,7 @@ struct AttendArgs {
   const float* sink;                // [H] or null
   float coef;                       // weight of every map after the first
   int unit_norm; float eps, out_scale;
-  const float* dist;                // [2, H] or null: r1, r2 of a penalty r1 ln(1 + r2 (p - s)) taken off each score
+  int kind; const float* dist; float cap;      // what happens to a scaled score (attention_scores.cuh)
 };
 
 template <typename T, int KPL, int VPL>
@@ -473,7 +475,7 @@ attention_maps_kernel(AttendArgs a) {
   const int* bt = a.block_table + (size_t)b * a.table_width;
   const T* kp = reinterpret_cast<const T*>(a.k_pages);
   const T* vp = reinterpret_cast<const T*>(a.v_pages);
-  const float r1 = a.dist != nullptr ? a.dist[h] : 0.f, r2 = a.dist != nullptr ? a.dist[a.H + h] : 0.f;
+  const float r1 = a.kind != SCORE_PLAIN ? a.dist[h] : 0.f, r2 = a.kind == SCORE_LOG ? a.dist[a.H + h] : 0.f;
   float total[VPL];
 #pragma unroll
   for (int j = 0; j < VPL; ++j) total[j] = 0.f;
@@ -500,7 +502,11 @@ attention_maps_kernel(AttendArgs a) {
         if (d < Dk) part += qr[j] * to_f32(kv[d]);
       }
       float score = warp_sum(part) * a.scale;
-      if (a.dist != nullptr) score -= r1 * log1pf(r2 * (float)(pos - s));
+      if (a.kind == SCORE_LOG) score -= r1 * log1pf(r2 * (float)(pos - s));
+      if (a.kind == SCORE_BOUND) {
+        if (a.cap > 0.f) score = a.cap * tanhf(score / a.cap);
+        score -= r1 * (float)(pos - s);
+      }
       const float m_new = fmaxf(mx, score);
       const float corr = expf(mx - m_new);   // exp(-inf) = 0 on the first key
       const float p = expf(score - m_new);
@@ -713,17 +719,18 @@ static int launch_attend(const AttendArgs& a, cudaStream_t stream) {
   return ab_launch_status();
 }
 
-// `dist`: float [2, H] or null (see AttendArgs).
+// `kind`, `dist`, `cap`: see AttendArgs.
 AB_API int ab_attention_maps_dist(const void* q, int q_stride, void* out, int dtype, const void* k_pages,
                                   const void* v_pages, const int* block_table, int table_width, const int* tok_pos,
                                   const int* tok_seq, int n_tokens, int H, int G, int M, int Dk, int Dv, int page_size,
                                   float scale, int window, const float* sink, float coef, int unit_norm, float eps,
-                                  float out_scale, const float* dist, cudaStream_t stream) {
+                                  float out_scale, int kind, const float* dist, float cap, cudaStream_t stream) {
   if (n_tokens <= 0) return AB_OK;
+  if (!score_kind_ok(kind, dist)) return AB_BAD_ARG;
   if (Dk <= 0 || Dk > AM_MAX_DIM || Dv <= 0 || Dv > AM_MAX_DIM || H <= 0 || G <= 0 || H % G || M <= 0 || page_size <= 0)
     return AB_BAD_ARG;
   AttendArgs a{q, q_stride, out, k_pages, v_pages, block_table, table_width, tok_pos, tok_seq, n_tokens, H, G, M, Dk,
-               Dv, page_size, scale, window, sink, coef, unit_norm, eps, out_scale, dist};
+               Dv, page_size, scale, window, sink, coef, unit_norm, eps, out_scale, kind, dist, cap};
   if (dtype == AB_F32) return launch_attend<float>(a, stream);
   if (dtype == AB_BF16) return launch_attend<bf16>(a, stream);
   return AB_BAD_ARG;
@@ -736,7 +743,7 @@ AB_API int ab_attention_maps(const void* q, int q_stride, void* out, int dtype, 
                              float out_scale, cudaStream_t stream) {
   return ab_attention_maps_dist(q, q_stride, out, dtype, k_pages, v_pages, block_table, table_width, tok_pos, tok_seq,
                                 n_tokens, H, G, M, Dk, Dv, page_size, scale, window, sink, coef, unit_norm, eps, out_scale,
-                                nullptr, stream);
+                                SCORE_PLAIN, nullptr, 0.f, stream);
 }
 
 

@@ -21,10 +21,11 @@
 // Scores: (q.k) * scale; key s is seen by a token at position p iff
 // lo <= s <= p, lo = max(0, p - window + 1) (window 0: all)
 // (alpacca/model.py:447-467).  Head sizes: multiples of 16 up to 256.
-// A penalty on distance may be taken off each scaled score (template parameter DIST): r1_h ln(1 + r2_h (p - s)), a head's
-// numbers from `dist` [2, heads] (r1 of all heads, then r2).  In the kernels' units (scores times log2 e) it is
-// r1 log2(1 + r2 (p - s)), one logarithm of the hardware's approximation (relative error 2^-22) per score.
+// A scaled score may be bounded and have a penalty on distance taken off (template parameter KIND, attention_scores.cuh).
+// In the kernels' units (scores times log2 e) the logarithmic penalty is r1 log2(1 + r2 (p - s)), one logarithm of the
+// hardware's approximation (relative error 2^-22) per score.
 #include "attention_common.cuh"
+#include "attention_scores.cuh"
 #include "launch.cuh"
 #include <cooperative_groups.h>
 #include <cuda_pipeline.h>
@@ -45,8 +46,9 @@ struct RowState {
   float l[2];   // running sum of 2^(score' - m)
 };
 
-// What the penalty on distance needs of one row or column: r1, r2 of its head and 1 + r2 * (its position - the tile's
-// first key), so that key number c of the tile costs one fused multiply-add and one logarithm.
+// What the penalty on distance needs of one row or column.  SCORE_LOG: r1, r2 of its head and 1 + r2 * (its position - the
+// tile's first key), so that key number c of the tile costs one fused multiply-add and one logarithm.  SCORE_BOUND: r1 =
+// slope * log2 e, base = its position - the tile's first key, an integer, so that the distance base - c is exact.
 struct DistRow {
   float r1, r2, base;
 };
@@ -56,7 +58,9 @@ __device__ __forceinline__ float fast_log2(float x) {
   return y;
 }
 // score - r1 log2(1 + r2 (distance - c)); negative distances (keys that are masked afterwards) may give NaN
+template <int KIND>
 __device__ __forceinline__ float less_distance(float score, const DistRow& d, float c) {
+  if (KIND == SCORE_BOUND) return fmaf(-d.r1, d.base - c, score);
   return fmaf(-d.r1, fast_log2(fmaf(-d.r2, c, d.base)), score);
 }
 
@@ -64,11 +68,11 @@ __device__ __forceinline__ float less_distance(float score, const DistRow& d, fl
 //   qs: this warp's 16 query rows in shared memory, pitch `pitch` elements
 //   ks, vs: the key tile [64][pitch] of D dims and the value tile [64][pitch_v] of Dv dims
 //   pos0/pos1, lo0/lo1: last and first visible key of rows g and g+8; key0: position of the tile's first key
-template <int DMAX, bool DIST>
+template <int DMAX, int KIND>
 __device__ __forceinline__ void attend_tile(RowState<DMAX>& st, const bf16* qs, const bf16* ks, const bf16* vs,
                                             int pitch, int pitch_v, int D, int Dv, float scale_log2, int key0,
                                             int pos0, int pos1, int lo0, int lo1, bool need_mask, const DistRow& d0,
-                                            const DistRow& d1) {
+                                            const DistRow& d1, const ScoreBound& bound) {
   const int lane = threadIdx.x & 31;
   const int t = lane & 3;
   float s[8][4];
@@ -100,7 +104,8 @@ __device__ __forceinline__ void attend_tile(RowState<DMAX>& st, const bf16* qs, 
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
       float v = s[nt][j] * scale_log2;
-      if (DIST) v = less_distance(v, j < 2 ? d0 : d1, (float)(nt * 8 + (j & 1)));     // the lane's 2t is in `base`
+      if (KIND == SCORE_BOUND) v = bounded_score(v, bound);
+      if (KIND) v = less_distance<KIND>(v, j < 2 ? d0 : d1, (float)(nt * 8 + (j & 1)));     // the lane's 2t is in `base`
       if (need_mask) {
         const int key = key0 + nt * 8 + 2 * t + (j & 1);
         const bool ok = (j < 2) ? (key <= pos0 && key >= lo0) : (key <= pos1 && key >= lo1);
@@ -188,12 +193,6 @@ __device__ __forceinline__ void load_tile_async(bf16* dst, const bf16* src, int 
   load_tile_async(dst, src, D, pitch, tid, nthreads, D);
 }
 
-// A sink: a learned logit per head whose exp joins the softmax's denominator and which has no value.  `m` is
-// the row's running maximum in the kernels' units (scaled scores times log2 e), `l` its sum of exp2(score - m).
-__device__ __forceinline__ float sum_with_sink(float l, float m, const float* __restrict__ sink, int h) {
-  return sink == nullptr ? l : l + exp2f(sink[h] * LOG2E - m);
-}
-
 // ---------------------------------------------------------------------------
 // prefill
 // ---------------------------------------------------------------------------
@@ -209,7 +208,7 @@ __device__ __forceinline__ float sum_with_sink(float l, float m, const float* __
 // for itself) and group c the columns c*group_cols .. (c+1)*group_cols of the launch's Dv: one copy of the key tile
 // and of a value tile of all Dv columns serves NG times the warps, where a value row is too wide for one warp's
 // registers.  DMAX then covers D and group_cols.
-template <int DMAX, int NG, bool DIST>
+template <int DMAX, int NG, int KIND>
 __global__ void __launch_bounds__(128 * NG)
 attention_prefill_kernel(const bf16* __restrict__ qkv, int q_stride, void* __restrict__ out_any, int out_f32,
                          const bf16* __restrict__ k_pages, const bf16* __restrict__ v_pages,
@@ -217,7 +216,7 @@ attention_prefill_kernel(const bf16* __restrict__ qkv, int q_stride, void* __res
                          const int* __restrict__ cu_q, const int* __restrict__ tok_seq,
                          const int* __restrict__ tile_seq, const int* __restrict__ tile_q0, int H, int K, int M, int D,
                          int Dv, float scale_log2, int window, int tokens_per_tile, const float* __restrict__ sink,
-                         int v_row, int v_col0, int group_cols, const float* __restrict__ dist) {
+                         int v_row, int v_col0, int group_cols, const float* __restrict__ dist, float cap) {
   extern __shared__ __align__(16) unsigned char smem_raw[];
   constexpr int NT = 128 * NG;
   const int pitch = D + 8, pitch_v = Dv + 8;
@@ -267,7 +266,12 @@ attention_prefill_kernel(const bf16* __restrict__ qkv, int q_stride, void* __res
   const int kb_end = pos_last / PAGE + 1;
   const int* bt = block_table + (size_t)b * table_width;
   float ra0 = 0.f, rb0 = 0.f, ra1 = 0.f, rb1 = 0.f;      // r1, r2 of the heads of this thread's two rows
-  if (DIST) {
+  const ScoreBound bound = score_bound(KIND == SCORE_BOUND ? cap : 0.f);
+  if (KIND == SCORE_BOUND) {
+    if (r0 < n_rows) ra0 = dist[grp * G + r0 % G] * LOG2E;
+    if (r1 < n_rows) ra1 = dist[grp * G + r1 % G] * LOG2E;
+  }
+  if (KIND == SCORE_LOG) {
     const int n_heads = H / M;
     if (r0 < n_rows) { ra0 = dist[grp * G + r0 % G]; rb0 = dist[n_heads + grp * G + r0 % G]; }
     if (r1 < n_rows) { ra1 = dist[grp * G + r1 % G]; rb1 = dist[n_heads + grp * G + r1 % G]; }
@@ -293,13 +297,17 @@ attention_prefill_kernel(const bf16* __restrict__ qkv, int q_stride, void* __res
     if (warp * 16 < n_rows && n_cols > 0) {
       const bool need_mask = (key0 + PAGE - 1 > pos_first) || (window > 0);
       DistRow d0{0.f, 0.f, 1.f}, d1{0.f, 0.f, 1.f};
-      if (DIST) {
+      if (KIND == SCORE_BOUND) {
+        d0 = DistRow{ra0, 0.f, (float)(pos0 - key0 - 2 * t4)};
+        d1 = DistRow{ra1, 0.f, (float)(pos1 - key0 - 2 * t4)};
+      }
+      if (KIND == SCORE_LOG) {
         d0 = DistRow{ra0, rb0, fmaf(rb0, (float)(pos0 - key0 - 2 * t4), 1.f)};
         d1 = DistRow{ra1, rb1, fmaf(rb1, (float)(pos1 - key0 - 2 * t4), 1.f)};
       }
-      attend_tile<DMAX, DIST>(st, qs + warp * 16 * pitch, kbuf + stage * 64 * pitch,
+      attend_tile<DMAX, KIND>(st, qs + warp * 16 * pitch, kbuf + stage * 64 * pitch,
                               vbuf + stage * 64 * pitch_v + col_first, pitch, pitch_v, D, n_cols, scale_log2, key0, pos0,
-                              pos1, lo0, lo1, need_mask, d0, d1);
+                              pos1, lo0, lo1, need_mask, d0, d1, bound);
     }
     __syncthreads();
   }
@@ -357,10 +365,11 @@ struct DecodeState {
 
 // One run of `nt` (1..DECODE_RUN) 16-key tiles; ks, vs: the run's keys and values [nt*16][pitch];
 // qb: Q^T as the second operand, per 16 columns of the head; key0: position of the run's first key.
-template <int DMAX, bool DIST>
+template <int DMAX, int KIND>
 __device__ __forceinline__ void attend_run(DecodeState<DMAX>& st, const uint32_t (&qb)[DMAX / 16][2], const bf16* ks,
                                            const bf16* vs, int pitch, int D, float scale_log2, int nt, int key0,
-                                           int pos, int lo, const DistRow& h0, const DistRow& h1) {
+                                           int pos, int lo, const DistRow& h0, const DistRow& h1,
+                                           const ScoreBound& bound) {
   const int lane = threadIdx.x & 31;
   const int g = lane >> 2;
   const int a_row = (lane & 7) + ((lane >> 3) & 1) * 8, a_col = (lane >> 4) * 8;
@@ -383,7 +392,11 @@ __device__ __forceinline__ void attend_run(DecodeState<DMAX>& st, const uint32_t
 #pragma unroll
       for (int j = 0; j < 4; ++j) {
         float v = s[i][j] * scale_log2;
-        if (DIST) {
+        if (KIND == SCORE_BOUND) {
+          const DistRow& hd = (j & 1) ? h1 : h0;
+          v = fmaf(-hd.r1, (float)(pos - (j < 2 ? ka : kb)), bounded_score(v, bound));
+        }
+        if (KIND == SCORE_LOG) {
           const DistRow& hd = (j & 1) ? h1 : h0;
           v = fmaf(-hd.r1, fast_log2(fmaf(hd.r2, (float)(pos - (j < 2 ? ka : kb)), 1.f)), v);
         }
@@ -466,7 +479,7 @@ __device__ __forceinline__ void load_run_async(bf16* ks, bf16* vs, const bf16* _
 // rotation kernel ran); 1 = this kernel rotates q; the step's key and value are in the cache (a layer
 // that reads the cache of another); 2 = this kernel rotates q and k, takes this step's key and value
 // from qkv and writes them to their place in the cache.
-template <int DMAX, int NWARPS, bool DIST>
+template <int DMAX, int NWARPS, int KIND>
 __global__ void __launch_bounds__(NWARPS * 32)
 attention_decode_kernel(const bf16* __restrict__ qkv, int q_stride, bf16* __restrict__ out,
                         float* __restrict__ part_o, float* __restrict__ part_ml, int* __restrict__ arrivals,
@@ -475,7 +488,7 @@ attention_decode_kernel(const bf16* __restrict__ qkv, int q_stride, bf16* __rest
                         const int* __restrict__ kv_len, int H, int K, int D, float scale_log2, int window,
                         int pages_per_cta, int n_chunks, int cluster_merge, bf16* k_out, bf16* v_out, const float* __restrict__ cos_t, const float* __restrict__ sin_t,
                         int n_rot, int pairing, int fuse, const float* __restrict__ sink,
-                        const float* __restrict__ dist) {
+                        const float* __restrict__ dist, float cap) {
   extern __shared__ __align__(16) unsigned char smem_raw[];
   const int pitch = D + 8;
   bf16* qs = reinterpret_cast<bf16*>(smem_raw);                 // [8][pitch] q, [2][pitch] this step's k, v
@@ -506,7 +519,13 @@ attention_decode_kernel(const bf16* __restrict__ qkv, int q_stride, bf16* __rest
   if (!active && !cluster_merge) { pdl_wait(); pdl_trigger(); return; }
   const int n_heads = min(8, G - rt * 8);
   DistRow hd0{0.f, 0.f, 1.f}, hd1{0.f, 0.f, 1.f};      // of this thread's two heads (columns 2t, 2t + 1 of the tiles)
-  if (DIST) {
+  const ScoreBound bound = score_bound(KIND == SCORE_BOUND ? cap : 0.f);
+  if (KIND == SCORE_BOUND) {
+    const int h = kh * G + rt * 8 + 2 * t4;
+    if (2 * t4 < n_heads) hd0.r1 = dist[h] * LOG2E;
+    if (2 * t4 + 1 < n_heads) hd1.r1 = dist[h + 1] * LOG2E;
+  }
+  if (KIND == SCORE_LOG) {
     const int h = kh * G + rt * 8 + 2 * t4;
     if (2 * t4 < n_heads) { hd0.r1 = dist[h]; hd0.r2 = dist[H + h]; }
     if (2 * t4 + 1 < n_heads) { hd1.r1 = dist[h + 1]; hd1.r2 = dist[H + h + 1]; }
@@ -612,7 +631,7 @@ attention_decode_kernel(const bf16* __restrict__ qkv, int q_stride, bf16* __rest
       }
     }
     __syncwarp();
-    if (t0 < t1) attend_run<DMAX, DIST>(st, qb, ks, vs, pitch, D, scale_log2, t1 - t0, t0 * 16, pos, lo, hd0, hd1);
+    if (t0 < t1) attend_run<DMAX, KIND>(st, qb, ks, vs, pitch, D, scale_log2, t1 - t0, t0 * 16, pos, lo, hd0, hd1, bound);
     __syncwarp();      // every lane is done reading the run before the next one overwrites it
   }
   float l0 = st.l[0], l1 = st.l[1];
@@ -761,15 +780,16 @@ AB_API int ab_attention_decode_round_pages(int D) { return ab_attention_decode_r
 // `v_row`, `v_col0`: columns v_col0 .. v_col0 + Dv of value rows and output vectors of v_row numbers (both multiples
 // of 8: 16-byte pieces).  `group_cols`: the columns of Dv that one group of four warps takes (a multiple of 16, up to
 // 256); ceil(Dv / group_cols) must be 1, 2 or 4 (four groups: D and group_cols up to 128).
-// `dist`: float [2, H / M] or null, the penalty on distance (one group of columns then).
+// `kind`, `dist`, `cap`: what happens to a scaled score, heads H / M (attention_scores.cuh; one group of columns then).
 AB_API int ab_attention_prefill_maps_dist_bf16(const void* qkv, int q_stride, void* out, int out_f32,
                                                const void* k_pages, const void* v_pages, const int* block_table,
                                                int table_width, const int* tok_pos, const int* cu_q,
                                                const int* tok_seq, const int* tile_seq, const int* tile_q0, int n_tiles,
                                                int tokens_per_tile, int H, int K, int M, int D, int Dv, float scale,
                                                int window, const float* sink, int v_row, int v_col0, int group_cols,
-                                               const float* dist, cudaStream_t stream) {
+                                               int kind, const float* dist, float cap, cudaStream_t stream) {
   if (n_tiles <= 0) return AB_OK;
+  if (!score_kind_ok(kind, dist)) return AB_BAD_ARG;
   if (D <= 0 || D > 256 || (D % 16) || Dv <= 0 || (Dv % 16) || K <= 0 || H % K || K > 65535 || M <= 0 || K % M)
     return AB_BAD_ARG;
   if (group_cols <= 0 || group_cols > 256 || (group_cols % 16)) return AB_BAD_ARG;
@@ -792,17 +812,24 @@ AB_API int ab_attention_prefill_maps_dist_bf16(const void* qkv, int q_stride, vo
     ab_launch(attention_prefill_kernel<DM, NG, DS>, grid, dim3(128 * NG), smem, stream,                             \
         (const bf16*)qkv, q_stride, out, out_f32, (const bf16*)k_pages, (const bf16*)v_pages, block_table,          \
         table_width, tok_pos, cu_q, tok_seq, tile_seq, tile_q0, H, K, M, D, Dv, sl, window, tokens_per_tile, sink,  \
-        v_row, v_col0, group_cols, dist);                                                                           \
+        v_row, v_col0, group_cols, dist, cap);                                                                      \
   }
-#define AB_GO(DM, NG) AB_GO_D(DM, NG, false)
+#define AB_GO(DM, NG) AB_GO_D(DM, NG, SCORE_PLAIN)
   const int widest = groups == 1 ? Dv : group_cols;
   const int dm = dmax_of(D > widest ? D : widest);
-  if (dist != nullptr) {
+  if (kind == SCORE_LOG) {
     if (groups != 1) return AB_BAD_ARG;
     switch (dm) {
-      case 64: AB_GO_D(64, 1, true); break;
-      case 128: AB_GO_D(128, 1, true); break;
-      default: AB_GO_D(256, 1, true); break;
+      case 64: AB_GO_D(64, 1, SCORE_LOG); break;
+      case 128: AB_GO_D(128, 1, SCORE_LOG); break;
+      default: AB_GO_D(256, 1, SCORE_LOG); break;
+    }
+  } else if (kind == SCORE_BOUND) {
+    if (groups != 1) return AB_BAD_ARG;
+    switch (dm) {
+      case 64: AB_GO_D(64, 1, SCORE_BOUND); break;
+      case 128: AB_GO_D(128, 1, SCORE_BOUND); break;
+      default: AB_GO_D(256, 1, SCORE_BOUND); break;
     }
   } else if (groups == 1) {
     switch (dm) {
@@ -830,7 +857,8 @@ AB_API int ab_attention_prefill_maps_groups_bf16(const void* qkv, int q_stride, 
                                                  cudaStream_t stream) {
   return ab_attention_prefill_maps_dist_bf16(qkv, q_stride, out, out_f32, k_pages, v_pages, block_table, table_width,
                                              tok_pos, cu_q, tok_seq, tile_seq, tile_q0, n_tiles, tokens_per_tile, H, K, M,
-                                             D, Dv, scale, window, sink, v_row, v_col0, group_cols, nullptr, stream);
+                                             D, Dv, scale, window, sink, v_row, v_col0, group_cols, SCORE_PLAIN, nullptr, 0.f,
+                                             stream);
 }
 
 // One group of warps: up to 256 columns per launch.
@@ -951,15 +979,17 @@ AB_API int ab_attention_decode_rope_bf16(const void* qkv, int q_stride, void* ou
                                        n_chunks, small, cos_t, sin_t, n_rot, pairing, fuse, nullptr, stream);
 }
 
-// The same with a sink per head in the softmax's denominator (`sink`: float [H] or null) and a penalty on distance
-// (`dist`: float [2, H] or null).
+// The same with a sink per head in the softmax's denominator (`sink`: float [H] or null); `kind`, `dist`, `cap`: what
+// happens to a scaled score (attention_scores.cuh).
 AB_API int ab_attention_decode_dist_bf16(const void* qkv, int q_stride, void* out, float* part_o, float* part_ml,
                                          int* arrivals, void* k_pages, void* v_pages, const int* block_table,
                                          int table_width, const int* tok_seq, const int* kv_len, int n_tokens, int H,
                                          int K, int D, float scale, int window, int pages_per_cta, int n_chunks,
                                          int small, const float* cos_t, const float* sin_t, int n_rot, int pairing,
-                                         int fuse, const float* sink, const float* dist, cudaStream_t stream) {
+                                         int fuse, const float* sink, int kind, const float* dist, float cap,
+                                         cudaStream_t stream) {
   if (n_tokens <= 0) return AB_OK;
+  if (!score_kind_ok(kind, dist)) return AB_BAD_ARG;
   if (D <= 0 || D > 256 || (D % 16) || H % K || n_chunks < 1 || n_chunks > 65535 || pages_per_cta < 1)
     return AB_BAD_ARG;
   if (small < 0 || small > 2) return AB_BAD_ARG;
@@ -973,7 +1003,12 @@ AB_API int ab_attention_decode_dist_bf16(const void* qkv, int q_stride, void* ou
   const float sl = scale * LOG2E;
   const int cluster_merge = (n_chunks > 1 && n_chunks <= AB_DECODE_MAX_CLUSTER) ? 1 : 0;
   dim3 grid(n_tokens, K * row_tiles, n_chunks);
-#define AB_GO(DM, NW) { if (dist != nullptr) AB_GO_D(DM, NW, true) else AB_GO_D(DM, NW, false) }
+#define AB_GO(DM, NW)                                                                                               \
+  {                                                                                                                 \
+    if (kind == SCORE_LOG) AB_GO_D(DM, NW, SCORE_LOG)                                                               \
+    else if (kind == SCORE_BOUND) AB_GO_D(DM, NW, SCORE_BOUND)                                                      \
+    else AB_GO_D(DM, NW, SCORE_PLAIN)                                                                               \
+  }
 #define AB_GO_D(DM, NW, DS)                                                                                         \
   {                                                                                                                 \
     size_t tiles = (size_t)(10 + NW * 2 * 16 * DECODE_RUN) * pitch * sizeof(bf16);                                  \
@@ -986,7 +1021,7 @@ AB_API int ab_attention_decode_dist_bf16(const void* qkv, int q_stride, void* ou
         cluster_merge ? (unsigned)n_chunks : 1u,                                                                    \
         (const bf16*)qkv, q_stride, (bf16*)out, part_o, part_ml, arrivals, (const bf16*)k_pages,                    \
         (const bf16*)v_pages, block_table, table_width, tok_seq, kv_len, H, K, D, sl, window, pages_per_cta,        \
-        n_chunks, cluster_merge, (bf16*)k_pages, (bf16*)v_pages, cos_t, sin_t, n_rot, pairing, fuse, sink, dist);   \
+        n_chunks, cluster_merge, (bf16*)k_pages, (bf16*)v_pages, cos_t, sin_t, n_rot, pairing, fuse, sink, dist, cap);   \
   }
   if (n_chunks > AB_DECODE_MAX_CLUSTER && (!part_o || !part_ml || !arrivals)) return AB_BAD_ARG;
   switch (dmax_of(D)) {
@@ -1014,7 +1049,7 @@ AB_API int ab_attention_decode_sink_bf16(const void* qkv, int q_stride, void* ou
                                          int fuse, const float* sink, cudaStream_t stream) {
   return ab_attention_decode_dist_bf16(qkv, q_stride, out, part_o, part_ml, arrivals, k_pages, v_pages, block_table,
                                        table_width, tok_seq, kv_len, n_tokens, H, K, D, scale, window, pages_per_cta,
-                                       n_chunks, small, cos_t, sin_t, n_rot, pairing, fuse, sink, nullptr, stream);
+                                       n_chunks, small, cos_t, sin_t, n_rot, pairing, fuse, sink, SCORE_PLAIN, nullptr, 0.f, stream);
 }
 
 // ---------------------------------------------------------------------------

@@ -22,12 +22,13 @@
 //   - the position rotation of q and k and the append of this step's k, v to the cache happen here
 //     (`fuse`), as in attention_mma.cu.
 //
-// A penalty on distance (template parameter DIST, numbers [2, H]) may be taken off each scaled score, as there.
+// A scaled score may be bounded and have a penalty on distance taken off, a sink may join the denominator, as there.
 // Head sizes 64 and 128 (rows of 128 bytes per swizzled panel); other sizes take attention_mma.cu.
 // Every wait on an mbarrier is bounded: after AS_SPIN tries the kernel records a code in `status`,
 // all roles fall through to the end and the output of that CTA is not valid (the host reads the
 // status where it synchronises).
 #include "attention_common.cuh"
+#include "attention_scores.cuh"
 #include "launch.cuh"
 #include <cooperative_groups.h>
 #include <cuda.h>
@@ -87,10 +88,10 @@ __device__ __forceinline__ float as_log2(float x) {
 }
 
 // 16 keys (rows r0 .. r0+15 of the stage's K and V tiles) against the group's heads.
-template <int HD, bool DIST>
+template <int HD, int KIND>
 __device__ __forceinline__ void attend_tile16(StreamState<HD>& st, const uint32_t (&qb)[HD / 16][2], uint32_t k_tile,
                                               uint32_t v_tile, int r0, float scale_log2, int key0, int pos, int lo,
-                                              const float (&r1)[2], const float (&r2)[2]) {
+                                              const float (&r1)[2], const float (&r2)[2], const ScoreBound& bound) {
   const int lane = threadIdx.x & 31;
   const int g = lane >> 2;
   const int a_row = r0 + (lane & 7) + ((lane >> 3) & 1) * 8, a_chunk = lane >> 4;
@@ -106,7 +107,8 @@ __device__ __forceinline__ void attend_tile16(StreamState<HD>& st, const uint32_
 #pragma unroll
   for (int j = 0; j < 4; ++j) {
     float v = s[j] * scale_log2;
-    if (DIST) v = fmaf(-r1[j & 1], as_log2(fmaf(r2[j & 1], (float)(pos - (j < 2 ? ka : kb)), 1.f)), v);
+    if (KIND == SCORE_BOUND) v = fmaf(-r1[j & 1], (float)(pos - (j < 2 ? ka : kb)), bounded_score(v, bound));
+    if (KIND == SCORE_LOG) v = fmaf(-r1[j & 1], as_log2(fmaf(r2[j & 1], (float)(pos - (j < 2 ? ka : kb)), 1.f)), v);
     s[j] = (j < 2 ? oka : okb) ? v : -INFINITY;
   }
   float mx0 = fmaxf(s[0], s[2]), mx1 = fmaxf(s[1], s[3]);
@@ -167,7 +169,7 @@ template <int HD, int STAGES> struct StreamSmem {
 // of a cluster; 2 = through scratch memory, the CTA that arrives last merges.
 // fuse: as in attention_mma.cu (0: q rotated and this step's k, v in the cache already; 1: this kernel
 // rotates q; 2: it rotates q and k and appends k, v to the cache).
-template <int HD, int STAGES, bool DIST>
+template <int HD, int STAGES, int KIND>
 __global__ void __launch_bounds__(AS_THREADS)
 attention_stream_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_v,
                         const bf16* __restrict__ qkv, int q_stride, bf16* __restrict__ out,
@@ -177,7 +179,8 @@ attention_stream_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
                         const int* __restrict__ row_order, int H, int K, float scale_log2, int window,
                         int pages_per_cta, int n_chunks, int merge, const float* __restrict__ cos_t,
                         const float* __restrict__ sin_t, int n_rot, int pairing, int fuse,
-                        int* __restrict__ status, const float* __restrict__ dist) {
+                        int* __restrict__ status, const float* __restrict__ dist, float cap,
+                        const float* __restrict__ sink) {
   using Sm = StreamSmem<HD, STAGES>;
   constexpr int D = HD;
   extern __shared__ unsigned char smem_raw[];
@@ -295,12 +298,13 @@ attention_stream_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
       }
     }
     float r1[2] = {0.f, 0.f}, r2[2] = {0.f, 0.f};      // of this thread's two heads
-    if (DIST) {
+    const ScoreBound bound = score_bound(KIND == SCORE_BOUND ? cap : 0.f);
+    if (KIND) {
 #pragma unroll
       for (int j = 0; j < 2; ++j)
         if (2 * t4 + j < n_heads) {
-          r1[j] = dist[kh * G + rt * 8 + 2 * t4 + j];
-          r2[j] = dist[H + kh * G + rt * 8 + 2 * t4 + j];
+          r1[j] = dist[kh * G + rt * 8 + 2 * t4 + j] * (KIND == SCORE_BOUND ? LOG2E : 1.f);
+          if (KIND == SCORE_LOG) r2[j] = dist[H + kh * G + rt * 8 + 2 * t4 + j];
         }
     }
     uint32_t qb[HD / 16][2];
@@ -329,7 +333,8 @@ attention_stream_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
           asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
           __syncwarp();
         }
-        attend_tile16<HD, DIST>(st, qb, smem_u32(stage), smem_u32(stage + Sm::TILE), r0, scale_log2, key0, pos, lo, r1, r2);
+        attend_tile16<HD, KIND>(st, qb, smem_u32(stage), smem_u32(stage + Sm::TILE), r0, scale_log2, key0, pos, lo, r1, r2,
+                                bound);
       }
       __syncwarp();      // every lane is done with the stage before it is given back
       if (lane == 0) as_arrive(empty + s);
@@ -394,6 +399,7 @@ attention_stream_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
         cta_o[r * D + d] = o;
         if (d == 0) { cta_ml[r * 2] = m; cta_ml[r * 2 + 1] = l; }
       } else if (single) {
+        l = sum_with_sink(l, m, sink, h);
         out[((size_t)tok * H + h) * D + d] = __float2bfloat16_rn(l > 0.f ? o / l : 0.f);
       } else {
         const size_t p = ((size_t)tok * H + h) * n_chunks + chunk;
@@ -432,6 +438,7 @@ attention_stream_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
           l += lc[j] * f;
           o += oc[j] * f;
         }
+        l = sum_with_sink(l, m, sink, kh * G + rt * 8 + r);
         out[((size_t)tok * H + kh * G + rt * 8 + r) * D + d] = __float2bfloat16_rn(l > 0.f ? o / l : 0.f);
       }
     }
@@ -490,6 +497,7 @@ attention_stream_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
       }
       m = top;
     }
+    l = sum_with_sink(l, m, sink, h);
     bf16* dst = out + ((size_t)tok * H + h) * D + d;
     *reinterpret_cast<__nv_bfloat162*>(dst) = __floats2bfloat162_rn(l > 0.f ? o.x / l : 0.f, l > 0.f ? o.y / l : 0.f);
     *reinterpret_cast<__nv_bfloat162*>(dst + 2) = __floats2bfloat162_rn(l > 0.f ? o.z / l : 0.f, l > 0.f ? o.w / l : 0.f);
@@ -552,14 +560,16 @@ AB_API int ab_attention_stream_stages(int D, int ring) {
 // n_chunks chunks of pages_per_cta pages cover the table; `ring`: see ab_attention_stream_stages.  merge_kind: 1 = cluster (2..8 chunks), 2 =
 // scratch: part_o float [n_tokens*H*n_chunks, D], part_ml float [n_tokens*H*n_chunks, 2], arrivals int
 // [n_tokens * K * ceil(G/8)], zero before the first launch and left zero by every launch.
-// `dist`: float [2, H] or null, the penalty on distance.
+// `sink`: float [H] or null, a logit per head that joins the denominator; `kind`, `dist`, `cap`: attention_scores.cuh.
 AB_API int ab_attention_stream_dist_bf16(const void* qkv, int q_stride, void* out, float* part_o, float* part_ml,
                                     int* arrivals, void* k_pages, void* v_pages, int n_pages,
                                     const int* block_table, int table_width, const int* tok_seq, const int* kv_len,
                                     const int* row_order, int n_tokens, int H, int K, int D, float scale, int window, int pages_per_cta,
                                     int n_chunks, int merge_kind, int ring, const float* cos_t, const float* sin_t,
-                                    int n_rot, int pairing, int fuse, const float* dist, cudaStream_t stream) {
+                                    int n_rot, int pairing, int fuse, const float* sink, int kind, const float* dist, float cap,
+                                    cudaStream_t stream) {
   if (n_tokens <= 0) return AB_OK;
+  if (!score_kind_ok(kind, dist)) return AB_BAD_ARG;
   if (!ab_attention_stream_supports(H, K, D) || n_chunks < 1 || n_chunks > 65535 || pages_per_cta < 1 || n_pages < 1)
     return AB_BAD_ARG;
   if (fuse < 0 || fuse > 2 || n_rot < 0 || n_rot > D || (n_rot % 16) || pairing < 0 || pairing > 1) return AB_BAD_ARG;
@@ -612,7 +622,12 @@ AB_API int ab_attention_stream_dist_bf16(const void* qkv, int q_stride, void* ou
   cfg.attrs = attr;
   cfg.numAttrs = n_attr;
   cudaError_t e;
-#define AS_GO(HDV, ST) { if (dist != nullptr) AS_GO_D(HDV, ST, true) else AS_GO_D(HDV, ST, false) }
+#define AS_GO(HDV, ST)                                                                                              \
+  {                                                                                                                 \
+    if (kind == SCORE_LOG) AS_GO_D(HDV, ST, SCORE_LOG)                                                              \
+    else if (kind == SCORE_BOUND) AS_GO_D(HDV, ST, SCORE_BOUND)                                                     \
+    else AS_GO_D(HDV, ST, SCORE_PLAIN)                                                                              \
+  }
 #define AS_GO_D(HDV, ST, DS)                                                                                        \
   {                                                                                                                 \
     cfg.dynamicSmemBytes = StreamSmem<HDV, ST>::TOTAL;                                                              \
@@ -622,7 +637,7 @@ AB_API int ab_attention_stream_dist_bf16(const void* qkv, int q_stride, void* ou
     e = cudaLaunchKernelEx(&cfg, attention_stream_kernel<HDV, ST, DS>, mk, mv, (const bf16*)qkv, q_stride, (bf16*)out,  \
                            part_o, part_ml, arrivals, (bf16*)k_pages, (bf16*)v_pages, block_table, table_width,     \
                            tok_seq, kv_len, row_order, H, K, sl, window, pages_per_cta, n_chunks, merge, cos_t, sin_t, n_rot,  \
-                           pairing, fuse, status, dist);                                                                  \
+                           pairing, fuse, status, dist, cap, sink);                                                                  \
   }
   if (D == 64) { if (ring <= 0) AS_GO(64, 3) else if (ring == 1) AS_GO(64, 6) else AS_GO(64, 12) }
   else { if (ring <= 0) AS_GO(128, 2) else if (ring == 1) AS_GO(128, 3) else AS_GO(128, 6) }
@@ -641,5 +656,5 @@ AB_API int ab_attention_stream_bf16(const void* qkv, int q_stride, void* out, fl
   return ab_attention_stream_dist_bf16(qkv, q_stride, out, part_o, part_ml, arrivals, k_pages, v_pages, n_pages, block_table,
                                        table_width, tok_seq, kv_len, row_order, n_tokens, H, K, D, scale, window,
                                        pages_per_cta, n_chunks, merge_kind, ring, cos_t, sin_t, n_rot, pairing, fuse, nullptr,
-                                       stream);
+                                       SCORE_PLAIN, nullptr, 0.f, stream);
 }

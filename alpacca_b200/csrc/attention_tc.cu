@@ -26,14 +26,15 @@
 // (q.k) * scale, key s visible to position p iff lo <= s <= p
 // (alpacca/model.py:457-467).
 //
-// A penalty on distance (template parameter DIST) is taken off each scaled score: r1_h ln(1 + r2_h (p - s)) with a head's
-// numbers from `dist` [2, H].  The exponentials already fill the unit that forms logarithms, so a tile's penalties are
+// A scaled score may be bounded and have a penalty on distance taken off (template parameter KIND, attention_scores.cuh).
+// The logarithmic penalty: the exponentials already fill the unit that forms logarithms, so a tile's penalties are
 // not formed per score: along a tile they depend on the head and on p - s alone, G x (tokens + 63) numbers instead of
 // 128 x 64.  The softmax threads form them for the next tile into one of two tables in shared memory, one named barrier
 // of their 128 threads per tile, and read one number per score (neighbouring rows meet different banks).
 //
 // Every mbarrier wait is bounded (see gemm_tc.cu): on a timeout the thread records a
 // code in `status` and all roles fall through to the end, where TMEM is given back.
+#include "attention_scores.cuh"
 #include "common.cuh"
 #include "launch.cuh"
 #include <cuda.h>
@@ -176,7 +177,7 @@ __device__ __forceinline__ float at_log2(float x) {
   return y;
 }
 
-template <int HD, bool DIST>
+template <int HD, int KIND>
 __global__ void __launch_bounds__(AT_THREADS, 2)
 attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                             const __grid_constant__ CUtensorMap map_v, bf16* __restrict__ out,
@@ -184,7 +185,8 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
                             const int* __restrict__ cu_q, const int* __restrict__ tile_seq,
                             const int* __restrict__ tile_q0, int H, int K, float scale_log2, int window,
                             int tokens_per_tile, int* __restrict__ status, const float* __restrict__ sink,
-                            const float* __restrict__ dist) {
+                            const float* __restrict__ dist, float cap) {
+  constexpr bool DIST = KIND == SCORE_LOG;      // penalties from tables
   extern __shared__ unsigned char smem_raw[];
   unsigned char* base = reinterpret_cast<unsigned char*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~(uintptr_t)1023);
   using Sm = AtSmem<HD>;
@@ -325,6 +327,8 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
       }
     };
     if (DIST && n_tiles > 0) form_penalties(0);
+    const ScoreBound bound = score_bound(KIND == SCORE_BOUND ? cap : 0.f);
+    const float slope = (KIND == SCORE_BOUND && row_ok) ? dist[kh * G + r % G] * AT_LOG2E : 0.f;
 
     for (int j = 0; j < n_tiles && (ok || DIST); ++j) {
       if (DIST) {
@@ -352,6 +356,30 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
 #pragma unroll
         for (int c = 0; c < AT_KEYS; ++c) sc[c] = fmaf(sc[c], scale_log2, pen[-c]);
       }
+      if (KIND == SCORE_BOUND) {
+        // less slope * (pos - key0 - c): the tile's share is formed once, the keys' is a constant times the slope
+        const float shift = fmaf(-slope, (float)((row_ok ? pos : key0) - key0), bound.c);
+        if (bound.c > 0.f) {
+          // c - 2 c / (1 + 2^x): four denominators share one reciprocal (2^x is cut at 2^30, where the fraction no longer
+          // counts, so that their product stays finite)
+          const float k = scale_log2 * bound.k, m2c = -2.0f * bound.c;
+#pragma unroll
+          for (int c = 0; c < AT_KEYS; c += 4) {
+            float d[4];
+#pragma unroll
+            for (int e = 0; e < 4; ++e) d[e] = 1.0f + at_exp2(fminf(sc[c + e] * k, 30.0f));
+            const float ab = d[0] * d[1], cd = d[2] * d[3], w = m2c * score_rcp(ab * cd);
+            const float wab = w * cd, wcd = w * ab;
+            sc[c] = fmaf(wab, d[1], fmaf(slope, (float)c, shift));
+            sc[c + 1] = fmaf(wab, d[0], fmaf(slope, (float)(c + 1), shift));
+            sc[c + 2] = fmaf(wcd, d[3], fmaf(slope, (float)(c + 2), shift));
+            sc[c + 3] = fmaf(wcd, d[2], fmaf(slope, (float)(c + 3), shift));
+          }
+        } else {
+#pragma unroll
+          for (int c = 0; c < AT_KEYS; ++c) sc[c] = fmaf(sc[c], scale_log2, fmaf(slope, (float)c, shift));
+        }
+      }
       if (need_mask) {
 #pragma unroll
         for (int c = 0; c < AT_KEYS; ++c)
@@ -365,7 +393,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
         mx4[2] = fmaxf(mx4[2], sc[c + 2]);
         mx4[3] = fmaxf(mx4[3], sc[c + 3]);
       }
-      const float mx = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3])) * (DIST ? 1.f : scale_log2);
+      const float mx = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3])) * (KIND ? 1.f : scale_log2);
       // move the reference only when the maximum has outgrown it by a lot (or there was none yet)
       const bool move = (mx > m_ref + AT_LAZY) || (m_ref == -INFINITY && mx > -INFINITY);
       float corr = 1.f;
@@ -398,7 +426,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
       uint32_t packed[AT_KEYS / 2];
 #pragma unroll
       for (int c = 0; c < AT_KEYS; c += 4) {
-        const float sl = DIST ? 1.f : scale_log2;
+        const float sl = KIND ? 1.f : scale_log2;
         const float p0 = at_exp2(fmaf(sc[c], sl, -sub)), p1 = at_exp2(fmaf(sc[c + 1], sl, -sub));
         const float p2 = at_exp2(fmaf(sc[c + 2], sl, -sub)), p3 = at_exp2(fmaf(sc[c + 3], sl, -sub));
         sum4[0] += p0; sum4[1] += p1; sum4[2] += p2; sum4[3] += p3;
@@ -501,23 +529,24 @@ AB_API int ab_attention_prefill_tc_supports(int H, int K, int D) {
 // (q part read); out [n_tokens, H*D], cache pages [n_pages, K, 64, D].  `sink`: float [H] or null, one more term
 // exp(sink_h) in every softmax's denominator.
 // tile_seq / tile_q0: the tiles of floor(128 / G) tokens (sequence, first packed token), as for the mma kernel.
-// `dist`: float [2, H] or null, the penalty on distance (G up to AT_DIST_MAX_GROUP: the tables' shared memory).
+// `kind`, `dist`, `cap`: attention_scores.cuh (SCORE_LOG: G up to AT_DIST_MAX_GROUP, the tables' shared memory).
 #define AT_DIST_MAX_GROUP 16
 AB_API int ab_attention_prefill_tc_dist_max_group() { return AT_DIST_MAX_GROUP; }
 AB_API int ab_attention_prefill_tc_dist(const void* qkv, int row_heads, int n_tokens, void* out, const void* k_pages,
                                         const void* v_pages, int n_pages, const int* block_table, int table_width,
                                         const int* tok_pos, const int* cu_q, const int* tile_seq, const int* tile_q0,
                                         int n_tiles, int H, int K, int D, float scale, int window, const float* sink,
-                                        const float* dist, cudaStream_t stream) {
+                                        int kind, const float* dist, float cap, cudaStream_t stream) {
   if (n_tiles <= 0) return AB_OK;
+  if (!score_kind_ok(kind, dist)) return AB_BAD_ARG;
   if (!ab_attention_prefill_tc_supports(H, K, D) || (long long)n_tiles * K > 0x7fffffffLL || row_heads < H)
     return AB_BAD_ARG;
   AtEncodeFn enc = at_encode_fn();
   int* status = at_status_word();
   if (!enc || !status) return AB_BAD_ARG;
   const int G = H / K, tpt = AT_ROWS / G;
-  if (dist != nullptr && G > AT_DIST_MAX_GROUP) return AB_BAD_ARG;
-  const size_t d_bytes = dist != nullptr ? (size_t)2 * G * at_dist_stride(tpt, G) * sizeof(float) : 0;
+  if (kind == SCORE_LOG && G > AT_DIST_MAX_GROUP) return AB_BAD_ARG;
+  const size_t d_bytes = kind == SCORE_LOG ? (size_t)2 * G * at_dist_stride(tpt, G) * sizeof(float) : 0;
   CUtensorMap mq, mk, mv;
   {
     cuuint64_t dims[3] = {(cuuint64_t)D, (cuuint64_t)row_heads, (cuuint64_t)n_tokens};
@@ -548,10 +577,11 @@ AB_API int ab_attention_prefill_tc_dist(const void* qkv, int row_heads, int n_to
     if (e != cudaSuccess) return AB_CUDA_ERR + (int)e;                                                              \
     e = ab_launch(attention_prefill_tc_kernel<HDV, DS>, dim3((unsigned)n_tiles * K), dim3(AT_THREADS), smem,        \
                   stream, mq, mk, mv, (bf16*)out, block_table, table_width, tok_pos, cu_q, tile_seq, tile_q0, H, K, \
-                  scale * AT_LOG2E, window, tpt, status, sink, dist);                                               \
+                  scale * AT_LOG2E, window, tpt, status, sink, dist, cap);                                          \
   }
-  if (dist != nullptr) { if (D == 64) AT_GO(64, true) else AT_GO(128, true) }
-  else { if (D == 64) AT_GO(64, false) else AT_GO(128, false) }
+  if (kind == SCORE_LOG) { if (D == 64) AT_GO(64, SCORE_LOG) else AT_GO(128, SCORE_LOG) }
+  else if (kind == SCORE_BOUND) { if (D == 64) AT_GO(64, SCORE_BOUND) else AT_GO(128, SCORE_BOUND) }
+  else { if (D == 64) AT_GO(64, SCORE_PLAIN) else AT_GO(128, SCORE_PLAIN) }
 #undef AT_GO
   if (e != cudaSuccess) return AB_CUDA_ERR + (int)e;
   return ab_launch_status();
@@ -563,8 +593,8 @@ AB_API int ab_attention_prefill_tc_sink(const void* qkv, int row_heads, int n_to
                                         int n_tiles, int H, int K, int D, float scale, int window, const float* sink,
                                         cudaStream_t stream) {
   return ab_attention_prefill_tc_dist(qkv, row_heads, n_tokens, out, k_pages, v_pages, n_pages, block_table, table_width,
-                                      tok_pos, cu_q, tile_seq, tile_q0, n_tiles, H, K, D, scale, window, sink, nullptr,
-                                      stream);
+                                      tok_pos, cu_q, tile_seq, tile_q0, n_tiles, H, K, D, scale, window, sink, SCORE_PLAIN,
+                                      nullptr, 0.f, stream);
 }
 
 // qkv [n_tokens, (H+2K)*D]: q | k | v of a token side by side; no sink.

@@ -2,7 +2,7 @@
 // sub-layers' outputs, whose mixers see the stream through a short causal convolution and whose results are averaged
 // over depth:
 //
-//   embed_positions  x[t] = table[token_t] + pos[place_t]                       token rows plus learned position rows
+//   embed_positions  x[t] = scale * table[token_t] + pos[place_t]               token rows plus learned position rows
 //   input_conv       h[t] = x[t] + sum_j w[:, j] x[t - taps + 1 + j]            per channel over time, zeros before the
 //                    sequence's start; a sequence's last taps - 1 rows of x are its state, kept from step to step
 //   post_norm_stream v = x[t] + y[t] / sqrt(mean(y[t]^2) + eps) * w             a sub-layer's output joins the stream;
@@ -48,7 +48,7 @@ __device__ __forceinline__ float dot4(float4 a, float4 b) { return (a.x * b.x + 
 // ---------------------------------------------------------------------------
 template <typename T, bool VEC>
 __global__ void embed_positions_kernel(const T* __restrict__ table, const T* __restrict__ pos, const int* __restrict__ tokens,
-                                       const int* __restrict__ tok_seq, const int* __restrict__ tok_pos,
+                                       const int* __restrict__ tok_seq, const int* __restrict__ tok_pos, float scale,
                                        float* __restrict__ out, int width) {
   pdl_wait();
   pdl_trigger();
@@ -63,20 +63,20 @@ __global__ void embed_positions_kernel(const T* __restrict__ table, const T* __r
   if (VEC) {
     for (int j = threadIdx.x * 4; j < width; j += blockDim.x * 4) {
       const float4 a = Quad<T>::load(e + j), b = Quad<T>::load(p + j);
-      *reinterpret_cast<float4*>(o + j) = make_float4(a.x + b.x, a.y + b.y, a.z + b.z, a.w + b.w);
+      *reinterpret_cast<float4*>(o + j) = axpy4(scale, a, b);
     }
   } else {
-    for (int j = threadIdx.x; j < width; j += blockDim.x) o[j] = to_f32(e[j]) + to_f32(p[j]);
+    for (int j = threadIdx.x; j < width; j += blockDim.x) o[j] = fmaf(scale, to_f32(e[j]), to_f32(p[j]));
   }
 }
 
 AB_API int ab_embed_positions(const void* table, const void* pos, int dtype, const int* tokens, const int* tok_seq,
-                              const int* tok_pos, float* out, int n_tokens, int width, cudaStream_t stream) {
+                              const int* tok_pos, float scale, float* out, int n_tokens, int width, cudaStream_t stream) {
   if (n_tokens <= 0 || width <= 0) return AB_OK;
   const int threads = width >= 1024 ? 256 : 128;
 #define AB_GO(T, V)                                                                                                    \
   ab_launch(embed_positions_kernel<T, V>, dim3((unsigned)n_tokens), dim3(threads), 0, stream, (const T*)table, (const T*)pos, \
-            tokens, tok_seq, tok_pos, out, width)
+            tokens, tok_seq, tok_pos, scale, out, width)
   if (dtype == AB_F32) { if (width % 4 == 0) AB_GO(float, true); else AB_GO(float, false); }
   else if (dtype == AB_BF16) { if (width % 4 == 0) AB_GO(bf16, true); else AB_GO(bf16, false); }
   else return AB_BAD_ARG;

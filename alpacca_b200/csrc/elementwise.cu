@@ -595,11 +595,13 @@ AB_API int ab_gated_act(const void* gu, void* act, int dtype, int n_rows, int F,
 __device__ __forceinline__ float gelu_exact(float z) { return 0.5f * z * (1.0f + erff(z * 0.70710678118654752440f)); }
 
 template <typename T>
-__global__ void act_kernel(T* __restrict__ y, size_t total) {
+__global__ void act_kernel(T* __restrict__ y, size_t total, int kind) {
   pdl_wait();
   pdl_trigger();
   const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
-  if (i < total) y[i] = from_f32<T>(gelu_exact(to_f32(y[i])));
+  if (i >= total) return;
+  const float v = to_f32(y[i]), r = fmaxf(v, 0.f);
+  y[i] = from_f32<T>(kind == 1 ? r * r : gelu_exact(v));
 }
 // The same for bfloat16 rows: erf by the rational approximation of Abramowitz and Stegun, "Handbook of Mathematical
 // Functions", 7.1.26 (absolute error 1.5e-7, far below the rounding of the result), with the hardware's approximate
@@ -611,6 +613,7 @@ __device__ __forceinline__ float gelu_fast(float y) {
   const float q = p * __expf(-x * x);                    // 1 - erf(x)
   return 0.5f * y * (y < 0.f ? q : 2.0f - q);
 }
+template <int KIND>
 __global__ void act_bf16x8_kernel(uint4* __restrict__ y, size_t n8) {
   pdl_wait();
   pdl_trigger();
@@ -620,7 +623,15 @@ __global__ void act_bf16x8_kernel(uint4* __restrict__ y, size_t n8) {
   uint32_t* w = reinterpret_cast<uint32_t*>(&v);
 #pragma unroll
   for (int j = 0; j < 4; ++j) {
-    __nv_bfloat162 r = __floats2bfloat162_rn(gelu_fast(__uint_as_float(w[j] << 16)), gelu_fast(__uint_as_float(w[j] & 0xffff0000u)));
+    float a = __uint_as_float(w[j] << 16), b = __uint_as_float(w[j] & 0xffff0000u);
+    if (KIND == 1) {
+      a = fmaxf(a, 0.f) * fmaxf(a, 0.f);
+      b = fmaxf(b, 0.f) * fmaxf(b, 0.f);
+    } else {
+      a = gelu_fast(a);
+      b = gelu_fast(b);
+    }
+    __nv_bfloat162 r = __floats2bfloat162_rn(a, b);
     w[j] = *reinterpret_cast<uint32_t*>(&r);
   }
   y[i] = v;
@@ -628,13 +639,13 @@ __global__ void act_bf16x8_kernel(uint4* __restrict__ y, size_t n8) {
 
 AB_API int ab_act(void* y, int dtype, long long total, int kind, cudaStream_t stream) {
   if (total <= 0) return AB_OK;
-  if (kind != 0) return AB_BAD_ARG;
+  if (kind != 0 && kind != 1) return AB_BAD_ARG;
   if (dtype == AB_BF16 && total % 8 == 0 && (((uintptr_t)y) & 15) == 0)
-    ab_launch(act_bf16x8_kernel, (unsigned)((total / 8 + 255) / 256), 256, 0, stream, (uint4*)y, (size_t)(total / 8));
+    ab_launch(kind == 1 ? act_bf16x8_kernel<1> : act_bf16x8_kernel<0>, (unsigned)((total / 8 + 255) / 256), 256, 0, stream, (uint4*)y, (size_t)(total / 8));
   else if (dtype == AB_BF16)
-    ab_launch(act_kernel<bf16>, (unsigned)((total + 255) / 256), 256, 0, stream, (bf16*)y, (size_t)total);
+    ab_launch(act_kernel<bf16>, (unsigned)((total + 255) / 256), 256, 0, stream, (bf16*)y, (size_t)total, kind);
   else if (dtype == AB_F32)
-    ab_launch(act_kernel<float>, (unsigned)((total + 255) / 256), 256, 0, stream, (float*)y, (size_t)total);
+    ab_launch(act_kernel<float>, (unsigned)((total + 255) / 256), 256, 0, stream, (float*)y, (size_t)total, kind);
   else
     return AB_BAD_ARG;
   return ab_launch_status();

@@ -7,6 +7,9 @@
 //       S <- g_t S;   u = beta_t (v_t - S^T k_t);   S <- S + k_t u^T;   o_t = S^T q_t      g_t, beta_t: one number
 //       per head and token; the read-out sees the token's own write
 //
+//   mode 2, one decay and one step size per head (a state-space model; csrc/state_space.cu has its other kernels):
+//       S <- g_t S + b_t k_t v_t^T;   o_t = S^T q_t + skip_h v_t       g_t, b_t: one number per head and token
+//
 // The walk (`recurrence_kernel`): a CTA per (sequence, head, tile of value columns); a column's D entries are spread
 // over 8, 16 or 32 neighbouring lanes' registers (a part of the rows each, read 16 bytes at a time), q, k and the decays of eight tokens at a time arrive in
 // shared memory by `cp.async` through a ring of four buffers (three rounds' rows are on their way while one is walked), a
@@ -98,6 +101,20 @@ __device__ __forceinline__ float walk_token(float (&S)[DR], const float4* __rest
       a2 += S[i + 2] * qq.z;
       a3 += S[i + 3] * qq.w;
     }
+  } else if (MODE == 2) {
+    const float u = bt * vj;
+#pragma unroll
+    for (int i = 0; i < DR; i += 4) {
+      const float4 kk = kr[i >> 2], qq = qr[i >> 2];
+      S[i] = g * S[i] + kk.x * u;
+      S[i + 1] = g * S[i + 1] + kk.y * u;
+      S[i + 2] = g * S[i + 2] + kk.z * u;
+      S[i + 3] = g * S[i + 3] + kk.w * u;
+      a0 += S[i] * qq.x;
+      a1 += S[i + 1] * qq.y;
+      a2 += S[i + 2] * qq.z;
+      a3 += S[i + 3] * qq.w;
+    }
   } else {
     float d0 = 0.f, d1 = 0.f, d2 = 0.f, d3 = 0.f;
 #pragma unroll
@@ -135,8 +152,8 @@ __device__ __forceinline__ float walk_token(float (&S)[DR], const float4* __rest
 template <int DR, int LANES, int MODE, int STAGES>
 __global__ void recurrence_kernel(const float* __restrict__ q, int ldq, const float* __restrict__ k, int ldk,
                                   const float* __restrict__ v, int ldv, const float* __restrict__ dvec, int ldd,
-                                  const float* __restrict__ dsc, const float* __restrict__ beta, float qscale,
-                                  float* __restrict__ state, float* __restrict__ out, const int* __restrict__ cu_q,
+                                  const float* __restrict__ dsc, const float* __restrict__ beta,
+                                  const float* __restrict__ skip, float qscale, float* __restrict__ state, float* __restrict__ out, const int* __restrict__ cu_q,
                                   const int* __restrict__ slots, int H, int Hk, int D, int V, int CV, int write_state,
                                   int vec) {
   extern __shared__ __align__(16) float rec_sm[];
@@ -147,6 +164,7 @@ __global__ void recurrence_kernel(const float* __restrict__ q, int ldq, const fl
   const int b = blockIdx.x, h = blockIdx.y, col0 = blockIdx.z * CV;
   const int slot = slots[b];
   if (slot < 0) return;
+  const float sk = (MODE == 2 && skip != nullptr) ? skip[h] : 0.f;
   const int kh = h / (H / Hk);
   const int tid = threadIdx.x, col = tid / LANES, r = tid % LANES;
   // a ring of buffers of a round's tokens: q, k (and the decays) of P4 floats each, CV values, two numbers per token
@@ -195,7 +213,7 @@ __global__ void recurrence_kernel(const float* __restrict__ q, int ldq, const fl
       stage_rows<DR>(rows, base + 2 * REC_TOKENS * P4, P4, dvec + (size_t)c0 * ldd + (size_t)h * D, ldd, n, D, vec);
     float* vs = base + NV * REC_TOKENS * P4;
     stage_rows<0>(vals, vs, CV, v + (size_t)c0 * ldv + (size_t)h * V + col0, ldv, n, cw, vec_v);
-    if (MODE == 1 && tid < n) {
+    if (MODE != 0 && tid < n) {
       float* sc = vs + REC_TOKENS * CV;
       copy_async4(sc + 2 * tid, dsc + (size_t)(c0 + tid) * H + h);
       copy_async4(sc + 2 * tid + 1, beta + (size_t)(c0 + tid) * H + h);
@@ -232,7 +250,8 @@ __global__ void recurrence_kernel(const float* __restrict__ q, int ldq, const fl
         sh[tt] = walk_token<DR, LANES, MODE>(S, reinterpret_cast<const float4*>(qs + tt * P4),
                                              reinterpret_cast<const float4*>(ks + tt * P4),
                                              reinterpret_cast<const float4*>(as + tt * P4), vs[tt * CV + col],
-                                             MODE == 1 ? sc[2 * tt] : 0.f, MODE == 1 ? sc[2 * tt + 1] : 0.f);
+                                             MODE != 0 ? sc[2 * tt] : 0.f, MODE != 0 ? sc[2 * tt + 1] : 0.f) +
+                 (MODE == 2 && r == 0 ? sk * vs[tt * CV + col] : 0.f);       // (the first lane of a column adds the skip)
 #pragma unroll
       for (int tt = 0; tt < REC_TOKENS; ++tt) mine[tt * CV * LANES] = sh[tt];
     } else {
@@ -240,7 +259,8 @@ __global__ void recurrence_kernel(const float* __restrict__ q, int ldq, const fl
         mine[tt * CV * LANES] = walk_token<DR, LANES, MODE>(S, reinterpret_cast<const float4*>(qs + tt * P4),
                                                             reinterpret_cast<const float4*>(ks + tt * P4),
                                                             reinterpret_cast<const float4*>(as + tt * P4), vs[tt * CV + col],
-                                                            MODE == 1 ? sc[2 * tt] : 0.f, MODE == 1 ? sc[2 * tt + 1] : 0.f);
+                                                            MODE != 0 ? sc[2 * tt] : 0.f, MODE != 0 ? sc[2 * tt + 1] : 0.f) +
+                                (MODE == 2 && r == 0 ? sk * vs[tt * CV + col] : 0.f);
     }
     __syncthreads();
     // a column's read-out: its lanes' shares, added in lane order
@@ -272,21 +292,22 @@ __global__ void recurrence_kernel(const float* __restrict__ q, int ldq, const fl
 }
 
 // One walk over the step's tokens.  q, k float32 rows with Hk heads of D (row strides ldq, ldk), v with H heads of V;
-// mode 0: dvec [T, H * D] (row stride ldd); mode 1: dsc, beta [T, H].  state [slots, H, D, V]; out [T, H * V].
+// mode 0: dvec [T, H * D] (row stride ldd); modes 1, 2: dsc, beta [T, H]; mode 2: skip [H] or null.  state [slots, H, D, V]; out [T, H * V].
 // `cols`: value columns per CTA (8, 16 or 32).  `one_round`: no sequence brings more than REC_TOKENS tokens.
 AB_API int ab_gated_recurrence(int mode, const float* q, int ldq, const float* k, int ldk, const float* v, int ldv,
-                               const float* dvec, int ldd, const float* dsc, const float* beta, float qscale, float* state,
+                               const float* dvec, int ldd, const float* dsc, const float* beta, const float* skip, float qscale,
+                               float* state,
                                float* out, const int* cu_q, const int* slots, int n_seqs, int H, int Hk, int D, int V,
                                int cols, int write_state, int one_round, cudaStream_t stream) {
   if (n_seqs <= 0) return AB_OK;
   if (H <= 0 || Hk <= 0 || H % Hk || D <= 0 || D > 256 || V <= 0 || (cols != 8 && cols != 16 && cols != 32)) return AB_BAD_ARG;
   if (!q || !k || !v || !state || !out || !cu_q || !slots) return AB_BAD_ARG;
-  if (mode == 0 ? !dvec : (mode != 1 || !dsc || !beta)) return AB_BAD_ARG;
+  if (mode == 0 ? !dvec : (mode < 0 || mode > 2 || !dsc || !beta)) return AB_BAD_ARG;
   // More lanes per column where few (sequence, head, column) triples would leave the schedulers with a warp or none
   // each: a walk is a chain of dependent steps per token, and what hides its latency is other warps.
   int lanes = 8;
   const long long threads8 = (long long)n_seqs * H * ((V + cols - 1) / cols) * cols * 8;
-  if (mode == 0 && D > 32 && threads8 < 600LL * 32) lanes = 16;      // (the delta rule's lanes exchange a sum per token)
+  if (mode != 1 && D > 32 && threads8 < 600LL * 32) lanes = 16;      // (the delta rule's lanes exchange a sum per token)
   const int per = (D + lanes - 1) / lanes;
   const int DR = per <= 4 ? 4 : (per <= 8 ? 8 : (per <= 16 ? 16 : 32));
   const int P4 = lanes * (DR > 4 ? DR + 4 : DR);
@@ -304,10 +325,12 @@ AB_API int ab_gated_recurrence(int mode, const float* q, int ldq, const float* k
     if (smem > 48 * 1024)                                                                                                 \
       cudaFuncSetAttribute(recurrence_kernel<DRV, L, M, ST>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);     \
     ab_launch(recurrence_kernel<DRV, L, M, ST>, grid, block, smem, stream, q, ldq, k, ldk, v, ldv, dvec, ldd, dsc, beta,  \
-              qscale, state, out, cu_q, slots, H, Hk, D, V, cols, write_state, vec);                                      \
+              skip, qscale, state, out, cu_q, slots, H, Hk, D, V, cols, write_state, vec);                                      \
     done = true;                                                                                                          \
   }
-#define AB_BOTH(DRV, L) AB_GO(DRV, L, 0, 1) AB_GO(DRV, L, 1, 1) AB_GO(DRV, L, 0, REC_STAGES) AB_GO(DRV, L, 1, REC_STAGES)
+#define AB_BOTH(DRV, L)                                                                                                   \
+  AB_GO(DRV, L, 0, 1) AB_GO(DRV, L, 1, 1) AB_GO(DRV, L, 2, 1)                                                             \
+  AB_GO(DRV, L, 0, REC_STAGES) AB_GO(DRV, L, 1, REC_STAGES) AB_GO(DRV, L, 2, REC_STAGES)
   AB_BOTH(4, 8) AB_BOTH(8, 8) AB_BOTH(16, 8) AB_BOTH(32, 8)
   AB_BOTH(4, 16) AB_BOTH(8, 16) AB_BOTH(16, 16)
   AB_BOTH(4, 32) AB_BOTH(8, 32)

@@ -47,6 +47,8 @@
 #define EPI_SWIGLU_BF16 2
 #define EPI_RELUGLU_BF16 3      // the same tail with max(g, 0) on the gate
 #define EPI_GELUGLU_BF16 4      // ... with the tanh form of GELU on the gate
+#define EPI_RELU2_BF16 5        // no gate: max(y, 0)^2, of y times a factor per row where there is one (persistent forms)
+#define EPI_GATED(E) ((E) >= EPI_SWIGLU_BF16 && (E) <= EPI_GELUGLU_BF16)
 
 __device__ __forceinline__ uint32_t smem_addr(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
 
@@ -130,13 +132,22 @@ template <int BN> struct TcShape {
 // The tail for 16 consecutive accumulator columns c0..c0+15 of row `row` of the tile.
 //   !SWAP: row = token (global row m), columns = features n0 + c
 //    SWAP: row = feature (global n), columns = batch rows c
+// max(f y, 0)^2 of 16 columns
+__device__ __forceinline__ void relu2_16(float* v, float f) {
+#pragma unroll
+  for (int c = 0; c < 16; ++c) {
+    const float r = fmaxf(f * v[c], 0.f);
+    v[c] = r * r;
+  }
+}
+
 template <int EPI, bool SWAP>
 __device__ __forceinline__ void tail16(const float* v, int row_g, int col0_g, int rows_total, int cols_total,
                                        const float* __restrict__ bias, void* __restrict__ Y, int ldy, int lane) {
   if (!SWAP) {
     const int m = row_g;
     if (m >= rows_total) return;
-    if (EPI >= EPI_SWIGLU_BF16) {
+    if (EPI_GATED(EPI)) {
       // columns col0..col0+7 gate, +8..+15 up of units (col0/16)*8 + 0..7
       if (col0_g + 16 > cols_total) return;
       bf16* y = reinterpret_cast<bf16*>(Y) + (size_t)m * ldy + (col0_g >> 1);
@@ -181,7 +192,7 @@ __device__ __forceinline__ void tail16(const float* v, int row_g, int col0_g, in
     // swapped: this thread's row is feature n; column c is batch row m = col0_g + c
     const int n = row_g;
     const float b = (bias && n < rows_total) ? bias[n] : 0.f;
-    if (EPI >= EPI_SWIGLU_BF16) {
+    if (EPI_GATED(EPI)) {
       // rows 16q..16q+7 gate, 16q+8..16q+15 up: lanes with bit 3 clear hold gates, their partner is lane + 8
       const int unit = (n >> 4) * 8 + (n & 7);
 #pragma unroll
@@ -406,7 +417,7 @@ __global__ void __launch_bounds__(TC_THREADS)
 gemm_tc_persistent_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant__ CUtensorMap map_w,
                           void* __restrict__ Y, const float* __restrict__ bias, int* __restrict__ status, int M, int N,
                           int K, int ldy, int tiles_m, int n_tiles, const int* __restrict__ tile_group,
-                          const int* __restrict__ row_tiles) {
+                          const int* __restrict__ row_tiles, const float* __restrict__ row_factor) {
   extern __shared__ unsigned char smem_raw[];
   unsigned char* base = reinterpret_cast<unsigned char*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~(uintptr_t)1023);
   uint64_t* full = reinterpret_cast<uint64_t*>(base + TP_STAGES * TP_STAGE_BYTES);
@@ -512,10 +523,13 @@ gemm_tc_persistent_kernel(const __grid_constant__ CUtensorMap map_x, const __gri
       ok = __all_sync(0xffffffffu, ok);      // tcgen05.ld below is warp-wide
       if (!ok) break;
       asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+      float factor = 1.f;
+      if (EPI == EPI_RELU2_BF16 && row_factor != nullptr && m0 + row < M) factor = row_factor[m0 + row];
 #pragma unroll 1
       for (int c0 = 0; c0 < TP_BN; c0 += 16) {
         float v[16];
         tmem_ld16(tmem + ((uint32_t)(quarter * 32) << 16) + (uint32_t)buf * TP_BN + c0, v);
+        if (EPI == EPI_RELU2_BF16) relu2_16(v, factor);
         tail16<EPI, false>(v, m0 + row, n0 + c0, M, N, bias, Y, ldy, lane);
       }
       asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
@@ -708,6 +722,7 @@ gemm_tc_pair_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_cons
       for (int c0 = 0; c0 < TP_BN; c0 += 16) {
         float v[16];
         tmem_ld16(tmem + ((uint32_t)(quarter * 32) << 16) + (uint32_t)buf * TP_BN + c0, v);
+        if (EPI == EPI_RELU2_BF16) relu2_16(v, 1.f);
         tail16<EPI, false>(v, m0 + (int)rank * TC_BM + row, n0 + c0, M, N, bias, Y, ldy, lane);
       }
       asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
@@ -815,7 +830,7 @@ AB_API int ab_gemm_tc(const void* X, const void* W, const float* bias, void* Y, 
                       cudaStream_t stream) {
   if (M <= 0 || N <= 0) return AB_OK;
   if (K <= 0 || (K % 8) || slices < 1) return AB_BAD_ARG;
-  if (epilogue_kind >= EPI_SWIGLU_BF16 && (N % 16)) return AB_BAD_ARG;
+  if (EPI_GATED(epilogue_kind) && (N % 16)) return AB_BAD_ARG;
   if (slices > 1 && (!partials || !arrivals)) return AB_BAD_ARG;
   int* status = status_word();
   if (!status) return AB_BAD_ARG;
@@ -835,13 +850,14 @@ AB_API int ab_gemm_tc(const void* X, const void* W, const float* bias, void* Y, 
   return AB_BAD_ARG;
 }
 
-// The persistent form (epilogue kinds 0 to 4: the gated tails also with ReLU or tanh-GELU on the gate):
+// The persistent form (epilogue kinds 0 to 5: the gated tails also with ReLU or tanh-GELU on the gate, the squared ReLU
+// without a bias):
 // Y = X[M,K] . W[N,K]^T for many rows, tiles of 128 x 256, one CTA per processor.
 AB_API int ab_gemm_tc_persistent(const void* X, const void* W, const float* bias, void* Y, int M, int N, int K,
                                  int ldy, int epilogue_kind, cudaStream_t stream) {
   if (M <= 0 || N <= 0) return AB_OK;
   if (K <= 0 || (K % 8)) return AB_BAD_ARG;
-  if (epilogue_kind >= EPI_SWIGLU_BF16 && (N % 16)) return AB_BAD_ARG;
+  if (EPI_GATED(epilogue_kind) && (N % 16)) return AB_BAD_ARG;
   int* status = status_word();
   if (!status) return AB_BAD_ARG;
   CUtensorMap mx, mw;
@@ -861,7 +877,8 @@ AB_API int ab_gemm_tc_persistent(const void* X, const void* W, const float* bias
     cudaError_t e = cudaFuncSetAttribute(gemm_tc_persistent_kernel<E, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, TP_SMEM); \
     if (e != cudaSuccess) return AB_CUDA_ERR + (int)e;                                                             \
     e = ab_launch(gemm_tc_persistent_kernel<E, false>, dim3(grid), dim3(TC_THREADS), (size_t)TP_SMEM, stream, mx, mw, Y, \
-                  bias, status, M, N, K, ldy, tiles_m, n_tiles, (const int*)nullptr, (const int*)nullptr);         \
+                  bias, status, M, N, K, ldy, tiles_m, n_tiles, (const int*)nullptr, (const int*)nullptr,          \
+                  (const float*)nullptr);                                                                          \
     if (e != cudaSuccess) return AB_CUDA_ERR + (int)e;                                                             \
     return ab_launch_status();                                                                                     \
   }
@@ -871,6 +888,7 @@ AB_API int ab_gemm_tc_persistent(const void* X, const void* W, const float* bias
     case EPI_SWIGLU_BF16: AB_GO(EPI_SWIGLU_BF16)
     case EPI_RELUGLU_BF16: AB_GO(EPI_RELUGLU_BF16)
     case EPI_GELUGLU_BF16: AB_GO(EPI_GELUGLU_BF16)
+    case EPI_RELU2_BF16: if (bias == nullptr) AB_GO(EPI_RELU2_BF16) else return AB_BAD_ARG;
   }
 #undef AB_GO
   return AB_BAD_ARG;
@@ -878,9 +896,10 @@ AB_API int ab_gemm_tc_persistent(const void* X, const void* W, const float* bias
 
 // Rows in groups with a matrix each (see the kernel): X [max_rows, K] in row tiles of 128 (max_rows a multiple of 128), W
 // [groups * N, K], Y [max_rows, ..]; tile_group int [max_rows / 128], row_tiles int [1] on the device.  Epilogue kinds 0
-// (bfloat16) and 2 (SwiGLU).
+// (bfloat16), 2 (SwiGLU) and 5 (squared ReLU, of the products times row_factor [max_rows] where it is given).
 AB_API int ab_gemm_tc_grouped(const void* X, const void* W, void* Y, int max_rows, int N, int K, int groups, int ldy,
-                              int epilogue_kind, const int* tile_group, const int* row_tiles, cudaStream_t stream) {
+                              int epilogue_kind, const int* tile_group, const int* row_tiles, const float* row_factor,
+                              cudaStream_t stream) {
   if (max_rows <= 0 || N <= 0) return AB_OK;
   if (K <= 0 || (K % 8) || groups <= 0 || (max_rows % TC_BM) || (long long)groups * N > 0x7fffffffLL || !tile_group || !row_tiles)
     return AB_BAD_ARG;
@@ -905,13 +924,15 @@ AB_API int ab_gemm_tc_grouped(const void* X, const void* W, void* Y, int max_row
     cudaError_t e = cudaFuncSetAttribute(gemm_tc_persistent_kernel<E, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, TP_SMEM); \
     if (e != cudaSuccess) return AB_CUDA_ERR + (int)e;                                                             \
     e = ab_launch(gemm_tc_persistent_kernel<E, true>, dim3(grid), dim3(TC_THREADS), (size_t)TP_SMEM, stream, mx, mw, Y, \
-                  (const float*)nullptr, status, max_rows, N, K, ldy, tiles_m, n_tiles, tile_group, row_tiles);    \
+                  (const float*)nullptr, status, max_rows, N, K, ldy, tiles_m, n_tiles, tile_group, row_tiles,     \
+                  row_factor);                                                                                     \
     if (e != cudaSuccess) return AB_CUDA_ERR + (int)e;                                                             \
     return ab_launch_status();                                                                                     \
   }
   switch (epilogue_kind) {
     case EPI_STORE_BF16: AB_GO(EPI_STORE_BF16)
     case EPI_SWIGLU_BF16: AB_GO(EPI_SWIGLU_BF16)
+    case EPI_RELU2_BF16: AB_GO(EPI_RELU2_BF16)
   }
 #undef AB_GO
   return AB_BAD_ARG;
@@ -922,7 +943,7 @@ AB_API int ab_gemm_tc_pair(const void* X, const void* W, const float* bias, void
                            int ldy, int epilogue_kind, cudaStream_t stream) {
   if (M <= 0 || N <= 0) return AB_OK;
   if (K <= 0 || (K % 8)) return AB_BAD_ARG;
-  if (epilogue_kind >= EPI_SWIGLU_BF16 && (N % 16)) return AB_BAD_ARG;
+  if (EPI_GATED(epilogue_kind) && (N % 16)) return AB_BAD_ARG;
   int* status = status_word();
   if (!status) return AB_BAD_ARG;
   CUtensorMap mx, mw;
@@ -965,6 +986,7 @@ AB_API int ab_gemm_tc_pair(const void* X, const void* W, const float* bias, void
     case EPI_SWIGLU_BF16: AB_GO(EPI_SWIGLU_BF16)
     case EPI_RELUGLU_BF16: AB_GO(EPI_RELUGLU_BF16)
     case EPI_GELUGLU_BF16: AB_GO(EPI_GELUGLU_BF16)
+    case EPI_RELU2_BF16: if (bias == nullptr) AB_GO(EPI_RELU2_BF16) else return AB_BAD_ARG;
   }
 #undef AB_GO
   return AB_BAD_ARG;

@@ -61,7 +61,7 @@
 #define EPI_STORE_F32 1
 #define EPI_SWIGLU_BF16 2
 #define EPI_RESIDUAL_BF16 3
-#define EPI_GELU_BF16 4      // a bfloat16 store behind GELU in its erf form
+#define EPI_ACT_BF16 4       // a bfloat16 store behind an activation: GELU in its erf form, or the square of ReLU
 #define EPI_CAP_F32 5        // a float32 store of cap * tanh(y / cap)
 
 // What the norm fusion adds to a launch; all null / 0 without it.
@@ -72,7 +72,8 @@ struct GemvNorm {
   float* residual;        // EPI_RESIDUAL: float32 [M, N], updated in place
   const float* norm_w;    // EPI_RESIDUAL: float32 [N], the weight of the norm that follows
   float* ss_out;          // EPI_RESIDUAL: float32 [M, ceil(N / 16)]
-  int gate_act;           // EPI_SWIGLU: the activation on the gate, 0 SiLU, 1 ReLU, 2 GELU in its tanh form
+  int gate_act;           // EPI_SWIGLU: the activation on the gate, 0 SiLU, 1 ReLU, 2 GELU in its tanh form;
+                          // EPI_ACT: 0 GELU (erf), 1 max(y, 0)^2
   float cap;              // EPI_CAP_F32
 };
 
@@ -170,7 +171,7 @@ __device__ __forceinline__ void epilogue(const float acc[4], int i, int ln, int 
       const int n = (j < 2) ? na : nb, m = m0 + (j & 1);
       if (n < N && m < M) {
         float v = c[j] + (bias ? bias[n] : 0.f);
-        if (EPI == EPI_GELU_BF16) v = 0.5f * v * (1.0f + erff(v * 0.70710678118654752440f));
+        if (EPI == EPI_ACT_BF16) v = nf.gate_act == 1 ? fmaxf(v, 0.f) * fmaxf(v, 0.f) : 0.5f * v * (1.0f + erff(v * 0.70710678118654752440f));
         if (EPI == EPI_CAP_F32) v = nf.cap * tanhf(v / nf.cap);
         if (EPI == EPI_STORE_F32 || EPI == EPI_CAP_F32) reinterpret_cast<float*>(Y)[(size_t)m * ldy + n] = v;
         else reinterpret_cast<bf16*>(Y)[(size_t)m * ldy + n] = __float2bfloat16_rn(v);
@@ -390,7 +391,7 @@ AB_API int ab_gemv_bf16_slices(int N, int K, int n_sms) {
 // slices > 1 needs scratch: partials float [ceil(N/16) * slices * 128 * (1, 2 or 4 for M <= 8, 16, 32)],
 // arrivals int [ceil(N/16)], zero before the first launch and left zero by every launch.
 // gate_act (epilogue 2): the activation on the gate, 0 SiLU, 1 ReLU, 2 GELU in its tanh form.
-// Epilogue 4: a bfloat16 store of GELU (erf) of the result; 5: a float32 store of cap * tanh(result / cap).
+// Epilogue 4: a bfloat16 store of GELU (erf; gate_act 0) or the squared ReLU (gate_act 1) of the result; 5: a float32 store of cap * tanh(result / cap).
 AB_API int ab_gemv_bf16_act(const void* X, const void* W, const float* bias, void* Y, float* partials,
                             int* arrivals, int M, int N, int K, int ldy, int epilogue_kind, int slices,
                             const float* ss_in, int n_part_in, float inv_width, float eps, float* residual,
@@ -414,7 +415,7 @@ AB_API int ab_gemv_bf16_act(const void* X, const void* W, const float* bias, voi
     case EPI_STORE_BF16: return launch<EPI_STORE_BF16>(X, W, bias, Y, partials, arrivals, M, N, K, ldy, slices, wide, nf, stream);
     case EPI_STORE_F32: return launch<EPI_STORE_F32>(X, W, bias, Y, partials, arrivals, M, N, K, ldy, slices, wide, nf, stream);
     case EPI_SWIGLU_BF16: return launch<EPI_SWIGLU_BF16>(X, W, bias, Y, partials, arrivals, M, N, K, ldy, slices, wide, nf, stream);
-    case EPI_GELU_BF16: return launch<EPI_GELU_BF16>(X, W, bias, Y, partials, arrivals, M, N, K, ldy, slices, wide, nf, stream);
+    case EPI_ACT_BF16: return launch<EPI_ACT_BF16>(X, W, bias, Y, partials, arrivals, M, N, K, ldy, slices, wide, nf, stream);
     case EPI_CAP_F32: return launch<EPI_CAP_F32>(X, W, bias, Y, partials, arrivals, M, N, K, ldy, slices, wide, nf, stream);
     case EPI_RESIDUAL_BF16: return launch<EPI_RESIDUAL_BF16>(X, W, bias, Y, partials, arrivals, M, N, K, ldy, slices, wide, nf, stream);
   }

@@ -298,7 +298,7 @@ AB_API int ab_moe_route_scores(const void* h, int dtype, int ld, const float* wr
                                int renorm, float scale, float* z, int* idx, float* wts, cudaStream_t stream) {
   if (n_tokens <= 0) return AB_OK;
   if (E <= 0 || E > MOE_MAX_EXPERTS || groups <= 0 || E % groups || keep <= 0 || keep > groups || top <= 0 ||
-      top > keep * (E / groups) || group_top <= 0 || E / groups > 128 || score_fn < 0 || score_fn > 1)
+      top > keep * (E / groups) || group_top <= 0 || (keep < groups && E / groups > 128) || score_fn < 0 || score_fn > 1)
     return AB_BAD_ARG;
   const int wpb = 4;
   const long long lw = (long long)n_tokens * E;
@@ -486,10 +486,13 @@ AB_API int ab_moe_weigh_all(void* up, int dtype, const int* idx, const float* wt
 }
 
 // ---------------------------------------------------------------------------
-// Gated experts behind any choice, with a shared expert.
+// Experts behind any choice, with a shared expert.
 //
 //   y_t = sum_k weight_k W_down[e_k] (silu(W_gate[e_k] h_t) * (W_up[e_k] h_t))
 //         + sigmoid(z_t) W_down_s (silu(W_gate_s h_t) * (W_up_s h_t))               (if there is a shared expert)
+//
+// without gates: W_down[e_k] act(W_up[e_k] h_t), gate_up then holds the up-projections alone, [E * ff, width].  With
+// `weight_in` weight_k multiplies expert k's input instead of its output.  z null: the shared expert's factor is 1.
 //
 // The choice comes from a router (`idx`, `wts`) or from the token's id: a row of a table names its experts, each with the
 // same constant weight (moe_choice.cuh).  Layouts (ff and fs multiples of 8): gate_up [E, 2 ff, width], an expert's rows in
@@ -552,15 +555,17 @@ __device__ __forceinline__ void lane_dot2(const float* __restrict__ x, const flo
 
 // act: [T, top * ff + fs].  A block of eight warps takes one unit of an expert for eight (token, choice) pairs, or one
 // unit of the shared expert for eight tokens, whose warps then read the same two rows at the same time.
-template <typename T>
+template <typename T, bool GATED>
 __global__ void __launch_bounds__(256)
 moe_shared_up_kernel(const T* __restrict__ h, int ld, const T* __restrict__ gate_up, const T* __restrict__ gate_up_s, Choice c,
-                     T* __restrict__ act, int n_tokens, int top, int width, int ff, int fs, int E, int activation, long long pair_blocks) {
+                     T* __restrict__ act, int n_tokens, int top, int width, int ff, int fs, int E, int activation, int weight_in,
+                     long long pair_blocks) {
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   pdl_wait();
   pdl_trigger();
   const int row_len = top * ff + fs;
   int t;
+  float wgt = 1.0f;
   size_t unit, dst;
   const T* w = gate_up;
   long long blk = blockIdx.x;
@@ -573,6 +578,7 @@ moe_shared_up_kernel(const T* __restrict__ h, int ld, const T* __restrict__ gate
     const int k = (int)(p - (long long)t * top);
     unit = (size_t)chosen_expert(c, t, k, top) * ff + j;
     dst = (size_t)t * row_len + (size_t)k * ff + j;
+    if (weight_in) wgt = chosen_weight(c, t, k, top);
   } else {
     blk -= pair_blocks;
     const int chunk = (int)(blk / fs), j = (int)(blk - (long long)chunk * fs);
@@ -582,12 +588,17 @@ moe_shared_up_kernel(const T* __restrict__ h, int ld, const T* __restrict__ gate
     w = gate_up_s;
     dst = (size_t)t * row_len + (size_t)top * ff + j;
   }
-  const T* gate = w + ((unit >> 3) * 16 + (unit & 7)) * width;
-  float pg, pu;
-  lane_dot2(h + (size_t)t * ld, gate, gate + (size_t)8 * width, width, lane, pg, pu);
-  pg = warp_sum(pg);
+  float pg = 0.f, pu;
+  if (GATED) {
+    const T* gate = w + ((unit >> 3) * 16 + (unit & 7)) * width;
+    lane_dot2(h + (size_t)t * ld, gate, gate + (size_t)8 * width, width, lane, pg, pu);
+    pg = warp_sum(pg);
+  } else {
+    pu = lane_dot(h + (size_t)t * ld, w + unit * width, width, lane);
+  }
   pu = warp_sum(pu);
-  if (lane == 0) act[dst] = from_f32<T>(activate(pg, activation) * pu);
+  // (a weight on the output is applied by the down-projection)
+  if (lane == 0) act[dst] = from_f32<T>(expert_inner<GATED>(pg, pu, wgt, 1, activation));
 }
 
 // out[t, i], float32 or T.  A block of eight warps takes one column i for eight tokens (the shared expert's row is then
@@ -595,7 +606,8 @@ moe_shared_up_kernel(const T* __restrict__ h, int ld, const T* __restrict__ gate
 template <typename T, typename TO>
 __global__ void __launch_bounds__(256)
 moe_shared_down_kernel(const T* __restrict__ act, const T* __restrict__ down, const T* __restrict__ down_s, Choice c,
-                       const float* __restrict__ z, TO* __restrict__ out, int n_tokens, int top, int width, int ff, int fs, int E) {
+                       const float* __restrict__ z, TO* __restrict__ out, int n_tokens, int top, int width, int ff, int fs, int E,
+                       int weight_in) {
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   pdl_wait();
   pdl_trigger();
@@ -607,11 +619,11 @@ moe_shared_down_kernel(const T* __restrict__ act, const T* __restrict__ down, co
   for (int k = 0; k < top; ++k) {
     const int e = chosen_expert(c, t, k, top);
     const float part = lane_dot(a + (size_t)k * ff, down + ((size_t)e * width + i) * ff, ff, lane);
-    total = fmaf(chosen_weight(c, t, k, top), part, total);
+    total = fmaf(weight_in ? 1.0f : chosen_weight(c, t, k, top), part, total);
   }
   if (fs > 0) {
     const float part = lane_dot(a + (size_t)top * ff, down_s + (size_t)i * fs, fs, lane);
-    total = fmaf(1.0f / (1.0f + expf(-z[t])), part, total);
+    total = fmaf(z != nullptr ? 1.0f / (1.0f + expf(-z[t])) : 1.0f, part, total);
   }
   total = warp_sum(total);
   if (lane == 0) out[(size_t)t * width + i] = from_f32<TO>(total);
@@ -621,11 +633,11 @@ moe_shared_down_kernel(const T* __restrict__ act, const T* __restrict__ down, co
 AB_API int ab_moe_shared_pairs(const void* h, int dtype, int ld, const void* gate_up, const void* down, const void* gate_up_s,
                                const void* down_s, const int* idx, const float* wts, const int* table, const int* tokens, float weight, const float* z, void* act,
                                void* out, int out_dtype, int n_tokens, int top, int width, int ff, int fs, int E,
-                               int activation, cudaStream_t stream) {
+                               int activation, int gated, int weight_in, cudaStream_t stream) {
   if (n_tokens <= 0) return AB_OK;
   const Choice c{idx, wts, table, tokens, weight};
-  if (top <= 0 || width <= 0 || ff <= 0 || ff % 8 || fs < 0 || fs % 8 || E <= 0 || (activation != 0 && activation != 1) || !choice_ok(c) ||
-      (fs > 0 && (!z || !gate_up_s || !down_s)))
+  if (top <= 0 || width <= 0 || ff <= 0 || ff % 8 || fs < 0 || fs % 8 || E <= 0 || activation < 0 || activation >= MOE_ACT_KINDS ||
+      !choice_ok(c) || (fs > 0 && (!gate_up_s || !down_s)))
     return AB_BAD_ARG;
   const long long pair_blocks = ((long long)n_tokens * top + 7) / 8 * ff;
   const long long blocks = pair_blocks + ((long long)n_tokens + 7) / 8 * fs;
@@ -633,10 +645,11 @@ AB_API int ab_moe_shared_pairs(const void* h, int dtype, int ld, const void* gat
   const dim3 dgrid((unsigned)width, (unsigned)((n_tokens + 7) / 8));
 #define AB_GO(T, TO)                                                                                                   \
   {                                                                                                                    \
-    ab_launch(moe_shared_up_kernel<T>, dim3((unsigned)blocks), dim3(256), 0, stream, (const T*)h, ld, (const T*)gate_up, \
-              (const T*)gate_up_s, c, (T*)act, n_tokens, top, width, ff, fs, E, activation, pair_blocks);                                      \
+    ab_launch(gated ? moe_shared_up_kernel<T, true> : moe_shared_up_kernel<T, false>, dim3((unsigned)blocks), dim3(256), 0, \
+              stream, (const T*)h, ld, (const T*)gate_up, (const T*)gate_up_s, c, (T*)act, n_tokens, top, width, ff, fs, E, \
+              activation, weight_in, pair_blocks);                                                                     \
     ab_launch(moe_shared_down_kernel<T, TO>, dgrid, dim3(256), 0, stream, (const T*)act, (const T*)down, (const T*)down_s, c, z, (TO*)out, \
-              n_tokens, top, width, ff, fs, E);                                                                        \
+              n_tokens, top, width, ff, fs, E, weight_in);                                                             \
   }
   if (dtype == AB_F32 && out_dtype == AB_F32) AB_GO(float, float)
   else if (dtype == AB_BF16 && out_dtype == AB_F32) AB_GO(bf16, float)
@@ -652,11 +665,11 @@ AB_API int ab_moe_shared_pairs(const void* h, int dtype, int ld, const void* gat
 #define MOE_TILE 128           // rows of a row tile of the grouped product
 
 // pos[t * top + k]: the row of a pair; an expert's rows start on a row tile.  tile_group[i]: the expert of row tile i,
-// row_tiles[0]: how many row tiles there are.  One block; the order of an expert's rows among themselves is whatever the
+// row_tiles[0]: how many row tiles there are.  row_weight (or null): a pair's weight, by its row.  One block; the order of an expert's rows among themselves is whatever the
 // counters give (a row's result does not depend on its place).
 __global__ void __launch_bounds__(1024)
 moe_plan_kernel(Choice c, int n_tokens, int top, int E, int* __restrict__ pos, int* __restrict__ tile_group,
-                int* __restrict__ row_tiles) {
+                int* __restrict__ row_tiles, float* __restrict__ row_weight) {
   __shared__ int count[MOE_MAX_EXPERTS], first[MOE_MAX_EXPERTS];
   pdl_wait();
   pdl_trigger();
@@ -708,7 +721,11 @@ moe_plan_kernel(Choice c, int n_tokens, int top, int E, int* __restrict__ pos, i
     }
 #pragma unroll
     for (int j = 0; j < 8; ++j)
-      if (e[j] >= 0) pos[p0 + j * blockDim.x] = atomicAdd(&first[e[j]], 1);
+      if (e[j] >= 0) {
+        const int p = p0 + j * blockDim.x, row = atomicAdd(&first[e[j]], 1);
+        pos[p] = row;
+        if (row_weight != nullptr) row_weight[row] = chosen_weight(c, p / top, p % top, top);
+      }
   }
 }
 
@@ -725,14 +742,15 @@ moe_gather_kernel(const bf16* __restrict__ h, const int* __restrict__ pos, bf16*
   }
 }
 
-// out[t] = sum_k weight_k y[pos[t, k]] + sigmoid(z_t) ys[t]   (ys null: no shared expert)
+// out[t] = sum_k weight_k y[pos[t, k]] + sigmoid(z_t) ys[t]   (ys null: no shared expert; z null: its factor is 1;
+// `weighed`: the rows of y carry their weights already)
 __global__ void __launch_bounds__(256)
 moe_combine_kernel(const bf16* __restrict__ y, const int* __restrict__ pos, Choice c, const bf16* __restrict__ ys,
-                   const float* __restrict__ z, float* __restrict__ out, int top, int width) {
+                   const float* __restrict__ z, float* __restrict__ out, int top, int width, int weighed) {
   pdl_wait();
   pdl_trigger();
   const int t = blockIdx.x;
-  const float g = ys != nullptr ? 1.0f / (1.0f + expf(-z[t])) : 0.f;
+  const float g = z != nullptr ? 1.0f / (1.0f + expf(-z[t])) : 1.0f;
   for (int i = threadIdx.x * 8; i < width; i += blockDim.x * 8) {
     float s[8];
 #pragma unroll
@@ -747,7 +765,7 @@ moe_combine_kernel(const bf16* __restrict__ y, const int* __restrict__ pos, Choi
       }
     };
 #pragma unroll 4
-    for (int k = 0; k < top; ++k) add(y + (size_t)pos[(size_t)t * top + k] * width + i, chosen_weight(c, t, k, top));
+    for (int k = 0; k < top; ++k) add(y + (size_t)pos[(size_t)t * top + k] * width + i, weighed ? 1.0f : chosen_weight(c, t, k, top));
     if (ys != nullptr) add(ys + (size_t)t * width + i, g);
     float4* o = reinterpret_cast<float4*>(out + (size_t)t * width + i);
     o[0] = make_float4(s[0], s[1], s[2], s[3]);
@@ -758,28 +776,29 @@ moe_combine_kernel(const bf16* __restrict__ y, const int* __restrict__ pos, Choi
 // pos int [n_tokens * top], tile_group int [n_tokens * top / 128 + E], row_tiles int [1]; rows bfloat16
 // [(n_tokens * top / 128 + E) * 128, width].
 AB_API int ab_moe_gather(const void* h, const int* idx, const float* wts, const int* table, const int* tokens, float weight,
-                         int* pos, int* tile_group, int* row_tiles, void* rows, int n_tokens, int top, int width, int E,
+                         int* pos, int* tile_group, int* row_tiles, float* row_weight, void* rows, int n_tokens, int top, int width, int E,
                          cudaStream_t stream) {
   if (n_tokens <= 0) return AB_OK;
   const Choice c{idx, wts, table, tokens, weight};
   if (top <= 0 || E <= 0 || E > MOE_MAX_EXPERTS || width <= 0 || width % 8 || !choice_ok(c) ||
       (long long)n_tokens * top > 0x3fffffffLL || ((((uintptr_t)h) | ((uintptr_t)rows)) & 15))
     return AB_BAD_ARG;
-  ab_launch(moe_plan_kernel, dim3(1), dim3(1024), 0, stream, c, n_tokens, top, E, pos, tile_group, row_tiles);
+  ab_launch(moe_plan_kernel, dim3(1), dim3(1024), 0, stream, c, n_tokens, top, E, pos, tile_group, row_tiles,
+            row_weight);
   ab_launch(moe_gather_kernel, dim3((unsigned)n_tokens), dim3(width >= 2048 ? 256 : 128), 0, stream, (const bf16*)h,
             (const int*)pos, (bf16*)rows, top, width);
   return ab_launch_status();
 }
 
 AB_API int ab_moe_combine(const void* y, const int* pos, const int* idx, const float* wts, const int* table, const int* tokens,
-                          float weight, const void* ys, const float* z, float* out, int n_tokens, int top, int width,
+                          float weight, const void* ys, const float* z, float* out, int n_tokens, int top, int width, int weighed,
                           cudaStream_t stream) {
   if (n_tokens <= 0) return AB_OK;
   const Choice c{idx, wts, table, tokens, weight};
-  if (top <= 0 || width <= 0 || width % 8 || !choice_ok(c) || (ys && !z) ||
+  if (top <= 0 || width <= 0 || width % 8 || !choice_ok(c) ||
       ((((uintptr_t)y) | ((uintptr_t)ys) | ((uintptr_t)out)) & 15))
     return AB_BAD_ARG;
   ab_launch(moe_combine_kernel, dim3((unsigned)n_tokens), dim3(width >= 2048 ? 256 : 128), 0, stream, (const bf16*)y, pos, c,
-            (const bf16*)ys, z, out, top, width);
+            (const bf16*)ys, z, out, top, width, weighed);
   return ab_launch_status();
 }

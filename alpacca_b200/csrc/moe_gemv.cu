@@ -1,4 +1,4 @@
-// Gated experts with a shared expert for bfloat16 steps of up to 32 tokens: two skinny products whose weights are read
+// Experts (gated or not) with a shared expert for bfloat16 steps of up to 32 tokens: two skinny products whose weights are read
 // once from memory, for all tokens that chose an expert together.  (The kernels of moe.cu read an expert's rows once per
 // (token, expert) pair: with several tokens per expert that is several times the weights' bytes through the L2.)
 //
@@ -7,7 +7,8 @@
 //         ended), leaves if there are none, and multiplies its rows with those tokens' rows on the tensor cores
 //         (mma.sync m16n8k16, the weights as the 16-row operand, the listed tokens as the columns; see gemv_bf16.cu for
 //         the loads and the permutation of k).  act[t, slot, unit] = weight * act(gate) * up, the weight being the
-//         choice's or, for the shared expert, sigmoid(z_t).
+//         choice's or, for the shared expert, sigmoid(z_t) (1 without z).  Without gates the 16 rows are 16 units,
+//         weight * act(up); with `weight_in` a chosen expert's weight multiplies its input instead.
 //   down  a CTA owns 16 columns of the output and walks the units of the experts that were chosen by any token, then the
 //         shared expert's; a token's column is zero where it did not choose the expert.  The walk is cut into slices, the
 //         CTAs of a cluster, whose sums the first of them adds in slice order.
@@ -43,20 +44,22 @@ __device__ __forceinline__ uint4 mg_act(const bf16* p) {
   return v;
 }
 
-template <int NT>
+template <int NT, bool GATED>
 __global__ void __launch_bounds__(256)
 moe_gemv_up_kernel(const bf16* __restrict__ X, const bf16* __restrict__ W, const bf16* __restrict__ Ws, Choice c, const float* __restrict__ z,
-                   bf16* __restrict__ act, int M, int K, int top, int ff, int fs, int E, int activation) {
+                   bf16* __restrict__ act, int M, int K, int top, int ff, int fs, int E, int activation,
+                   int weight_in) {
+  constexpr int UNITS = GATED ? 8 : 16;        // of a slab of 16 rows
   constexpr int WARPS = 8;
   __shared__ float red[WARPS][NT][32][4];
   __shared__ int list[NT * 8];                  // token * top + slot (the shared expert: token * top + top, one slot more)
   __shared__ int n_list;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int g = lane >> 2, t = lane & 3;
-  const int slab = blockIdx.x, per_expert = ff >> 3;
+  const int slab = blockIdx.x, per_expert = ff / UNITS;
   const bool shared = slab >= E * per_expert;
   const int e = shared ? E : slab / per_expert;
-  const int unit0 = (shared ? slab - E * per_expert : slab - e * per_expert) * 8;      // within the expert
+  const int unit0 = (shared ? slab - E * per_expert : slab - e * per_expert) * UNITS;      // within the expert
   bool waited = false;
   if (c.idx != nullptr) { pdl_wait(); pdl_trigger(); waited = true; }      // a router's choice is the kernel's before this one
   if (warp == 0) {
@@ -139,11 +142,18 @@ moe_gemv_up_kernel(const bf16* __restrict__ X, const bf16* __restrict__ W, const
   const int row_len = top * ff + fs;
 #pragma unroll
   for (int j = 0; j < 2; ++j) {
-    const int at = i * 8 + 2 * t + j;          // columns 2t, 2t + 1: listed tokens; s[j] the gate of unit g, s[2 + j] its up
+    const int at = i * 8 + 2 * t + j;          // columns 2t, 2t + 1: listed tokens; s[j], s[2 + j]: rows g and g + 8
     if (at >= n) continue;
     const int tok = list[at] / (top + 1), slot = list[at] - tok * (top + 1);
-    const float wgt = shared ? 1.0f / (1.0f + expf(-z[tok])) : chosen_weight(c, tok, slot, top);
-    act[(size_t)tok * row_len + (size_t)slot * ff + unit0 + g] = __float2bfloat16_rn(wgt * activate(s[j], activation) * s[2 + j]);
+    const float wgt = !shared ? chosen_weight(c, tok, slot, top) : z != nullptr ? 1.0f / (1.0f + expf(-z[tok])) : 1.0f;
+    const int in = shared ? 0 : weight_in;
+    bf16* dst = act + (size_t)tok * row_len + (size_t)slot * ff + unit0 + g;
+    if (GATED) {
+      *dst = __float2bfloat16_rn(expert_inner<true>(s[j], s[2 + j], wgt, in, activation));
+    } else {
+      dst[0] = __float2bfloat16_rn(expert_inner<false>(0.f, s[j], wgt, in, activation));
+      dst[8] = __float2bfloat16_rn(expert_inner<false>(0.f, s[2 + j], wgt, in, activation));
+    }
   }
 }
 
@@ -288,20 +298,23 @@ moe_gemv_down_kernel(const bf16* __restrict__ act, const bf16* __restrict__ W, c
 AB_API int ab_moe_gemv_max_tokens() { return MG_MAX_TOKENS; }
 AB_API int ab_moe_gemv_max_experts() { return MG_MAX_EXPERTS; }
 
+// Without `gated`, gate_up holds the up-projections alone, [E * ff, width] (ff and fs multiples of 16).
 // act: scratch bfloat16 [M, top * ff + fs]; out: float32 [M, width].  `slices` (1, 2, 4 or 8): CTAs per 16 output columns.
 AB_API int ab_moe_gemv_max_top() { return MG_MAX_TOP; }
 AB_API int ab_moe_gemv(const void* h, const void* gate_up, const void* down, const void* gate_up_s, const void* down_s, const int* idx, const float* wts, const int* table,
                        const int* tokens, float weight, const float* z, void* act, float* out, int M, int top, int width, int ff,
-                       int fs, int E, int activation, int slices, cudaStream_t stream) {
+                       int fs, int E, int activation, int gated, int weight_in, int slices, cudaStream_t stream) {
   if (M <= 0) return AB_OK;
   const Choice c{idx, wts, table, tokens, weight};
   if (M > MG_MAX_TOKENS || E <= 0 || E > MG_MAX_EXPERTS || top <= 0 || top > MG_MAX_TOP || top > E || width <= 0 || width % 8 || ff <= 0 ||
-      ff % 8 || fs < 0 || fs % 8 || (activation != 0 && activation != 1) || !choice_ok(c) || (fs > 0 && (!z || !gate_up_s || !down_s)))
+      ff % 8 || fs < 0 || fs % 8 || activation < 0 || activation >= MOE_ACT_KINDS || !choice_ok(c) || (fs > 0 && (!gate_up_s || !down_s)) ||
+      (!gated && (ff % 16 || fs % 16)))
     return AB_BAD_ARG;
   if (slices != 1 && slices != 2 && slices != 4 && slices != 8) return AB_BAD_ARG;
   if ((((uintptr_t)h) | ((uintptr_t)gate_up) | ((uintptr_t)down) | ((uintptr_t)gate_up_s) | ((uintptr_t)down_s) |
        ((uintptr_t)act)) & 15) return AB_BAD_ARG;
-  const unsigned up_blocks = (unsigned)(E * (ff / 8) + fs / 8);
+  const int units = gated ? 8 : 16;
+  const unsigned up_blocks = (unsigned)(E * (ff / units) + fs / units);
   cudaLaunchConfig_t cfg = {};
   cfg.gridDim = dim3((unsigned)((width + 15) / 16), (unsigned)slices);
   cfg.stream = stream;
@@ -324,8 +337,9 @@ AB_API int ab_moe_gemv(const void* h, const void* gate_up, const void* down, con
   cudaError_t e = cudaSuccess;
 #define AB_GO(NT, WARPS)                                                                                               \
   {                                                                                                                    \
-    ab_launch(moe_gemv_up_kernel<NT>, dim3(up_blocks), dim3(256), 0, stream, (const bf16*)h, (const bf16*)gate_up, \
-              (const bf16*)gate_up_s, c, z, (bf16*)act, M, width, top, ff, fs, E, activation);                                                       \
+    ab_launch(gated ? moe_gemv_up_kernel<NT, true> : moe_gemv_up_kernel<NT, false>, dim3(up_blocks), dim3(256), 0, stream, \
+              (const bf16*)h, (const bf16*)gate_up, (const bf16*)gate_up_s, c, z, (bf16*)act, M, width, top, ff, fs, E,   \
+              activation, weight_in);                                                                                  \
     cfg.blockDim = dim3(WARPS * 32);                                                                                   \
     e = cudaLaunchKernelEx(&cfg, moe_gemv_down_kernel<NT, WARPS>, (const bf16*)act, (const bf16*)down, (const bf16*)down_s, c, out, \
                            M, width, top, ff, fs, E, slices);                                                                         \

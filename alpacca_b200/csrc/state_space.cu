@@ -1,0 +1,744 @@
+// A state-space mixer with one decay and one step size per head and token (Dao and Gu, "Transformers are SSMs:
+// Generalized Models and Efficient Algorithms Through Structured State Space Duality").
+//
+// A token's projected row (float32) holds [z | x | B | C | dt]: z and x H heads of V, B and C G groups of N, dt H numbers.
+//   x, B, C  pass a causal convolution per channel over `taps` tokens (with a bias) and SiLU; a sequence's last taps - 1
+//            inputs are state
+//   dt       softplus(dt + bias_h);   a = exp(-exp(A_log_h) dt)                 head h reads group h // (H / G)
+//   S        <- a S + dt B x^T   [N, V] float32 per (sequence, head);   y = S^T C + skip_h x
+//   out      = (y silu(z)) in `parts` equal parts, each divided by its own root mean square, times w
+//
+// Three forms of the recurrence, the same sums up to rounding:
+//   ssm_step    one token per sequence: convolution, step size, decay, update and read-out in one kernel.  A CTA takes a
+//               (sequence, head, tile of value columns); the tile of S is asked for, 16 bytes per thread and row, before the
+//               wait for the projection, and goes back once.
+//   ssm_chunks  prompts in bfloat16: 64 tokens at a time on the tensor cores (mma.sync), S in the accumulators of a CTA that
+//               walks one sequence's chunks for one (head, tile of columns).  With L_t the running sum of the chunk's log
+//               decays,  y_t = exp(L_t) S^T C_t + sum_(s <= t) exp(L_t - L_s) dt_s (C_t . B_s) x_s  and
+//               S <- exp(L_end) S + sum_s exp(L_end - L_s) dt_s B_s x_s^T.  B, C and x are the convolution's outputs rounded
+//               to bfloat16; everything else that meets them (S, the weights of the scores, the weighted x) is split into
+//               two bfloat16 numbers, high and low, and multiplied twice, so that it enters with 16 bits.
+//   otherwise   ssm_prepare leaves float32 rows and the walk of csrc/gated_recurrence.cu (mode 2) does the rest.
+// Around them: ssm_prepare (convolution, step sizes, decays for many tokens), ssm_gate_norm (the gate and the norm; after
+// ssm_step it moves the convolution's inputs on, since every CTA of that kernel has read them by then).
+#include "attention_common.cuh"
+#include "launch.cuh"
+
+#define SSM_MAX_TAPS 17
+#define SSM_RUN 8            // tokens that a thread of ssm_prepare walks
+
+__device__ __forceinline__ float ssm_softplus(float x) { return x > 20.f ? x : log1pf(expf(x)); }
+__device__ __forceinline__ float ssm_silu(float x) { return x / (1.0f + expf(-x)); }
+
+struct SsmSizes {
+  int H, G, N, V, taps;
+  __host__ __device__ int inner() const { return H * V; }
+  __host__ __device__ int channels() const { return H * V + 2 * G * N; }      // x | B | C, convolved
+  __host__ __device__ int off_x() const { return H * V; }
+  __host__ __device__ int off_dt() const { return 2 * H * V + 2 * G * N; }
+};
+
+template <int W> struct Lanes { float v[W]; };
+template <int W> __device__ __forceinline__ Lanes<W> load_lanes(const float* p) {
+  Lanes<W> r;
+  if (W == 4) {
+    const float4 q = *reinterpret_cast<const float4*>(p);
+    r.v[0] = q.x; r.v[1 % W] = q.y; r.v[2 % W] = q.z; r.v[3 % W] = q.w;
+  } else r.v[0] = *p;
+  return r;
+}
+template <int W> __device__ __forceinline__ void store_lanes(float* p, const Lanes<W>& r) {
+  if (W == 4) *reinterpret_cast<float4*>(p) = make_float4(r.v[0], r.v[1 % W], r.v[2 % W], r.v[3 % W]);
+  else *p = r.v[0];
+}
+template <int W> __device__ __forceinline__ void store_lanes(bf16* p, const Lanes<W>& r) {
+  if (W == 4) *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16(r.v[0], r.v[1 % W]), pack_bf16(r.v[2 % W], r.v[3 % W]));
+  else *p = __float2bfloat16_rn(r.v[0]);
+}
+
+// ---------------------------------------------------------------------------
+// many tokens: convolution, step sizes, decays
+// ---------------------------------------------------------------------------
+// A thread takes W neighbouring channels of SSM_RUN tokens (blocks with blockIdx.y < chan_blocks) or the heads' numbers.
+// K > 0: the number of taps, the last K - 1 inputs in registers; K = 0: any number, inputs fetched per tap.
+// conv_w is [taps, channels]; conv_state [slots, taps - 1, channels], oldest first.
+template <typename TO, int W, int K>
+__global__ void __launch_bounds__(128)
+ssm_prepare_kernel(const float* __restrict__ proj, int ld, const float* __restrict__ conv_w, const float* __restrict__ conv_b,
+                   const float* __restrict__ conv_state, const float* __restrict__ A_log, const float* __restrict__ dt_bias,
+                   TO* __restrict__ xbc, float* __restrict__ decay, float* __restrict__ dt, int log_decay,
+                   const int* __restrict__ tok_seq, const int* __restrict__ cu_q, const int* __restrict__ slots,
+                   int n_tokens, SsmSizes z, int chan_blocks) {
+  pdl_wait();
+  pdl_trigger();
+  const int t0 = blockIdx.x * SSM_RUN, t1 = min(n_tokens, t0 + SSM_RUN);
+  const int Cc = z.channels(), taps = K ? K : z.taps;
+  if ((int)blockIdx.y >= chan_blocks) {
+    const int h = (blockIdx.y - chan_blocks) * blockDim.x + threadIdx.x;
+    if (h >= z.H) return;
+    const float ea = expf(A_log[h]), bias = dt_bias[h];
+    for (int t = t0; t < t1; ++t) {
+      if (tok_seq[t] < 0) continue;
+      const float d = ssm_softplus(proj[(size_t)t * ld + z.off_dt() + h] + bias);
+      dt[(size_t)t * z.H + h] = d;
+      decay[(size_t)t * z.H + h] = log_decay ? -ea * d : expf(-ea * d);
+    }
+    return;
+  }
+  const int c = (blockIdx.y * blockDim.x + threadIdx.x) * W;
+  if (c >= Cc) return;
+  const float* x = proj + z.off_x() + c;
+  const Lanes<W> bias = load_lanes<W>(conv_b + c);
+  Lanes<W> w[K ? K : 1], past[K > 1 ? K - 1 : 1];
+#pragma unroll
+  for (int j = 0; j < K; ++j) w[j] = load_lanes<W>(conv_w + (size_t)j * Cc + c);
+  for (int t = t0; t < t1; ++t) {
+    const int b = tok_seq[t];
+    if (b < 0) continue;
+    const int i = t - cu_q[b];
+    const float* held = conv_state + (size_t)slots[b] * (taps - 1) * Cc + c;
+    if (K) {
+      if (t == t0 || i == 0) {
+#pragma unroll
+        for (int j = 0; j < K - 1; ++j) {
+          const int src = i - (K - 1) + j;
+          past[j] = src >= 0 ? load_lanes<W>(x + (size_t)(t - (K - 1) + j) * ld) : load_lanes<W>(held + (size_t)(K - 1 + src) * Cc);
+        }
+      }
+    }
+    const Lanes<W> now = load_lanes<W>(x + (size_t)t * ld);
+    Lanes<W> acc = bias;
+    if (K) {
+#pragma unroll
+      for (int j = 0; j < K - 1; ++j)
+#pragma unroll
+        for (int e = 0; e < W; ++e) acc.v[e] = fmaf(w[j].v[e], past[j].v[e], acc.v[e]);
+#pragma unroll
+      for (int e = 0; e < W; ++e) acc.v[e] = fmaf(w[K ? K - 1 : 0].v[e], now.v[e], acc.v[e]);
+#pragma unroll
+      for (int j = 0; j + 1 < K - 1; ++j) past[j] = past[j + 1];
+      if (K > 1) past[K > 1 ? K - 2 : 0] = now;
+    } else {
+      for (int j = 0; j < taps; ++j) {
+        const int src = i - (taps - 1) + j;
+        const Lanes<W> in = src >= 0 ? load_lanes<W>(x + (size_t)(t - (taps - 1) + j) * ld)
+                                     : load_lanes<W>(held + (size_t)(taps - 1 + src) * Cc);
+        const Lanes<W> wj = load_lanes<W>(conv_w + (size_t)j * Cc + c);
+#pragma unroll
+        for (int e = 0; e < W; ++e) acc.v[e] = fmaf(wj.v[e], in.v[e], acc.v[e]);
+      }
+    }
+#pragma unroll
+    for (int e = 0; e < W; ++e) acc.v[e] = ssm_silu(acc.v[e]);
+    store_lanes<W>(xbc + (size_t)t * Cc + c, acc);
+  }
+}
+
+// conv_state[slot] <- the sequence's last taps - 1 inputs: a thread per (sequence, channel) reads what it keeps first
+__global__ void ssm_conv_move_kernel(const float* __restrict__ proj, int ld, float* __restrict__ conv_state,
+                                     const int* __restrict__ cu_q, const int* __restrict__ slots, int n_seqs, SsmSizes z) {
+  pdl_wait();
+  pdl_trigger();
+  const int Cc = z.channels(), keep = z.taps - 1;
+  const long long id = (long long)blockIdx.x * blockDim.x + threadIdx.x;
+  if (id >= (long long)n_seqs * Cc) return;
+  const int b = (int)(id / Cc), c = (int)(id - (long long)b * Cc);
+  const int slot = slots[b];
+  if (slot < 0) return;
+  const int t0 = cu_q[b], n = cu_q[b + 1] - t0;
+  const float* x = proj + z.off_x() + c;
+  float* held = conv_state + (size_t)slot * keep * Cc + c;
+  float now[SSM_MAX_TAPS - 1];
+#pragma unroll
+  for (int s = 0; s < SSM_MAX_TAPS - 1; ++s)
+    if (s < keep) {
+      const int i = n - keep + s;
+      now[s] = i >= 0 ? x[(size_t)(t0 + i) * ld] : held[(size_t)(s + n) * Cc];
+    }
+#pragma unroll
+  for (int s = 0; s < SSM_MAX_TAPS - 1; ++s)
+    if (s < keep) held[(size_t)s * Cc] = now[s];
+}
+
+static bool ssm_sizes_ok(const SsmSizes& z) {
+  return z.H > 0 && z.G > 0 && z.H % z.G == 0 && z.N > 0 && z.N <= 256 && z.V > 0 && z.taps >= 1 && z.taps <= SSM_MAX_TAPS;
+}
+
+// xbc [T, channels] float32 or bfloat16; decay, dt [T, H] float32 (decay: exp(..), or its logarithm with `log_decay`)
+AB_API int ab_ssm_prepare(const float* proj, int ld, const float* conv_w, const float* conv_b, float* conv_state,
+                          const float* A_log, const float* dt_bias, void* xbc, int xbc_dtype, float* decay, float* dt,
+                          int log_decay, const int* tok_seq, const int* cu_q, const int* slots, int n_tokens, int n_seqs,
+                          int H, int G, int N, int V, int taps, int write_state, cudaStream_t stream) {
+  if (n_tokens <= 0) return AB_OK;
+  const SsmSizes z{H, G, N, V, taps};
+  if (!ssm_sizes_ok(z) || !proj || !conv_w || !conv_b || !A_log || !dt_bias || !xbc || !decay || !dt || (taps > 1 && !conv_state))
+    return AB_BAD_ARG;
+  const int Cc = z.channels();
+  auto al = [](const void* p) { return ((uintptr_t)p & 15) == 0; };
+  const bool vec = Cc % 4 == 0 && ld % 4 == 0 && z.off_x() % 4 == 0 && al(proj) && al(conv_w) && al(conv_b) && al(conv_state) && al(xbc);
+  const int per = 128 * (vec ? 4 : 1), chan_blocks = (Cc + per - 1) / per;
+  const dim3 grid((unsigned)((n_tokens + SSM_RUN - 1) / SSM_RUN), (unsigned)(chan_blocks + (H + 127) / 128));
+#define AB_GO(TO, W, K)                                                                                                \
+  ab_launch(ssm_prepare_kernel<TO, W, K>, grid, dim3(128), 0, stream, proj, ld, conv_w, conv_b, (const float*)conv_state, \
+            A_log, dt_bias, (TO*)xbc, decay, dt, log_decay, tok_seq, cu_q, slots, n_tokens, z, chan_blocks)
+#define AB_K(TO, W)                                                                                                    \
+  {                                                                                                                    \
+    if (taps == 2) AB_GO(TO, W, 2); else if (taps == 3) AB_GO(TO, W, 3); else if (taps == 4) AB_GO(TO, W, 4);          \
+    else AB_GO(TO, W, 0);                                                                                              \
+  }
+  if (xbc_dtype == AB_F32) { if (vec) AB_K(float, 4) else AB_K(float, 1) }
+  else if (xbc_dtype == AB_BF16) { if (vec) AB_K(bf16, 4) else AB_K(bf16, 1) }
+  else return AB_BAD_ARG;
+#undef AB_K
+#undef AB_GO
+  int rc = ab_launch_status();
+  if (rc || !write_state || taps == 1) return rc;
+  const long long total = (long long)n_seqs * Cc;
+  ab_launch(ssm_conv_move_kernel, dim3((unsigned)((total + 127) / 128)), dim3(128), 0, stream, proj, ld, conv_state, cu_q,
+            slots, n_seqs, z);
+  return ab_launch_status();
+}
+
+// ---------------------------------------------------------------------------
+// one token per sequence
+// ---------------------------------------------------------------------------
+// 256 threads: CV / 4 of them side by side on a row of the tile, R rows each.  What a thread asks for before the wait (the
+// tile of S, the convolution's kept inputs and weights) was written a step ago or never.
+template <int CV, int R>
+__global__ void __launch_bounds__(256)
+ssm_step_kernel(const float* __restrict__ proj, int ld, const float* __restrict__ conv_w, const float* __restrict__ conv_b,
+                const float* __restrict__ conv_state, const float* __restrict__ A_log, const float* __restrict__ dt_bias,
+                const float* __restrict__ skip, float* __restrict__ state, float* __restrict__ y,
+                const int* __restrict__ tok_seq, const int* __restrict__ slots, SsmSizes z, int write_state) {
+  constexpr int C4 = CV / 4, RS = 256 / C4, MAXC = (512 + CV + 255) / 256;
+  __shared__ __align__(16) float row[512 + CV];          // B | C | x of this CTA, after convolution and SiLU
+  __shared__ __align__(16) float red[8][CV];
+  const int t = blockIdx.x, h = blockIdx.y, col0 = blockIdx.z * CV;
+  const int N = z.N, V = z.V, Cc = z.channels(), taps = z.taps;
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  const int b = tok_seq[t];
+  float* yr = y + (size_t)t * z.inner() + (size_t)h * V + col0;
+  const int cw = min(CV, V - col0);
+  if (b < 0) {
+    pdl_wait();
+    pdl_trigger();
+    for (int j = tid; j < cw; j += 256) yr[j] = 0.f;
+    return;
+  }
+  const int slot = slots[b];
+  const int c4 = (tid % C4) * 4, r0 = tid / C4;
+  const bool col_ok = c4 < cw;
+  float* st = state + (((size_t)slot * z.H + h) * N) * V + col0 + c4;
+  float4 S[R];
+#pragma unroll
+  for (int i = 0; i < R; ++i) {
+    const int n = r0 + i * RS;
+    S[i] = (n < N && col_ok) ? *reinterpret_cast<const float4*>(st + (size_t)n * V) : make_float4(0.f, 0.f, 0.f, 0.f);
+  }
+  const int g = h / (z.H / z.G), n_ch = 2 * N + cw;
+  const float* held = conv_state + (size_t)slot * (taps - 1) * Cc;
+  int ch[MAXC];
+  float acc[MAXC], last[MAXC];
+#pragma unroll
+  for (int k = 0; k < MAXC; ++k) {
+    const int i = tid + k * 256;
+    ch[k] = -1;
+    if (i < n_ch) {
+      const int c = i < N ? z.inner() + g * N + i : i < 2 * N ? z.inner() + z.G * N + g * N + i - N : h * V + col0 + i - 2 * N;
+      ch[k] = c;
+      acc[k] = conv_b[c];
+      for (int j = 0; j < taps - 1; ++j) acc[k] = fmaf(conv_w[(size_t)j * Cc + c], held[(size_t)j * Cc + c], acc[k]);
+      last[k] = conv_w[(size_t)(taps - 1) * Cc + c];
+    }
+  }
+  const float ea = expf(A_log[h]), bias = dt_bias[h], sk = skip[h];
+  pdl_wait();
+  pdl_trigger();
+  const float* p = proj + (size_t)t * ld;
+  const float raw_dt = p[z.off_dt() + h];
+#pragma unroll
+  for (int k = 0; k < MAXC; ++k)
+    if (ch[k] >= 0) row[tid + k * 256] = ssm_silu(fmaf(last[k], p[z.off_x() + ch[k]], acc[k]));
+  const float dt = ssm_softplus(raw_dt + bias), a = expf(-ea * dt);
+  __syncthreads();
+  const float* xs = row + 2 * N;
+  float4 x4 = make_float4(0.f, 0.f, 0.f, 0.f);
+  if (col_ok) x4 = make_float4(xs[c4] * dt, xs[c4 + 1] * dt, xs[c4 + 2] * dt, xs[c4 + 3] * dt);
+  float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+  for (int i = 0; i < R; ++i) {
+    const int n = r0 + i * RS;
+    if (n < N) {
+      const float kb = row[n], qc = row[N + n];
+      S[i].x = fmaf(a, S[i].x, kb * x4.x);
+      S[i].y = fmaf(a, S[i].y, kb * x4.y);
+      S[i].z = fmaf(a, S[i].z, kb * x4.z);
+      S[i].w = fmaf(a, S[i].w, kb * x4.w);
+      o.x = fmaf(S[i].x, qc, o.x);
+      o.y = fmaf(S[i].y, qc, o.y);
+      o.z = fmaf(S[i].z, qc, o.z);
+      o.w = fmaf(S[i].w, qc, o.w);
+      if (write_state && col_ok) *reinterpret_cast<float4*>(st + (size_t)n * V) = S[i];
+    }
+  }
+#pragma unroll
+  for (int d = C4; d < 32; d <<= 1) {
+    o.x += __shfl_xor_sync(0xffffffffu, o.x, d);
+    o.y += __shfl_xor_sync(0xffffffffu, o.y, d);
+    o.z += __shfl_xor_sync(0xffffffffu, o.z, d);
+    o.w += __shfl_xor_sync(0xffffffffu, o.w, d);
+  }
+  if (lane < C4) *reinterpret_cast<float4*>(&red[warp][c4]) = o;
+  __syncthreads();
+  if (tid < cw) {
+    float s = 0.f;
+#pragma unroll
+    for (int w = 0; w < 8; ++w) s += red[w][tid];
+    yr[tid] = fmaf(sk, xs[tid], s);
+  }
+}
+
+// 1 if ssm_step takes the sizes: value sizes in steps of 4
+AB_API int ab_ssm_step_supports(int N, int V) { return N > 0 && N <= 256 && V > 0 && V % 4 == 0 ? 1 : 0; }
+
+// `cols`: value columns per CTA (16, 32 or 64).  The convolution's kept inputs are left as they are (ab_ssm_gate_norm
+// moves them on).
+AB_API int ab_ssm_step(const float* proj, int ld, const float* conv_w, const float* conv_b, const float* conv_state,
+                       const float* A_log, const float* dt_bias, const float* skip, float* state, float* y,
+                       const int* tok_seq, const int* slots, int n_tokens, int H, int G, int N, int V, int taps, int cols,
+                       int write_state, cudaStream_t stream) {
+  if (n_tokens <= 0) return AB_OK;
+  const SsmSizes z{H, G, N, V, taps};
+  if (!ssm_sizes_ok(z) || !ab_ssm_step_supports(N, V) || H > 65535 || (((uintptr_t)state) & 15)) return AB_BAD_ARG;
+  const dim3 grid((unsigned)n_tokens, (unsigned)H, (unsigned)((V + cols - 1) / cols));
+#define AB_GO(CV, R)                                                                                                   \
+  ab_launch(ssm_step_kernel<CV, R>, grid, dim3(256), 0, stream, proj, ld, conv_w, conv_b, conv_state, A_log, dt_bias, skip, \
+            state, y, tok_seq, slots, z, write_state)
+  if (cols == 64) {
+    if (N <= 16) AB_GO(64, 1); else if (N <= 32) AB_GO(64, 2); else if (N <= 64) AB_GO(64, 4);
+    else if (N <= 128) AB_GO(64, 8); else AB_GO(64, 16);
+  } else if (cols == 32) {
+    if (N <= 32) AB_GO(32, 1); else if (N <= 64) AB_GO(32, 2); else if (N <= 128) AB_GO(32, 4); else AB_GO(32, 8);
+  } else if (cols == 16) {
+    if (N <= 64) AB_GO(16, 1); else if (N <= 128) AB_GO(16, 2); else AB_GO(16, 4);
+  } else
+    return AB_BAD_ARG;
+#undef AB_GO
+  return ab_launch_status();
+}
+
+// ---------------------------------------------------------------------------
+// gate and norm
+// ---------------------------------------------------------------------------
+// A block per (token, part): out = cast(u / rms(u) * w), u = y silu(z), over the part's n numbers.  NV > 0: n and the row
+// strides are multiples of 4 and the part fits NV quads per thread; NV = 0: any size, u formed twice.
+// `conv_state` (or null): the token's convolution inputs become the newest of what its sequence keeps (one token per
+// sequence; the blocks of a token share the channels).
+template <typename TO, int NV>
+__global__ void __launch_bounds__(512)
+ssm_gate_norm_kernel(const float* __restrict__ y, const float* __restrict__ proj, int ld, const float* __restrict__ w,
+                     TO* __restrict__ out, float* __restrict__ conv_state, const int* __restrict__ tok_seq,
+                     const int* __restrict__ slots, int n, float eps, SsmSizes z) {
+  __shared__ float scratch[32];
+  const int t = blockIdx.x, base = blockIdx.y * n;
+  pdl_wait();
+  pdl_trigger();
+  const int b = tok_seq[t];
+  TO* o = out + (size_t)t * z.inner() + base;
+  if (b < 0) {
+    for (int j = threadIdx.x; j < n; j += blockDim.x) o[j] = from_f32<TO>(0.f);
+    return;
+  }
+  const float* yr = y + (size_t)t * z.inner() + base;
+  const float* zr = proj + (size_t)t * ld + base;
+  const float* wr = w + base;
+  float ss = 0.f;
+  if (NV > 0) {
+    Lanes<4> u[NV > 0 ? NV : 1], wv[NV > 0 ? NV : 1];
+#pragma unroll
+    for (int k = 0; k < NV; ++k) {
+      const int j = (threadIdx.x + k * blockDim.x) * 4;
+      if (j < n) {
+        u[k] = load_lanes<4>(yr + j);
+        const Lanes<4> g = load_lanes<4>(zr + j);
+        wv[k] = load_lanes<4>(wr + j);
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          u[k].v[e] *= ssm_silu(g.v[e]);
+          ss += u[k].v[e] * u[k].v[e];
+        }
+      }
+    }
+    ss = block_sum(ss, scratch);
+    const float inv = 1.0f / sqrtf(ss / (float)n + eps);
+#pragma unroll
+    for (int k = 0; k < NV; ++k) {
+      const int j = (threadIdx.x + k * blockDim.x) * 4;
+      if (j < n) {
+#pragma unroll
+        for (int e = 0; e < 4; ++e) u[k].v[e] *= inv * wv[k].v[e];
+        store_lanes<4>(o + j, u[k]);
+      }
+    }
+  } else {
+    for (int j = threadIdx.x; j < n; j += blockDim.x) {
+      const float u = yr[j] * ssm_silu(zr[j]);
+      ss += u * u;
+    }
+    ss = block_sum(ss, scratch);
+    const float inv = 1.0f / sqrtf(ss / (float)n + eps);
+    for (int j = threadIdx.x; j < n; j += blockDim.x) o[j] = from_f32<TO>(yr[j] * ssm_silu(zr[j]) * (inv * wr[j]));
+  }
+  if (conv_state != nullptr) {
+    const int Cc = z.channels(), keep = z.taps - 1;
+    float* held = conv_state + (size_t)slots[b] * keep * Cc;
+    const float* x = proj + (size_t)t * ld + z.off_x();
+    for (int c = blockIdx.y * blockDim.x + threadIdx.x; c < Cc; c += gridDim.y * blockDim.x) {
+      for (int s = 0; s + 1 < keep; ++s) held[(size_t)s * Cc + c] = held[(size_t)(s + 1) * Cc + c];
+      held[(size_t)(keep - 1) * Cc + c] = x[c];
+    }
+  }
+}
+
+AB_API int ab_ssm_gate_norm(const float* y, const float* proj, int ld, const float* w, void* out, int out_dtype,
+                            float* conv_state, const int* tok_seq, const int* slots, int n_tokens, int parts, float eps,
+                            int H, int G, int N, int V, int taps, cudaStream_t stream) {
+  if (n_tokens <= 0) return AB_OK;
+  const SsmSizes z{H, G, N, V, taps};
+  if (!ssm_sizes_ok(z) || parts <= 0 || z.inner() % parts || parts > 65535 || (taps == 1 && conv_state)) return AB_BAD_ARG;
+  const int n = z.inner() / parts;
+  auto al = [](const void* p) { return ((uintptr_t)p & 15) == 0; };
+  const bool vec = n % 4 == 0 && ld % 4 == 0 && al(y) && al(proj) && al(w) && al(out) && n <= 512 * 4 * 4;
+  const int threads = n >= 4096 ? 512 : n >= 1024 ? 256 : n >= 256 ? 128 : 64;
+  const int nv = vec ? (n / 4 + threads - 1) / threads : 0;
+  const dim3 grid((unsigned)n_tokens, (unsigned)parts);
+#define AB_GO(TO, NV)                                                                                                  \
+  ab_launch(ssm_gate_norm_kernel<TO, NV>, grid, dim3(threads), 0, stream, y, proj, ld, w, (TO*)out, conv_state, tok_seq, slots, \
+            n, eps, z)
+#define AB_NV(TO)                                                                                                      \
+  { if (nv == 0) AB_GO(TO, 0); else if (nv == 1) AB_GO(TO, 1); else if (nv == 2) AB_GO(TO, 2); else AB_GO(TO, 4); }
+  if (out_dtype == AB_F32) AB_NV(float)
+  else if (out_dtype == AB_BF16) AB_NV(bf16)
+  else return AB_BAD_ARG;
+#undef AB_NV
+#undef AB_GO
+  return ab_launch_status();
+}
+
+// ---------------------------------------------------------------------------
+// prompts: chunks of 64 tokens on the tensor cores
+// ---------------------------------------------------------------------------
+#define SC_T 64
+
+__device__ __forceinline__ void sc_async16(void* dst, const void* src) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;\n" ::"r"(smem_u32(dst)), "l"(src));
+}
+__device__ __forceinline__ void sc_async4(void* dst, const void* src) {
+  asm volatile("cp.async.ca.shared.global [%0], [%1], 4;\n" ::"r"(smem_u32(dst)), "l"(src));
+}
+// v = hi + lo up to 2^-17: two bfloat16 numbers each
+__device__ __forceinline__ void split2(float a, float b, uint32_t& hi, uint32_t& lo) {
+  hi = pack_bf16(a, b);
+  lo = pack_bf16(a - __uint_as_float(hi << 16), b - __uint_as_float(hi & 0xffff0000u));
+}
+
+template <int CV> struct ChunkSmem {
+  static constexpr int PV = CV + 8;                      // pitch of rows of value columns
+  // float offsets are kept in bytes; N is the state size
+  __host__ __device__ static size_t bc(int N) { return (size_t)SC_T * (N + 8) * 2; }      // one buffer of B or C
+  __host__ __device__ static size_t total(int N) {
+    return 4 * bc(N) + 2 * (size_t)SC_T * PV * 2 + 2 * (size_t)N * PV * 2 + 2 * (size_t)SC_T * PV * 2 +
+           (size_t)SC_T * (CV + 4) * 4 + 4 * SC_T * 4 + 4 * SC_T * 4 + 16;
+  }
+};
+
+// RT: row tiles of S (16 rows) per warp; eight warps cover N <= 128 * RT rows.
+template <int CV, int RT>
+__global__ void __launch_bounds__(256)
+ssm_chunks_kernel(const bf16* __restrict__ xbc, const float* __restrict__ la, const float* __restrict__ dt,
+                  const float* __restrict__ skip, float* __restrict__ state, float* __restrict__ y,
+                  const int* __restrict__ cu_q, const int* __restrict__ slots, SsmSizes z, int write_state) {
+  constexpr int PV = ChunkSmem<CV>::PV, NT = CV / 8;
+  extern __shared__ __align__(16) unsigned char sm[];
+  const int N = z.N, V = z.V, H = z.H, Cc = z.channels(), PN = N + 8;
+  bf16* Bs = reinterpret_cast<bf16*>(sm);                       // [2][64][PN]
+  bf16* Cs = Bs + 2 * SC_T * PN;                                // [2][64][PN]
+  bf16* xs = Cs + 2 * SC_T * PN;                                // [2][64][PV]
+  bf16* Sh = xs + 2 * SC_T * PV;                                // [N][PV] the state before the chunk, high parts
+  bf16* Sl = Sh + N * PV;
+  bf16* wh = Sl + N * PV;                                       // [64][PV] exp(L_end - L_s) dt_s x_s, high parts
+  bf16* wl = wh + SC_T * PV;
+  float* Yx = reinterpret_cast<float*>(wl + SC_T * PV);         // [64][CV + 4]
+  float* las = Yx + SC_T * (CV + 4);                            // [2][64]
+  float* dts = las + 2 * SC_T;                                  // [2][64]
+  float* cs = dts + 2 * SC_T;                                   // [64] L_s
+  float* ecs = cs + SC_T;                                       // exp(L_s)
+  float* wsm = ecs + SC_T;                                      // exp(L_end - L_s) dt_s
+  float* endp = wsm + SC_T;                                     // exp(L_end)
+  const int b = blockIdx.x, h = blockIdx.y, col0 = blockIdx.z * CV;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int g = lane >> 2, t4 = lane & 3;
+  const int slot = slots[b], t0 = cu_q[b], t1 = cu_q[b + 1];
+  if (slot < 0 || t1 <= t0) { pdl_wait(); pdl_trigger(); return; }
+  const int n_rt = N >> 4, grp = h / (H / z.G);
+  float* st = state + ((size_t)slot * H + h) * N * V + col0;
+  float S[RT][NT][4];
+#pragma unroll
+  for (int r = 0; r < RT; ++r)
+#pragma unroll
+    for (int nt = 0; nt < NT; ++nt) {
+      const int n = (warp + 8 * r) * 16 + g, c = nt * 8 + 2 * t4;
+      const bool in = warp + 8 * r < n_rt && col0 + c < V;
+      const float2 lo = in ? *reinterpret_cast<const float2*>(st + (size_t)n * V + c) : make_float2(0.f, 0.f);
+      const float2 hi = in ? *reinterpret_cast<const float2*>(st + (size_t)(n + 8) * V + c) : make_float2(0.f, 0.f);
+      S[r][nt][0] = lo.x; S[r][nt][1] = lo.y; S[r][nt][2] = hi.x; S[r][nt][3] = hi.y;
+    }
+  pdl_wait();
+  pdl_trigger();
+  const float sk = skip[h];
+  const int pn = N >> 3;
+  const bf16* xg = xbc + (size_t)h * V + col0;
+  const bf16* Bg = xbc + z.inner() + (size_t)grp * N;
+  const bf16* Cg = Bg + (size_t)z.G * N;
+  auto load = [&](int buf, int c0) {
+    const int n = min(SC_T, t1 - c0);
+    for (int i = tid; i < SC_T * pn; i += 256) {
+      const int r = i / pn, c = (i - r * pn) * 8;
+      bf16 *db = Bs + ((size_t)buf * SC_T + r) * PN + c, *dc = Cs + ((size_t)buf * SC_T + r) * PN + c;
+      if (r < n) {
+        sc_async16(db, Bg + (size_t)(c0 + r) * Cc + c);
+        sc_async16(dc, Cg + (size_t)(c0 + r) * Cc + c);
+      } else {
+        *reinterpret_cast<uint4*>(db) = make_uint4(0, 0, 0, 0);
+        *reinterpret_cast<uint4*>(dc) = make_uint4(0, 0, 0, 0);
+      }
+    }
+    for (int i = tid; i < SC_T * (CV / 8); i += 256) {
+      const int r = i / (CV / 8), c = (i - r * (CV / 8)) * 8;
+      bf16* d = xs + ((size_t)buf * SC_T + r) * PV + c;
+      if (r < n && col0 + c < V) sc_async16(d, xg + (size_t)(c0 + r) * Cc + c);
+      else *reinterpret_cast<uint4*>(d) = make_uint4(0, 0, 0, 0);
+    }
+    if (tid < 2 * SC_T) {
+      const int r = tid & (SC_T - 1);
+      float* d = (tid < SC_T ? las : dts) + buf * SC_T + r;
+      if (r < n) sc_async4(d, (tid < SC_T ? la : dt) + (size_t)(c0 + r) * H + h);
+      else *d = 0.f;                       // no decay, no weight
+    }
+    asm volatile("cp.async.commit_group;\n" ::);
+  };
+  load(0, t0);
+  const int a_row = (lane & 7) + ((lane >> 3) & 1) * 8, a_col = (lane >> 4) * 8;       // first operand, rows of k
+  const int b_row = (lane & 7) + (lane >> 4) * 8, b_col = ((lane >> 3) & 1) * 8;       // second operand, rows of k
+  const int v_row = a_row, v_col = a_col;                                              // second operand, rows of n (transposed)
+  const int s_tok = (lane & 7) + (lane >> 4) * 8, s_n = ((lane >> 3) & 1) * 8;         // first operand, rows of m (transposed)
+  int buf = 0;
+  for (int c0 = t0; c0 < t1; c0 += SC_T, buf ^= 1) {
+    asm volatile("cp.async.wait_group 0;\n" ::);
+    __syncthreads();                       // A: the chunk has arrived; everything of the chunk before has been read
+    if (c0 + SC_T < t1) load(buf ^ 1, c0 + SC_T);
+    if (warp == 0) {                       // running sums of the log decays, two tokens per lane
+      const float v0 = las[buf * SC_T + 2 * lane], v1 = las[buf * SC_T + 2 * lane + 1];
+      float incl = v0 + v1;
+#pragma unroll
+      for (int o = 1; o < 32; o <<= 1) {
+        const float up = __shfl_up_sync(0xffffffffu, incl, o);
+        if (lane >= o) incl += up;
+      }
+      float before = __shfl_up_sync(0xffffffffu, incl, 1);
+      if (lane == 0) before = 0.f;
+      const float end = __shfl_sync(0xffffffffu, incl, 31);
+      const float l0 = before + v0, l1 = incl;
+      cs[2 * lane] = l0;
+      cs[2 * lane + 1] = l1;
+      ecs[2 * lane] = expf(l0);
+      ecs[2 * lane + 1] = expf(l1);
+      wsm[2 * lane] = expf(end - l0) * dts[buf * SC_T + 2 * lane];
+      wsm[2 * lane + 1] = expf(end - l1) * dts[buf * SC_T + 2 * lane + 1];
+      if (lane == 0) *endp = expf(end);
+    }
+#pragma unroll
+    for (int r = 0; r < RT; ++r) {
+      if (warp + 8 * r < n_rt) {
+        const int n = (warp + 8 * r) * 16 + g;
+#pragma unroll
+        for (int nt = 0; nt < NT; ++nt) {
+          uint32_t hi, lo;
+          split2(S[r][nt][0], S[r][nt][1], hi, lo);
+          *reinterpret_cast<uint32_t*>(Sh + n * PV + nt * 8 + 2 * t4) = hi;
+          *reinterpret_cast<uint32_t*>(Sl + n * PV + nt * 8 + 2 * t4) = lo;
+          split2(S[r][nt][2], S[r][nt][3], hi, lo);
+          *reinterpret_cast<uint32_t*>(Sh + (n + 8) * PV + nt * 8 + 2 * t4) = hi;
+          *reinterpret_cast<uint32_t*>(Sl + (n + 8) * PV + nt * 8 + 2 * t4) = lo;
+        }
+      }
+    }
+    __syncthreads();                       // B
+    const bf16* xb = xs + (size_t)buf * SC_T * PV;
+    for (int i = tid; i < SC_T * (CV / 2); i += 256) {
+      const int r = i / (CV / 2), c = (i - r * (CV / 2)) * 2;
+      const uint32_t v = *reinterpret_cast<const uint32_t*>(xb + r * PV + c);
+      const float w = wsm[r];
+      uint32_t hi, lo;
+      split2(w * __uint_as_float(v << 16), w * __uint_as_float(v & 0xffff0000u), hi, lo);
+      *reinterpret_cast<uint32_t*>(wh + r * PV + c) = hi;
+      *reinterpret_cast<uint32_t*>(wl + r * PV + c) = lo;
+    }
+    __syncthreads();                       // C
+    const bf16 *Bb = Bs + (size_t)buf * SC_T * PN, *Cb = Cs + (size_t)buf * SC_T * PN;
+    const int m0 = (warp & 3) * 16;
+    float Y[NT][4];
+#pragma unroll
+    for (int nt = 0; nt < NT; ++nt) Y[nt][0] = Y[nt][1] = Y[nt][2] = Y[nt][3] = 0.f;
+    if (warp < 4) {
+      // the chunk's own tokens: scores of 16 rows against the columns up to them
+      float p[8][4];
+#pragma unroll
+      for (int nt = 0; nt < 8; ++nt) p[nt][0] = p[nt][1] = p[nt][2] = p[nt][3] = 0.f;
+      for (int k = 0; k < N; k += 16) {
+        uint32_t a0, a1, a2, a3;
+        ldmatrix_x4(a0, a1, a2, a3, smem_u32(Cb + (m0 + a_row) * PN + k + a_col));
+#pragma unroll
+        for (int np = 0; np < 4; ++np) {
+          if (np * 16 <= m0) {
+            uint32_t b0, b1, b2, b3;
+            ldmatrix_x4(b0, b1, b2, b3, smem_u32(Bb + (np * 16 + b_row) * PN + k + b_col));
+            mma_bf16(p[2 * np], a0, a1, a2, a3, b0, b1);
+            mma_bf16(p[2 * np + 1], a0, a1, a2, a3, b2, b3);
+          }
+        }
+      }
+      const float l0 = cs[m0 + g], l1 = cs[m0 + g + 8];
+#pragma unroll
+      for (int nt = 0; nt < 8; ++nt)
+        if (nt * 8 <= m0 + 15) {
+#pragma unroll
+          for (int j = 0; j < 4; ++j) {
+            const int s = nt * 8 + 2 * t4 + (j & 1), row = m0 + g + (j < 2 ? 0 : 8);
+            p[nt][j] = s <= row ? p[nt][j] * (expf((j < 2 ? l0 : l1) - cs[s]) * dts[buf * SC_T + s]) : 0.f;
+          }
+        }
+#pragma unroll
+      for (int ks = 0; ks < 4; ++ks) {
+        if (ks * 16 <= m0) {
+          uint32_t h0, h1, h2, h3, q0, q1, q2, q3;
+          split2(p[2 * ks][0], p[2 * ks][1], h0, q0);
+          split2(p[2 * ks][2], p[2 * ks][3], h1, q1);
+          split2(p[2 * ks + 1][0], p[2 * ks + 1][1], h2, q2);
+          split2(p[2 * ks + 1][2], p[2 * ks + 1][3], h3, q3);
+#pragma unroll
+          for (int np = 0; np < NT / 2; ++np) {
+            uint32_t b0, b1, b2, b3;
+            ldmatrix_x4_trans(b0, b1, b2, b3, smem_u32(xb + (ks * 16 + v_row) * PV + np * 16 + v_col));
+            mma_bf16(Y[2 * np], h0, h1, h2, h3, b0, b1);
+            mma_bf16(Y[2 * np + 1], h0, h1, h2, h3, b2, b3);
+            mma_bf16(Y[2 * np], q0, q1, q2, q3, b0, b1);
+            mma_bf16(Y[2 * np + 1], q0, q1, q2, q3, b2, b3);
+          }
+        }
+      }
+    } else {
+      // what the state before the chunk gives: exp(L_t) S^T C_t
+      for (int k = 0; k < N; k += 16) {
+        uint32_t a0, a1, a2, a3;
+        ldmatrix_x4(a0, a1, a2, a3, smem_u32(Cb + (m0 + a_row) * PN + k + a_col));
+#pragma unroll
+        for (int np = 0; np < NT / 2; ++np) {
+          uint32_t b0, b1, b2, b3;
+          ldmatrix_x4_trans(b0, b1, b2, b3, smem_u32(Sh + (k + v_row) * PV + np * 16 + v_col));
+          mma_bf16(Y[2 * np], a0, a1, a2, a3, b0, b1);
+          mma_bf16(Y[2 * np + 1], a0, a1, a2, a3, b2, b3);
+          ldmatrix_x4_trans(b0, b1, b2, b3, smem_u32(Sl + (k + v_row) * PV + np * 16 + v_col));
+          mma_bf16(Y[2 * np], a0, a1, a2, a3, b0, b1);
+          mma_bf16(Y[2 * np + 1], a0, a1, a2, a3, b2, b3);
+        }
+      }
+      const float e0 = ecs[m0 + g], e1 = ecs[m0 + g + 8];
+#pragma unroll
+      for (int nt = 0; nt < NT; ++nt) {
+        *reinterpret_cast<float2*>(Yx + (m0 + g) * (CV + 4) + nt * 8 + 2 * t4) = make_float2(Y[nt][0] * e0, Y[nt][1] * e0);
+        *reinterpret_cast<float2*>(Yx + (m0 + g + 8) * (CV + 4) + nt * 8 + 2 * t4) = make_float2(Y[nt][2] * e1, Y[nt][3] * e1);
+      }
+    }
+    const float keep = *endp;
+#pragma unroll
+    for (int r = 0; r < RT; ++r) {
+      if (warp + 8 * r < n_rt) {
+#pragma unroll
+        for (int nt = 0; nt < NT; ++nt) { S[r][nt][0] *= keep; S[r][nt][1] *= keep; S[r][nt][2] *= keep; S[r][nt][3] *= keep; }
+#pragma unroll
+        for (int ks = 0; ks < 4; ++ks) {
+          uint32_t a0, a1, a2, a3;
+          ldmatrix_x4_trans(a0, a1, a2, a3, smem_u32(Bb + (ks * 16 + s_tok) * PN + (warp + 8 * r) * 16 + s_n));
+#pragma unroll
+          for (int np = 0; np < NT / 2; ++np) {
+            uint32_t b0, b1, b2, b3;
+            ldmatrix_x4_trans(b0, b1, b2, b3, smem_u32(wh + (ks * 16 + v_row) * PV + np * 16 + v_col));
+            mma_bf16(S[r][2 * np], a0, a1, a2, a3, b0, b1);
+            mma_bf16(S[r][2 * np + 1], a0, a1, a2, a3, b2, b3);
+            ldmatrix_x4_trans(b0, b1, b2, b3, smem_u32(wl + (ks * 16 + v_row) * PV + np * 16 + v_col));
+            mma_bf16(S[r][2 * np], a0, a1, a2, a3, b0, b1);
+            mma_bf16(S[r][2 * np + 1], a0, a1, a2, a3, b2, b3);
+          }
+        }
+      }
+    }
+    __syncthreads();                       // D
+    if (warp < 4) {
+      const int n = min(SC_T, t1 - c0);
+#pragma unroll
+      for (int half = 0; half < 2; ++half) {
+        const int row = m0 + g + half * 8;
+        if (row >= n) continue;
+        float* o = y + (size_t)(c0 + row) * z.inner() + (size_t)h * V + col0;
+#pragma unroll
+        for (int nt = 0; nt < NT; ++nt) {
+          const int c = nt * 8 + 2 * t4;
+          if (col0 + c >= V) continue;
+          const float2 inter = *reinterpret_cast<const float2*>(Yx + row * (CV + 4) + c);
+          const uint32_t v = *reinterpret_cast<const uint32_t*>(xb + row * PV + c);
+          *reinterpret_cast<float2*>(o + c) =
+              make_float2(fmaf(sk, __uint_as_float(v << 16), Y[nt][2 * half] + inter.x),
+                          fmaf(sk, __uint_as_float(v & 0xffff0000u), Y[nt][2 * half + 1] + inter.y));
+        }
+      }
+    }
+  }
+  if (!write_state) return;
+#pragma unroll
+  for (int r = 0; r < RT; ++r)
+#pragma unroll
+    for (int nt = 0; nt < NT; ++nt) {
+      const int n = (warp + 8 * r) * 16 + g, c = nt * 8 + 2 * t4;
+      if (warp + 8 * r >= n_rt || col0 + c >= V) continue;
+      *reinterpret_cast<float2*>(st + (size_t)n * V + c) = make_float2(S[r][nt][0], S[r][nt][1]);
+      *reinterpret_cast<float2*>(st + (size_t)(n + 8) * V + c) = make_float2(S[r][nt][2], S[r][nt][3]);
+    }
+}
+
+// 1 if ssm_chunks takes the sizes: state sizes in steps of 16, value sizes in steps of 8, both up to 256
+AB_API int ab_ssm_chunks_supports(int N, int V) { return N > 0 && N <= 256 && N % 16 == 0 && V > 0 && V <= 256 && V % 8 == 0 ? 1 : 0; }
+
+// xbc bfloat16 [T, channels] (x | B | C), la and dt float32 [T, H] (log decays, step sizes), y float32 [T, H * V].
+// `cols`: value columns per CTA (16 or 32).
+AB_API int ab_ssm_chunks(const void* xbc, const float* la, const float* dt, const float* skip, float* state, float* y,
+                         const int* cu_q, const int* slots, int n_seqs, int H, int G, int N, int V, int cols, int write_state,
+                         cudaStream_t stream) {
+  if (n_seqs <= 0) return AB_OK;
+  const SsmSizes z{H, G, N, V, 1};
+  if (!ssm_sizes_ok(z) || !ab_ssm_chunks_supports(N, V) || H > 65535 || ((((uintptr_t)xbc) | ((uintptr_t)state)) & 15)) return AB_BAD_ARG;
+  const dim3 grid((unsigned)n_seqs, (unsigned)H, (unsigned)((V + cols - 1) / cols));
+#define AB_GO(CV, RT)                                                                                                  \
+  {                                                                                                                    \
+    const size_t smem = ChunkSmem<CV>::total(N);                                                                       \
+    cudaError_t e = cudaFuncSetAttribute(ssm_chunks_kernel<CV, RT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
+    if (e != cudaSuccess) return AB_CUDA_ERR + (int)e;                                                                 \
+    ab_launch(ssm_chunks_kernel<CV, RT>, grid, dim3(256), smem, stream, (const bf16*)xbc, la, dt, skip, state, y, cu_q, slots, \
+              z, write_state);                                                                                         \
+  }
+  if (cols == 32) { if (N <= 128) AB_GO(32, 1) else AB_GO(32, 2) }
+  else if (cols == 16) { if (N <= 128) AB_GO(16, 1) else AB_GO(16, 2) }
+  else return AB_BAD_ARG;
+#undef AB_GO
+  return ab_launch_status();
+}

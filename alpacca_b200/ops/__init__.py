@@ -338,7 +338,7 @@ def _sm_count(device) -> int:
     return n
 
 
-PLAIN_ACTIVATIONS = {None: 0, "gelu": 1}      # on a product without a gate ("gelu": the erf form)
+PLAIN_ACTIVATIONS = {None: 0, "gelu": 1, "relu2": 2}      # on a product without a gate ("gelu": the erf form; the square of ReLU)
 
 
 def gemv_bf16(x, w, out, bias=None, n_rows=None, swiglu=False, slices=None, start_early=True, owed=None,
@@ -414,7 +414,8 @@ def gemv_bf16(x, w, out, bias=None, n_rows=None, swiglu=False, slices=None, star
         _check(lib.ab_gemv_bf16_act(_p(x), _p(w), _p(bias), _p(out), _p(partials), _p(arrivals), n, N, K,
                                     out.shape[-1], epi, slices, _p(ss_in), n_part, ctypes.c_float(inv_width),
                                     ctypes.c_float(eps), _p(residual), _p(norm_weight), _p(ss_out),
-                                    GATE_ACTIVATIONS[activation], ctypes.c_float(cap), _stream()),
+                                    PLAIN_ACTIVATIONS[act] - 1 if act is not None else GATE_ACTIVATIONS[activation],
+                                    ctypes.c_float(cap), _stream()),
                "gemv_bf16")
     finally:
         if not start_early:
@@ -518,24 +519,38 @@ def _stream_scratch(device, n_partial: int, n_counters: int):
     return have
 
 
-def _check_dist(dist, H):
-    """The penalty on distance of H heads: float32 [2, H], r1 of all heads and then r2."""
+def _score_args(dist, bound, H):
+    """What happens to the scaled scores of H heads, as the entry points take it (kind, numbers, cap): `dist` float32
+    [2, H], r1 of all heads and then r2 (a logarithmic penalty on distance), or `bound` = (slopes float32 [H], cap): scores
+    bounded to cap * tanh(score / cap) (cap 0: not), then less slope_h times the distance."""
+    _need(dist is None or bound is None, "a score takes one kind of penalty on distance")
     if dist is not None:
         _cuda(dist)
         _need(dist.dtype == torch.float32 and dist.is_contiguous() and tuple(dist.shape) == (2, H),
               f"the penalty on distance must be float32 [2, {H}]")
+        return 1, _p(dist), ctypes.c_float(0.0)
+    if bound is not None:
+        slopes, cap = bound
+        _cuda(slopes)
+        _need(slopes.dtype == torch.float32 and slopes.is_contiguous() and tuple(slopes.shape) == (H,) and float(cap) >= 0,
+              f"the slopes of a penalty on distance must be float32 [{H}], the scores' bound must not be negative")
+        return 2, _p(slopes), ctypes.c_float(cap)
+    return 0, None, ctypes.c_float(0.0)
 
 
 def attention_stream(qkv, out, cache, ctx, H, K, D, scale, window=0, rot=None, fuse=0, pages_per_cta=8,
-                     merge="memory", ring=1, dist=None):
+                     merge="memory", ring=1, dist=None, bound=None, sink=None):
     """Decode attention that streams the cache through a ring of pages filled by TMA
     (csrc/attention_stream.cu): head sizes 64 and 128, bfloat16.  A CTA takes `pages_per_cta` pages of
     one (sequence, KV head); the chunks of a sequence are merged in chunk order, through scratch memory
     (`merge` "memory") or inside a cluster of up to 8 ("cluster").  `ring`: 0 a short ring (four CTAs per
     processor), 1 the usual one (two), 2 a deep one (one).  `fuse` as for the other decode kernel: 1 rotates q, 2 also rotates k
-    and appends k, v to the cache.  `dist` (float32 [2, H]): a penalty on distance, see `attention_maps`."""
+    and appends k, v to the cache.  `dist`, `bound`, `sink`: see `attention_maps`."""
     lib = _lib("attention_stream")
-    _check_dist(dist, H)
+    score = _score_args(dist, bound, H)
+    if sink is not None:
+        _cuda(sink)
+        _need(sink.dtype == torch.float32 and sink.numel() == H and sink.is_contiguous(), "sink must be float32 [H]")
     k_pages, v_pages, table = cache.k, cache.v, cache.block_table
     _cuda(qkv, out, k_pages, v_pages, table)
     T = ctx.n_tokens
@@ -576,7 +591,7 @@ def attention_stream(qkv, out, cache, ctx, H, K, D, scale, window=0, rot=None, f
         _p(qkv), qkv.shape[-1], _p(out), _p(part_o), _p(part_ml), _p(arrivals), _p(k_pages), _p(v_pages),
         k_pages.shape[0], _p(table), table.shape[1], _p(ctx.tok_seq), _p(ctx.kv_len), _p(order), T, H, K, D,
         ctypes.c_float(scale), int(window or 0), ppc, n_chunks, kind, int(ring), _p(cos), _p(sin), n_rot,
-        pairing, fuse, _p(dist), _stream()), "attention_stream")
+        pairing, fuse, _p(sink), *score, _stream()), "attention_stream")
     return out
 
 
@@ -763,7 +778,7 @@ def softcap(y, cap, n_rows=None):
 
 
 def plain_act(y, activation, n_rows=None):
-    """y[:n] = act(y[:n]) in place ("gelu": the erf form); y [M, N]."""
+    """y[:n] = act(y[:n]) in place ("gelu": the erf form; "relu2": the square of ReLU); y [M, N]."""
     _cuda(y)
     n = y.shape[0] if n_rows is None else n_rows
     _need(activation in PLAIN_ACTIVATIONS and activation is not None,
@@ -873,12 +888,13 @@ def decode_advance(tokens, tok_pos, kv_len, rng_step, tok_seq, sampled, recent, 
 
 
 def gemm_tc(x, w, out, bias=None, n_rows=None, swiglu=False, swap=None, bn=None, slices=None, persistent=True,
-            pair=None, activation="silu"):
+            pair=None, activation="silu", relu2=False):
     """out[:n] = x[:n] @ w^T (+ bias) on the tcgen05 tensor cores (TMA-fed, TMEM accumulators).
 
     x [M,K], w [N,K] bfloat16; out bfloat16 or float32 [M,N]; with `swiglu`, w is the 8-row
     interleaved gate|up matrix and out is bfloat16 [M, N/2] (`activation` on the gate: "silu"; "relu" and
-    "gelu_tanh" in the persistent forms only).  `swap` puts the weights on the
+    "gelu_tanh" in the persistent forms only).  `relu2`: out = max(x @ w^T, 0)^2 in bfloat16 (persistent forms, no bias).
+    `swap` puts the weights on the
     128-row side of the MMA (the batch, up to 256 rows, becomes the columns): the shape for decode
     steps.  `bn` is the MMA's column count per tile, `slices` the number of K slices.  Without `swap`,
     256-wide tiles and one slice run as the persistent kernel (one CTA per SM walks the tiles) unless
@@ -907,6 +923,10 @@ def gemm_tc(x, w, out, bias=None, n_rows=None, swiglu=False, swap=None, bn=None,
     else:
         _need(out.shape[-1] == N and out.dtype in (torch.bfloat16, torch.float32), "gemm_tc: out [M,N]")
         epi = 1 if out.dtype == torch.float32 else 0
+        if relu2:
+            _need(epi == 0 and bias is None and not swap and bn == 256 and slices in (None, 1) and persistent,
+                  "gemm_tc: the squared ReLU runs in the persistent forms, bfloat16 without a bias")
+            epi = 5
     if bias is not None:
         _need(bias.dtype == torch.float32 and bias.numel() == N and bias.is_contiguous(), "gemm_tc: bias f32 [N]")
     _tc_unchecked["gemm_tc"] = True
@@ -1170,7 +1190,7 @@ def latent_attention(q, out, cache, ctx, H, C, R, scale, sink=None, window=0):
     return out
 
 
-MOE_ACTIVATIONS = {"gelu": 0, "silu": 1}
+MOE_ACTIVATIONS = {"gelu": 0, "silu": 1, "relu2": 2}      # ("relu2", the square of ReLU: `moe_shared_experts` alone)
 
 
 MOE_SCORES = {"softmax": None, "logit": 0, "sigmoid": 1}
@@ -1203,7 +1223,7 @@ def moe_route(h, router, n_tokens, groups, keep, top, scale, bias=None, score="s
     wts = torch.empty((max(n_tokens, 1), top), dtype=torch.float32, device=h.device)
     z = torch.empty((max(n_tokens, 1), E), dtype=torch.float32, device=h.device)
     if score != "softmax":
-        _need(group_top >= 1 and E // groups <= 128, "moe_route: groups of up to 128 experts, group_top >= 1")
+        _need(group_top >= 1 and (keep == groups or E // groups <= 128), "moe_route: groups of up to 128 experts, group_top >= 1")
         _check(_lib("moe").ab_moe_route_scores(
             _p(h), _dt(h), width, _p(router), _p(bias), _p(correction), n_tokens, width, E, groups, keep, int(group_top),
             top, MOE_SCORES[score], 1 if renorm else 0, ctypes.c_float(scale), _p(z), _p(idx), _p(wts), _stream()),
@@ -1453,13 +1473,14 @@ def attention_prepare(buf, offsets, H, G, M, Dk, Dv, cache, ctx, q_weight=None, 
 
 
 def attention_maps(q, q_stride, out, cache, ctx, H, G, M, Dk, Dv, scale, window=0, sink=None, coef=0.0,
-                   unit_norm=False, eps=0.0, out_scale=1.0, dist=None):
+                   unit_norm=False, eps=0.0, out_scale=1.0, dist=None, bound=None):
     """Attention of every token over its sequence's cached keys and values, one warp per (token, head), 32-bit
     arithmetic (csrc/attention_maps.cu): M score maps per head, combined as a_0 + coef * (a_1 + ..), optionally
     divided by the head's root mean square, times `out_scale`.  q: the prepared rows (query vectors at the
     start of each row of `q_stride` elements); out [T, H*Dv] of q's dtype.  `dist` (float32 [2, H], r1 and r2): a
-    penalty r1_h ln(1 + r2_h (p - s)) is taken off the scaled score of a key at s for a token at p."""
-    _check_dist(dist, H)
+    penalty r1_h ln(1 + r2_h (p - s)) is taken off the scaled score of a key at s for a token at p.  `bound` (slopes
+    float32 [H], cap): a scaled score becomes cap * tanh(score / cap) (cap 0: stays), less slope_h (p - s)."""
+    score = _score_args(dist, bound, H)
     k_pages, v_pages, table = cache.k, cache.v, cache.block_table
     _cuda(q, out, k_pages, v_pages, table, sink)
     T = ctx.n_tokens
@@ -1481,7 +1502,7 @@ def attention_maps(q, q_stride, out, cache, ctx, H, G, M, Dk, Dv, scale, window=
     _check(_lib("attention_maps").ab_attention_maps_dist(
         _p(q), q_stride, _p(out), _dt(q), _p(k_pages), _p(v_pages), _p(table), table.shape[1], _p(ctx.tok_pos),
         _p(ctx.tok_seq), T, H, G, M, Dk, Dv, page, ctypes.c_float(scale), int(window or 0), _p(sink),
-        ctypes.c_float(coef), 1 if unit_norm else 0, ctypes.c_float(eps), ctypes.c_float(out_scale), _p(dist), _stream()),
+        ctypes.c_float(coef), 1 if unit_norm else 0, ctypes.c_float(eps), ctypes.c_float(out_scale), *score, _stream()),
         "attention_maps")
     return out
 
@@ -1510,13 +1531,13 @@ def _row_index(device, n: int):
 
 
 def attention_maps_mma(q, q_stride, out, cache, ctx, H, G, M, Dk, Dv, scale, window=0, sink=None, coef=0.0,
-                       unit_norm=False, eps=0.0, out_scale=1.0, dist=None):
+                       unit_norm=False, eps=0.0, out_scale=1.0, dist=None, bound=None):
     """`attention_maps` on the tensor-core kernels (bfloat16 operands, float32 scores, softmax and sums): q holds
     the prepared query vectors at the start of each row, keys and values are in the cache already.  One map with
     equal key and value sizes in a step of one token each takes the decode kernel; everything else the kernel that
     tiles query rows (a step of one token each then has one token per tile).  Several maps leave their outputs
-    in float32 and are combined by `ab_maps_combine`.  `dist`: see `attention_maps`."""
-    _check_dist(dist, H)
+    in float32 and are combined by `ab_maps_combine`.  `dist`, `bound`: see `attention_maps`."""
+    score = _score_args(dist, bound, H)
     k_pages, v_pages, table = cache.k, cache.v, cache.block_table
     _cuda(q, out, k_pages, v_pages, table, sink)
     T = ctx.n_tokens
@@ -1537,16 +1558,16 @@ def attention_maps_mma(q, q_stride, out, cache, ctx, H, G, M, Dk, Dv, scale, win
     _i32(ctx.tok_seq, T, "tok_seq")
     if ctx.is_decode and M == 1 and Dk == Dv:
         width = max(int(table.shape[1]), 1)
-        plan = _stream_plan(T, H, G, Dk, width, _sm_count(q.device)) if dist is not None and sink is None else None
+        plan = _stream_plan(T, H, G, Dk, width, _sm_count(q.device)) if score[0] else None
         if plan is not None:
             return attention_stream(q, out, cache, ctx, H, G, Dk, scale, window, pages_per_cta=plan[0], merge=plan[1],
-                                    ring=plan[2], dist=dist)
+                                    ring=plan[2], dist=dist, bound=bound, sink=sink)
         small, n_chunks = _decode_attention_plan(T * G * -(-(H // G) // 8), width, Dk, _sm_count(q.device))
         _i32(ctx.kv_len, ctx.n_seqs, "kv_len")
         _check(lib.ab_attention_decode_dist_bf16(
             _p(q), q_stride, _p(out), None, None, None, _p(k_pages), _p(v_pages), _p(table), table.shape[1],
             _p(ctx.tok_seq), _p(ctx.kv_len), T, H, G, Dk, ctypes.c_float(scale), int(window or 0),
-            -(-width // n_chunks), n_chunks, small, None, None, 0, 0, 0, _p(sink), _p(dist), _stream()), "attention_decode")
+            -(-width // n_chunks), n_chunks, small, None, None, 0, 0, 0, _p(sink), *score, _stream()), "attention_decode")
         return out
     _i32(ctx.tok_pos, T, "tok_pos")
     _i32(ctx.cu_q, ctx.n_seqs + 1, "cu_q")
@@ -1561,7 +1582,7 @@ def attention_maps_mma(q, q_stride, out, cache, ctx, H, G, M, Dk, Dv, scale, win
             _check(tc.ab_attention_prefill_tc_dist(
                 _p(q), q_stride // Dk, T, _p(out), _p(k_pages), _p(v_pages), k_pages.shape[0], _p(table), table.shape[1],
                 _p(ctx.tok_pos), _p(ctx.cu_q), _p(tile_seq), _p(tile_q0), n_tiles, H, G, Dk, ctypes.c_float(scale),
-                int(window or 0), _p(sink), _p(dist), _stream()), "attention_prefill_tc")
+                int(window or 0), _p(sink), *score, _stream()), "attention_prefill_tc")
             return out
     if ctx.is_decode:
         # one token per sequence: a tile per token; the rows are the batch rows themselves
@@ -1573,7 +1594,7 @@ def attention_maps_mma(q, q_stride, out, cache, ctx, H, G, M, Dk, Dv, scale, win
     _check(lib.ab_attention_prefill_maps_dist_bf16(
         _p(q), q_stride, _p(maps), 0 if M == 1 else 1, _p(k_pages), _p(v_pages), _p(table), table.shape[1],
         _p(ctx.tok_pos), _p(ctx.cu_q), _p(ctx.tok_seq), _p(tile_seq), _p(tile_q0), n_tiles, tpt, H * M, G * M, M, Dk, Dv,
-        ctypes.c_float(scale), int(window or 0), _p(sink), Dv, 0, Dv, _p(dist), _stream()), "attention_prefill")
+        ctypes.c_float(scale), int(window or 0), _p(sink), Dv, 0, Dv, *score, _stream()), "attention_prefill")
     if M > 1:
         _check(_lib("attention_maps").ab_maps_combine(
             _p(maps), _p(out), _dt(out), _p(ctx.tok_seq), T, H, M, Dv, ctypes.c_float(coef),
@@ -1896,14 +1917,19 @@ def _f32_rows(t, n, name):
     return t.stride(0)
 
 
-def gated_recurrence(mode, q, k, v, state, out, ctx, H, Hk, D, V, qscale=1.0, decay=None, beta=None, write_state=True):
+def gated_recurrence(mode, q, k, v, state, out, ctx, H, Hk, D, V, qscale=1.0, decay=None, beta=None, skip=None,
+                     write_state=True):
     """One walk of a recurrent mixer over the step's tokens; q, k [T, Hk * D] and v [T, H * V] float32 (views with a
     row stride are fine), state float32 [slots, H, D, V], out float32 [T, H * V].
     mode "channel": S <- diag(a_t) S + k_t v_t^T, o_t = S^T (q_t qscale), decay a [T, H * D];
-    mode "delta": S <- g_t S; u = beta_t (v_t - S^T k_t); S <- S + k_t u^T; o_t = S^T (q_t qscale), decay g and beta [T, H]."""
-    _cuda(q, k, v, state, out, decay, beta)
+    mode "delta": S <- g_t S; u = beta_t (v_t - S^T k_t); S <- S + k_t u^T; o_t = S^T (q_t qscale), decay g and beta [T, H];
+    mode "scalar": S <- g_t S + beta_t k_t v_t^T, o_t = S^T q_t + skip_h v_t, decay g and beta [T, H], skip [H] or None."""
+    _cuda(q, k, v, state, out, decay, beta, skip)
     T = ctx.n_tokens
-    _need(mode in ("channel", "delta"), "gated_recurrence: mode channel or delta")
+    _need(mode in ("channel", "delta", "scalar"), "gated_recurrence: mode channel, delta or scalar")
+    _need(skip is None or (mode == "scalar" and skip.dtype == torch.float32 and skip.is_contiguous() and skip.numel() == H),
+          "gated_recurrence: skip float32 [H], in mode scalar")
+    _need(mode != "scalar" or qscale == 1.0, "gated_recurrence: mode scalar reads q as it is")
     _need(0 < D <= RECURRENCE_MAX_DIM and H % Hk == 0, f"gated_recurrence: {D} dims per head are outside 1..{RECURRENCE_MAX_DIM}")
     ldq, ldk, ldv = _f32_rows(q, T, "q"), _f32_rows(k, T, "k"), _f32_rows(v, T, "v")
     _need(q.shape[0] >= T and k.shape[0] >= T and v.shape[0] >= T and q.shape[1] == Hk * D and k.shape[1] == Hk * D
@@ -1925,7 +1951,8 @@ def gated_recurrence(mode, q, k, v, state, out, ctx, H, Hk, D, V, qscale=1.0, de
     _i32(ctx.slots, ctx.n_seqs, "slots")
     cols = _recurrence_cols(ctx.n_seqs, H, V)
     _check(_lib("gated_recurrence").ab_gated_recurrence(
-        0 if mode == "channel" else 1, _p(q), ldq, _p(k), ldk, _p(v), ldv, _p(dvec), ldd, _p(dsc), _p(beta),
+        {"channel": 0, "delta": 1, "scalar": 2}[mode], _p(q), ldq, _p(k), ldk, _p(v), ldv, _p(dvec), ldd, _p(dsc), _p(beta),
+        _p(skip),
         ctypes.c_float(qscale), _p(state), _p(out), _p(ctx.cu_q), _p(ctx.slots), ctx.n_seqs, H, Hk, D, V, cols,
         1 if write_state else 0, 1 if ctx.max_q_len <= RECURRENCE_ROUND else 0, _stream()), "gated_recurrence")
     return out
@@ -2017,8 +2044,8 @@ def head_norm_gate(o, weight, gate, gate_act, eps, out, ctx, H, V):
 # blocks whose norms act on the sub-layers' outputs, whose mixers see the stream through a short convolution and whose
 # results are averaged over depth (csrc/depth_stream.cu); experts chosen by token id and a shared expert (csrc/moe.cu)
 
-def embed_positions(table, pos, out, ctx):
-    """out[t] = table[token of t] + pos[place of t in its sequence] as float32; table [V, E], pos [P, E] of one dtype."""
+def embed_positions(table, pos, out, ctx, scale=1.0):
+    """out[t] = scale * table[token of t] + pos[place of t in its sequence] as float32; table [V, E], pos [P, E] of one dtype."""
     _cuda(table, pos, out)
     T, E = ctx.n_tokens, table.shape[1]
     _need(table.dim() == 2 and pos.dim() == 2 and table.is_contiguous() and pos.is_contiguous() and pos.shape[1] == E
@@ -2029,7 +2056,8 @@ def embed_positions(table, pos, out, ctx):
     for t, name in ((ctx.tokens, "tokens"), (ctx.tok_seq, "tok_seq"), (ctx.tok_pos, "tok_pos")):
         _i32(t, T, name)
     _check(_lib("depth_stream").ab_embed_positions(_p(table), _p(pos), _dt(table), _p(ctx.tokens), _p(ctx.tok_seq),
-                                                   _p(ctx.tok_pos), _p(out), T, E, _stream()), "embed_positions")
+                                                   _p(ctx.tok_pos), ctypes.c_float(scale), _p(out), T, E, _stream()),
+           "embed_positions")
     return out
 
 
@@ -2118,12 +2146,15 @@ def row_dots(h, w, n_tokens):
 MOE_GEMV_MAX_ROWS = 32             # up to here the skinny products of csrc/moe_gemv.cu
 
 
-def gemm_tc_grouped(x, w, out, n_groups, tile_group, row_tiles, swiglu=False):
+def gemm_tc_grouped(x, w, out, n_groups, tile_group, row_tiles, swiglu=False, relu2=False, row_factor=None):
     """Rows in groups with a matrix each, on the tcgen05 tensor cores: row tile i (128 rows) of x [R, K] belongs to group
     tile_group[i] and is multiplied with w [n_groups * N, K]'s rows of that group; out [R, N], or [R, N / 2] with `swiglu`
     (an 8-row interleaved gate|up matrix per group).  row_tiles int32 [1]: how many row tiles there are, on the device;
-    rows past them are left alone.  All bfloat16."""
-    _cuda(x, w, out, tile_group, row_tiles)
+    rows past them are left alone.  `relu2`: out = max(y, 0)^2 of the products y, each first multiplied by its row's
+    number of row_factor (float32 [R]) if that is given.  All bfloat16."""
+    _cuda(x, w, out, tile_group, row_tiles, row_factor)
+    _need(row_factor is None or (relu2 and row_factor.dtype == torch.float32 and row_factor.is_contiguous()
+                                 and row_factor.numel() >= x.shape[0]), "gemm_tc_grouped: row_factor float32 [R], with relu2")
     R, K = x.shape
     N = w.shape[0] // n_groups
     _need(x.dtype == w.dtype == out.dtype == torch.bfloat16 and x.is_contiguous() and w.is_contiguous() and out.is_contiguous()
@@ -2134,17 +2165,20 @@ def gemm_tc_grouped(x, w, out, n_groups, tile_group, row_tiles, swiglu=False):
     _i32(tile_group, R // 128, "tile_group")
     _i32(row_tiles, 1, "row_tiles")
     _tc_unchecked["gemm_tc"] = True
-    _check(_lib("gemm_tc").ab_gemm_tc_grouped(_p(x), _p(w), _p(out), R, N, K, n_groups, out.shape[1], 2 if swiglu else 0,
-                                              _p(tile_group), _p(row_tiles), _stream()), "gemm_tc_grouped")
+    _check(_lib("gemm_tc").ab_gemm_tc_grouped(_p(x), _p(w), _p(out), R, N, K, n_groups, out.shape[1],
+                                              5 if relu2 else 2 if swiglu else 0, _p(tile_group), _p(row_tiles),
+                                              _p(row_factor), _stream()), "gemm_tc_grouped")
     return out
 
 
 def moe_shared_experts(h, gate_up, down, n_experts, top, out, ctx, activation="silu", choice=None, table=None, shared=None,
-                       gate_logits=None):
-    """Gated experts and a shared expert: out[t] = sum_k weight_k E_(e_k)(h[t]) + sigmoid(gate_logits[t]) S(h[t]), an expert
+                       gate_logits=None, gated=True, weight_in=False):
+    """Experts and a shared expert: out[t] = sum_k weight_k E_(e_k)(h[t]) + sigmoid(gate_logits[t]) S(h[t]), an expert
     W_down (act(W_gate h) * (W_up h)).  gate_up [n_experts * 2 ff, width]: an expert's rows in groups of 16, the gates of 8
     units and then their up-projections; down [n_experts * width, ff].  `shared` = (gate_up [2 fs, width], down [width, fs])
-    likewise, or None.  The choice is `choice` = (experts int32 [T, top], weights float32 [T, top]), or row token_t of
+    likewise, or None; without `gate_logits` its factor is 1.  Without `gated` an expert is W_down act(W_up h), gate_up
+    [n_experts * ff, width] its up-projections alone (likewise the shared expert's).  `weight_in`: weight_k multiplies
+    expert k's input instead of its output.  The choice is `choice` = (experts int32 [T, top], weights float32 [T, top]), or row token_t of
     `table` int32 [vocab, top] with weight 1 / top each.  out [T, width] float32.
 
     bfloat16: up to MOE_GEMV_MAX_ROWS tokens two skinny products that read the chosen experts' weights once; more tokens
@@ -2155,15 +2189,17 @@ def moe_shared_experts(h, gate_up, down, n_experts, top, out, ctx, activation="s
     _cuda(h, gate_up, down, out, idx, wts, table, gate_logits, gate_up_s, down_s)
     T, width = ctx.n_tokens, h.shape[-1]
     ff, fs = down.shape[1], 0 if shared is None else down_s.shape[1]
-    _need(tuple(gate_up.shape) == (n_experts * 2 * ff, width) and tuple(down.shape) == (n_experts * width, ff) and ff % 8 == 0
+    rpu = 2 if gated else 1          # rows of gate_up per unit
+    _need(tuple(gate_up.shape) == (n_experts * rpu * ff, width) and tuple(down.shape) == (n_experts * width, ff) and ff % 8 == 0
           and gate_up.is_contiguous() and down.is_contiguous() and gate_up.dtype == h.dtype and down.dtype == h.dtype,
-          "moe_shared_experts: gate_up [experts * 2 ff, width], down [experts * width, ff] of h's dtype, ff a multiple of 8")
+          "moe_shared_experts: gate_up [experts * 2 ff, width] (ungated: [experts * ff, width]), down [experts * width, ff] of "
+          "h's dtype, ff a multiple of 8")
     if shared is not None:
-        _need(tuple(gate_up_s.shape) == (2 * fs, width) and tuple(down_s.shape) == (width, fs) and fs % 8 == 0
+        _need(tuple(gate_up_s.shape) == (rpu * fs, width) and tuple(down_s.shape) == (width, fs) and fs % 8 == 0
               and gate_up_s.is_contiguous() and down_s.is_contiguous() and gate_up_s.dtype == h.dtype and down_s.dtype == h.dtype,
               "moe_shared_experts: the shared expert's gate_up [2 fs, width], down [width, fs] of h's dtype, fs a multiple of 8")
-        _need(gate_logits is not None and gate_logits.dtype == torch.float32 and gate_logits.is_contiguous()
-              and gate_logits.numel() >= T, "moe_shared_experts: the shared expert's gate logits float32 [T]")
+        _need(gate_logits is None or (gate_logits.dtype == torch.float32 and gate_logits.is_contiguous()
+                                      and gate_logits.numel() >= T), "moe_shared_experts: the shared expert's gate logits float32 [T]")
     _need(h.is_contiguous() and h.numel() >= T * width and out.is_contiguous() and out.shape[-1] == width
           and out.numel() >= T * width and out.dtype == torch.float32, "moe_shared_experts: h [T, width], out float32 [T, width]")
     _need((choice is None) != (table is None), "moe_shared_experts: the choice is a router's or a table's")
@@ -2177,37 +2213,173 @@ def moe_shared_experts(h, gate_up, down, n_experts, top, out, ctx, activation="s
               "the experts' table must be contiguous int32 [vocab, top]")
     by = (_p(idx), _p(wts), _p(table), _p(ctx.tokens) if table is not None else None, ctypes.c_float(1.0 / top))
     z = _p(gate_logits) if shared is not None else None
+    inward = 1 if weight_in else 0
     dev, code = h.device, MOE_ACTIVATIONS[activation]
     fast = h.dtype == torch.bfloat16 and width % 8 == 0
-    if fast and T > MOE_GEMV_MAX_ROWS and activation == "silu":
+    if fast and T > MOE_GEMV_MAX_ROWS and (activation == "silu" and not weight_in if gated else activation == "relu2"):
         n_tiles = T * top // 128 + n_experts
         pos = torch.empty(T * top, dtype=torch.int32, device=dev)
         plan = torch.empty(n_tiles + 1, dtype=torch.int32, device=dev)
         rows = torch.empty((n_tiles * 128, width), dtype=h.dtype, device=dev)
-        _check(_lib("moe").ab_moe_gather(_p(h), *by, _p(pos), _p(plan), _p(plan[n_tiles:]), _p(rows), T, top, width, n_experts,
-                                         _stream()), "moe_gather", kernels=2)
+        row_w = torch.empty(n_tiles * 128, dtype=torch.float32, device=dev) if weight_in else None
+        _check(_lib("moe").ab_moe_gather(_p(h), *by, _p(pos), _p(plan), _p(plan[n_tiles:]), _p(row_w), _p(rows), T, top, width,
+                                         n_experts, _stream()), "moe_gather", kernels=2)
         act = torch.empty((n_tiles * 128, ff), dtype=h.dtype, device=dev)
-        gemm_tc_grouped(rows, gate_up, act, n_experts, plan[:n_tiles], plan[n_tiles:], swiglu=True)
+        gemm_tc_grouped(rows, gate_up, act, n_experts, plan[:n_tiles], plan[n_tiles:], swiglu=gated, relu2=not gated,
+                        row_factor=row_w)
         gemm_tc_grouped(act, down, rows, n_experts, plan[:n_tiles], plan[n_tiles:])
         ys = None
         if shared is not None:
             act_s = torch.empty((T, fs), dtype=h.dtype, device=dev)
-            if T >= TC_PERSISTENT_MIN_ROWS:
+            if not gated:
+                if T >= TC_PERSISTENT_MIN_ROWS:
+                    gemm_tc(h, gate_up_s, act_s, n_rows=T, swap=False, relu2=True)
+                else:
+                    linear_bf16(h, gate_up_s, act_s, n_rows=T, act="relu2")
+            elif T >= TC_PERSISTENT_MIN_ROWS:
                 gemm_tc(h, gate_up_s, act_s, n_rows=T, swiglu=True, swap=False)
             else:
                 gated_act(linear_bf16(h, gate_up_s, torch.empty((T, 2 * fs), dtype=h.dtype, device=dev), n_rows=T), act_s, n_rows=T)
             ys = linear_bf16(act_s, down_s, torch.empty((T, width), dtype=h.dtype, device=dev), n_rows=T)
-        _check(_lib("moe").ab_moe_combine(_p(rows), _p(pos), *by, _p(ys), z, _p(out), T, top, width, _stream()), "moe_combine")
+        _check(_lib("moe").ab_moe_combine(_p(rows), _p(pos), *by, _p(ys), z, _p(out), T, top, width, inward, _stream()),
+               "moe_combine")
         return out
     act = torch.empty((max(T, 1), top * ff + fs), dtype=h.dtype, device=dev)
-    if fast and T <= MOE_GEMV_MAX_ROWS and n_experts <= 512 and top <= 32:
+    if fast and T <= MOE_GEMV_MAX_ROWS and n_experts <= 512 and top <= 32 and (gated or (ff % 16 == 0 and fs % 16 == 0)):
         slabs, slices = -(-width // 16), 1
         while slices < 8 and slabs * slices * 4 < 3 * _sm_count(dev):
             slices *= 2
         _check(_lib("moe_gemv").ab_moe_gemv(_p(h), _p(gate_up), _p(down), _p(gate_up_s), _p(down_s), *by, z, _p(act), _p(out), T,
-                                            top, width, ff, fs, n_experts, code, slices, _stream()), "moe_experts", kernels=2)
+                                            top, width, ff, fs, n_experts, code, 1 if gated else 0, inward, slices, _stream()), "moe_experts", kernels=2)
         return out
     _check(_lib("moe").ab_moe_shared_pairs(_p(h), _dt(h), width, _p(gate_up), _p(down), _p(gate_up_s), _p(down_s), *by, z, _p(act),
-                                           _p(out), _dt(out), T, top, width, ff, fs, n_experts, code, _stream()),
+                                           _p(out), _dt(out), T, top, width, ff, fs, n_experts, code, 1 if gated else 0, inward, _stream()),
            "moe_experts", kernels=2)
+    return out
+
+
+# ---------------------------------------------------------------------------
+# the state-space mixer (csrc/state_space.cu)
+
+SSM_MAX_TAPS = 17
+SSM_CHUNKS_FROM = 16             # tokens per sequence (on average) from which a bfloat16 step runs in chunks of 64
+
+
+def _ssm_check(proj, conv_w, conv_state, H, G, N, V, T):
+    """The sizes that the kernels around the recurrence share; returns (channels, taps)."""
+    _need(H > 0 and G > 0 and H % G == 0 and 0 < N <= RECURRENCE_MAX_DIM and V > 0,
+          f"state-space mixer: {H} heads in {G} groups, state {N} (up to {RECURRENCE_MAX_DIM}), values {V}")
+    Cc = H * V + 2 * G * N
+    taps = conv_w.shape[0]
+    _need(conv_w.dtype == torch.float32 and conv_w.is_contiguous() and conv_w.dim() == 2 and conv_w.shape[1] == Cc
+          and 1 <= taps <= SSM_MAX_TAPS, f"state-space mixer: convolution float32 [1..{SSM_MAX_TAPS} taps, {Cc}]")
+    _need(proj.dtype == torch.float32 and proj.is_contiguous() and proj.dim() == 2 and proj.shape[0] >= T
+          and proj.shape[1] >= H * V + Cc + H, "state-space mixer: projected rows float32 [T, z | x | B | C | dt]")
+    if taps > 1:
+        _need(conv_state is not None and conv_state.dtype == torch.float32 and conv_state.is_contiguous()
+              and tuple(conv_state.shape[1:]) == (taps - 1, Cc), f"state-space mixer: kept inputs float32 [slots, {taps - 1}, {Cc}]")
+    return Cc, taps
+
+
+def _ssm_vectors(H, **vectors):
+    for name, t in vectors.items():
+        _need(t.dtype == torch.float32 and t.is_contiguous() and t.numel() == H, f"state-space mixer: {name} float32 [{H}]")
+
+
+def ssm_prepare(proj, conv_w, conv_b, conv_state, A_log, dt_bias, xbc, decay, dt, ctx, H, G, N, V, log_decay, write_state=True):
+    """From projected rows float32 [T, z | x | B | C | dt]: xbc [T, channels] (float32 or bfloat16), the causal convolution
+    (conv_w [taps, channels], conv_b) of x | B | C with SiLU; dt [T, H] = softplus(row + dt_bias); decay [T, H] =
+    exp(-exp(A_log) dt), or its logarithm.  conv_state [slots, taps - 1, channels] is read and, with `write_state`, moved on."""
+    _cuda(proj, conv_w, conv_b, conv_state, A_log, dt_bias, xbc, decay, dt)
+    T = ctx.n_tokens
+    Cc, taps = _ssm_check(proj, conv_w, conv_state, H, G, N, V, T)
+    _ssm_vectors(H, A_log=A_log, dt_bias=dt_bias)
+    _need(conv_b.dtype == torch.float32 and conv_b.is_contiguous() and conv_b.numel() == Cc and xbc.is_contiguous()
+          and xbc.shape[-1] == Cc and xbc.numel() >= T * Cc, "ssm_prepare: conv_b [channels], xbc [T, channels]")
+    for t in (decay, dt):
+        _need(t.dtype == torch.float32 and t.is_contiguous() and t.numel() >= T * H, "ssm_prepare: decay, dt float32 [T, H]")
+    _i32(ctx.tok_seq, T, "tok_seq")
+    _i32(ctx.cu_q, ctx.n_seqs + 1, "cu_q")
+    _i32(ctx.slots, ctx.n_seqs, "slots")
+    _check(_lib("state_space").ab_ssm_prepare(
+        _p(proj), proj.shape[1], _p(conv_w), _p(conv_b), _p(conv_state), _p(A_log), _p(dt_bias), _p(xbc), _dt(xbc), _p(decay),
+        _p(dt), 1 if log_decay else 0, _p(ctx.tok_seq), _p(ctx.cu_q), _p(ctx.slots), T, ctx.n_seqs, H, G, N, V, taps,
+        1 if write_state else 0, _stream()), "ssm_prepare", kernels=2 if write_state and taps > 1 else 1)
+
+
+def ssm_step_supports(N, V) -> bool:
+    return _lib("state_space").ab_ssm_step_supports(N, V) == 1
+
+
+def ssm_step(proj, conv_w, conv_b, conv_state, A_log, dt_bias, skip, state, y, ctx, H, G, N, V, write_state=True):
+    """A step of one token per sequence: convolution, step size, decay, S <- a S + dt B x^T and y = S^T C + skip x in one
+    kernel; state float32 [slots, H, N, V], y float32 [T, H * V].  conv_state is left to `ssm_gate_norm`."""
+    _cuda(proj, conv_w, conv_b, conv_state, A_log, dt_bias, skip, state, y)
+    T = ctx.n_tokens
+    _need(ctx.is_decode, "ssm_step: one token per sequence")
+    Cc, taps = _ssm_check(proj, conv_w, conv_state, H, G, N, V, T)
+    _ssm_vectors(H, A_log=A_log, dt_bias=dt_bias, skip=skip)
+    _need(conv_b.dtype == torch.float32 and conv_b.is_contiguous() and conv_b.numel() == Cc, "ssm_step: conv_b [channels]")
+    _need(state.dtype == torch.float32 and state.is_contiguous() and tuple(state.shape[1:]) == (H, N, V)
+          and y.dtype == torch.float32 and y.is_contiguous() and y.shape[-1] == H * V and y.numel() >= T * H * V,
+          "ssm_step: state float32 [slots, H, N, V], y float32 [T, H * V]")
+    _i32(ctx.tok_seq, T, "tok_seq")
+    _i32(ctx.slots, ctx.n_seqs, "slots")
+    cols = 64
+    while cols > 16 and (cols >= 2 * V or T * H * -(-V // cols) < 2 * _sm_count(y.device)):
+        cols //= 2
+    _check(_lib("state_space").ab_ssm_step(
+        _p(proj), proj.shape[1], _p(conv_w), _p(conv_b), _p(conv_state), _p(A_log), _p(dt_bias), _p(skip), _p(state), _p(y),
+        _p(ctx.tok_seq), _p(ctx.slots), T, H, G, N, V, taps, cols, 1 if write_state else 0, _stream()), "ssm_step")
+    return y
+
+
+def ssm_chunks_supports(N, V, H, G) -> bool:
+    """Whether `ssm_chunks` takes the sizes (its rows must start on 16 bytes)."""
+    return _lib("state_space").ab_ssm_chunks_supports(N, V) == 1 and (H * V) % 8 == 0 and (G * N) % 8 == 0
+
+
+def ssm_chunks(xbc, log_decay, dt, skip, state, y, ctx, H, G, N, V, write_state=True):
+    """The recurrence over many tokens, 64 at a time on the tensor cores: xbc bfloat16 [T, x | B | C], log_decay and dt float32
+    [T, H]; state float32 [slots, H, N, V] is carried on, y float32 [T, H * V]."""
+    _cuda(xbc, log_decay, dt, skip, state, y)
+    T = ctx.n_tokens
+    _need(ssm_chunks_supports(N, V, H, G), f"ssm_chunks: state {N}, values {V} not supported")
+    _need(xbc.dtype == torch.bfloat16 and xbc.is_contiguous() and xbc.shape[-1] == H * V + 2 * G * N and xbc.shape[0] >= T,
+          "ssm_chunks: xbc bfloat16 [T, x | B | C]")
+    for t in (log_decay, dt):
+        _need(t.dtype == torch.float32 and t.is_contiguous() and t.numel() >= T * H, "ssm_chunks: log_decay, dt float32 [T, H]")
+    _ssm_vectors(H, skip=skip)
+    _need(state.dtype == torch.float32 and state.is_contiguous() and tuple(state.shape[1:]) == (H, N, V)
+          and y.dtype == torch.float32 and y.is_contiguous() and y.shape[-1] == H * V and y.numel() >= T * H * V,
+          "ssm_chunks: state float32 [slots, H, N, V], y float32 [T, H * V]")
+    _i32(ctx.cu_q, ctx.n_seqs + 1, "cu_q")
+    _i32(ctx.slots, ctx.n_seqs, "slots")
+    cols = 32 if V > 16 else 16
+    _check(_lib("state_space").ab_ssm_chunks(_p(xbc), _p(log_decay), _p(dt), _p(skip), _p(state), _p(y), _p(ctx.cu_q),
+                                             _p(ctx.slots), ctx.n_seqs, H, G, N, V, cols, 1 if write_state else 0, _stream()),
+           "ssm_chunks")
+    return y
+
+
+def ssm_gate_norm(y, proj, weight, parts, eps, out, ctx, H, G, N, V, taps, conv_state=None):
+    """out = cast(u / rms(u) * weight), u = y silu(z), in `parts` equal parts of the H * V columns, each by its own root mean
+    square; z stands at the start of the projected rows.  `conv_state`: after `ssm_step`, the kept inputs to move on."""
+    _cuda(y, proj, weight, out, conv_state)
+    T = ctx.n_tokens
+    inner = H * V
+    _need(parts > 0 and inner % parts == 0, f"ssm_gate_norm: {inner} columns in {parts} parts")
+    _need(y.dtype == torch.float32 and y.is_contiguous() and y.shape[-1] == inner and y.numel() >= T * inner
+          and proj.dtype == torch.float32 and proj.is_contiguous() and proj.shape[0] >= T and proj.shape[1] >= 2 * inner + 2 * G * N
+          and weight.dtype == torch.float32 and weight.is_contiguous() and weight.numel() == inner and out.is_contiguous()
+          and out.shape[-1] == inner and out.numel() >= T * inner, "ssm_gate_norm: y, out [T, H * V], weight [H * V]")
+    if conv_state is not None:
+        _need(ctx.is_decode and taps > 1 and conv_state.dtype == torch.float32 and conv_state.is_contiguous()
+              and tuple(conv_state.shape[1:]) == (taps - 1, inner + 2 * G * N),
+              "ssm_gate_norm: kept inputs are moved on in steps of one token per sequence")
+    _i32(ctx.tok_seq, T, "tok_seq")
+    _i32(ctx.slots, ctx.n_seqs, "slots")
+    _check(_lib("state_space").ab_ssm_gate_norm(
+        _p(y), _p(proj), proj.shape[1], _p(weight), _p(out), _dt(out), _p(conv_state), _p(ctx.tok_seq), _p(ctx.slots), T,
+        int(parts), ctypes.c_float(eps), H, G, N, V, taps, _stream()), "ssm_gate_norm")
     return out

@@ -64,8 +64,8 @@ class TokenEmbedding(Part):
         if norm is not None and (pairs is not None or self.scale != 1.0):
             raise ValueError(f"{name}: a normed embedding has no factor and no pair table")
         self.positions = positions
-        if positions is not None and (norm is not None or pairs is not None or self.scale != 1.0):
-            raise ValueError(f"{name}: an embedding with learned positions has no norm, factor or pair table")
+        if positions is not None and (norm is not None or pairs is not None):
+            raise ValueError(f"{name}: an embedding with learned positions has no norm or pair table")
 
     @property
     def needs_context(self) -> bool:
@@ -89,7 +89,7 @@ class TokenEmbedding(Part):
         if self.positions is not None:
             if ctx is None:
                 raise ValueError(f"{self.name}: the embedding needs the step's context")
-            return ops.embed_positions(self.weight, self.positions.weight, out, ctx)
+            return ops.embed_positions(self.weight, self.positions.weight, out, ctx, self.scale)
         if self.pairs is not None or self.scale != 1.0:
             if ctx is None or (self.pairs is not None and cache is None):
                 raise ValueError(f"{self.name}: the embedding needs the step's context (and the sequences' last tokens)")

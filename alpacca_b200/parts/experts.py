@@ -174,3 +174,75 @@ class TableExperts(FeedForward):
         out = torch.empty((h.shape[0], self.width), dtype=torch.float32, device=h.device)
         return ops.moe_shared_experts(h, self.gate_up, self.down, self.E, self.top, out, ctx, activation=self.activation,
                                       table=self.table, shared=self.shared_weights(), gate_logits=gate_logits)
+
+
+class ScoredExperts(FeedForward):
+    """Experts chosen by a router's scores, beside an optional shared expert that runs for every token.  The output is float32.
+
+        z = W_r h (32-bit);  s = score(z);  the `top` largest s are chosen, their weights are s as they are
+        (`renorm`: divided by their sum)
+        out = sum_k E_(e_k)(s_k h) + S(h)             `weight_in`: the weight multiplies the expert's input
+        out = sum_k s_k E_(e_k)(h) + S(h)             otherwise
+        E(h) = W_down act(W_up h), or with gates (`expert_names` of three) W_down (act(W_gate h) * (W_up h))
+
+    The experts' matrices are stacked, inner sizes padded with zero units to multiples of 16 (act(0) = 0); gates and
+    up-projections are interleaved in groups of 8 rows.  The kernels are those of `TableExperts`."""
+
+    def __init__(self, opts: BuildOptions, width: int, inner: int, n_experts: int, top: int, prefix: str, activation: str = "relu2",
+                 score: str = "sigmoid", renorm: bool = False, weight_in: bool = False, shared_inner: int = 0,
+                 router_name: str = "router", expert_names=("e{}.up", "e{}.down"), shared_names=("shared.up", "shared.down")):
+        if activation not in ops.MOE_ACTIVATIONS:
+            raise ValueError(f"activation must be one of {tuple(ops.MOE_ACTIVATIONS)}, got {activation!r}")
+        if score not in ("sigmoid", "logit"):
+            raise ValueError(f"{prefix}: score {score!r} is not one of this part's")
+        if not 0 < top <= n_experts:
+            raise ValueError(f"{prefix}: {top} of {n_experts} experts cannot be chosen")
+        if len(expert_names) != len(shared_names) or len(expert_names) not in (2, 3):
+            raise ValueError(f"{prefix}: experts have two matrices, or three with a gate, and the shared one likewise")
+        self.opts, self.width, self.inner, self.E, self.top = opts, int(width), int(inner), int(n_experts), int(top)
+        self.prefix, self.activation, self.score, self.renorm = prefix, activation, score, bool(renorm)
+        self.weight_in, self.shared_inner, self.gated = bool(weight_in), int(shared_inner), len(expert_names) == 3
+        self.router_name, self.expert_names, self.shared_names = router_name, expert_names, shared_names
+        self.router = self.up = self.down = self.shared_up = self.shared_down = None
+
+    def _specs_of(self, names, inner):
+        shapes = [(inner, self.width)] * (len(names) - 1) + [(self.width, inner)]
+        return [ParamSpec(f"{self.prefix}.{n}", s) for n, s in zip(names, shapes)]
+
+    def own_param_specs(self):
+        specs = [ParamSpec(f"{self.prefix}.{self.router_name}", (self.E, self.width), "vector", "normal")]
+        for e in range(self.E):
+            specs += self._specs_of([n.format(e) for n in self.expert_names], self.inner)
+        if self.shared_inner:
+            specs += self._specs_of(self.shared_names, self.shared_inner)
+        return specs
+
+    def load_own(self, fetch):
+        specs, n = self.own_param_specs(), len(self.expert_names)
+        self.router = fetch(specs[0])
+        ff = -(-self.inner // 16) * 16
+        for e in range(self.E):
+            up, down = self._laid_out(*(fetch(s) for s in specs[1 + n * e:1 + n * (e + 1)]))
+            if e == 0:
+                self.up = torch.empty((self.E, *up.shape), dtype=up.dtype, device=up.device)
+                self.down = torch.empty((self.E, *down.shape), dtype=down.dtype, device=down.device)
+            self.up[e], self.down[e] = up, down
+        self.up, self.down = self.up.view(-1, self.width), self.down.view(-1, ff)
+        if self.shared_inner:
+            self.shared_up, self.shared_down = self._laid_out(*(fetch(s) for s in specs[1 + n * self.E:]))
+
+    def _laid_out(self, *matrices):
+        """(gate|up in groups of 16 rows, or up; down), the inner size padded to a multiple of 16."""
+        *first, down = matrices
+        more = -down.shape[1] % 16
+        first = [torch.nn.functional.pad(w, (0, 0, 0, more)) for w in first]
+        if self.gated:
+            first = [torch.cat([w.view(-1, 8, self.width) for w in first], dim=1).reshape(-1, self.width)]
+        return first[0].contiguous(), torch.nn.functional.pad(down, (0, more)).contiguous()
+
+    def forward(self, h, ctx):
+        choice = ops.moe_route(h, self.router, ctx.n_tokens, 1, 1, self.top, 1.0, score=self.score, renorm=self.renorm)
+        out = torch.empty((h.shape[0], self.width), dtype=torch.float32, device=h.device)
+        shared = (self.shared_up, self.shared_down) if self.shared_inner else None
+        return ops.moe_shared_experts(h, self.up, self.down, self.E, self.top, out, ctx, activation=self.activation,
+                                      choice=choice, shared=shared, gated=self.gated, weight_in=self.weight_in)

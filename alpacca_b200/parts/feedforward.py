@@ -19,15 +19,15 @@ from .linear import Linear
 class SwiGLU(FeedForward):
     def __init__(self, opts: BuildOptions, width: int, inner: int, prefix: str, bias: bool = False,
                  names=("gate_proj", "up_proj", "down_proj"), weight_suffix: str = ".weight",
-                 out_dtype=None, activation: str = "silu"):
+                 out_dtype=None, activation: str = "silu", bias_suffix: str = ".bias"):
         if activation not in ops.GATE_ACTIVATIONS:
             raise ValueError(f"activation {activation!r} is not one of {tuple(ops.GATE_ACTIVATIONS)}")
         self.opts, self.width, self.inner, self.activation = opts, int(width), int(inner), activation
         g, u, d = names
         self.gate_up = Linear(opts, width, [(f"{prefix}.{g}", inner), (f"{prefix}.{u}", inner)], bias=bias,
-                              interleave8=True, weight_suffix=weight_suffix, pad_rows_to=8)
+                              interleave8=True, weight_suffix=weight_suffix, pad_rows_to=8, bias_suffix=bias_suffix)
         self.down = Linear(opts, inner, [(f"{prefix}.{d}", width)], bias=bias, weight_suffix=weight_suffix,
-                           out_dtype=out_dtype, pad_in_to=8)
+                           out_dtype=out_dtype, pad_in_to=8, bias_suffix=bias_suffix)
 
     adds_to_residual = True
 

@@ -33,6 +33,11 @@ Options, each a constructor argument:
                      vectors, with weights of those sizes (tensors `<prefix>.<q>.norm` [H*M*dim], `<prefix>.<k>.norm`)
     distance         names of two tensors [H], r1 and r2: r1_h ln(1 + r2_h (p - s)) is taken off each scaled score (Chi et
                      al., "KERPLE: Kernelized Relative Positional Embedding for Length Extrapolation")
+    softcap          a scaled score becomes softcap * tanh(score / softcap), before any penalty on distance
+    slopes           H numbers: slope_h (p - s) is taken off each scaled (and bounded) score (Press et al., "Train Short, Test
+                     Long: Attention with Linear Biases Enables Input Length Extrapolation"); `alibi_slopes(H)` gives
+                     2^(-8 (h + 1) / H)
+    fixed_sink       a sink whose logit is this number in every head (no tensor): 0 adds one to every denominator
     own_kv           off: the layer has no W_k and W_v (nor a key norm); it reads the keys, as cached, and values of another
                      layer with the same key/value heads and sizes (the schedule's run names that layer's run), with its
                      own queries, window and penalty
@@ -56,6 +61,11 @@ from .base import BuildOptions, KVSpec, Mixer, PositionEncoding
 from .linear import Linear
 
 
+def alibi_slopes(n_heads: int) -> list[float]:
+    """A slope per head, 2^(-8 (h + 1) / n_heads)."""
+    return [2.0 ** (-8.0 * (h + 1) / n_heads) for h in range(n_heads)]
+
+
 class MapsAttention(Mixer):
     def __init__(self, opts: BuildOptions, width: int, n_heads: int, n_kv_heads: int, dim: int, vdim: int | None,
                  position: PositionEncoding | None, prefix: str, scale: float, eps: float, window: int | None = None,
@@ -64,7 +74,8 @@ class MapsAttention(Mixer):
                  weight_suffix: str = "", bias_suffix: str = ".b", out_dtype=None, qk_norm_weight: bool = True,
                  value_norm: bool = False, head_mix: str | None = None, gate: str | None = None,
                  head_gate: str | None = None, qk_norm_rows: bool = False, distance: tuple | None = None,
-                 own_kv: bool = True, keep_window: int | str | None = None):
+                 own_kv: bool = True, keep_window: int | str | None = None, softcap: float | None = None,
+                 slopes=None, fixed_sink: float | None = None):
         if n_heads % n_kv_heads:
             raise ValueError(f"{prefix}: {n_heads} heads cannot share {n_kv_heads} key/value heads")
         self.opts, self.prefix = opts, prefix
@@ -105,6 +116,19 @@ class MapsAttention(Mixer):
             raise ValueError(f"{prefix}: a layer that reads another layer's keys has a query norm over whole rows")
         if distance is not None and head_mix is not None:
             raise ValueError(f"{prefix}: a penalty on distance does not go with mixed heads")
+        if fixed_sink is not None and (sink or head_mix is not None):
+            raise ValueError(f"{prefix}: a sink is learned or fixed, and does not go with mixed heads")
+        if (softcap is not None or slopes is not None) and (head_mix is not None or distance is not None):
+            raise ValueError(f"{prefix}: bounded scores and slopes go neither with mixed heads nor with another penalty on distance")
+        if softcap is not None and not softcap > 0:
+            raise ValueError(f"{prefix}: the scores' bound must be positive, got {softcap}")
+        if slopes is not None and len(slopes) != n_heads:
+            raise ValueError(f"{prefix}: {len(slopes)} slopes for {n_heads} heads")
+        self.bound = None
+        if softcap is not None or slopes is not None:
+            self.bound = (torch.tensor([0.0] * n_heads if slopes is None else [float(x) for x in slopes],
+                                       dtype=torch.float32, device=opts.device), float(softcap or 0.0))
+        self.fixed_sink = None if fixed_sink is None else float(fixed_sink)
         self.scale, self.eps = float(scale), float(eps)
         self.position, self.qk_norm, self.has_sink = position, bool(qk_norm), bool(sink)
         self.difference = None if difference is None else float(difference)
@@ -172,6 +196,8 @@ class MapsAttention(Mixer):
             self.talk = got[self.head_mix].contiguous()
         if self.has_sink:
             self.sink = got["sink"]
+        elif self.fixed_sink is not None:
+            self.sink = torch.full((self.H,), self.fixed_sink, dtype=torch.float32, device=self.opts.device)
         if self.distance is not None:
             self.penalty = torch.stack([got[n] for n in self.distance]).contiguous()
 
@@ -221,7 +247,7 @@ class MapsAttention(Mixer):
         attend = ops.attention_maps_mma if self._on_tensor_cores(buf) else ops.attention_maps
         attend(buf, buf.shape[-1], att, cache, ctx, self.H, self.G, self.M, self.Dk, self.Dv, self.scale,
                self.window or 0, self.sink, coef=self.coef, unit_norm=unit, eps=self.eps,
-               out_scale=(1.0 - self.difference) if unit else 1.0, dist=self.penalty)
+               out_scale=(1.0 - self.difference) if unit else 1.0, dist=self.penalty, bound=self.bound)
         if self.head_gate is not None:
             ops.head_gate(att, buf.reshape(-1)[self.gate_offset:], buf.shape[-1], T, self.H, self.Dv)
         # after a kernel that fills the processors' shared memory the product starts when that kernel has ended

@@ -7,7 +7,10 @@ float32, when the weight is loaded.  With `scalar` the checkpoint keeps ONE numb
 for all columns (a tensor without dimensions); it is spread over the width when it
 is loaded, so every kernel that takes a weight per column serves it.  `scale`
 multiplies the weight once at load (a constant factor on what reads the norm, such
-as a factor on the logits after the last norm).
+as a factor on the logits after the last norm).  `columns` names a second tensor
+[width] that multiplies the norm's result column by column (a layer scale on a
+sub-layer's output, Touvron et al., "Going deeper with Image Transformers"); it is
+taken into the weight at load, in float32.
 """
 from __future__ import annotations
 
@@ -20,15 +23,18 @@ from .base import BuildOptions, Norm
 
 class RMSNorm(Norm):
     def __init__(self, opts: BuildOptions, width: int, eps: float, name: str, weight_suffix: str = ".weight",
-                 unit_offset: bool = False, scalar: bool = False, scale: float = 1.0):
+                 unit_offset: bool = False, scalar: bool = False, scale: float = 1.0,
+                 columns: str | None = None):
         self.opts, self.width, self.eps, self.name = opts, int(width), float(eps), name
         self.weight_suffix, self.unit_offset = weight_suffix, bool(unit_offset)
         self.scalar, self.scale = bool(scalar), float(scale)
+        self.columns = columns
         self.weight = None
 
     def own_param_specs(self):
+        more = [ParamSpec(self.columns, (self.width,), "vector", "one_plus_normal")] if self.columns is not None else []
         return [ParamSpec(f"{self.name}{self.weight_suffix}", () if self.scalar else (self.width,), "vector",
-                          "normal" if self.unit_offset else "one_plus_normal")]
+                          "normal" if self.unit_offset else "one_plus_normal")] + more
 
     def load_own(self, fetch):
         self.weight = fetch(self.own_param_specs()[0])
@@ -36,6 +42,8 @@ class RMSNorm(Norm):
             self.weight = self.weight.reshape(1).expand(self.width).contiguous()
         if self.unit_offset:
             self.weight = (self.weight + 1.0).contiguous()
+        if self.columns is not None:
+            self.weight = (self.weight * fetch(self.own_param_specs()[1])).contiguous()
         if self.scale != 1.0:
             self.weight = (self.weight * self.scale).contiguous()
 
