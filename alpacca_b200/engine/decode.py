@@ -161,9 +161,10 @@ class GraphDecoder:
                            sh.history, sh.counter, sh.rows, host_ring=sh.host_ring)
 
     def _capture(self, sh: _Shape):
-        # with every row marked as padding the step touches neither cache nor counters, so the
-        # warm-up run that must precede a capture is harmless
+        # with every row marked as padding the step touches neither cache nor states nor counters, so the
+        # warm-up run that must precede a capture is harmless (recurrences go by the slots, not by tok_seq)
         sh.d("tok_seq").fill_(-1)
+        sh.d("slots").fill_(-1)
         sh.d("cu_q").copy_(torch.arange(sh.rows + 1, dtype=torch.int32))
         sh.d("want_rows").copy_(torch.arange(sh.rows, dtype=torch.int32))
         sh.d("row_order").copy_(torch.arange(sh.rows, dtype=torch.int32))

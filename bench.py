@@ -551,7 +551,7 @@ def run_reference(args):
 
 
 # ---------------------------------------------------------------------------------------------------------
-# --design lefatar | buguzen | sazepel | mavidra | ponusun: that decoder beside the Llama decoder of the same width, depth and dense
+# --design lefatar | buguzen | sazepel | mavidra | ponusun | nagavik: that decoder beside the Llama decoder of the same width, depth and dense
 # feed-forward, at sizes that resemble a real model's layers (random weights).
 
 def _lefatar_layers(E, mlstm, latent, dense_ff, moe, n_layers):
@@ -672,6 +672,21 @@ def _ponusun_config(z):
             "canon": {"taps": 4}, "logit_softcap": 30.0, "layers": layers}
 
 
+def _nagavik_config(z):
+    """Eight layers, every fourth one attention with bounded scores and slopes, the others state-space mixers of twice the
+    width; a dense feed-forward in the first layer, then ungated experts of the inner size of the other decoders' beside a
+    shared one of twice that size."""
+    rt = z["moe"]["router"]
+    ff = z["moe"]["expert"]["ff"]
+    moe = {"kind": "moe", "expert": {"ff": ff}, "router": {"experts": rt["experts"], "top": rt["top"]}, "shared": {"ff": 2 * ff}}
+    ssm = {"type": "mamba2", "mixer": {"heads": z["width"] // 32, "vdim": 64, "state": 128, "groups": 4, "conv": 4, "norm_groups": 4}}
+    att = {"type": "attention", "mixer": {"heads": z["heads"], "kv_heads": z["kv_heads"], "dim": z["head_dim"], "vdim": z["head_dim"],
+                                          "scale": z["head_dim"] ** -0.5, "softcap": 20.0}}
+    layers = [dict(att if i % 4 == 3 else ssm, mlp=moe if i else {"kind": "dense", "ff": z["dense_ff"]}) for i in range(z["layers"])]
+    return {"architecture": "Nagavik", "vocab": z["vocab"], "width": z["width"], "max_positions": 8192, "norm": {"eps": 1e-6},
+            "embedding": {"scale": 4.0}, "logit_softcap": 30.0, "layers": layers}
+
+
 def design_configs(size, design="lefatar"):
     z = DESIGN_SIZES[size]
     llama = {"architectures": ["LlamaForCausalLM"], "num_hidden_layers": z["layers"], "hidden_size": z["width"],
@@ -689,6 +704,8 @@ def design_configs(size, design="lefatar"):
         return {"mavidra": _mavidra_config(z), "sazepel": _sazepel_config(z), "lefatar": lefatar, "llama": llama}
     if design == "ponusun":
         return {"ponusun": _ponusun_config(z), "sazepel": _sazepel_config(z), "buguzen": _buguzen_config(z), "llama": llama}
+    if design == "nagavik":
+        return {"nagavik": _nagavik_config(z), "mavidra": _mavidra_config(z), "ponusun": _ponusun_config(z), "llama": llama}
     return {"lefatar": lefatar, "llama": llama}
 
 
@@ -769,7 +786,7 @@ def main():
                     help="with --only decode: equal prompts of this many tokens instead of the workload's")
     ap.add_argument("--prefill-tokens", type=int, default=0,
                     help="with --only prefill: one prompt of this many tokens instead of the workload's")
-    ap.add_argument("--design", default="", choices=["", "lefatar", "buguzen", "sazepel", "mavidra", "ponusun"],
+    ap.add_argument("--design", default="", choices=["", "lefatar", "buguzen", "sazepel", "mavidra", "ponusun", "nagavik"],
                     help="instead of the benchmark workload: prefill and decode throughput of this design beside the "
                          "Llama decoder of the same width and depth (random weights), one JSON line")
     ap.add_argument("--size", default="", choices=[""] + sorted(DESIGN_SIZES), help="with --design: one size only")
