@@ -206,20 +206,12 @@ AB_API int ab_moe_route(const void* h, int dtype, int ld, const float* wr, int n
 //   Groups: a group's score is the sum of its `group_top` largest c; experts outside the `keep` best groups cannot be
 //   chosen whatever their c (choice scores may be negative, so they are struck out with minus infinity).
 // The lower index wins a tie, among groups and among experts.
-__global__ void moe_route_scores_kernel(const float* __restrict__ z, const float* __restrict__ correction, int n_tokens,
-                                        int E, int groups, int keep, int group_top, int top, int score_fn, int renorm,
-                                        float scale, int* __restrict__ idx, float* __restrict__ wts) {
-  extern __shared__ float sm[];           // per warp: E scores, E choice scores, `groups` group scores
-  pdl_wait();
-  pdl_trigger();
-  const int lane = threadIdx.x & 31, wib = threadIdx.x >> 5;
-  const int t = blockIdx.x * (blockDim.x >> 5) + wib;
-  if (t >= n_tokens) return;
-  float* s = sm + (size_t)wib * (2 * E + groups);
-  float* c = s + E;
-  float* gs = c + E;
+// (one token, by one warp: z its logits, s, c, gs scratch of E, E and `groups` numbers, idx and wts its `top` choices)
+__device__ __forceinline__ void choose_by_scores(const float* z, const float* __restrict__ correction, int E, int groups, int keep,
+                                                 int group_top, int top, int score_fn, int renorm, float scale, float* s, float* c,
+                                                 float* gs, int* __restrict__ idx, float* __restrict__ wts, int lane) {
   for (int e = lane; e < E; e += 32) {
-    const float v = z[(size_t)t * E + e];
+    const float v = z[e];
     const float sc = score_fn == 1 ? 1.0f / (1.0f + expf(-v)) : v;
     s[e] = sc;
     c[e] = sc + (correction != nullptr ? correction[e] : 0.f);
@@ -280,8 +272,8 @@ __global__ void moe_route_scores_kernel(const float* __restrict__ z, const float
     const float w = s[be];
     chosen_sum += w;
     if (lane == 0) {
-      idx[(size_t)t * top + pick] = be;
-      wts[(size_t)t * top + pick] = w;
+      idx[pick] = be;
+      wts[pick] = w;
     }
     __syncwarp();
     if (lane == 0) c[be] = -INFINITY;                  // taken
@@ -289,18 +281,71 @@ __global__ void moe_route_scores_kernel(const float* __restrict__ z, const float
   }
   if (lane == 0) {
     const float f = renorm ? scale / (chosen_sum + 1e-20f) : scale;
-    for (int j = 0; j < top; ++j) wts[(size_t)t * top + j] *= f;
+    for (int j = 0; j < top; ++j) wts[j] *= f;
   }
+}
+
+__global__ void moe_route_scores_kernel(const float* __restrict__ z, const float* __restrict__ correction, int n_tokens,
+                                        int E, int groups, int keep, int group_top, int top, int score_fn, int renorm,
+                                        float scale, int* __restrict__ idx, float* __restrict__ wts) {
+  extern __shared__ float sm[];           // per warp: E scores, E choice scores, `groups` group scores
+  pdl_wait();
+  pdl_trigger();
+  const int lane = threadIdx.x & 31, wib = threadIdx.x >> 5;
+  const int t = blockIdx.x * (blockDim.x >> 5) + wib;
+  if (t >= n_tokens) return;
+  float* s = sm + (size_t)wib * (2 * E + groups);
+  choose_by_scores(z + (size_t)t * E, correction, E, groups, keep, group_top, top, score_fn, renorm, scale, s, s + E, s + 2 * E,
+                   idx + (size_t)t * top, wts + (size_t)t * top, lane);
+}
+
+// Logits and choice of a few tokens in one kernel: a block per token, a warp per expert in turn; the router's rows are asked
+// of the L2 before the wait.
+template <typename T, typename TW>
+__global__ void __launch_bounds__(512)
+moe_route_small_kernel(const T* __restrict__ h, int ld, const TW* __restrict__ wr, const float* __restrict__ bias,
+                       const float* __restrict__ correction, int width, int E, int groups, int keep, int group_top, int top,
+                       int score_fn, int renorm, float scale, int* __restrict__ idx, float* __restrict__ wts) {
+  extern __shared__ float sm[];           // E logits, E scores, E choice scores, `groups` group scores
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, t = blockIdx.x;
+  const char* rows = reinterpret_cast<const char*>(wr);
+  for (size_t at = (size_t)threadIdx.x * 128; at < (size_t)E * width * sizeof(TW); at += (size_t)blockDim.x * 128)
+    asm volatile("prefetch.global.L2 [%0];" ::"l"(rows + at));
+  pdl_wait();
+  pdl_trigger();
+  for (int e = warp; e < E; e += blockDim.x >> 5) {
+    const float part = warp_sum(lane_dot(h + (size_t)t * ld, wr + (size_t)e * width, width, lane));
+    if (lane == 0) sm[e] = part + (bias != nullptr ? bias[e] : 0.f);
+  }
+  __syncthreads();
+  if (warp == 0)
+    choose_by_scores(sm, correction, E, groups, keep, group_top, top, score_fn, renorm, scale, sm + E, sm + 2 * E, sm + 3 * E,
+                     idx + (size_t)t * top, wts + (size_t)t * top, lane);
+}
+
+static bool route_ok(int E, int groups, int keep, int group_top, int top, int score_fn) {
+  return E > 0 && E <= MOE_MAX_EXPERTS && groups > 0 && E % groups == 0 && keep > 0 && keep <= groups && top > 0 &&
+         top <= keep * (E / groups) && group_top > 0 && !(keep < groups && E / groups > 128) && score_fn >= 0 && score_fn <= 1;
+}
+
+// The choice of every token from its logits z [T, E].
+AB_API int ab_moe_route_logits(const float* z, const float* correction, int n_tokens, int E, int groups, int keep, int group_top,
+                               int top, int score_fn, int renorm, float scale, int* idx, float* wts, cudaStream_t stream) {
+  if (n_tokens <= 0) return AB_OK;
+  if (!route_ok(E, groups, keep, group_top, top, score_fn)) return AB_BAD_ARG;
+  const int wpb = 4;
+  const unsigned blocks = (unsigned)((n_tokens + wpb - 1) / wpb);
+  const size_t smem = (size_t)wpb * (2 * E + groups) * sizeof(float);
+  ab_launch(moe_route_scores_kernel, dim3(blocks), dim3(wpb * 32), smem, stream, z, correction, n_tokens, E, groups, keep, group_top,
+            top, score_fn, renorm, scale, idx, wts);
+  return ab_launch_status();
 }
 
 AB_API int ab_moe_route_scores(const void* h, int dtype, int ld, const float* wr, const float* bias, const float* correction,
                                int n_tokens, int width, int E, int groups, int keep, int group_top, int top, int score_fn,
                                int renorm, float scale, float* z, int* idx, float* wts, cudaStream_t stream) {
   if (n_tokens <= 0) return AB_OK;
-  if (E <= 0 || E > MOE_MAX_EXPERTS || groups <= 0 || E % groups || keep <= 0 || keep > groups || top <= 0 ||
-      top > keep * (E / groups) || group_top <= 0 || (keep < groups && E / groups > 128) || score_fn < 0 || score_fn > 1)
-    return AB_BAD_ARG;
-  const int wpb = 4;
+  if (!route_ok(E, groups, keep, group_top, top, score_fn)) return AB_BAD_ARG;
   const long long lw = (long long)n_tokens * E;
   const unsigned lblocks = (unsigned)((lw + 7) / 8);
   if (dtype == AB_F32)
@@ -311,13 +356,26 @@ AB_API int ab_moe_route_scores(const void* h, int dtype, int ld, const float* wr
     return AB_BAD_ARG;
   int rc = ab_launch_status();
   if (rc) return rc;
-  const unsigned blocks = (unsigned)((n_tokens + wpb - 1) / wpb);
-  const size_t smem = (size_t)wpb * (2 * E + groups) * sizeof(float);
-  ab_launch(moe_route_scores_kernel, dim3(blocks), dim3(wpb * 32), smem, stream, (const float*)z, correction, n_tokens, E,
-            groups, keep, group_top, top, score_fn, renorm, scale, idx, wts);
-  return ab_launch_status();
+  return ab_moe_route_logits(z, correction, n_tokens, E, groups, keep, group_top, top, score_fn, renorm, scale, idx, wts, stream);
 }
 
+// Both in one kernel, for a few tokens; wr of wr_dtype (bfloat16 with bfloat16 rows of h only).
+AB_API int ab_moe_route_small(const void* h, int dtype, int ld, const void* wr, int wr_dtype, const float* bias,
+                              const float* correction, int n_tokens, int width, int E, int groups, int keep, int group_top, int top,
+                              int score_fn, int renorm, float scale, int* idx, float* wts, cudaStream_t stream) {
+  if (n_tokens <= 0) return AB_OK;
+  if (!route_ok(E, groups, keep, group_top, top, score_fn) || width <= 0) return AB_BAD_ARG;
+  const size_t smem = (size_t)(3 * E + groups) * sizeof(float);
+#define AB_GO(T, TW)                                                                                                   \
+  ab_launch(moe_route_small_kernel<T, TW>, dim3((unsigned)n_tokens), dim3(512), smem, stream, (const T*)h, ld, (const TW*)wr, bias, \
+            correction, width, E, groups, keep, group_top, top, score_fn, renorm, scale, idx, wts)
+  if (dtype == AB_F32 && wr_dtype == AB_F32) AB_GO(float, float);
+  else if (dtype == AB_BF16 && wr_dtype == AB_F32) AB_GO(bf16, float);
+  else if (dtype == AB_BF16 && wr_dtype == AB_BF16) AB_GO(bf16, bf16);
+  else return AB_BAD_ARG;
+#undef AB_GO
+  return ab_launch_status();
+}
 
 // act[p, j] = f(W_up[e_p][j] . h[t_p]) for pair p = t * top + k, or, gated (w_gate given),
 // f(W_gate[e_p][j] . h[t_p]) * (W_up[e_p][j] . h[t_p]).  One warp per (pair, j).

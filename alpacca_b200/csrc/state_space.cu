@@ -333,19 +333,37 @@ AB_API int ab_ssm_step(const float* proj, int ld, const float* conv_w, const flo
 // A block per (token, part): out = cast(u / rms(u) * w), u = y silu(z), over the part's n numbers.  NV > 0: n and the row
 // strides are multiples of 4 and the part fits NV quads per thread; NV = 0: any size, u formed twice.
 // `conv_state` (or null): the token's convolution inputs become the newest of what its sequence keeps (one token per
-// sequence; the blocks of a token share the channels).
+// sequence), by the blocks behind a token's parts.  What is asked for before the wait is older than the kernel before.
 template <typename TO, int NV>
 __global__ void __launch_bounds__(512)
 ssm_gate_norm_kernel(const float* __restrict__ y, const float* __restrict__ proj, int ld, const float* __restrict__ w,
                      TO* __restrict__ out, float* __restrict__ conv_state, const int* __restrict__ tok_seq,
-                     const int* __restrict__ slots, int n, float eps, SsmSizes z) {
+                     const int* __restrict__ slots, int n, float eps, int parts, SsmSizes z) {
   __shared__ float scratch[32];
   const int t = blockIdx.x, base = blockIdx.y * n;
-  pdl_wait();
-  pdl_trigger();
   const int b = tok_seq[t];
+  if ((int)blockIdx.y >= parts) {
+    const int Cc = z.channels(), keep = z.taps - 1, c = ((int)blockIdx.y - parts) * blockDim.x + threadIdx.x;
+    float* held = conv_state + (b < 0 ? 0 : (size_t)slots[b] * keep * Cc) + c;
+    float now[SSM_MAX_TAPS - 1];
+    if (b >= 0 && c < Cc) {
+#pragma unroll
+      for (int s = 0; s < SSM_MAX_TAPS - 1; ++s)
+        if (s < keep) now[s] = s + 1 < keep ? held[(size_t)(s + 1) * Cc] : proj[(size_t)t * ld + z.off_x() + c];
+    }
+    pdl_wait();
+    pdl_trigger();
+    if (b >= 0 && c < Cc) {
+#pragma unroll
+      for (int s = 0; s < SSM_MAX_TAPS - 1; ++s)
+        if (s < keep) held[(size_t)s * Cc] = now[s];
+    }
+    return;
+  }
   TO* o = out + (size_t)t * z.inner() + base;
   if (b < 0) {
+    pdl_wait();
+    pdl_trigger();
     for (int j = threadIdx.x; j < n; j += blockDim.x) o[j] = from_f32<TO>(0.f);
     return;
   }
@@ -354,17 +372,28 @@ ssm_gate_norm_kernel(const float* __restrict__ y, const float* __restrict__ proj
   const float* wr = w + base;
   float ss = 0.f;
   if (NV > 0) {
-    Lanes<4> u[NV > 0 ? NV : 1], wv[NV > 0 ? NV : 1];
+    Lanes<4> u[NV > 0 ? NV : 1], wv[NV > 0 ? NV : 1], gv[NV > 0 ? NV : 1];
 #pragma unroll
     for (int k = 0; k < NV; ++k) {
       const int j = (threadIdx.x + k * blockDim.x) * 4;
       if (j < n) {
-        u[k] = load_lanes<4>(yr + j);
-        const Lanes<4> g = load_lanes<4>(zr + j);
+        gv[k] = load_lanes<4>(zr + j);
         wv[k] = load_lanes<4>(wr + j);
+      }
+    }
+    pdl_wait();
+    pdl_trigger();
+#pragma unroll
+    for (int k = 0; k < NV; ++k) {
+      const int j = (threadIdx.x + k * blockDim.x) * 4;
+      if (j < n) u[k] = load_lanes<4>(yr + j);
+    }
+#pragma unroll
+    for (int k = 0; k < NV; ++k) {
+      if ((threadIdx.x + k * blockDim.x) * 4 < n) {
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
-          u[k].v[e] *= ssm_silu(g.v[e]);
+          u[k].v[e] *= ssm_silu(gv[k].v[e]);
           ss += u[k].v[e] * u[k].v[e];
         }
       }
@@ -381,6 +410,8 @@ ssm_gate_norm_kernel(const float* __restrict__ y, const float* __restrict__ proj
       }
     }
   } else {
+    pdl_wait();
+    pdl_trigger();
     for (int j = threadIdx.x; j < n; j += blockDim.x) {
       const float u = yr[j] * ssm_silu(zr[j]);
       ss += u * u;
@@ -389,15 +420,6 @@ ssm_gate_norm_kernel(const float* __restrict__ y, const float* __restrict__ proj
     const float inv = 1.0f / sqrtf(ss / (float)n + eps);
     for (int j = threadIdx.x; j < n; j += blockDim.x) o[j] = from_f32<TO>(yr[j] * ssm_silu(zr[j]) * (inv * wr[j]));
   }
-  if (conv_state != nullptr) {
-    const int Cc = z.channels(), keep = z.taps - 1;
-    float* held = conv_state + (size_t)slots[b] * keep * Cc;
-    const float* x = proj + (size_t)t * ld + z.off_x();
-    for (int c = blockIdx.y * blockDim.x + threadIdx.x; c < Cc; c += gridDim.y * blockDim.x) {
-      for (int s = 0; s + 1 < keep; ++s) held[(size_t)s * Cc + c] = held[(size_t)(s + 1) * Cc + c];
-      held[(size_t)(keep - 1) * Cc + c] = x[c];
-    }
-  }
 }
 
 AB_API int ab_ssm_gate_norm(const float* y, const float* proj, int ld, const float* w, void* out, int out_dtype,
@@ -405,16 +427,17 @@ AB_API int ab_ssm_gate_norm(const float* y, const float* proj, int ld, const flo
                             int H, int G, int N, int V, int taps, cudaStream_t stream) {
   if (n_tokens <= 0) return AB_OK;
   const SsmSizes z{H, G, N, V, taps};
-  if (!ssm_sizes_ok(z) || parts <= 0 || z.inner() % parts || parts > 65535 || (taps == 1 && conv_state)) return AB_BAD_ARG;
+  if (!ssm_sizes_ok(z) || parts <= 0 || z.inner() % parts || parts > 32767 || (taps == 1 && conv_state)) return AB_BAD_ARG;
   const int n = z.inner() / parts;
   auto al = [](const void* p) { return ((uintptr_t)p & 15) == 0; };
   const bool vec = n % 4 == 0 && ld % 4 == 0 && al(y) && al(proj) && al(w) && al(out) && n <= 512 * 4 * 4;
   const int threads = n >= 4096 ? 512 : n >= 1024 ? 256 : n >= 256 ? 128 : 64;
   const int nv = vec ? (n / 4 + threads - 1) / threads : 0;
-  const dim3 grid((unsigned)n_tokens, (unsigned)parts);
+  const int movers = conv_state != nullptr ? (z.channels() + threads - 1) / threads : 0;
+  const dim3 grid((unsigned)n_tokens, (unsigned)(parts + movers));
 #define AB_GO(TO, NV)                                                                                                  \
   ab_launch(ssm_gate_norm_kernel<TO, NV>, grid, dim3(threads), 0, stream, y, proj, ld, w, (TO*)out, conv_state, tok_seq, slots, \
-            n, eps, z)
+            n, eps, parts, z)
 #define AB_NV(TO)                                                                                                      \
   { if (nv == 0) AB_GO(TO, 0); else if (nv == 1) AB_GO(TO, 1); else if (nv == 2) AB_GO(TO, 2); else AB_GO(TO, 4); }
   if (out_dtype == AB_F32) AB_NV(float)
@@ -433,9 +456,6 @@ AB_API int ab_ssm_gate_norm(const float* y, const float* proj, int ld, const flo
 __device__ __forceinline__ void sc_async16(void* dst, const void* src) {
   asm volatile("cp.async.cg.shared.global [%0], [%1], 16;\n" ::"r"(smem_u32(dst)), "l"(src));
 }
-__device__ __forceinline__ void sc_async4(void* dst, const void* src) {
-  asm volatile("cp.async.ca.shared.global [%0], [%1], 4;\n" ::"r"(smem_u32(dst)), "l"(src));
-}
 // v = hi + lo up to 2^-17: two bfloat16 numbers each
 __device__ __forceinline__ void split2(float a, float b, uint32_t& hi, uint32_t& lo) {
   hi = pack_bf16(a, b);
@@ -444,21 +464,29 @@ __device__ __forceinline__ void split2(float a, float b, uint32_t& hi, uint32_t&
 
 template <int CV> struct ChunkSmem {
   static constexpr int PV = CV + 8;                      // pitch of rows of value columns
-  // float offsets are kept in bytes; N is the state size
   __host__ __device__ static size_t bc(int N) { return (size_t)SC_T * (N + 8) * 2; }      // one buffer of B or C
   __host__ __device__ static size_t total(int N) {
-    return 4 * bc(N) + 2 * (size_t)SC_T * PV * 2 + 2 * (size_t)N * PV * 2 + 2 * (size_t)SC_T * PV * 2 +
-           (size_t)SC_T * (CV + 4) * 4 + 4 * SC_T * 4 + 4 * SC_T * 4 + 16;
+    return 4 * bc(N) + 2 * (size_t)SC_T * PV * 2 + 2 * (size_t)N * PV * 2 + 2 * (size_t)SC_T * PV * 2 + 2 * (4 * SC_T + 4) * 4;
   }
 };
 
-// RT: row tiles of S (16 rows) per warp; eight warps cover N <= 128 * RT rows.
+// What a chunk's step sizes and log decays come to, in powers of two: L_t, the running sum of the log decays (times log2 e).
+struct ChunkScales {
+  float L[SC_T];          // L_t
+  float q[SC_T];          // L_s - log2 dt_s: a key's score is multiplied by 2^(L_t - q_s)
+  float e[SC_T];          // 2^(L_t)
+  float w[SC_T];          // 2^(L_end - L_s) dt_s
+  float end[4];           // 2^(L_end)
+};
+
+// Eight warps: warp w takes the 16 tokens from 16 (w & 3) on and half w / 4 of the tile's CV columns of the outputs, and the
+// row tiles w, w + 8, .. (RT of them) of S with all columns.
 template <int CV, int RT>
-__global__ void __launch_bounds__(256)
+__global__ void __launch_bounds__(256, 2)
 ssm_chunks_kernel(const bf16* __restrict__ xbc, const float* __restrict__ la, const float* __restrict__ dt,
                   const float* __restrict__ skip, float* __restrict__ state, float* __restrict__ y,
                   const int* __restrict__ cu_q, const int* __restrict__ slots, SsmSizes z, int write_state) {
-  constexpr int PV = ChunkSmem<CV>::PV, NT = CV / 8;
+  constexpr int PV = ChunkSmem<CV>::PV, NT = CV / 8, HT = CV / 16;      // column tiles of 8: of S, of a warp's outputs
   extern __shared__ __align__(16) unsigned char sm[];
   const int N = z.N, V = z.V, H = z.H, Cc = z.channels(), PN = N + 8;
   bf16* Bs = reinterpret_cast<bf16*>(sm);                       // [2][64][PN]
@@ -466,15 +494,9 @@ ssm_chunks_kernel(const bf16* __restrict__ xbc, const float* __restrict__ la, co
   bf16* xs = Cs + 2 * SC_T * PN;                                // [2][64][PV]
   bf16* Sh = xs + 2 * SC_T * PV;                                // [N][PV] the state before the chunk, high parts
   bf16* Sl = Sh + N * PV;
-  bf16* wh = Sl + N * PV;                                       // [64][PV] exp(L_end - L_s) dt_s x_s, high parts
+  bf16* wh = Sl + N * PV;                                       // [64][PV] w_s x_s, high parts
   bf16* wl = wh + SC_T * PV;
-  float* Yx = reinterpret_cast<float*>(wl + SC_T * PV);         // [64][CV + 4]
-  float* las = Yx + SC_T * (CV + 4);                            // [2][64]
-  float* dts = las + 2 * SC_T;                                  // [2][64]
-  float* cs = dts + 2 * SC_T;                                   // [64] L_s
-  float* ecs = cs + SC_T;                                       // exp(L_s)
-  float* wsm = ecs + SC_T;                                      // exp(L_end - L_s) dt_s
-  float* endp = wsm + SC_T;                                     // exp(L_end)
+  ChunkScales* scales = reinterpret_cast<ChunkScales*>(wl + SC_T * PV);      // [2]
   const int b = blockIdx.x, h = blockIdx.y, col0 = blockIdx.z * CV;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int g = lane >> 2, t4 = lane & 3;
@@ -500,6 +522,7 @@ ssm_chunks_kernel(const bf16* __restrict__ xbc, const float* __restrict__ la, co
   const bf16* xg = xbc + (size_t)h * V + col0;
   const bf16* Bg = xbc + z.inner() + (size_t)grp * N;
   const bf16* Cg = Bg + (size_t)z.G * N;
+  // who copies what of a chunk, worked out once: pieces of 16 bytes
   auto load = [&](int buf, int c0) {
     const int n = min(SC_T, t1 - c0);
     for (int i = tid; i < SC_T * pn; i += 256) {
@@ -519,44 +542,50 @@ ssm_chunks_kernel(const bf16* __restrict__ xbc, const float* __restrict__ la, co
       if (r < n && col0 + c < V) sc_async16(d, xg + (size_t)(c0 + r) * Cc + c);
       else *reinterpret_cast<uint4*>(d) = make_uint4(0, 0, 0, 0);
     }
-    if (tid < 2 * SC_T) {
-      const int r = tid & (SC_T - 1);
-      float* d = (tid < SC_T ? las : dts) + buf * SC_T + r;
-      if (r < n) sc_async4(d, (tid < SC_T ? la : dt) + (size_t)(c0 + r) * H + h);
-      else *d = 0.f;                       // no decay, no weight
-    }
     asm volatile("cp.async.commit_group;\n" ::);
   };
+  // the first warp's lanes hold two tokens' numbers each; tokens past the end have no decay and no weight
+  float l0 = 0.f, l1 = 0.f, d0 = 0.f, d1 = 0.f;
+  auto fetch = [&](int c0) {
+    const int a = c0 + 2 * lane;
+    l0 = a < t1 ? la[(size_t)a * H + h] : 0.f;
+    d0 = a < t1 ? dt[(size_t)a * H + h] : 0.f;
+    l1 = a + 1 < t1 ? la[(size_t)(a + 1) * H + h] : 0.f;
+    d1 = a + 1 < t1 ? dt[(size_t)(a + 1) * H + h] : 0.f;
+  };
+  auto scan = [&](ChunkScales& s) {
+    const float v0 = l0 * LOG2E, v1 = l1 * LOG2E;
+    float incl = v0 + v1;
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+      const float up = __shfl_up_sync(0xffffffffu, incl, o);
+      if (lane >= o) incl += up;
+    }
+    float before = __shfl_up_sync(0xffffffffu, incl, 1);
+    if (lane == 0) before = 0.f;
+    const float end = __shfl_sync(0xffffffffu, incl, 31), La = before + v0;
+    *reinterpret_cast<float2*>(s.L + 2 * lane) = make_float2(La, incl);
+    *reinterpret_cast<float2*>(s.q + 2 * lane) = make_float2(La - log2f(d0), incl - log2f(d1));
+    *reinterpret_cast<float2*>(s.e + 2 * lane) = make_float2(fast_exp2(La), fast_exp2(incl));
+    *reinterpret_cast<float2*>(s.w + 2 * lane) = make_float2(fast_exp2(end - La) * d0, fast_exp2(end - incl) * d1);
+    if (lane == 0) s.end[0] = fast_exp2(end);
+  };
   load(0, t0);
+  if (warp == 0) { fetch(t0); scan(scales[0]); }
   const int a_row = (lane & 7) + ((lane >> 3) & 1) * 8, a_col = (lane >> 4) * 8;       // first operand, rows of k
   const int b_row = (lane & 7) + (lane >> 4) * 8, b_col = ((lane >> 3) & 1) * 8;       // second operand, rows of k
-  const int v_row = a_row, v_col = a_col;                                              // second operand, rows of n (transposed)
   const int s_tok = (lane & 7) + (lane >> 4) * 8, s_n = ((lane >> 3) & 1) * 8;         // first operand, rows of m (transposed)
+  const int m0 = (warp & 3) * 16, oc = (warp >> 2) * (CV / 2);                         // this warp's tokens and columns
   int buf = 0;
   for (int c0 = t0; c0 < t1; c0 += SC_T, buf ^= 1) {
     asm volatile("cp.async.wait_group 0;\n" ::);
-    __syncthreads();                       // A: the chunk has arrived; everything of the chunk before has been read
-    if (c0 + SC_T < t1) load(buf ^ 1, c0 + SC_T);
-    if (warp == 0) {                       // running sums of the log decays, two tokens per lane
-      const float v0 = las[buf * SC_T + 2 * lane], v1 = las[buf * SC_T + 2 * lane + 1];
-      float incl = v0 + v1;
-#pragma unroll
-      for (int o = 1; o < 32; o <<= 1) {
-        const float up = __shfl_up_sync(0xffffffffu, incl, o);
-        if (lane >= o) incl += up;
-      }
-      float before = __shfl_up_sync(0xffffffffu, incl, 1);
-      if (lane == 0) before = 0.f;
-      const float end = __shfl_sync(0xffffffffu, incl, 31);
-      const float l0 = before + v0, l1 = incl;
-      cs[2 * lane] = l0;
-      cs[2 * lane + 1] = l1;
-      ecs[2 * lane] = expf(l0);
-      ecs[2 * lane + 1] = expf(l1);
-      wsm[2 * lane] = expf(end - l0) * dts[buf * SC_T + 2 * lane];
-      wsm[2 * lane + 1] = expf(end - l1) * dts[buf * SC_T + 2 * lane + 1];
-      if (lane == 0) *endp = expf(end);
+    __syncthreads();                       // the chunk and its scales have arrived; everything of the chunk before has been read
+    if (c0 + SC_T < t1) {
+      load(buf ^ 1, c0 + SC_T);
+      if (warp == 0) fetch(c0 + SC_T);
     }
+    const ChunkScales& sc = scales[buf];
+    const bf16* xb = xs + (size_t)buf * SC_T * PV;
 #pragma unroll
     for (int r = 0; r < RT; ++r) {
       if (warp + 8 * r < n_rt) {
@@ -573,94 +602,86 @@ ssm_chunks_kernel(const bf16* __restrict__ xbc, const float* __restrict__ la, co
         }
       }
     }
-    __syncthreads();                       // B
-    const bf16* xb = xs + (size_t)buf * SC_T * PV;
-    for (int i = tid; i < SC_T * (CV / 2); i += 256) {
-      const int r = i / (CV / 2), c = (i - r * (CV / 2)) * 2;
-      const uint32_t v = *reinterpret_cast<const uint32_t*>(xb + r * PV + c);
-      const float w = wsm[r];
-      uint32_t hi, lo;
-      split2(w * __uint_as_float(v << 16), w * __uint_as_float(v & 0xffff0000u), hi, lo);
-      *reinterpret_cast<uint32_t*>(wh + r * PV + c) = hi;
-      *reinterpret_cast<uint32_t*>(wl + r * PV + c) = lo;
+#pragma unroll
+    for (int k = 0; k < SC_T * (CV / 4) / 256; ++k) {
+      const int i = tid + k * 256, r = i / (CV / 4), c = (i - r * (CV / 4)) * 4;
+      const uint2 v = *reinterpret_cast<const uint2*>(xb + r * PV + c);
+      const float w = sc.w[r];
+      uint2 hi, lo;
+      split2(w * __uint_as_float(v.x << 16), w * __uint_as_float(v.x & 0xffff0000u), hi.x, lo.x);
+      split2(w * __uint_as_float(v.y << 16), w * __uint_as_float(v.y & 0xffff0000u), hi.y, lo.y);
+      *reinterpret_cast<uint2*>(wh + r * PV + c) = hi;
+      *reinterpret_cast<uint2*>(wl + r * PV + c) = lo;
     }
-    __syncthreads();                       // C
+    __syncthreads();
     const bf16 *Bb = Bs + (size_t)buf * SC_T * PN, *Cb = Cs + (size_t)buf * SC_T * PN;
-    const int m0 = (warp & 3) * 16;
-    float Y[NT][4];
+    // the scores of the warp's tokens against those up to them, and what the state before the chunk gives, S^T C_t
+    float p[8][4], Y[HT][4];
 #pragma unroll
-    for (int nt = 0; nt < NT; ++nt) Y[nt][0] = Y[nt][1] = Y[nt][2] = Y[nt][3] = 0.f;
-    if (warp < 4) {
-      // the chunk's own tokens: scores of 16 rows against the columns up to them
-      float p[8][4];
+    for (int nt = 0; nt < 8; ++nt) p[nt][0] = p[nt][1] = p[nt][2] = p[nt][3] = 0.f;
 #pragma unroll
-      for (int nt = 0; nt < 8; ++nt) p[nt][0] = p[nt][1] = p[nt][2] = p[nt][3] = 0.f;
-      for (int k = 0; k < N; k += 16) {
-        uint32_t a0, a1, a2, a3;
-        ldmatrix_x4(a0, a1, a2, a3, smem_u32(Cb + (m0 + a_row) * PN + k + a_col));
+    for (int nt = 0; nt < HT; ++nt) Y[nt][0] = Y[nt][1] = Y[nt][2] = Y[nt][3] = 0.f;
+#pragma unroll 2
+    for (int k = 0; k < N; k += 16) {
+      uint32_t a0, a1, a2, a3;
+      ldmatrix_x4(a0, a1, a2, a3, smem_u32(Cb + (m0 + a_row) * PN + k + a_col));
 #pragma unroll
-        for (int np = 0; np < 4; ++np) {
-          if (np * 16 <= m0) {
-            uint32_t b0, b1, b2, b3;
-            ldmatrix_x4(b0, b1, b2, b3, smem_u32(Bb + (np * 16 + b_row) * PN + k + b_col));
-            mma_bf16(p[2 * np], a0, a1, a2, a3, b0, b1);
-            mma_bf16(p[2 * np + 1], a0, a1, a2, a3, b2, b3);
-          }
-        }
-      }
-      const float l0 = cs[m0 + g], l1 = cs[m0 + g + 8];
-#pragma unroll
-      for (int nt = 0; nt < 8; ++nt)
-        if (nt * 8 <= m0 + 15) {
-#pragma unroll
-          for (int j = 0; j < 4; ++j) {
-            const int s = nt * 8 + 2 * t4 + (j & 1), row = m0 + g + (j < 2 ? 0 : 8);
-            p[nt][j] = s <= row ? p[nt][j] * (expf((j < 2 ? l0 : l1) - cs[s]) * dts[buf * SC_T + s]) : 0.f;
-          }
-        }
-#pragma unroll
-      for (int ks = 0; ks < 4; ++ks) {
-        if (ks * 16 <= m0) {
-          uint32_t h0, h1, h2, h3, q0, q1, q2, q3;
-          split2(p[2 * ks][0], p[2 * ks][1], h0, q0);
-          split2(p[2 * ks][2], p[2 * ks][3], h1, q1);
-          split2(p[2 * ks + 1][0], p[2 * ks + 1][1], h2, q2);
-          split2(p[2 * ks + 1][2], p[2 * ks + 1][3], h3, q3);
-#pragma unroll
-          for (int np = 0; np < NT / 2; ++np) {
-            uint32_t b0, b1, b2, b3;
-            ldmatrix_x4_trans(b0, b1, b2, b3, smem_u32(xb + (ks * 16 + v_row) * PV + np * 16 + v_col));
-            mma_bf16(Y[2 * np], h0, h1, h2, h3, b0, b1);
-            mma_bf16(Y[2 * np + 1], h0, h1, h2, h3, b2, b3);
-            mma_bf16(Y[2 * np], q0, q1, q2, q3, b0, b1);
-            mma_bf16(Y[2 * np + 1], q0, q1, q2, q3, b2, b3);
-          }
-        }
-      }
-    } else {
-      // what the state before the chunk gives: exp(L_t) S^T C_t
-      for (int k = 0; k < N; k += 16) {
-        uint32_t a0, a1, a2, a3;
-        ldmatrix_x4(a0, a1, a2, a3, smem_u32(Cb + (m0 + a_row) * PN + k + a_col));
-#pragma unroll
-        for (int np = 0; np < NT / 2; ++np) {
+      for (int np = 0; np < 4; ++np) {
+        if (np * 16 <= m0) {
           uint32_t b0, b1, b2, b3;
-          ldmatrix_x4_trans(b0, b1, b2, b3, smem_u32(Sh + (k + v_row) * PV + np * 16 + v_col));
-          mma_bf16(Y[2 * np], a0, a1, a2, a3, b0, b1);
-          mma_bf16(Y[2 * np + 1], a0, a1, a2, a3, b2, b3);
-          ldmatrix_x4_trans(b0, b1, b2, b3, smem_u32(Sl + (k + v_row) * PV + np * 16 + v_col));
-          mma_bf16(Y[2 * np], a0, a1, a2, a3, b0, b1);
-          mma_bf16(Y[2 * np + 1], a0, a1, a2, a3, b2, b3);
+          ldmatrix_x4(b0, b1, b2, b3, smem_u32(Bb + (np * 16 + b_row) * PN + k + b_col));
+          mma_bf16(p[2 * np], a0, a1, a2, a3, b0, b1);
+          mma_bf16(p[2 * np + 1], a0, a1, a2, a3, b2, b3);
         }
       }
-      const float e0 = ecs[m0 + g], e1 = ecs[m0 + g + 8];
-#pragma unroll
-      for (int nt = 0; nt < NT; ++nt) {
-        *reinterpret_cast<float2*>(Yx + (m0 + g) * (CV + 4) + nt * 8 + 2 * t4) = make_float2(Y[nt][0] * e0, Y[nt][1] * e0);
-        *reinterpret_cast<float2*>(Yx + (m0 + g + 8) * (CV + 4) + nt * 8 + 2 * t4) = make_float2(Y[nt][2] * e1, Y[nt][3] * e1);
+      if (HT == 2) {
+        uint32_t b0, b1, b2, b3;
+        ldmatrix_x4_trans(b0, b1, b2, b3, smem_u32(Sh + (k + a_row) * PV + oc + a_col));
+        mma_bf16(Y[0], a0, a1, a2, a3, b0, b1);
+        mma_bf16(Y[HT - 1], a0, a1, a2, a3, b2, b3);
+        ldmatrix_x4_trans(b0, b1, b2, b3, smem_u32(Sl + (k + a_row) * PV + oc + a_col));
+        mma_bf16(Y[0], a0, a1, a2, a3, b0, b1);
+        mma_bf16(Y[HT - 1], a0, a1, a2, a3, b2, b3);
+      } else {
+        // eight columns: the high parts' two pieces of k and the low parts' in one load
+        uint32_t b0, b1, b2, b3;
+        ldmatrix_x4_trans(b0, b1, b2, b3, smem_u32((lane < 16 ? Sh : Sl) + (k + a_row) * PV + oc));
+        mma_bf16(Y[0], a0, a1, a2, a3, b0, b1);
+        mma_bf16(Y[0], a0, a1, a2, a3, b2, b3);
       }
     }
-    const float keep = *endp;
+    const float La = sc.L[m0 + g], Lb = sc.L[m0 + g + 8], ea = sc.e[m0 + g], eb = sc.e[m0 + g + 8];
+#pragma unroll
+    for (int nt = 0; nt < HT; ++nt) { Y[nt][0] *= ea; Y[nt][1] *= ea; Y[nt][2] *= eb; Y[nt][3] *= eb; }
+#pragma unroll
+    for (int nt = 0; nt < 8; ++nt)
+      if (nt * 8 <= m0 + 15) {
+        const float2 q = *reinterpret_cast<const float2*>(sc.q + nt * 8 + 2 * t4);
+        const int s = nt * 8 + 2 * t4, row = m0 + g;
+        p[nt][0] = s <= row ? p[nt][0] * fast_exp2(La - q.x) : 0.f;
+        p[nt][1] = s + 1 <= row ? p[nt][1] * fast_exp2(La - q.y) : 0.f;
+        p[nt][2] = s <= row + 8 ? p[nt][2] * fast_exp2(Lb - q.x) : 0.f;
+        p[nt][3] = s + 1 <= row + 8 ? p[nt][3] * fast_exp2(Lb - q.y) : 0.f;
+      }
+#pragma unroll
+    for (int ks = 0; ks < 4; ++ks) {
+      if (ks * 16 <= m0) {
+        uint32_t h0, h1, h2, h3, q0, q1, q2, q3, b0, b1, b2, b3;
+        split2(p[2 * ks][0], p[2 * ks][1], h0, q0);
+        split2(p[2 * ks][2], p[2 * ks][3], h1, q1);
+        split2(p[2 * ks + 1][0], p[2 * ks + 1][1], h2, q2);
+        split2(p[2 * ks + 1][2], p[2 * ks + 1][3], h3, q3);
+        ldmatrix_x4_trans(b0, b1, b2, b3, smem_u32(xb + (ks * 16 + a_row) * PV + oc + (HT == 2 ? a_col : 0)));
+        mma_bf16(Y[0], h0, h1, h2, h3, b0, b1);
+        mma_bf16(Y[0], q0, q1, q2, q3, b0, b1);
+        if (HT == 2) {
+          mma_bf16(Y[HT - 1], h0, h1, h2, h3, b2, b3);
+          mma_bf16(Y[HT - 1], q0, q1, q2, q3, b2, b3);
+        }
+      }
+    }
+    // S <- 2^(L_end) S + sum_s B_s (w_s x_s)^T
+    const float keep = sc.end[0];
 #pragma unroll
     for (int r = 0; r < RT; ++r) {
       if (warp + 8 * r < n_rt) {
@@ -673,36 +694,32 @@ ssm_chunks_kernel(const bf16* __restrict__ xbc, const float* __restrict__ la, co
 #pragma unroll
           for (int np = 0; np < NT / 2; ++np) {
             uint32_t b0, b1, b2, b3;
-            ldmatrix_x4_trans(b0, b1, b2, b3, smem_u32(wh + (ks * 16 + v_row) * PV + np * 16 + v_col));
+            ldmatrix_x4_trans(b0, b1, b2, b3, smem_u32(wh + (ks * 16 + a_row) * PV + np * 16 + a_col));
             mma_bf16(S[r][2 * np], a0, a1, a2, a3, b0, b1);
             mma_bf16(S[r][2 * np + 1], a0, a1, a2, a3, b2, b3);
-            ldmatrix_x4_trans(b0, b1, b2, b3, smem_u32(wl + (ks * 16 + v_row) * PV + np * 16 + v_col));
+            ldmatrix_x4_trans(b0, b1, b2, b3, smem_u32(wl + (ks * 16 + a_row) * PV + np * 16 + a_col));
             mma_bf16(S[r][2 * np], a0, a1, a2, a3, b0, b1);
             mma_bf16(S[r][2 * np + 1], a0, a1, a2, a3, b2, b3);
           }
         }
       }
     }
-    __syncthreads();                       // D
-    if (warp < 4) {
-      const int n = min(SC_T, t1 - c0);
+    const int n = min(SC_T, t1 - c0);
 #pragma unroll
-      for (int half = 0; half < 2; ++half) {
-        const int row = m0 + g + half * 8;
-        if (row >= n) continue;
-        float* o = y + (size_t)(c0 + row) * z.inner() + (size_t)h * V + col0;
+    for (int half = 0; half < 2; ++half) {
+      const int row = m0 + g + half * 8;
+      if (row >= n) continue;
+      float* o = y + (size_t)(c0 + row) * z.inner() + (size_t)h * V + col0;
 #pragma unroll
-        for (int nt = 0; nt < NT; ++nt) {
-          const int c = nt * 8 + 2 * t4;
-          if (col0 + c >= V) continue;
-          const float2 inter = *reinterpret_cast<const float2*>(Yx + row * (CV + 4) + c);
-          const uint32_t v = *reinterpret_cast<const uint32_t*>(xb + row * PV + c);
-          *reinterpret_cast<float2*>(o + c) =
-              make_float2(fmaf(sk, __uint_as_float(v << 16), Y[nt][2 * half] + inter.x),
-                          fmaf(sk, __uint_as_float(v & 0xffff0000u), Y[nt][2 * half + 1] + inter.y));
-        }
+      for (int nt = 0; nt < HT; ++nt) {
+        const int c = oc + nt * 8 + 2 * t4;
+        if (col0 + c >= V) continue;
+        const uint32_t v = *reinterpret_cast<const uint32_t*>(xb + row * PV + c);
+        *reinterpret_cast<float2*>(o + c) = make_float2(fmaf(sk, __uint_as_float(v << 16), Y[nt][2 * half]),
+                                                        fmaf(sk, __uint_as_float(v & 0xffff0000u), Y[nt][2 * half + 1]));
       }
     }
+    if (warp == 0 && c0 + SC_T < t1) scan(scales[buf ^ 1]);
   }
   if (!write_state) return;
 #pragma unroll

@@ -1196,15 +1196,22 @@ MOE_ACTIVATIONS = {"gelu": 0, "silu": 1, "relu2": 2}      # ("relu2", the square
 MOE_SCORES = {"softmax": None, "logit": 0, "sigmoid": 1}
 
 
+MOE_ROUTE_SMALL_MAX_ROWS = 64      # up to here logits and choice in one kernel (scores that are no softmax)
+
+
 def moe_route(h, router, n_tokens, groups, keep, top, scale, bias=None, score="softmax", correction=None, group_top=1,
-              renorm=True):
+              renorm=True, router16=None):
     """(experts int32 [T, top], weights float32 [T, top]) of every token: softmax over all experts, the `keep`
     best of `groups` groups of neighbours, the `top` best experts of those, weights renormalised times `scale`.
     `bias` float32 [E] is added to the logits.  (One group, scale 1: the softmax over the chosen logits alone.)
     `score` "sigmoid" (or "logit"): the scores are sigmoid(z) (or z); the choice is made by score + `correction`
     (float32 [E], if given), a group's score is the sum of its `group_top` largest choice scores, and the weights are
-    the chosen experts' scores without the correction, divided by their sum only if `renorm`."""
-    _cuda(h, router, bias, correction)
+    the chosen experts' scores without the correction, divided by their sum only if `renorm`.
+    `router16`: the router's matrix in bfloat16, where that holds it exactly: bfloat16 rows then run a library product with a
+    float32 result (many tokens; the products are exact, the sums 32-bit), or read half the bytes (few)."""
+    _cuda(h, router, bias, correction, router16)
+    _need(router16 is None or (router16.dtype == torch.bfloat16 and router16.shape == router.shape and router16.is_contiguous()),
+          "moe_route: router16 bfloat16 [experts, width]")
     _need(score in MOE_SCORES, f"moe_route: score must be one of {tuple(MOE_SCORES)}")
     _need(score != "softmax" or (correction is None and group_top == 1 and renorm),
           "moe_route: the softmax router has no correction, takes a group's largest score and renormalises")
@@ -1221,9 +1228,22 @@ def moe_route(h, router, n_tokens, groups, keep, top, scale, bias=None, score="s
           f"moe_route: {E} experts in {groups} groups, {keep} kept, {top} chosen cannot be routed")
     idx = torch.empty((max(n_tokens, 1), top), dtype=torch.int32, device=h.device)
     wts = torch.empty((max(n_tokens, 1), top), dtype=torch.float32, device=h.device)
-    z = torch.empty((max(n_tokens, 1), E), dtype=torch.float32, device=h.device)
     if score != "softmax":
         _need(group_top >= 1 and (keep == groups or E // groups <= 128), "moe_route: groups of up to 128 experts, group_top >= 1")
+        how = (E, groups, keep, int(group_top), top, MOE_SCORES[score], 1 if renorm else 0, ctypes.c_float(scale))
+        w16 = router16 if h.dtype == torch.bfloat16 else None
+        if n_tokens <= MOE_ROUTE_SMALL_MAX_ROWS:
+            w = router if w16 is None else w16
+            _check(_lib("moe").ab_moe_route_small(_p(h), _dt(h), width, _p(w), _dt(w), _p(bias), _p(correction), n_tokens, width,
+                                                  *how, _p(idx), _p(wts), _stream()), "moe_route")
+            return idx, wts
+        if w16 is not None and bias is None:
+            z = torch.mm(h.view(-1, width)[:n_tokens], w16.t(), out_dtype=torch.float32)
+            _mark("library product")
+            _check(_lib("moe").ab_moe_route_logits(_p(z), _p(correction), n_tokens, *how, _p(idx), _p(wts), _stream()), "moe_route")
+            return idx, wts
+    z = torch.empty((max(n_tokens, 1), E), dtype=torch.float32, device=h.device)
+    if score != "softmax":
         _check(_lib("moe").ab_moe_route_scores(
             _p(h), _dt(h), width, _p(router), _p(bias), _p(correction), n_tokens, width, E, groups, keep, int(group_top),
             top, MOE_SCORES[score], 1 if renorm else 0, ctypes.c_float(scale), _p(z), _p(idx), _p(wts), _stream()),

@@ -203,7 +203,7 @@ class ScoredExperts(FeedForward):
         self.prefix, self.activation, self.score, self.renorm = prefix, activation, score, bool(renorm)
         self.weight_in, self.shared_inner, self.gated = bool(weight_in), int(shared_inner), len(expert_names) == 3
         self.router_name, self.expert_names, self.shared_names = router_name, expert_names, shared_names
-        self.router = self.up = self.down = self.shared_up = self.shared_down = None
+        self.router = self.router16 = self.up = self.down = self.shared_up = self.shared_down = None
 
     def _specs_of(self, names, inner):
         shapes = [(inner, self.width)] * (len(names) - 1) + [(self.width, inner)]
@@ -220,6 +220,8 @@ class ScoredExperts(FeedForward):
     def load_own(self, fetch):
         specs, n = self.own_param_specs(), len(self.expert_names)
         self.router = fetch(specs[0])
+        w16 = self.router.to(torch.bfloat16)
+        self.router16 = w16.contiguous() if self.opts.dtype == torch.bfloat16 and torch.equal(w16.float(), self.router) else None
         ff = -(-self.inner // 16) * 16
         for e in range(self.E):
             up, down = self._laid_out(*(fetch(s) for s in specs[1 + n * e:1 + n * (e + 1)]))
@@ -241,7 +243,8 @@ class ScoredExperts(FeedForward):
         return first[0].contiguous(), torch.nn.functional.pad(down, (0, more)).contiguous()
 
     def forward(self, h, ctx):
-        choice = ops.moe_route(h, self.router, ctx.n_tokens, 1, 1, self.top, 1.0, score=self.score, renorm=self.renorm)
+        choice = ops.moe_route(h, self.router, ctx.n_tokens, 1, 1, self.top, 1.0, score=self.score, renorm=self.renorm,
+                               router16=self.router16)
         out = torch.empty((h.shape[0], self.width), dtype=torch.float32, device=h.device)
         shared = (self.shared_up, self.shared_down) if self.shared_inner else None
         return ops.moe_shared_experts(h, self.up, self.down, self.E, self.top, out, ctx, activation=self.activation,
