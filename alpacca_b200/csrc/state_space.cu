@@ -462,13 +462,11 @@ __device__ __forceinline__ void split2(float a, float b, uint32_t& hi, uint32_t&
   lo = pack_bf16(a - __uint_as_float(hi << 16), b - __uint_as_float(hi & 0xffff0000u));
 }
 
-template <int CV> struct ChunkSmem {
-  static constexpr int PV = CV + 8;                      // pitch of rows of value columns
-  __host__ __device__ static size_t bc(int N) { return (size_t)SC_T * (N + 8) * 2; }      // one buffer of B or C
-  __host__ __device__ static size_t total(int N) {
-    return 4 * bc(N) + 2 * (size_t)SC_T * PV * 2 + 2 * (size_t)N * PV * 2 + 2 * (size_t)SC_T * PV * 2 + 2 * (4 * SC_T + 4) * 4;
-  }
-};
+#define SC_CV 32               // value columns per CTA
+#define SC_PV (SC_CV + 8)      // pitch of rows of value columns
+#define SC_PP (SC_T + 8)       // pitch of rows of weights
+#define SC_WORKERS 512         // threads that hold S and outputs; one more warp forms the scales
+#define SC_THREADS (SC_WORKERS + 32)
 
 // What a chunk's step sizes and log decays come to, in powers of two: L_t, the running sum of the log decays (times log2 e).
 struct ChunkScales {
@@ -479,72 +477,85 @@ struct ChunkScales {
   float end[4];           // 2^(L_end)
 };
 
-// Eight warps: warp w takes the 16 tokens from 16 (w & 3) on and half w / 4 of the tile's CV columns of the outputs, and the
-// row tiles w, w + 8, .. (RT of them) of S with all columns.
-template <int CV, int RT>
-__global__ void __launch_bounds__(256, 2)
+static size_t chunk_smem(int N) {
+  return sizeof(bf16) * (4 * (size_t)SC_T * (N + 8) + 2 * (size_t)SC_T * SC_PV + 2 * (size_t)N * SC_PV + 2 * (size_t)SC_T * SC_PV +
+                         2 * (size_t)SC_T * SC_PP) + 2 * sizeof(ChunkScales);
+}
+
+// Sixteen warps.  Warp w takes tokens 16 (w / 4) .. + 15 of the chunk and, of them, the scores against tokens 16 (w % 4) .. + 15
+// and the output columns 8 (w % 4) .. + 7; of S the row tiles w % 8, w % 8 + 8, .. (RT of them) and columns 16 (w / 8) .. + 15.
+// A seventeenth warp forms the next chunk's scales.  Two barriers per chunk: (1) S and the weighted x of the chunk lie in
+// shared memory, split; (2) so do the weights of its scores, and the next chunk's rows and scales have arrived.
+template <int RT>
+__global__ void __launch_bounds__(SC_THREADS)
 ssm_chunks_kernel(const bf16* __restrict__ xbc, const float* __restrict__ la, const float* __restrict__ dt,
                   const float* __restrict__ skip, float* __restrict__ state, float* __restrict__ y,
                   const int* __restrict__ cu_q, const int* __restrict__ slots, SsmSizes z, int write_state) {
-  constexpr int PV = ChunkSmem<CV>::PV, NT = CV / 8, HT = CV / 16;      // column tiles of 8: of S, of a warp's outputs
   extern __shared__ __align__(16) unsigned char sm[];
   const int N = z.N, V = z.V, H = z.H, Cc = z.channels(), PN = N + 8;
   bf16* Bs = reinterpret_cast<bf16*>(sm);                       // [2][64][PN]
   bf16* Cs = Bs + 2 * SC_T * PN;                                // [2][64][PN]
   bf16* xs = Cs + 2 * SC_T * PN;                                // [2][64][PV]
-  bf16* Sh = xs + 2 * SC_T * PV;                                // [N][PV] the state before the chunk, high parts
-  bf16* Sl = Sh + N * PV;
-  bf16* wh = Sl + N * PV;                                       // [64][PV] w_s x_s, high parts
-  bf16* wl = wh + SC_T * PV;
-  ChunkScales* scales = reinterpret_cast<ChunkScales*>(wl + SC_T * PV);      // [2]
-  const int b = blockIdx.x, h = blockIdx.y, col0 = blockIdx.z * CV;
+  bf16* Sh = xs + 2 * SC_T * SC_PV;                             // [N][PV] the state before the chunk, high and low parts
+  bf16* Sl = Sh + N * SC_PV;
+  bf16* wh = Sl + N * SC_PV;                                    // [64][PV] w_s x_s
+  bf16* wl = wh + SC_T * SC_PV;
+  bf16* Ph = wl + SC_T * SC_PV;                                 // [64][PP] scores times their weights
+  bf16* Pl = Ph + SC_T * SC_PP;
+  ChunkScales* scales = reinterpret_cast<ChunkScales*>(Pl + SC_T * SC_PP);      // [2]
+  const int b = blockIdx.x, h = blockIdx.y, col0 = blockIdx.z * SC_CV;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int g = lane >> 2, t4 = lane & 3;
   const int slot = slots[b], t0 = cu_q[b], t1 = cu_q[b + 1];
   if (slot < 0 || t1 <= t0) { pdl_wait(); pdl_trigger(); return; }
-  const int n_rt = N >> 4, grp = h / (H / z.G);
-  float* st = state + ((size_t)slot * H + h) * N * V + col0;
-  float S[RT][NT][4];
+  const int grp = h / (H / z.G);
+  const int srow = (warp & 7) * 16, scol = ((warp >> 3) & 1) * 16;                    // this warp's part of S
+  float* st = state + ((size_t)slot * H + h) * N * V + col0 + scol;
+  float S[RT][2][4];
 #pragma unroll
   for (int r = 0; r < RT; ++r)
 #pragma unroll
-    for (int nt = 0; nt < NT; ++nt) {
-      const int n = (warp + 8 * r) * 16 + g, c = nt * 8 + 2 * t4;
-      const bool in = warp + 8 * r < n_rt && col0 + c < V;
+    for (int nt = 0; nt < 2; ++nt) {
+      const int n = srow + 128 * r + g, c = nt * 8 + 2 * t4;
+      const bool in = warp < 16 && srow + 128 * r < N && col0 + scol + c < V;
       const float2 lo = in ? *reinterpret_cast<const float2*>(st + (size_t)n * V + c) : make_float2(0.f, 0.f);
       const float2 hi = in ? *reinterpret_cast<const float2*>(st + (size_t)(n + 8) * V + c) : make_float2(0.f, 0.f);
       S[r][nt][0] = lo.x; S[r][nt][1] = lo.y; S[r][nt][2] = hi.x; S[r][nt][3] = hi.y;
     }
+  // who copies what of a chunk: a thread keeps its 16-byte column of B and C and walks down the rows; the first 256 one piece of x
+  const int pn = N >> 3, per_pass = SC_WORKERS / pn, br = tid / pn, bc = (tid - br * pn) * 8;
+  const bool worker = warp < 16, copies = worker && br < per_pass;
+  const int xr = tid >> 2, xc = (tid & 3) * 8;
   pdl_wait();
   pdl_trigger();
   const float sk = skip[h];
-  const int pn = N >> 3;
-  const bf16* xg = xbc + (size_t)h * V + col0;
-  const bf16* Bg = xbc + z.inner() + (size_t)grp * N;
-  const bf16* Cg = Bg + (size_t)z.G * N;
-  // who copies what of a chunk, worked out once: pieces of 16 bytes
+  const bf16* Bg = xbc + z.inner() + (size_t)grp * N + bc;
+  const bf16* xg = xbc + (size_t)h * V + col0 + xc;
+  const size_t c_ahead = (size_t)z.G * N;
   auto load = [&](int buf, int c0) {
     const int n = min(SC_T, t1 - c0);
-    for (int i = tid; i < SC_T * pn; i += 256) {
-      const int r = i / pn, c = (i - r * pn) * 8;
-      bf16 *db = Bs + ((size_t)buf * SC_T + r) * PN + c, *dc = Cs + ((size_t)buf * SC_T + r) * PN + c;
-      if (r < n) {
-        sc_async16(db, Bg + (size_t)(c0 + r) * Cc + c);
-        sc_async16(dc, Cg + (size_t)(c0 + r) * Cc + c);
-      } else {
-        *reinterpret_cast<uint4*>(db) = make_uint4(0, 0, 0, 0);
-        *reinterpret_cast<uint4*>(dc) = make_uint4(0, 0, 0, 0);
+    if (copies) {
+      const bf16* src = Bg + (size_t)(c0 + br) * Cc;
+      bf16* db = Bs + (buf * SC_T + br) * PN + bc;
+      for (int r = br; r < SC_T; r += per_pass, src += (size_t)per_pass * Cc, db += per_pass * PN) {
+        bf16* dc = db + 2 * SC_T * PN;
+        if (r < n) {
+          sc_async16(db, src);
+          sc_async16(dc, src + c_ahead);
+        } else {
+          *reinterpret_cast<uint4*>(db) = make_uint4(0, 0, 0, 0);
+          *reinterpret_cast<uint4*>(dc) = make_uint4(0, 0, 0, 0);
+        }
       }
     }
-    for (int i = tid; i < SC_T * (CV / 8); i += 256) {
-      const int r = i / (CV / 8), c = (i - r * (CV / 8)) * 8;
-      bf16* d = xs + ((size_t)buf * SC_T + r) * PV + c;
-      if (r < n && col0 + c < V) sc_async16(d, xg + (size_t)(c0 + r) * Cc + c);
+    if (tid < SC_T * (SC_CV / 8)) {
+      bf16* d = xs + (buf * SC_T + xr) * SC_PV + xc;
+      if (xr < n && col0 + xc < V) sc_async16(d, xg + (size_t)(c0 + xr) * Cc);
       else *reinterpret_cast<uint4*>(d) = make_uint4(0, 0, 0, 0);
     }
     asm volatile("cp.async.commit_group;\n" ::);
   };
-  // the first warp's lanes hold two tokens' numbers each; tokens past the end have no decay and no weight
+  // the last warp's lanes hold two tokens' numbers each; tokens past the end have no decay and no weight
   float l0 = 0.f, l1 = 0.f, d0 = 0.f, d1 = 0.f;
   auto fetch = [&](int c0) {
     const int a = c0 + 2 * lane;
@@ -570,164 +581,189 @@ ssm_chunks_kernel(const bf16* __restrict__ xbc, const float* __restrict__ la, co
     *reinterpret_cast<float2*>(s.w + 2 * lane) = make_float2(fast_exp2(end - La) * d0, fast_exp2(end - incl) * d1);
     if (lane == 0) s.end[0] = fast_exp2(end);
   };
-  load(0, t0);
-  if (warp == 0) { fetch(t0); scan(scales[0]); }
   const int a_row = (lane & 7) + ((lane >> 3) & 1) * 8, a_col = (lane >> 4) * 8;       // first operand, rows of k
   const int b_row = (lane & 7) + (lane >> 4) * 8, b_col = ((lane >> 3) & 1) * 8;       // second operand, rows of k
-  const int s_tok = (lane & 7) + (lane >> 4) * 8, s_n = ((lane >> 3) & 1) * 8;         // first operand, rows of m (transposed)
-  const int m0 = (warp & 3) * 16, oc = (warp >> 2) * (CV / 2);                         // this warp's tokens and columns
-  int buf = 0;
-  for (int c0 = t0; c0 < t1; c0 += SC_T, buf ^= 1) {
-    asm volatile("cp.async.wait_group 0;\n" ::);
-    __syncthreads();                       // the chunk and its scales have arrived; everything of the chunk before has been read
-    if (c0 + SC_T < t1) {
-      load(buf ^ 1, c0 + SC_T);
-      if (warp == 0) fetch(c0 + SC_T);
-    }
-    const ChunkScales& sc = scales[buf];
-    const bf16* xb = xs + (size_t)buf * SC_T * PV;
+  const int mi = (warp >> 2) & 3, mj = warp & 3, m0 = mi * 16;                         // tokens; scores' tokens and columns
+  // shared-memory addresses of this lane's matrix rows, in bytes, without what moves with the loops
+  const uint32_t aC = smem_u32(Cs + (m0 + a_row) * PN + a_col), aB = smem_u32(Bs + (mj * 16 + b_row) * PN + b_col);
+  const uint32_t aS = smem_u32((lane < 16 ? Sh : Sl) + a_row * SC_PV + mj * 8);
+  const uint32_t aBt = smem_u32(Bs + b_row * PN + srow + b_col);
+  const uint32_t aW = smem_u32(wh + a_row * SC_PV + scol + a_col), to_wl = SC_T * SC_PV * 2;      // wl lies behind wh
+  const uint32_t aP = smem_u32(Ph + (m0 + a_row) * SC_PP + a_col), to_pl = SC_T * SC_PP * 2;      // and Pl behind Ph
+  const uint32_t aX = smem_u32(xs + lane * SC_PV + mj * 8);                            // 32 rows of x, eight columns
+  const uint32_t bytes_bc = SC_T * PN * 2, bytes_x = SC_T * SC_PV * 2;                 // from one buffer to the other
+  // S and the weighted x of the chunk in buffer `buf`, as pairs of bfloat16 numbers
+  auto lay_out = [&](int buf) {
 #pragma unroll
     for (int r = 0; r < RT; ++r) {
-      if (warp + 8 * r < n_rt) {
-        const int n = (warp + 8 * r) * 16 + g;
+      if (srow + 128 * r < N) {
+        const int at = (srow + 128 * r + g) * SC_PV + scol + 2 * t4;
 #pragma unroll
-        for (int nt = 0; nt < NT; ++nt) {
+        for (int nt = 0; nt < 2; ++nt) {
           uint32_t hi, lo;
           split2(S[r][nt][0], S[r][nt][1], hi, lo);
-          *reinterpret_cast<uint32_t*>(Sh + n * PV + nt * 8 + 2 * t4) = hi;
-          *reinterpret_cast<uint32_t*>(Sl + n * PV + nt * 8 + 2 * t4) = lo;
+          *reinterpret_cast<uint32_t*>(Sh + at + nt * 8) = hi;
+          *reinterpret_cast<uint32_t*>(Sl + at + nt * 8) = lo;
           split2(S[r][nt][2], S[r][nt][3], hi, lo);
-          *reinterpret_cast<uint32_t*>(Sh + (n + 8) * PV + nt * 8 + 2 * t4) = hi;
-          *reinterpret_cast<uint32_t*>(Sl + (n + 8) * PV + nt * 8 + 2 * t4) = lo;
+          *reinterpret_cast<uint32_t*>(Sh + at + 8 * SC_PV + nt * 8) = hi;
+          *reinterpret_cast<uint32_t*>(Sl + at + 8 * SC_PV + nt * 8) = lo;
         }
       }
     }
+    const int row = tid >> 3, c = (tid & 7) * 4;
+    const uint2 v = *reinterpret_cast<const uint2*>(xs + (buf * SC_T + row) * SC_PV + c);
+    const float w = scales[buf].w[row];
+    uint2 hi, lo;
+    split2(w * __uint_as_float(v.x << 16), w * __uint_as_float(v.x & 0xffff0000u), hi.x, lo.x);
+    split2(w * __uint_as_float(v.y << 16), w * __uint_as_float(v.y & 0xffff0000u), hi.y, lo.y);
+    *reinterpret_cast<uint2*>(wh + row * SC_PV + c) = hi;
+    *reinterpret_cast<uint2*>(wl + row * SC_PV + c) = lo;
+  };
+  if (worker) {
+    load(0, t0);
+  } else {
+    fetch(t0);
+    scan(scales[0]);
+    fetch(t0 + SC_T);
+  }
+  asm volatile("cp.async.wait_group 0;\n" ::);
+  __syncthreads();
+  if (worker) lay_out(0);
+  int buf = 0;
+  for (int c0 = t0; c0 < t1; c0 += SC_T, buf ^= 1) {
+    const bool more = c0 + SC_T < t1;
+    float Y[4] = {0.f, 0.f, 0.f, 0.f}, Y2[4] = {0.f, 0.f, 0.f, 0.f};
+    __syncthreads();                       // (1)
+    if (!worker) {
+      if (more) {
+        scan(scales[buf ^ 1]);
+        fetch(c0 + 2 * SC_T);
+      }
+    } else {
+      if (more) load(buf ^ 1, c0 + SC_T);
+      const ChunkScales& sc = scales[buf];
+      const uint32_t off = buf * bytes_bc;
+      // a tile of scores C_t . B_s (none above the diagonal), and what the state before the chunk gives, S^T C_t: eight columns
+      // of S, the high parts' two pieces of k and the low parts' in one load.  The next step's operands are on their way.
+      float p[2][4];
 #pragma unroll
-    for (int k = 0; k < SC_T * (CV / 4) / 256; ++k) {
-      const int i = tid + k * 256, r = i / (CV / 4), c = (i - r * (CV / 4)) * 4;
-      const uint2 v = *reinterpret_cast<const uint2*>(xb + r * PV + c);
-      const float w = sc.w[r];
-      uint2 hi, lo;
-      split2(w * __uint_as_float(v.x << 16), w * __uint_as_float(v.x & 0xffff0000u), hi.x, lo.x);
-      split2(w * __uint_as_float(v.y << 16), w * __uint_as_float(v.y & 0xffff0000u), hi.y, lo.y);
-      *reinterpret_cast<uint2*>(wh + r * PV + c) = hi;
-      *reinterpret_cast<uint2*>(wl + r * PV + c) = lo;
-    }
-    __syncthreads();
-    const bf16 *Bb = Bs + (size_t)buf * SC_T * PN, *Cb = Cs + (size_t)buf * SC_T * PN;
-    // the scores of the warp's tokens against those up to them, and what the state before the chunk gives, S^T C_t
-    float p[8][4], Y[HT][4];
-#pragma unroll
-    for (int nt = 0; nt < 8; ++nt) p[nt][0] = p[nt][1] = p[nt][2] = p[nt][3] = 0.f;
-#pragma unroll
-    for (int nt = 0; nt < HT; ++nt) Y[nt][0] = Y[nt][1] = Y[nt][2] = Y[nt][3] = 0.f;
-#pragma unroll 2
-    for (int k = 0; k < N; k += 16) {
-      uint32_t a0, a1, a2, a3;
-      ldmatrix_x4(a0, a1, a2, a3, smem_u32(Cb + (m0 + a_row) * PN + k + a_col));
-#pragma unroll
-      for (int np = 0; np < 4; ++np) {
-        if (np * 16 <= m0) {
-          uint32_t b0, b1, b2, b3;
-          ldmatrix_x4(b0, b1, b2, b3, smem_u32(Bb + (np * 16 + b_row) * PN + k + b_col));
-          mma_bf16(p[2 * np], a0, a1, a2, a3, b0, b1);
-          mma_bf16(p[2 * np + 1], a0, a1, a2, a3, b2, b3);
+      for (int nt = 0; nt < 2; ++nt) p[nt][0] = p[nt][1] = p[nt][2] = p[nt][3] = 0.f;
+      uint32_t a[2][4], bb[2][4], ss[2][4];
+      auto ask = [&](int w, int k) {
+        ldmatrix_x4(a[w][0], a[w][1], a[w][2], a[w][3], aC + off + k * 2);
+        if (mj <= mi) ldmatrix_x4(bb[w][0], bb[w][1], bb[w][2], bb[w][3], aB + off + k * 2);
+        ldmatrix_x4_trans(ss[w][0], ss[w][1], ss[w][2], ss[w][3], aS + k * (SC_PV * 2));
+      };
+      auto use = [&](int w) {
+        if (mj <= mi) {
+          mma_bf16(p[0], a[w][0], a[w][1], a[w][2], a[w][3], bb[w][0], bb[w][1]);
+          mma_bf16(p[1], a[w][0], a[w][1], a[w][2], a[w][3], bb[w][2], bb[w][3]);
         }
+        mma_bf16(Y, a[w][0], a[w][1], a[w][2], a[w][3], ss[w][0], ss[w][1]);
+        mma_bf16(Y2, a[w][0], a[w][1], a[w][2], a[w][3], ss[w][2], ss[w][3]);
+      };
+      ask(0, 0);
+      for (int k = 0; k < N; k += 32) {
+        if (k + 16 < N) ask(1, k + 16);
+        use(0);
+        if (k + 32 < N) ask(0, k + 32);
+        if (k + 16 < N) use(1);
       }
-      if (HT == 2) {
-        uint32_t b0, b1, b2, b3;
-        ldmatrix_x4_trans(b0, b1, b2, b3, smem_u32(Sh + (k + a_row) * PV + oc + a_col));
-        mma_bf16(Y[0], a0, a1, a2, a3, b0, b1);
-        mma_bf16(Y[HT - 1], a0, a1, a2, a3, b2, b3);
-        ldmatrix_x4_trans(b0, b1, b2, b3, smem_u32(Sl + (k + a_row) * PV + oc + a_col));
-        mma_bf16(Y[0], a0, a1, a2, a3, b0, b1);
-        mma_bf16(Y[HT - 1], a0, a1, a2, a3, b2, b3);
-      } else {
-        // eight columns: the high parts' two pieces of k and the low parts' in one load
-        uint32_t b0, b1, b2, b3;
-        ldmatrix_x4_trans(b0, b1, b2, b3, smem_u32((lane < 16 ? Sh : Sl) + (k + a_row) * PV + oc));
-        mma_bf16(Y[0], a0, a1, a2, a3, b0, b1);
-        mma_bf16(Y[0], a0, a1, a2, a3, b2, b3);
-      }
-    }
-    const float La = sc.L[m0 + g], Lb = sc.L[m0 + g + 8], ea = sc.e[m0 + g], eb = sc.e[m0 + g + 8];
+      // S <- 2^(L_end) S + sum_s B_s (w_s x_s)^T
+      const float keep = sc.end[0];
 #pragma unroll
-    for (int nt = 0; nt < HT; ++nt) { Y[nt][0] *= ea; Y[nt][1] *= ea; Y[nt][2] *= eb; Y[nt][3] *= eb; }
+      for (int r = 0; r < RT; ++r) {
+        if (srow + 128 * r < N) {
 #pragma unroll
-    for (int nt = 0; nt < 8; ++nt)
-      if (nt * 8 <= m0 + 15) {
-        const float2 q = *reinterpret_cast<const float2*>(sc.q + nt * 8 + 2 * t4);
-        const int s = nt * 8 + 2 * t4, row = m0 + g;
-        p[nt][0] = s <= row ? p[nt][0] * fast_exp2(La - q.x) : 0.f;
-        p[nt][1] = s + 1 <= row ? p[nt][1] * fast_exp2(La - q.y) : 0.f;
-        p[nt][2] = s <= row + 8 ? p[nt][2] * fast_exp2(Lb - q.x) : 0.f;
-        p[nt][3] = s + 1 <= row + 8 ? p[nt][3] * fast_exp2(Lb - q.y) : 0.f;
-      }
+          for (int nt = 0; nt < 2; ++nt) { S[r][nt][0] *= keep; S[r][nt][1] *= keep; S[r][nt][2] *= keep; S[r][nt][3] *= keep; }
 #pragma unroll
-    for (int ks = 0; ks < 4; ++ks) {
-      if (ks * 16 <= m0) {
-        uint32_t h0, h1, h2, h3, q0, q1, q2, q3, b0, b1, b2, b3;
-        split2(p[2 * ks][0], p[2 * ks][1], h0, q0);
-        split2(p[2 * ks][2], p[2 * ks][3], h1, q1);
-        split2(p[2 * ks + 1][0], p[2 * ks + 1][1], h2, q2);
-        split2(p[2 * ks + 1][2], p[2 * ks + 1][3], h3, q3);
-        ldmatrix_x4_trans(b0, b1, b2, b3, smem_u32(xb + (ks * 16 + a_row) * PV + oc + (HT == 2 ? a_col : 0)));
-        mma_bf16(Y[0], h0, h1, h2, h3, b0, b1);
-        mma_bf16(Y[0], q0, q1, q2, q3, b0, b1);
-        if (HT == 2) {
-          mma_bf16(Y[HT - 1], h0, h1, h2, h3, b2, b3);
-          mma_bf16(Y[HT - 1], q0, q1, q2, q3, b2, b3);
-        }
-      }
-    }
-    // S <- 2^(L_end) S + sum_s B_s (w_s x_s)^T
-    const float keep = sc.end[0];
+          for (int k2 = 0; k2 < 2; ++k2) {
+            uint32_t h[2][4];
 #pragma unroll
-    for (int r = 0; r < RT; ++r) {
-      if (warp + 8 * r < n_rt) {
+            for (int w = 0; w < 2; ++w) {
+              const int ks = 2 * k2 + w;
+              ldmatrix_x4_trans(a[w][0], a[w][1], a[w][2], a[w][3], aBt + off + (ks * 16 * PN + 128 * r) * 2);
+              ldmatrix_x4_trans(bb[w][0], bb[w][1], bb[w][2], bb[w][3], aW + ks * (16 * SC_PV * 2));
+              ldmatrix_x4_trans(h[w][0], h[w][1], h[w][2], h[w][3], aW + to_wl + ks * (16 * SC_PV * 2));
+            }
 #pragma unroll
-        for (int nt = 0; nt < NT; ++nt) { S[r][nt][0] *= keep; S[r][nt][1] *= keep; S[r][nt][2] *= keep; S[r][nt][3] *= keep; }
-#pragma unroll
-        for (int ks = 0; ks < 4; ++ks) {
-          uint32_t a0, a1, a2, a3;
-          ldmatrix_x4_trans(a0, a1, a2, a3, smem_u32(Bb + (ks * 16 + s_tok) * PN + (warp + 8 * r) * 16 + s_n));
-#pragma unroll
-          for (int np = 0; np < NT / 2; ++np) {
-            uint32_t b0, b1, b2, b3;
-            ldmatrix_x4_trans(b0, b1, b2, b3, smem_u32(wh + (ks * 16 + a_row) * PV + np * 16 + a_col));
-            mma_bf16(S[r][2 * np], a0, a1, a2, a3, b0, b1);
-            mma_bf16(S[r][2 * np + 1], a0, a1, a2, a3, b2, b3);
-            ldmatrix_x4_trans(b0, b1, b2, b3, smem_u32(wl + (ks * 16 + a_row) * PV + np * 16 + a_col));
-            mma_bf16(S[r][2 * np], a0, a1, a2, a3, b0, b1);
-            mma_bf16(S[r][2 * np + 1], a0, a1, a2, a3, b2, b3);
+            for (int w = 0; w < 2; ++w) {
+              mma_bf16(S[r][0], a[w][0], a[w][1], a[w][2], a[w][3], bb[w][0], bb[w][1]);
+              mma_bf16(S[r][1], a[w][0], a[w][1], a[w][2], a[w][3], bb[w][2], bb[w][3]);
+              mma_bf16(S[r][0], a[w][0], a[w][1], a[w][2], a[w][3], h[w][0], h[w][1]);
+              mma_bf16(S[r][1], a[w][0], a[w][1], a[w][2], a[w][3], h[w][2], h[w][3]);
+            }
           }
         }
       }
+      if (mj <= mi) {
+        const float La = sc.L[m0 + g], Lb = sc.L[m0 + g + 8];
+#pragma unroll
+        for (int nt = 0; nt < 2; ++nt) {
+          const int s = mj * 16 + nt * 8 + 2 * t4, row = m0 + g;
+          const float2 q = *reinterpret_cast<const float2*>(sc.q + s);
+          p[nt][0] = s <= row ? p[nt][0] * fast_exp2(La - q.x) : 0.f;
+          p[nt][1] = s + 1 <= row ? p[nt][1] * fast_exp2(La - q.y) : 0.f;
+          p[nt][2] = s <= row + 8 ? p[nt][2] * fast_exp2(Lb - q.x) : 0.f;
+          p[nt][3] = s + 1 <= row + 8 ? p[nt][3] * fast_exp2(Lb - q.y) : 0.f;
+          uint32_t hi, lo;
+          split2(p[nt][0], p[nt][1], hi, lo);
+          *reinterpret_cast<uint32_t*>(Ph + row * SC_PP + s) = hi;
+          *reinterpret_cast<uint32_t*>(Pl + row * SC_PP + s) = lo;
+          split2(p[nt][2], p[nt][3], hi, lo);
+          *reinterpret_cast<uint32_t*>(Ph + (row + 8) * SC_PP + s) = hi;
+          *reinterpret_cast<uint32_t*>(Pl + (row + 8) * SC_PP + s) = lo;
+        }
+      }
+      const float ea = sc.e[m0 + g], eb = sc.e[m0 + g + 8];
+      Y[0] *= ea; Y[1] *= ea; Y[2] *= eb; Y[3] *= eb;
+      Y2[0] *= ea; Y2[1] *= ea; Y2[2] *= eb; Y2[3] *= eb;
+      asm volatile("cp.async.wait_group 0;\n" ::);
     }
-    const int n = min(SC_T, t1 - c0);
+    __syncthreads();                       // (2)
+    if (!worker) continue;
+    // the chunk's own tokens: the weighted scores times x
 #pragma unroll
-    for (int half = 0; half < 2; ++half) {
-      const int row = m0 + g + half * 8;
-      if (row >= n) continue;
-      float* o = y + (size_t)(c0 + row) * z.inner() + (size_t)h * V + col0;
-#pragma unroll
-      for (int nt = 0; nt < HT; ++nt) {
-        const int c = oc + nt * 8 + 2 * t4;
-        if (col0 + c >= V) continue;
-        const uint32_t v = *reinterpret_cast<const uint32_t*>(xb + row * PV + c);
-        *reinterpret_cast<float2*>(o + c) = make_float2(fmaf(sk, __uint_as_float(v << 16), Y[nt][2 * half]),
-                                                        fmaf(sk, __uint_as_float(v & 0xffff0000u), Y[nt][2 * half + 1]));
+    for (int k2 = 0; k2 < 2; ++k2) {
+      if (2 * k2 <= mi) {
+        uint32_t b0, b1, b2, b3, h[2][4], l[2][4];
+        ldmatrix_x4_trans(b0, b1, b2, b3, aX + buf * bytes_x + k2 * (32 * SC_PV * 2));      // 32 tokens, eight columns
+        ldmatrix_x4(h[0][0], h[0][1], h[0][2], h[0][3], aP + k2 * 64);
+        ldmatrix_x4(l[0][0], l[0][1], l[0][2], l[0][3], aP + to_pl + k2 * 64);
+        if (2 * k2 + 1 <= mi) {
+          ldmatrix_x4(h[1][0], h[1][1], h[1][2], h[1][3], aP + k2 * 64 + 32);
+          ldmatrix_x4(l[1][0], l[1][1], l[1][2], l[1][3], aP + to_pl + k2 * 64 + 32);
+        }
+        mma_bf16(Y, h[0][0], h[0][1], h[0][2], h[0][3], b0, b1);
+        mma_bf16(Y2, l[0][0], l[0][1], l[0][2], l[0][3], b0, b1);
+        if (2 * k2 + 1 <= mi) {
+          mma_bf16(Y, h[1][0], h[1][1], h[1][2], h[1][3], b2, b3);
+          mma_bf16(Y2, l[1][0], l[1][1], l[1][2], l[1][3], b2, b3);
+        }
       }
     }
-    if (warp == 0 && c0 + SC_T < t1) scan(scales[buf ^ 1]);
+    if (more) lay_out(buf ^ 1);
+    const int n = min(SC_T, t1 - c0), c = mj * 8 + 2 * t4;
+    if (col0 + c < V) {
+#pragma unroll
+      for (int half = 0; half < 2; ++half) {
+        const int row = m0 + g + half * 8;
+        if (row >= n) continue;
+        const uint32_t v = *reinterpret_cast<const uint32_t*>(xs + (buf * SC_T + row) * SC_PV + c);
+        *reinterpret_cast<float2*>(y + (size_t)(c0 + row) * z.inner() + (size_t)h * V + col0 + c) =
+            make_float2(fmaf(sk, __uint_as_float(v << 16), Y[2 * half] + Y2[2 * half]),
+                        fmaf(sk, __uint_as_float(v & 0xffff0000u), Y[2 * half + 1] + Y2[2 * half + 1]));
+      }
+    }
   }
+  if (!worker) return;
   if (!write_state) return;
 #pragma unroll
   for (int r = 0; r < RT; ++r)
 #pragma unroll
-    for (int nt = 0; nt < NT; ++nt) {
-      const int n = (warp + 8 * r) * 16 + g, c = nt * 8 + 2 * t4;
-      if (warp + 8 * r >= n_rt || col0 + c >= V) continue;
+    for (int nt = 0; nt < 2; ++nt) {
+      const int n = srow + 128 * r + g, c = nt * 8 + 2 * t4;
+      if (srow + 128 * r >= N || col0 + scol + c >= V) continue;
       *reinterpret_cast<float2*>(st + (size_t)n * V + c) = make_float2(S[r][nt][0], S[r][nt][1]);
       *reinterpret_cast<float2*>(st + (size_t)(n + 8) * V + c) = make_float2(S[r][nt][2], S[r][nt][3]);
     }
@@ -737,25 +773,23 @@ ssm_chunks_kernel(const bf16* __restrict__ xbc, const float* __restrict__ la, co
 AB_API int ab_ssm_chunks_supports(int N, int V) { return N > 0 && N <= 256 && N % 16 == 0 && V > 0 && V <= 256 && V % 8 == 0 ? 1 : 0; }
 
 // xbc bfloat16 [T, channels] (x | B | C), la and dt float32 [T, H] (log decays, step sizes), y float32 [T, H * V].
-// `cols`: value columns per CTA (16 or 32).
 AB_API int ab_ssm_chunks(const void* xbc, const float* la, const float* dt, const float* skip, float* state, float* y,
-                         const int* cu_q, const int* slots, int n_seqs, int H, int G, int N, int V, int cols, int write_state,
+                         const int* cu_q, const int* slots, int n_seqs, int H, int G, int N, int V, int write_state,
                          cudaStream_t stream) {
   if (n_seqs <= 0) return AB_OK;
   const SsmSizes z{H, G, N, V, 1};
   if (!ssm_sizes_ok(z) || !ab_ssm_chunks_supports(N, V) || H > 65535 || ((((uintptr_t)xbc) | ((uintptr_t)state)) & 15)) return AB_BAD_ARG;
-  const dim3 grid((unsigned)n_seqs, (unsigned)H, (unsigned)((V + cols - 1) / cols));
-#define AB_GO(CV, RT)                                                                                                  \
+  if ((H * V) % 8 || (G * N) % 8) return AB_BAD_ARG;              // rows of 16-byte pieces
+  const dim3 grid((unsigned)n_seqs, (unsigned)H, (unsigned)((V + SC_CV - 1) / SC_CV));
+  const size_t smem = chunk_smem(N);
+#define AB_GO(RT)                                                                                                      \
   {                                                                                                                    \
-    const size_t smem = ChunkSmem<CV>::total(N);                                                                       \
-    cudaError_t e = cudaFuncSetAttribute(ssm_chunks_kernel<CV, RT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
+    cudaError_t e = cudaFuncSetAttribute(ssm_chunks_kernel<RT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
     if (e != cudaSuccess) return AB_CUDA_ERR + (int)e;                                                                 \
-    ab_launch(ssm_chunks_kernel<CV, RT>, grid, dim3(256), smem, stream, (const bf16*)xbc, la, dt, skip, state, y, cu_q, slots, \
+    ab_launch(ssm_chunks_kernel<RT>, grid, dim3(SC_THREADS), smem, stream, (const bf16*)xbc, la, dt, skip, state, y, cu_q, slots, \
               z, write_state);                                                                                         \
   }
-  if (cols == 32) { if (N <= 128) AB_GO(32, 1) else AB_GO(32, 2) }
-  else if (cols == 16) { if (N <= 128) AB_GO(16, 1) else AB_GO(16, 2) }
-  else return AB_BAD_ARG;
+  if (N <= 128) AB_GO(1) else AB_GO(2)
 #undef AB_GO
   return ab_launch_status();
 }

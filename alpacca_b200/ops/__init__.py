@@ -2375,10 +2375,8 @@ def ssm_chunks(xbc, log_decay, dt, skip, state, y, ctx, H, G, N, V, write_state=
           "ssm_chunks: state float32 [slots, H, N, V], y float32 [T, H * V]")
     _i32(ctx.cu_q, ctx.n_seqs + 1, "cu_q")
     _i32(ctx.slots, ctx.n_seqs, "slots")
-    cols = 32 if V > 16 else 16
     _check(_lib("state_space").ab_ssm_chunks(_p(xbc), _p(log_decay), _p(dt), _p(skip), _p(state), _p(y), _p(ctx.cu_q),
-                                             _p(ctx.slots), ctx.n_seqs, H, G, N, V, cols, 1 if write_state else 0, _stream()),
-           "ssm_chunks")
+                                             _p(ctx.slots), ctx.n_seqs, H, G, N, V, 1 if write_state else 0, _stream()), "ssm_chunks")
     return y
 
 

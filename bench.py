@@ -45,6 +45,11 @@ two mixers side by side, routed gated experts of the same sizes, norms around ev
 layer reading the keys of the layer before; experts chosen by token id beside a shared one; norms on the sub-layers'
 outputs, an input convolution and an average over depth in every layer), beside the Sazepel decoder (routed gated
 experts of the same sizes), the Buguzen decoder (attention with a window and a query/key norm) and the Llama decoder.
+`--design nagavik` does the same for the Nagavik decoder (state-space mixers, every fourth layer attention with bounded scores
+and a slope per head; ungated experts chosen by sigmoid scores beside a shared one; norms around every sub-layer), beside the
+Mavidra decoder (the closest: recurrences with decays that depend on the token, short convolutions, a sink attention, experts
+with sigmoid scores, norms around every sub-layer), the Ponusun decoder (the same experts' kernels with gates, attention with
+a penalty on distance) and the Llama decoder.
 
 One JSON line goes to standard output.  With --gpus N > 1 it prints a line that says so and exits
 with 2: this library runs on one GPU.

@@ -464,3 +464,14 @@ def test_layer_scale_after_the_norm(dtype, width):
     h = plain.rms_norm(f64(x), w["n1"], 1e-4)
     want = plain.rms_norm(h, w["n1b"], 1e-4) * w["ls"]
     close(stream.residual.double().cpu().numpy() - f64(x), want, dtype, "layer scale", tol=(3e-5, 3e-6) if dtype == "float32" else (0.03, 0.004))
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("n", [1, 8, 14, 60])
+def test_plain_feed_forward_with_the_square_of_relu(dtype, n):
+    from alpacca_b200.parts import PlainFeedForward
+    part = PlainFeedForward(opts_of(dtype), 48, 37, "m", activation="relu2", out_dtype=torch.float32)
+    w = short(load_part(part, seed=n, dtype=dtype, std=0.3), "m")
+    x, x64 = hidden(np.random.default_rng(n), n, 48, dtype)
+    close(part.forward(x, Ctx(n)).float().cpu().numpy()[:n], plain.expert(x64, w["up"], w["down"]), dtype, "squared ReLU",
+          tol=None if dtype == "float32" else (0.1, 0.01))
