@@ -282,11 +282,26 @@ __global__ void add_bias_kernel(T* __restrict__ y, const float* __restrict__ bia
   y[i] = from_f32<T>(to_f32(y[i]) + bias[i % width]);
 }
 
+// the same for float32 rows of whole quads, 16 bytes per thread
+__global__ void add_bias4_kernel(float4* __restrict__ y, const float4* __restrict__ bias, unsigned total4, unsigned width4) {
+  pdl_wait();
+  pdl_trigger();
+  const unsigned i = blockIdx.x * blockDim.x + threadIdx.x;
+  if (i >= total4) return;
+  const float4 b = bias[i % width4];
+  float4 v = y[i];
+  v.x += b.x; v.y += b.y; v.z += b.z; v.w += b.w;
+  y[i] = v;
+}
+
 AB_API int ab_add_bias(void* y, int dtype, const float* bias, int n_rows, int width, cudaStream_t stream) {
   size_t total = (size_t)n_rows * width;
   if (total == 0) return AB_OK;
   unsigned blocks = (unsigned)((total + 255) / 256);
-  if (dtype == AB_F32)
+  if (dtype == AB_F32 && width % 4 == 0 && total / 4 < 0x7fffffffULL && ((((uintptr_t)y) | ((uintptr_t)bias)) & 15) == 0)
+    ab_launch(add_bias4_kernel, (unsigned)((total / 4 + 255) / 256), 256, 0, stream, (float4*)y, (const float4*)bias,
+              (unsigned)(total / 4), (unsigned)(width / 4));
+  else if (dtype == AB_F32)
     ab_launch(add_bias_kernel<float>, blocks, 256, 0, stream, (float*)y, bias, total, width);
   else if (dtype == AB_BF16)
     ab_launch(add_bias_kernel<bf16>, blocks, 256, 0, stream, (bf16*)y, bias, total, width);

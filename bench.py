@@ -686,10 +686,10 @@ def _nagavik_config(z):
     moe = {"kind": "moe", "expert": {"ff": ff}, "router": {"experts": rt["experts"], "top": rt["top"]}, "shared": {"ff": 2 * ff}}
     ssm = {"type": "mamba2", "mixer": {"heads": z["width"] // 32, "vdim": 64, "state": 128, "groups": 4, "conv": 4, "norm_groups": 4}}
     att = {"type": "attention", "mixer": {"heads": z["heads"], "kv_heads": z["kv_heads"], "dim": z["head_dim"], "vdim": z["head_dim"],
-                                          "scale": z["head_dim"] ** -0.5, "softcap": 20.0}}
+                                          "scale": z["head_dim"] ** -0.5, "softcap": 16.0}}
     layers = [dict(att if i % 4 == 3 else ssm, mlp=moe if i else {"kind": "dense", "ff": z["dense_ff"]}) for i in range(z["layers"])]
     return {"architecture": "Nagavik", "vocab": z["vocab"], "width": z["width"], "max_positions": 8192, "norm": {"eps": 1e-6},
-            "embedding": {"scale": 4.0}, "logit_softcap": 30.0, "layers": layers}
+            "embedding": {"scale": 4.0}, "logit_softcap": 40.0, "layers": layers}
 
 
 def design_configs(size, design="lefatar"):

@@ -322,7 +322,7 @@ def planted(shape, dtype, places, asking, n, slopes, score):
 
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("decode", [False, True])
-@pytest.mark.parametrize("shape", [(4, 2, 64, 64), (4, 2, 128, 128), (2, 2, 32, 32), (2, 1, 16, 32), (3, 1, 24, 24), (8, 2, 48, 80)])
+@pytest.mark.parametrize("shape", [(4, 2, 64, 64), (4, 2, 128, 128), (2, 2, 32, 32), (2, 1, 16, 32), (3, 1, 24, 24), (10, 2, 48, 112)])
 def test_planted_keys_fall_with_their_distance(dtype, decode, shape):
     """Keys on the first token, at page borders, next to the asking one and 668 tokens back, each alone: its weight is
     e^s / (1 + sum), s the bounded score less slope times distance, beside the other keys (score 0 less the same penalty) and
